@@ -5,7 +5,7 @@
 //
 // writes /some/dir/pid<N>/launches.jsonl, one JSON object per line:
 //
-//     {"kind":"module", "t_ns", "handle", "sha256", "bytes", "format": "elf"|"fatbin"|"text"}
+//     {"kind":"module", "t_ns", "handle", "sha256", "bytes"}
 //     {"kind":"alloc",  "t_ns", "ptr", "bytes"}          {"kind":"free", "t_ns", "ptr"}
 //     {"kind":"tensormap", "t_ns", "id", "hex" (the 128 encoded bytes), "dtype", "rank", "address", "dims", "strides",
 //      "box", "elem_strides", "interleave", "swizzle", "l2_promotion", "oob_fill"}
@@ -16,8 +16,10 @@
 // The staged bytes of every parameter are recorded as the launch call holds them (its offset and size come from the
 // driver's own description of the function); an 8-byte word that points into a live allocation is marked with the
 // allocation it falls into, and a 128-byte run equal to a descriptor that the process encoded is marked with that
-// descriptor's record, wherever in a struct it sits. Module images are hashed, never stored: a manifest pins a module by
-// the sha256 of its file, which is what the hash of a loaded image reproduces.
+// descriptor's record, wherever in a struct it sits. Module images are never read: a program that wants its launches
+// tied to the modules it built names them through `kern_capture_module` (the runtime here does: it hashes the files it
+// loads anyway; the library leaves the function's address in the environment as KERN_CAPTURE_MODULE_HOOK). Launches out
+// of any other module carry `"module": null`.
 //
 // The library subscribes to the driver-API callback domain of the profiling interface, which it opens at run time
 // (`KERN_CUPTI_LIB` names the file if the loader cannot find one) and tells calls apart by the name the callback
@@ -43,8 +45,6 @@
 #include <string>
 #include <vector>
 
-#include "common/sha256.hpp"
-
 namespace {
 
 // ---- the slice of the profiling interface this file uses (layouts are part of its public ABI) ----
@@ -68,7 +68,6 @@ struct LaunchCoopArgs { void* f; unsigned gx, gy, gz, bx, by, bz, smem; void* st
 struct LaunchAttr { int id; int pad; unsigned char value[64]; };
 struct LaunchConfig { unsigned gx, gy, gz, bx, by, bz, smem; void* stream; LaunchAttr* attrs; unsigned n_attrs; };
 struct LaunchExArgs { const LaunchConfig* config; void* f; void** params; void** extra; };
-struct ModuleLoadDataArgs { void** module; const void* image; };
 struct MemAllocArgs { uint64_t* dptr; size_t bytes; };
 struct MemFreeArgs { uint64_t dptr; };
 struct AddressReserveArgs { uint64_t* ptr; size_t size; size_t alignment; uint64_t addr; unsigned long long flags; };
@@ -119,52 +118,6 @@ std::string quoted(const char* s) {
   return o + "\"";
 }
 
-// How many bytes a module image spans, from its own header, and which kind it is.
-size_t image_size(const void* image, const char** format) {
-  const unsigned char* p = static_cast<const unsigned char*>(image);
-  uint32_t magic;
-  memcpy(&magic, p, 4);
-  if (magic == 0x466243B1u) {                   // a wrapper {magic, version, const void* data, ...}: follow it
-    const void* data;
-    memcpy(&data, p + 8, sizeof data);
-    return data ? image_size(data, format) : 0;
-  }
-  if (magic == 0xBA55ED50u) {                   // fat binary: {magic, u16 version, u16 header size, u64 payload size}
-    uint16_t header;
-    uint64_t payload;
-    memcpy(&header, p + 6, 2);
-    memcpy(&payload, p + 8, 8);
-    *format = "fatbin";
-    return (size_t)header + (size_t)payload;
-  }
-  if (memcmp(p, "\x7f" "ELF", 4) == 0 && p[4] == 2) {   // ELF64: the furthest byte any table or section reaches
-    uint64_t shoff, phoff;
-    uint16_t shentsize, shnum, phentsize, phnum;
-    memcpy(&phoff, p + 0x20, 8);
-    memcpy(&shoff, p + 0x28, 8);
-    memcpy(&phentsize, p + 0x36, 2);
-    memcpy(&phnum, p + 0x38, 2);
-    memcpy(&shentsize, p + 0x3A, 2);
-    memcpy(&shnum, p + 0x3C, 2);
-    uint64_t end = 64;
-    if (shoff) end = std::max<uint64_t>(end, shoff + (uint64_t)shentsize * shnum);
-    if (phoff) end = std::max<uint64_t>(end, phoff + (uint64_t)phentsize * phnum);
-    for (uint16_t i = 0; shoff && i < shnum; ++i) {
-      const unsigned char* sh = p + shoff + (uint64_t)i * shentsize;
-      uint32_t type;
-      uint64_t off, size;
-      memcpy(&type, sh + 4, 4);
-      memcpy(&off, sh + 0x18, 8);
-      memcpy(&size, sh + 0x20, 8);
-      if (type != 8) end = std::max(end, off + size);   // 8: a section that occupies no file bytes
-    }
-    *format = "elf";
-    return (size_t)end;
-  }
-  *format = "text";
-  return strnlen(reinterpret_cast<const char*>(p), (size_t)1 << 28);
-}
-
 void emit(const std::string& line) {
   if (!g_out) return;
   fputs(line.c_str(), g_out);
@@ -179,23 +132,15 @@ std::string list_of(const T* v, size_t n) {
   return o + "]";
 }
 
-void on_module(const void* image, void* handle) {
-  if (!image) return;
-  const char* format = "?";
-  const size_t n = image_size(image, &format);
-  uint32_t magic;
-  memcpy(&magic, image, 4);
-  const void* bytes = image;
-  if (magic == 0x466243B1u) memcpy(&bytes, static_cast<const unsigned char*>(image) + 8, sizeof bytes);
-  kern::Sha256 h;
-  h.update(bytes, n);
-  const std::string sha = kern::Sha256::hex(h.finish());
+// A module the launching program loaded and names itself: the program read the file it was built into and knows its
+// hash. The images that other programs and libraries hand to the driver are not looked at.
+void on_module(void* handle, const char* sha, size_t bytes) {
   char b[64];
   snprintf(b, sizeof b, "\"0x%" PRIx64 "\"", (uint64_t)(uintptr_t)handle);
   std::lock_guard<std::mutex> g(g_mu);
   g_modules[handle] = sha;
   emit("{\"kind\":\"module\",\"t_ns\":" + std::to_string(now_ns()) + ",\"handle\":" + b + ",\"sha256\":\"" + sha +
-       "\",\"bytes\":" + std::to_string(n) + ",\"format\":\"" + format + "\"}");
+       "\",\"bytes\":" + std::to_string(bytes) + "}");
 }
 
 void on_alloc(uint64_t ptr, uint64_t bytes) {
@@ -352,10 +297,7 @@ void callback(void*, int domain, uint32_t, const void* data) {
       on_free(static_cast<const MemFreeArgs*>(d.params)->dptr);
     }
   } else if (ok) {
-    if (is(fn, "cuModuleLoadData") || is(fn, "cuModuleLoadDataEx") || is(fn, "cuModuleLoadFatBinary") || is(fn, "cuLibraryLoadData")) {
-      const auto& a = *static_cast<const ModuleLoadDataArgs*>(d.params);
-      on_module(a.image, a.module ? *a.module : nullptr);
-    } else if (is(fn, "cuMemAlloc") || is(fn, "cuMemAllocAsync") || is(fn, "cuMemAllocManaged") || is(fn, "cuMemAllocFromPoolAsync")) {
+    if (is(fn, "cuMemAlloc") || is(fn, "cuMemAllocAsync") || is(fn, "cuMemAllocManaged") || is(fn, "cuMemAllocFromPoolAsync")) {
       const auto& a = *static_cast<const MemAllocArgs*>(d.params);
       if (a.dptr) on_alloc(*a.dptr, a.bytes);
     } else if (is(fn, "cuMemAddressReserve")) {
@@ -403,9 +345,17 @@ extern "C" void kern_capture_feed(const char* function_name, int site, const voi
   callback(nullptr, kDomainDriver, 0, &d);
 }
 
+// The launching program's word about a module it loaded: its handle, the sha256 of its file, the file's size.
+extern "C" void kern_capture_module(void* handle, const char* sha256, size_t bytes) {
+  if (sha256) on_module(handle, sha256, bytes);
+}
+
 // The driver calls this once, when the process initialises CUDA with CUDA_INJECTION64_PATH naming this file.
 extern "C" int InitializeInjection(void) {
   if (!open_output()) return 0;
+  char hook[32];
+  snprintf(hook, sizeof hook, "%" PRIxPTR, reinterpret_cast<uintptr_t>(&kern_capture_module));
+  setenv("KERN_CAPTURE_MODULE_HOOK", hook, 1);
 
   if (void* cuda = dlopen("libcuda.so.1", RTLD_NOW | RTLD_GLOBAL)) {
     cuFuncGetParamInfo_ = reinterpret_cast<decltype(cuFuncGetParamInfo_)>(dlsym(cuda, "cuFuncGetParamInfo"));
