@@ -2,6 +2,7 @@
 //
 //   kern_moe_route_f32      router scores -> top-k expert ids and weights per token (sigmoid or softmax scoring,
 //                           optional selection bias, renormalise, scale)
+//   kern_moe_route_logits   the same by the logits plus a bias: top-k largest, softmax over the chosen
 //   kern_moe_plan           counts per expert -> row offsets, the permuted row of every (token, choice), and the
 //                           M-tile table the grouped GEMM walks; experts outside [e_lo, e_hi) belong to another rank
 //   kern_moe_gather_bf16    x_perm[perm[t, j]] = x[t]
@@ -84,6 +85,51 @@ extern "C" __global__ void __launch_bounds__(128)
     const float w = renorm ? my_w / (wsum + 1e-20f) : my_w;
     topk_ids[(size_t)t * k + lane] = my_id;
     topk_w[(size_t)t * k + lane] = w * scale;
+  }
+}
+
+// Routing on the logits themselves: z = logits + bias (bf16, one per expert, may be null), the k largest are chosen (ties:
+// the lower id) and weigh in by the softmax over the chosen ones. One warp per token; E <= 1024, k <= 32.
+extern "C" __global__ void __launch_bounds__(128)
+    kern_moe_route_logits(const float* logits, const __nv_bfloat16* bias, int* topk_ids, float* topk_w, int tokens, int experts,
+                          int k, int ld) {
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * 4 + warp;
+  if (t >= tokens) return;
+  constexpr int PER = 32;
+  float z[PER];
+  const float* row = logits + (size_t)t * ld;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int e = i * 32 + lane;
+    z[i] = e < experts ? row[e] + (bias ? __bfloat162float(bias[e]) : 0.f) : -INFINITY;
+  }
+  float my_z = -INFINITY, top = 0.f;
+  int my_id = 0;
+  for (int j = 0; j < k; ++j) {
+    float best = -INFINITY;
+    int bi = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (z[i] > best) { best = z[i]; bi = i * 32 + lane; }
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+    }
+    if (bi >= experts) bi = 0;                     // no logit is a number: still a valid row
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (i * 32 + lane == bi) z[i] = -INFINITY;
+    if (j == 0) top = best;
+    if (lane == j) { my_z = best; my_id = bi; }
+  }
+  const float e = lane < k ? expf(my_z - top) : 0.f;
+  const float sum = warp_sum(e);
+  if (lane < k) {
+    topk_ids[(size_t)t * k + lane] = my_id;
+    topk_w[(size_t)t * k + lane] = e / sum;
   }
 }
 

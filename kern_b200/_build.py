@@ -70,23 +70,33 @@ def kernels_dir(checked_build: bool | None = None) -> Path:
     return KOUT_CHECKED if (checked() if checked_build is None else checked_build) else KOUT
 
 
-def build_kernels(force: bool = False, verbose: bool = False, checked_build: bool = False) -> dict[str, dict]:
-    """Compile every kernel source to ``kernels/<stem>.cubin`` (``kernels_checked/`` with -DKERN_CHECKED for the checked
-    build); return the module index."""
+def nvcc_flags(src: Path) -> list[str]:
+    """A source whose first line says ``// build: precise`` is compiled without the fast-math substitutions."""
+    with open(src) as f:
+        precise = f.readline().strip() == "// build: precise"
+    return [x for x in NVCC_FLAGS if not (precise and x == "--use_fast_math")]
+
+
+def build_kernels(force: bool = False, verbose: bool = False, checked_build: bool = False, only=None) -> dict[str, dict]:
+    """Compile every kernel source (or those named by ``only``) to ``kernels/<stem>.cubin`` (``kernels_checked/`` with
+    -DKERN_CHECKED for the checked build); return the module index, which lists what is compiled and current."""
     KOUT = kernels_dir(checked_build)
     KOUT.mkdir(parents=True, exist_ok=True)
     headers = sorted(KSRC.glob("*.cuh"))
-    jobs = []
+    jobs, stale = [], set()
     for src in kernel_sources():
         out = KOUT / (src.stem + ".cubin")
         # a source that includes another kernel source (the GEMM body shared by several modules) depends on it too
         included = [KSRC / m for m in re.findall(r'#include\s+"([\w.]+\.cu)"', src.read_text())]
         if force or _newer([src, *headers, *included], out):
-            jobs.append((src, out))
+            if only is None or src.stem in only:
+                jobs.append((src, out))
+            else:
+                stale.add(src.stem)
 
     def one(job):
         src, out = job
-        cmd = [NVCC, *ARCH, *NVCC_FLAGS, *(["-DKERN_CHECKED"] if checked_build else []), "-cubin", "-I", str(KSRC), "-o", str(out), str(src)]
+        cmd = [NVCC, *ARCH, *nvcc_flags(src), *(["-DKERN_CHECKED"] if checked_build else []), "-cubin", "-I", str(KSRC), "-o", str(out), str(src)]
         text = _run(cmd, BUILD / ("ptxas_checked" if checked_build else "ptxas") / (src.stem + ".log"))
         if verbose:
             print(text)
@@ -96,6 +106,8 @@ def build_kernels(force: bool = False, verbose: bool = False, checked_build: boo
             list(ex.map(one, jobs))
     index = {}
     for src in kernel_sources():
+        if src.stem in stale:
+            continue
         out = KOUT / (src.stem + ".cubin")
         data = out.read_bytes()
         index[src.stem] = {"source": out.name, "sha256": hashlib.sha256(data).hexdigest()}
@@ -216,9 +228,33 @@ def build_all(force: bool = False, verbose: bool = False) -> None:
             fcntl.flock(lock, fcntl.LOCK_UN)
 
 
+def on_demand() -> bool:
+    """KERN_B200_BUILD=demand: importing the package builds the C++ core only, and a manifest's kernel modules are
+    compiled when the manifest is generated."""
+    return os.environ.get("KERN_B200_BUILD") == "demand"
+
+
+def _locked(what):
+    BUILD.mkdir(exist_ok=True)
+    with open(BUILD / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        try:
+            return what()
+        finally:
+            fcntl.flock(lock, fcntl.LOCK_UN)
+
+
+def build_some(modules) -> dict[str, dict]:
+    """The named kernel modules; returns the index of everything that is compiled."""
+    return _locked(lambda: build_kernels(only=set(modules), checked_build=checked()))
+
+
 def ensure_built() -> None:
     """Build whatever is missing or stale. Cheap when everything is current."""
     try:
+        if on_demand():
+            _locked(build_native)
+            return
         build_all(False)
     except FileNotFoundError as e:  # no compiler on this machine: use what is in the tree
         if not native_path().exists():

@@ -29,19 +29,22 @@ if hasattr(torch, "float8_e4m3fn"):
     _ST_DTYPES[torch.float8_e4m3fn] = "F8_E4M3"
 
 
-def kernel_index() -> dict:
-    """sha256 pins of the in-tree cubins, written by the build."""
+def kernel_index(names=None) -> dict:
+    """sha256 pins of the in-tree cubins, written by the build. `names`: the modules that must be current (on-demand
+    builds compile just those)."""
     from .. import _build
 
+    if names is not None and _build.on_demand():
+        return _build.build_some(names)
     _build.ensure_built()
     return json.loads((KERNELS_DIR / "index.json").read_text())
 
 
 def modules_for(names) -> dict:
-    idx = kernel_index()
     names = list(names)
     if "gemm_bf16" in names and "gemv_bf16" not in names:
         names.append("gemv_bf16")          # every gemm_op carries the weight-streaming launches for a handful of rows
+    idx = kernel_index(names)
     return {n: {"source": idx[n]["source"], "sha256": idx[n]["sha256"], "multicast": False} for n in names}
 
 
