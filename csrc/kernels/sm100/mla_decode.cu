@@ -27,13 +27,22 @@ namespace {
 constexpr int MW = 8;                    // math warps: 512 / MW value columns each for O
 constexpr int TKM = 64;                  // tokens per tile
 constexpr int SW = TKM / 8;              // warps that take part in S = Q K^T, 8 tokens of the tile each
-constexpr int DQK = 576, DVV = 512;
 constexpr int HM = 16;                   // heads per CTA
-constexpr int kTileBytes = TKM * DQK * 2;
-constexpr int kStagesM = TKM == 48 ? 3 : 2;   // 48-token tiles (54 KB) three deep, or 64-token tiles two deep
-constexpr int ON = DVV / MW / 8;             // 8-column accumulator tiles per warp
-constexpr int kQStride = DQK + 8, kPStride = TKM + 8;
-constexpr int kQBytes = HM * kQStride * 2, kPBytes = HM * kPStride * 2;
+constexpr int kPStride = TKM + 8, kPBytes = HM * kPStride * 2;
+constexpr int DQK = 576;                 // row of the 512 + 64 form
+
+// QB / VB: 64-column blocks of a cached row that serve as key / value. The 512 + 64 form is <9, 8>; a latent without
+// rotary columns is <B, B>, its last block filled up with zeros by the copy when the width is not a multiple of 64.
+template <int QB, int VB>
+struct MlaCfg {
+  static constexpr int kQ = QB * 64;
+  static constexpr int kTileBytes = TKM * kQ * 2;
+  // 64-token tiles of 72 KB two deep; narrower rows go deeper, up to about 144 KB
+  static constexpr int kStages = QB >= 8 ? 2 : (QB >= 5 ? 3 : (QB >= 3 ? 4 : 6));
+  static constexpr int kON = VB;         // 8-column accumulator tiles per warp
+  static constexpr int kQStride = kQ + 8;
+  static constexpr int kQBytes = HM * kQStride * 2;
+};
 
 KERN_DEVICE void ldsm4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
@@ -54,15 +63,17 @@ KERN_DEVICE void math_bar() { asm volatile("bar.sync 1, %0;" ::"n"(MW * 32) : "m
 
 }  // namespace
 
-// grid [ceil(H / 16), seqs, splits], block 32 MW + 32, dynamic shared memory MLA_SMEM bytes.
+// grid [ceil(H / 16), seqs, splits], block 32 MW + 32, dynamic shared memory: 1024 + stages + queries + probabilities +
+// 1024 + 256 bytes. `q_cols` / `v_cols`: the columns a head's query / result row really has.
 // `splits` packs (launch splits | first slot << 8 | slots per (row, head) << 16) as the GQA decode kernel does.
-constexpr int MLA_SMEM = 1024 + kStagesM * kTileBytes + kQBytes + kPBytes + 2 * MW * HM * 4 + 128;
-
-extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)
-    kern_mla_decode_bf16(const __grid_constant__ CUtensorMap lat_map, const __nv_bfloat16* q, __nv_bfloat16* out, float* ws_o,
-                         float* ws_ml, const int* block_table, const int* seq_lens, int seqs, int heads, int q_stride,
-                         int out_stride, int max_pages, int page_size, int splits, int pool_pages, float scale_log2, int* err,
-                         const int* row_seq) {
+template <int QB, int VB>
+__device__ __forceinline__ void mla_body(const CUtensorMap* lat_map, const __nv_bfloat16* q, __nv_bfloat16* out, float* ws_o,
+                                         float* ws_ml, const int* block_table, const int* seq_lens, int seqs, int heads,
+                                         int q_stride, int out_stride, int max_pages, int page_size, int splits, int pool_pages,
+                                         float scale_log2, int* err, const int* row_seq, int q_cols, int v_cols) {
+  using Cfg = MlaCfg<QB, VB>;
+  constexpr int kStagesM = Cfg::kStages, kTileBytes = Cfg::kTileBytes, kQBytes = Cfg::kQBytes, kQStride = Cfg::kQStride;
+  constexpr int ON = Cfg::kON;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* stages = smem;
@@ -83,7 +94,7 @@ extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)
     }
     *abort_flag = 0;
     mbar_fence_init();
-    tma_prefetch_desc(&lat_map);
+    tma_prefetch_desc(lat_map);
   }
   __syncthreads();
   pdl_wait();
@@ -105,10 +116,11 @@ extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)
   const int ntiles = tile_hi - tile_lo;
 
   // the 16 query rows (one per head) -> shared
-  for (int i = threadIdx.x; i < HM * (DQK / 8); i += blockDim.x) {
-    const int r = i / (DQK / 8), c = i % (DQK / 8);
+  for (int i = threadIdx.x; i < HM * (QB * 8); i += blockDim.x) {
+    const int r = i / (QB * 8), c = i % (QB * 8);
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < valid_rows) v = *reinterpret_cast<const uint4*>(q + (size_t)seq * q_stride + (size_t)(head0 + r) * DQK + c * 8);
+    if (r < valid_rows && c * 8 < q_cols)
+      v = *reinterpret_cast<const uint4*>(q + (size_t)seq * q_stride + (size_t)(head0 + r) * q_cols + c * 8);
     *reinterpret_cast<uint4*>(qs + r * kQStride + c * 8) = v;
   }
   __syncthreads();
@@ -144,8 +156,8 @@ extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)
           }
           const int row = page * page_size + in_page;
 #pragma unroll
-          for (int cb = 0; cb < DQK / 64; ++cb)
-            tma_load_2d(sk + cb * (TKM * 128) + b * box_rows * 128, &lat_map, cb * 64, row, &full_bar[stage]);
+          for (int cb = 0; cb < QB; ++cb)
+            tma_load_2d(sk + cb * (TKM * 128) + b * box_rows * 128, lat_map, cb * 64, row, &full_bar[stage]);
         }
         if (++stage == kStagesM) { stage = 0; phase ^= 1; }
       }
@@ -179,7 +191,7 @@ extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)
       const bool scoring = live && warp < SW;
       if (scoring) {
 #pragma unroll 2
-        for (int kk = 0; kk < DQK / 16; kk += 2) {
+        for (int kk = 0; kk < QB * 4; kk += 2) {
           uint32_t qa[2][4];
           ldsm4(q_addr + kk * 32, qa[0][0], qa[0][1], qa[0][2], qa[0][3]);
           ldsm4(q_addr + kk * 32 + 32, qa[1][0], qa[1][1], qa[1][2], qa[1][3]);
@@ -244,11 +256,13 @@ extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)
           ldsm4(p_addr + ks * 32, a0, a1, a2, a3);
           const int tok = ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
 #pragma unroll
-          for (int dn = 0; dn < ON / 2; ++dn) {
+          for (int dn = 0; dn < (ON + 1) / 2; ++dn) {
+            // an odd last tile loads its own columns twice and uses the first copy
+            const int chunk = warp * ON + min(dn * 2 + (lane >> 4), ON - 1);
             uint32_t b0, b1, b2, b3;
-            ldsm4_t(sk + lat_off(tok, warp * ON + dn * 2 + (lane >> 4)), b0, b1, b2, b3);
+            ldsm4_t(sk + lat_off(tok, chunk), b0, b1, b2, b3);
             mma16816(o[dn * 2], a0, a1, a2, a3, b0, b1);
-            mma16816(o[dn * 2 + 1], a0, a1, a2, a3, b2, b3);
+            if (dn * 2 + 1 < ON) mma16816(o[dn * 2 + 1 < ON ? dn * 2 + 1 : 0], a0, a1, a2, a3, b2, b3);
           }
         }
         __syncwarp();
@@ -270,11 +284,12 @@ extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)
       const float iA = lA > 0.f ? 1.f / lA : 0.f, iB = lB > 0.f ? 1.f / lB : 0.f;
 #pragma unroll
       for (int i = 0; i < ON; ++i) {
-        const int c = warp * (DVV / MW) + i * 8 + 2 * (lane & 3);
+        const int c = warp * (ON * 8) + i * 8 + 2 * (lane & 3);
+        if (c >= v_cols) continue;
         if (rA < valid_rows)
-          *reinterpret_cast<uint32_t*>(out + (size_t)seq * out_stride + (size_t)(head0 + rA) * DVV + c) = pack_bf16x2(o[i][0] * iA, o[i][1] * iA);
+          *reinterpret_cast<uint32_t*>(out + (size_t)seq * out_stride + (size_t)(head0 + rA) * v_cols + c) = pack_bf16x2(o[i][0] * iA, o[i][1] * iA);
         if (rB < valid_rows)
-          *reinterpret_cast<uint32_t*>(out + (size_t)seq * out_stride + (size_t)(head0 + rB) * DVV + c) = pack_bf16x2(o[i][2] * iB, o[i][3] * iB);
+          *reinterpret_cast<uint32_t*>(out + (size_t)seq * out_stride + (size_t)(head0 + rB) * v_cols + c) = pack_bf16x2(o[i][2] * iB, o[i][3] * iB);
       }
     } else {
 #pragma unroll
@@ -284,8 +299,8 @@ extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)
         const size_t base = ((size_t)seq * heads + head0 + r) * split_total + split_base + split;
 #pragma unroll
         for (int i = 0; i < ON; ++i) {
-          const int c = warp * (DVV / MW) + i * 8 + 2 * (lane & 3);
-          *reinterpret_cast<float2*>(ws_o + base * DVV + c) = make_float2(o[i][2 * hh], o[i][2 * hh + 1]);
+          const int c = warp * (ON * 8) + i * 8 + 2 * (lane & 3);
+          if (c < v_cols) *reinterpret_cast<float2*>(ws_o + base * v_cols + c) = make_float2(o[i][2 * hh], o[i][2 * hh + 1]);
         }
         if (warp == 0 && (lane & 3) == 0) {
           ws_ml[base * 2] = m_run[hh];
@@ -296,6 +311,34 @@ extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)
   }
   pdl_launch_dependents();
 }
+
+extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)
+    kern_mla_decode_bf16(const __grid_constant__ CUtensorMap lat_map, const __nv_bfloat16* q, __nv_bfloat16* out, float* ws_o,
+                         float* ws_ml, const int* block_table, const int* seq_lens, int seqs, int heads, int q_stride,
+                         int out_stride, int max_pages, int page_size, int splits, int pool_pages, float scale_log2, int* err,
+                         const int* row_seq) {
+  mla_body<9, 8>(&lat_map, q, out, ws_o, ws_ml, block_table, seq_lens, seqs, heads, q_stride, out_stride, max_pages, page_size,
+                 splits, pool_pages, scale_log2, err, row_seq, 576, 512);
+}
+
+// latents without rotary columns, `rank` columns in B blocks of 64
+#define KERN_LATENT_DECODE(B)                                                                                                \
+  extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)                                                              \
+      kern_latent_decode_bf16_b##B(const __grid_constant__ CUtensorMap lat_map, const __nv_bfloat16* q, __nv_bfloat16* out,  \
+                                   float* ws_o, float* ws_ml, const int* block_table, const int* seq_lens, int seqs,         \
+                                   int heads, int q_stride, int out_stride, int max_pages, int page_size, int splits,        \
+                                   int pool_pages, float scale_log2, int* err, const int* row_seq, int rank) {               \
+    mla_body<B, B>(&lat_map, q, out, ws_o, ws_ml, block_table, seq_lens, seqs, heads, q_stride, out_stride, max_pages,       \
+                   page_size, splits, pool_pages, scale_log2, err, row_seq, rank, rank);                                     \
+  }
+KERN_LATENT_DECODE(1)
+KERN_LATENT_DECODE(2)
+KERN_LATENT_DECODE(3)
+KERN_LATENT_DECODE(4)
+KERN_LATENT_DECODE(5)
+KERN_LATENT_DECODE(6)
+KERN_LATENT_DECODE(7)
+KERN_LATENT_DECODE(8)
 
 // ---- the steps around the attention of a latent-attention layer ----------------------------------------------------
 // kern_mla_rope_append_bf16: grid = tokens, block 128. Per token: RMS-norm of the 512 compressed columns (weight w),

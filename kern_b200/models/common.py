@@ -1114,13 +1114,22 @@ def mla_rows_op() -> dict:
         "args": [{"param": 0}, {"param": 1}, {"param": 4}, {"param": 5}, {"param": 2}, {"param": 3}]}]}}
 
 
+def latent_smem(blocks: int) -> int:
+    """Shared memory of the latent decode kernel for rows of `blocks` 64-column blocks."""
+    stages = 2 if blocks >= 8 else (3 if blocks >= 5 else (4 if blocks >= 3 else 6))
+    return 1024 + stages * 64 * blocks * 128 + 16 * (blocks * 64 + 8) * 2 + 16 * (64 + 8) * 2 + 2 * 8 * 16 * 4 + 256
+
+
 def mla_attn_op(heads: int, page_size: int, table_width: int, ragged: bool, head_width: int = 192, seqs_max: int = 0,
-                sms: int = SMS) -> dict:
+                sms: int = SMS, rank: int = 0, scale: float | None = None) -> dict:
     """Absorbed latent attention: every head attends over the shared 576-wide latent rows, values their first 512
     columns. One row per sequence: interface [q, latent state, out, block_table, seq_lens, err], the context split over
     CTAs by `when` ranges of the batch (partials merged by a second launch) so that a few long sequences still fill
     the machine; ragged rows bring [.., row_len, err, row_seq] — a row reads its sequence's table row and attends over
-    its own causal reach."""
+    its own causal reach. `rank`: latent rows of that many columns (no rotary part), keys and values alike, scores times
+    `scale`; 0 is the 512 + 64 form."""
+    dq, dv = (rank, rank) if rank else (MLA_DQK, MLA_DV)
+    scale = head_width ** -0.5 if scale is None else scale
     assert page_size % 64 == 0 or 64 % page_size == 0
     iface = ["in buffer<bf16>", "in state", "out buffer<bf16>", "in buffer<i32>", "in buffer<i32>", "out buffer<i32>"]
     if ragged:
@@ -1150,23 +1159,26 @@ def mla_attn_op(heads: int, page_size: int, table_width: int, ragged: bool, head
               "out buffer<f32>" if part else "i64", "in buffer<i32>", "in buffer<i32>"] + ["i32"] * 8 + \
              ["f32", "out buffer<i32>", "in buffer<i32>" if ragged else "i64"]
         ws = [{"scratch": "ws_o"}, {"scratch": "ws_ml"}] if part else [{"i64": 0}, {"i64": 0}]
-        args = [_kv_map(MLA_DQK, page_size, 1), {"param": 0}, {"param": 2}, *ws, {"param": 3}, {"param": 4},
-                {"i32": I32_MAX}, {"i32": heads}, {"i32": heads * MLA_DQK}, {"i32": heads * MLA_DV}, {"i32": table_width},
-                {"i32": page_size}, {"i32": splits}, {"i32": I32_MAX}, {"f32": (head_width ** -0.5) * 1.4426950408889634},
+        args = [_kv_map(dq, page_size, 1), {"param": 0}, {"param": 2}, *ws, {"param": 3}, {"param": 4},
+                {"i32": I32_MAX}, {"i32": heads}, {"i32": heads * dq}, {"i32": heads * dv}, {"i32": table_width},
+                {"i32": page_size}, {"i32": splits}, {"i32": I32_MAX}, {"f32": scale * 1.4426950408889634},
                 {"param": 5}, {"param": 6} if ragged else {"i64": 0}]
-        launch = {"module": "mla_decode", "entry": "kern_mla_decode_bf16", "block": [288, 1, 1],
-                  "grid": [blocks, "tokens" if ragged else "seqs", splits], "shared_mem": MLA_SMEM, "params": lp, "args": args}
+        if rank:
+            lp, args = lp + ["i32"], args + [{"i32": rank}]
+        launch = {"module": "mla_decode", "entry": f"kern_latent_decode_bf16_b{-(-rank // 64)}" if rank else "kern_mla_decode_bf16",
+                  "block": [288, 1, 1], "grid": [blocks, "tokens" if ragged else "seqs", splits],
+                  "shared_mem": latent_smem(-(-rank // 64)) if rank else MLA_SMEM, "params": lp, "args": args}
         merge = {"module": "attn_paged", "entry": "kern_attn_merge_splits", "block": [256, 1, 1],
                  "grid": [{"mul": ["tokens", heads]}, 1, 1],
                  "params": ["in buffer<f32>", "in buffer<f32>", "out buffer<bf16>", "i32", "i32", "i32", "i32", "i32"],
                  "args": [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, {"param": 2}, {"i32": I32_MAX}, {"i32": heads},
-                          {"i32": MLA_DV}, {"i32": splits}, {"i32": heads * MLA_DV}]}
+                          {"i32": dv}, {"i32": splits}, {"i32": heads * dv}]}
         for l in ([launch, merge] if part else [launch]):
             if len(when) > 1:
                 l["when"] = when
             launches.append(l)
     impl = {"launches": launches}
     if max_splits > 1:
-        impl["scratch"] = {"ws_o": {"dtype": "f32", "shape": ["tokens", heads * max_splits * MLA_DV]},
+        impl["scratch"] = {"ws_o": {"dtype": "f32", "shape": ["tokens", heads * max_splits * dv]},
                            "ws_ml": {"dtype": "f32", "shape": ["tokens", heads * max_splits * 2]}}
     return {"params": iface, "impl": impl}
