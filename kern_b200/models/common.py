@@ -920,29 +920,31 @@ def gdn_line_bytes(hk: int, hv: int, dk: int, dv: int, width: int = 4) -> tuple[
     return s_off + hv * dv * dk * 4, s_off
 
 
-def gdn_conv_op(conv_dim: int, width: int, x_stride: int, line_bytes: int, ragged: bool) -> dict:
+def gdn_conv_op(conv_dim: int, width: int, x_stride: int, line_bytes: int, ragged: bool, bias: bool = False) -> dict:
     """Causal conv + SiLU over the first `conv_dim` channels of a row (row-parallel), then the windows kept in the
-    state lines advance. Interface [x, y, state, lines, (cu_seqlens,) w, seqs, rows]."""
+    state lines advance. Interface [x, y, state, lines, (cu_seqlens,) w, (bias,) seqs, rows]."""
     assert conv_dim % 4 == 0 and x_stride % 4 == 0, "the conv kernel moves four channels (8 bytes) per thread"
     iface = ["in buffer<bf16>", "out buffer<bf16>", "inout state", "in buffer<i32>"]
     if ragged:
         iface.append("in buffer<i32>")
-    iface += ["in buffer<bf16>", "i32", "i32"]
-    w_at = len(iface) - 3
+    w_at = len(iface)
+    iface += ["in buffer<bf16>"] * (2 if bias else 1) + ["i32", "i32"]
+    n_at = len(iface) - 2
+    b_t, b_a = ("in buffer<bf16>", {"param": w_at + 1}) if bias else ("i64", {"i64": 0})
     if not ragged:      # one row per sequence: the conv and the window shift in one launch
         step = {"module": "gdn", "entry": "kern_gdn_conv_step_bf16", "block": [256, 1, 1], "grid": ["seqs", -(-conv_dim // 1024), 1],
-                "params": ["in buffer<bf16>", "out buffer<bf16>", "inout state", "in buffer<i32>", "in buffer<bf16>", "i64", "i32",
+                "params": ["in buffer<bf16>", "out buffer<bf16>", "inout state", "in buffer<i32>", "in buffer<bf16>", b_t, "i32",
                            "i32", "i32", "i32", "i64"],
-                "args": [{"param": 0}, {"param": 1}, {"param": 2}, {"param": 3}, {"param": w_at}, {"i64": 0}, {"param": w_at + 1},
+                "args": [{"param": 0}, {"param": 1}, {"param": 2}, {"param": 3}, {"param": w_at}, b_a, {"param": n_at},
                          {"i32": conv_dim}, {"i32": width}, {"i32": x_stride}, {"i64": line_bytes}]}
         return {"params": iface, "impl": {"launches": [step]}}
     cu_t, cu_a = ("in buffer<i32>", {"param": 4}) if ragged else ("i64", {"i64": 0})
     conv = {"module": "gdn", "entry": "kern_gdn_conv_bf16", "block": [256, 1, 1],
             "grid": [{"ceil_div": ["tokens", 16]} if ragged else "tokens", -(-conv_dim // 1024), 1],
-            "params": ["in buffer<bf16>", "out buffer<bf16>", "in state", "in buffer<i32>", cu_t, "in buffer<bf16>", "i64",
+            "params": ["in buffer<bf16>", "out buffer<bf16>", "in state", "in buffer<i32>", cu_t, "in buffer<bf16>", b_t,
                        "i32", "i32", "i32", "i32", "i32", "i64", "i32"],
-            "args": [{"param": 0}, {"param": 1}, {"param": 2}, {"param": 3}, cu_a, {"param": w_at}, {"i64": 0},
-                     {"param": w_at + 1}, {"param": w_at + 2}, {"i32": conv_dim}, {"i32": width}, {"i32": x_stride},
+            "args": [{"param": 0}, {"param": 1}, {"param": 2}, {"param": 3}, cu_a, {"param": w_at}, b_a,
+                     {"param": n_at}, {"param": n_at + 1}, {"i32": conv_dim}, {"i32": width}, {"i32": x_stride},
                      {"i64": line_bytes}, {"i32": 16 if ragged else 1}]}
     upd = {"module": "gdn", "entry": "kern_gdn_conv_state", "block": [256, 1, 1], "grid": ["seqs", -(-conv_dim // 256), 1],
            "params": ["in buffer<bf16>", "inout state", "in buffer<i32>", cu_t, "i32", "i32", "i32", "i32", "i64"],
