@@ -124,3 +124,127 @@ def row_norm_op(width: int, eps: float, src_rows: int, act: str = "bf16", pick: 
     return _op(iface, _launch("hyper", f"kern_row_norm_f32_{act}", [256, 1, 1], ["wanted" if pick == "listed" else "seqs", 1, 1],
                               [iface[0], cu[0], rows[0], iface[1], iface[2], "i32", "i32", "f32"],
                               [P(0), cu[1], rows[1], P(1), P(2), I(src_rows), I(width), {"f32": eps}], shared_mem=width * 4))
+
+
+# ---- Mamba-2 (state-space duality) ----------------------------------------------------------------------
+def ssd_line_bytes(heads: int, vdim: int, state: int, channels: int, taps: int, act: str = "bf16") -> tuple[int, int]:
+    """(bytes of one per-sequence line, offset of the recurrent matrix in it)."""
+    s_off = ((taps - 1) * channels * ACT_BYTES[act] + 255) // 256 * 256
+    return (s_off + heads * vdim * state * 4 + 255) // 256 * 256, s_off
+
+
+def short_conv_op(channels: int, taps: int, x_stride: int, line_bytes: int, ragged: bool, act: str = "bf16", x_off: int = 0) -> dict:
+    """Causal convolution with bias, then SiLU, for any taps / channels; the window at the start of the state line
+    advances with it. `x_off`: elements before the channels in a row (decides whether the aligned kernels apply).
+    Interface [x, y, state, lines, (cu_seqlens,) w, bias, seqs, rows]."""
+    if act == "bf16" and 2 <= taps <= 4 and channels % 4 == 0 and x_stride % 4 == 0 and x_off % 4 == 0:
+        return C.gdn_conv_op(channels, taps, x_stride, line_bytes, ragged, bias=True)
+    iface = [f"in buffer<{act}>", f"out buffer<{act}>", "inout state", "in buffer<i32>"] + (["in buffer<i32>"] if ragged else [])
+    w = len(iface)
+    iface += ["in buffer<bf16>", "in buffer<bf16>", "i32", "i32"]
+    cu_t, cu_a = ("in buffer<i32>", P(4)) if ragged else NULL
+    cols = -(-channels // 256)
+    conv = _launch("ssd", f"kern_ssd_conv_{act}", [256, 1, 1], ["tokens", cols, 1],
+                   [iface[0], iface[1], "in state", "in buffer<i32>", cu_t, "in buffer<bf16>", "in buffer<bf16>"] + ["i32"] * 5 + ["i64"],
+                   [P(0), P(1), P(2), P(3), cu_a, P(w), P(w + 1), P(w + 2), P(w + 3), I(channels), I(taps), I(x_stride), L(line_bytes)])
+    upd = _launch("ssd", f"kern_ssd_conv_state_{act}", [256, 1, 1], ["seqs", cols, 1],
+                  [iface[0], "inout state", "in buffer<i32>", cu_t] + ["i32"] * 4 + ["i64"],
+                  [P(0), P(2), P(3), cu_a, P(w + 2), I(channels), I(taps), I(x_stride), L(line_bytes)])
+    return _op(iface, conv, upd)
+
+
+def ssd_rule_op(heads: int, vdim: int, state: int, groups: int, dt_stride: int, line_bytes: int, s_off: int, ragged: bool,
+                act: str = "bf16") -> dict:
+    """The recurrence. Interface [xbc, dt, y (f32), state, lines, (cu_seqlens,) A_log, dt_bias, D, seqs]."""
+    if heads % groups or state > 512:
+        raise ValueError(f"{heads} heads in {groups} groups with {state} state columns: heads split evenly, at most 512 columns")
+    iface = [f"in buffer<{act}>", f"in buffer<{act}>", "out buffer<f32>", "inout state", "in buffer<i32>"] + (["in buffer<i32>"] if ragged else [])
+    w = len(iface)
+    iface += ["in buffer<bf16>"] * 3 + ["i32"]
+    cu_t, cu_a = ("in buffer<i32>", P(5)) if ragged else NULL
+    nl = next(n for n in (32, 64, 128, 256, 512) if state <= n)
+    tb = (32 if nl <= 128 else 8) if ragged else 1
+    return _op(iface, _launch(
+        "ssd", f"kern_ssd_rule_{act}_n{nl}", [256, 1, 1], [heads * -(-vdim // 16), "seqs", 1],
+        iface[:5] + [cu_t] + ["in buffer<bf16>"] * 3 + ["i32"] * 6 + ["i64", "i32", "i32"],
+        [*map(P, range(5)), cu_a, *map(P, range(w, w + 4)), I(heads), I(vdim), I(state), I(groups), I(dt_stride), L(line_bytes), I(s_off), I(tb)],
+        shared_mem=tb * (2 * state + 16 + 2) * 4))
+
+
+def ssd_gate_norm_op(inner: int, parts: int, z_stride: int, eps: float, act: str = "bf16") -> dict:
+    """out = rms_norm per part of (y * silu(z)), times w. Interface [y (f32), z, w, out]."""
+    if inner % parts:
+        raise ValueError(f"{inner} columns do not split into {parts} norm groups")
+    iface = ["in buffer<f32>", f"in buffer<{act}>", "in buffer<bf16>", f"out buffer<{act}>"]
+    return _op(iface, _launch("ssd", f"kern_ssd_gate_norm_{act}", [256, 1, 1], ["tokens", parts, 1], iface + ["i32", "i32", "i32", "f32"],
+                              [*map(P, range(4)), I(inner), I(parts), I(z_stride), {"f32": eps}], shared_mem=inner // parts * 4))
+
+
+# ---- latent attention without positions -----------------------------------------------------------------
+def latent_append_op(rank: int, stride: int, eps: float, act: str = "bf16") -> dict:
+    """RMS norm of a token's latent into its row of the paged cache. Interface [latent columns, state, slots, norm w]."""
+    iface = [f"in buffer<{act}>", "inout state", "in buffer<i64>", "in buffer<bf16>"]
+    return _op(iface, _launch("latent", f"kern_latent_append_{act}", [128, 1, 1], ["tokens", 1, 1], iface + ["i32", "i32", "f32"],
+                              [*map(P, range(4)), I(rank), I(stride), {"f32": eps}]))
+
+
+def latent_attn_op(heads: int, rank: int, scale: float, page_size: int, table_width: int, ragged: bool, act: str = "bf16",
+                   seqs_max: int = 0) -> dict:
+    """Every head attends over the shared latent rows, which are keys and values alike.
+    Interface [q, state, out, block_table, lens, err] (+ [row_seq] for ragged rows: one attention row per token). bf16
+    latents of up to 512 aligned columns take the tensor-core kernel, others one block per (row, head)."""
+    if act == "bf16" and tiles_fit(rank) and rank <= 512 and (page_size % 64 == 0 or 64 % page_size == 0):
+        return C.mla_attn_op(heads, page_size, table_width, ragged, seqs_max=seqs_max, rank=rank, scale=scale)
+    if rank > 1024:
+        raise ValueError(f"latent rows of {rank} columns (at most 1024)")
+    iface = [f"in buffer<{act}>", "in state", f"out buffer<{act}>", "in buffer<i32>", "in buffer<i32>", "out buffer<i32>"]
+    iface += ["in buffer<i32>"] if ragged else []
+    w = next(n for n in (64, 128, 256, 512, 1024) if rank <= n)
+    return _op(iface, _launch("latent", f"kern_latent_attn_{act}_w{w}", [128, 1, 1], [heads, "tokens" if ragged else "seqs", 1],
+                              iface[:5] + ["in buffer<i32>" if ragged else "i64", "i32", "i32", "i32", "i32", "f32", "out buffer<i32>"],
+                              [*map(P, range(5)), P(6) if ragged else NULL[1], I(heads), I(rank), I(table_width), I(page_size),
+                               {"f32": scale}, P(5)], shared_mem=(4 * rank + 8) * 4))
+
+
+# ---- routed experts ---------------------------------------------------------------------------------------
+def route_logits_op(experts: int, top: int, bias: bool = True) -> dict:
+    """The `top` largest of logits + bias, weighed by the softmax over them. Interface [logits, (bias,) ids, weights, tokens]."""
+    if not (1 <= top <= min(32, experts) and experts <= 1024):
+        raise ValueError(f"{top} of {experts} experts per token (at most 32 of 1024)")
+    iface = ["in buffer<f32>"] + (["in buffer<bf16>"] if bias else []) + ["out buffer<i32>", "out buffer<f32>", "i32"]
+    b_t, b_a = (iface[1], P(1)) if bias else NULL
+    o = 2 if bias else 1
+    return _op(iface, _launch("moe", "kern_moe_route_logits", [128, 1, 1], [{"ceil_div": ["tokens", 4]}, 1, 1],
+                              ["in buffer<f32>", b_t, "out buffer<i32>", "out buffer<f32>", "i32", "i32", "i32", "i32"],
+                              [P(0), b_a, P(o), P(o + 1), P(o + 2), I(experts), I(top), I(experts)]))
+
+
+def routed_tile_rows(act: str, width: int, ff: int) -> int:
+    """Rows of a tile of the planner's table: 128 for the tensor-core kernels, 64 for the generic one."""
+    return C.BM if act == "bf16" and tiles_fit(width, ff) else 64
+
+
+def routed_ops(width: int, ff: int, experts: int, top: int, tokens_max: int, act: str = "bf16") -> dict:
+    """plan / gather / fc1 / fc2 of routed SwiGLU experts under the interfaces of `moe._moe_ops`."""
+    from . import moe
+
+    cfg = moe.MoeConfig(hidden=width, moe_intermediate=ff, experts=experts, top_k=top, max_tokens=tokens_max)
+    ops = moe._moe_ops(cfg, 0, experts)
+    if routed_tile_rows(act, width, ff) == C.BM:
+        return {k: ops[k] for k in ("moe_plan", "moe_gather", "moe_fc1", "moe_fc2")}
+    bm = routed_tile_rows(act, width, ff)
+    plan = ops["moe_plan"]["impl"]["launches"][0]
+    plan["args"][9], plan["args"][10] = I(bm), I(tokens_max * top // bm + experts)
+    b = f"buffer<{act}>"
+    gather = _op(["in " + b, "in buffer<i32>", "out " + b, "i32"],
+                 _launch("linear", f"kern_rows_scatter_{act}", [256, 1, 1], [{"mul": ["tokens", top]}, 1, 1],
+                         ["in " + b, "in buffer<i32>", "out " + b, "i32", "i32", "i32"], [P(0), P(1), P(2), P(3), I(top), I(width)]))
+
+    def routed(n, k, swiglu):
+        return _op(["in " + b, "in buffer<bf16>", "out " + b, "in buffer<i32>", "in buffer<i32>", "i32", "out buffer<i32>"],
+                   _launch("linear", f"kern_linear_grouped_{act}" + ("_swiglu" if swiglu else ""), [256, 1, 1],
+                           [-(-n // 64), {"clamp": [{"add": [{"ceil_div": [{"mul": ["tokens", top]}, bm]}, experts]}, 0, 4096]}, 1],
+                           ["in " + b, "in buffer<bf16>", "out " + b, "in buffer<i32>", "in buffer<i32>", "i32", "i32", "i32", "i64", "out buffer<i32>"],
+                           [P(0), P(1), P(2), P(3), P(4), P(5), I(n), I(k), L((2 if swiglu else 1) * n * k), P(6)]))
+
+    return {"moe_plan": ops["moe_plan"], "moe_gather": gather, "moe_fc1": routed(ff, width, True), "moe_fc2": routed(width, ff, False)}
