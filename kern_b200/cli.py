@@ -63,7 +63,7 @@ def make_runtime(args, manifest=None):
     if model and not manifest:
         from .models import registry
 
-        over = {k: getattr(args, k, None) or None for k in ("layers", "max_tokens", "max_seqs", "max_context")}
+        over = {k: getattr(args, k, None) or None for k in ("layers", "max_tokens", "max_seqs", "max_context", "dtype")}
         cfg, build, load, make = registry.resolve(model, **over)
         doc = build(cfg)
         # state slots only for models with per-sequence state: a lease that holds a slot makes its checkpoints usable
@@ -691,7 +691,8 @@ def main(argv=None) -> int:
         p.add_argument("--gpu", type=int); p.add_argument("--capacity", type=int, help="token capacity of the paged states")
         p.add_argument("--cpu", action="store_true", help="run on the host-memory executor instead of a GPU")
         p.add_argument("--chunk", type=int); p.add_argument("--max-seqs", type=int, default=0)
-        p.add_argument("--model", help="a built-in model family with random-init weights instead of --manifest/--weights")
+        p.add_argument("--model", help="a built-in model family with random-init weights, or a checkpoint folder (config.json + safetensors), instead of --manifest/--weights")
+        p.add_argument("--dtype", choices=["bf16", "f32"], help="with --model: activations of a family that has a 32-bit form")
         p.add_argument("--layers", type=int); p.add_argument("--max-tokens", type=int); p.add_argument("--max-context", type=int)
 
     v = sub.add_parser("verify"); v.add_argument("manifest")

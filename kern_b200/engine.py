@@ -48,7 +48,10 @@ class Engine:
         self.page_tables = p["page_tables"]
         self.unit = rt.page_unit
         row_pages = min((t["width"] * t["stride"] // self.unit for t in self.page_tables), default=0)
-        self.pool = pool or _native.Pool(self.unit, rt.pages, rt.slots, row_pages)
+        pages = rt.pages
+        if not self.page_tables and not pages:      # no paged state: leases only hand out slots, the pages stand for nothing
+            self.unit, pages = 64, 1 << 16
+        self.pool = pool or _native.Pool(self.unit, pages, rt.slots, row_pages)
         self.forwards = p["forwards"]
         self._pinned: dict[str, torch.Tensor] = {}
         self._out: dict[str, torch.Tensor] = {}
@@ -65,6 +68,10 @@ class Engine:
         if lease.slot >= 0:
             self.rt.zero_slot(lease.slot)
         return Sequence(lease=lease, sampling=sampling or Sampling())
+
+    def grow(self, seq: Sequence, tokens_capacity: int) -> None:
+        """Make a sequence's lease hold ``tokens_capacity`` positions in all (pages are added as they are needed)."""
+        self.pool.extend(seq.lease, tokens_capacity)
 
     def close(self, seq: Sequence) -> None:
         seq.lease.release()
@@ -154,6 +161,49 @@ class Engine:
             self.d2h_bytes += b * cnt.itemsize
             return [toks[i, : int(cnt[i])].tolist() for i in range(b)]
         return [toks[i, :1].tolist() for i in range(b)]
+
+    # ---- logits of any rows (manifests with a `logits` program) ----
+    def logits(self, rows: list[int]) -> np.ndarray:
+        """Logits [len(rows), vocab] (f32) of the last call's rows with these indices, counted over the whole call. The manifest's
+        `logits` program projects rows of what the last forward left behind: `want_rows` in, `want_logits` out, over var
+        `wanted`."""
+        doc = self.rt.doc
+        if "logits" not in doc["programs"]:
+            raise ValueError(f"model `{doc['model']}` has no `logits` program")
+        most, vocab = doc["vars"]["wanted"]["max"], doc["buffers"]["want_logits"]["shape"][1]
+        out = np.empty((len(rows), vocab), np.float32)
+        for at in range(0, len(rows), most):
+            part = np.asarray(rows[at:at + most], np.int32)
+            self._write("want_rows", "i32", part)
+            self.rt.issue("logits", {"wanted": len(part), self.p["rows"]["var"]: 1, self.p["groups"]["var"]: 1})
+            out[at:at + len(part)] = self.rt.read("want_logits", len(part) * vocab).reshape(len(part), vocab)
+        return out
+
+    def feed(self, batch: list[tuple[Sequence, list[int]]], want: list[list[int]]) -> np.ndarray:
+        """One batch of any size: every sequence takes its tokens (leases grow as needed), in as few calls as the manifest's
+        row and group limits allow; returns the logits at `want[i]` (places among entry i's tokens), entry by entry."""
+        for s, new in batch:
+            self.grow(s, s.length + len(new))
+        got: dict[tuple[int, int], np.ndarray] = {}
+        at = [0] * len(batch)
+        while True:
+            call, rows, used = [], [], 0
+            for i, (s, new) in enumerate(batch):
+                n = min(len(new) - at[i], self.rows_max - used)
+                if n <= 0 or len(call) == self.groups_max:
+                    continue
+                call.append((s, new[at[i]:at[i] + n]))
+                rows += [(i, w, used + w - at[i]) for w in want[i] if at[i] <= w < at[i] + n]
+                at[i] += n
+                used += n
+            if not call:
+                break
+            self.step(call, read=False)
+            if rows:
+                out = self.logits([r for _, _, r in rows])
+                got.update({(i, w): out[k] for k, (i, w, _) in enumerate(rows)})
+        flat = [got[i, w] for i, ws in enumerate(want) for w in ws]
+        return np.stack(flat) if flat else np.zeros((0, 0), np.float32)
 
     # ---- whole-sequence helpers (the single-sequence `Caller`) ----
     def generate(self, prompt: list[int], steps: int, chunk: int | None = None, sampling: Sampling | None = None) -> list[int]:

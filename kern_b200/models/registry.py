@@ -5,10 +5,30 @@ random-init checkpoint on the device (no files), which is how the benchmarks run
 from __future__ import annotations
 
 import dataclasses
+import json
+from pathlib import Path
+
+ARCHITECTURES = {"Gafapel": "gafapel"}      # config.json's `architecture` -> the module of its family
+
+
+def is_folder(name: str) -> bool:
+    return (Path(name) / "config.json").is_file()
+
+
+def from_folder(path, **overrides):
+    """A checkpoint folder (config.json + safetensors) -> (config with overrides applied, manifest builder); the family is
+    the one config.json's `architecture` names."""
+    import importlib
+
+    arch = json.loads((Path(path) / "config.json").read_text()).get("architecture")
+    if arch not in ARCHITECTURES:
+        raise KeyError(f"{path}: unknown architecture `{arch}`; known: {', '.join(sorted(ARCHITECTURES))}")
+    mod = importlib.import_module(f".{ARCHITECTURES[arch]}", __package__)
+    return mod.from_folder(path, **{k: v for k, v in overrides.items() if v is not None}), mod.build_manifest
 
 
 def families() -> dict:
-    from . import dense, hybrid, latent, moe
+    from . import dense, gafapel, hybrid, latent, moe
 
     out = {}
     for cfg in (dense.TOY, dense.TINY, dense.DENSE_8B):
@@ -20,6 +40,8 @@ def families() -> dict:
     for cfg in (latent.TINY_LATENT, latent.TINY_LATENT_K128, latent.TINY_LATENT_MOE, latent.LATENT_48B):
         out[cfg.name] = (cfg, latent.build_manifest, latent.load_random_weights,
                          lambda cfg, **kw: latent.folded(cfg, latent.random_weights(cfg, **kw)))
+    for cfg in (gafapel.TINY_GAFAPEL, gafapel.GAFAPEL_LARGE):
+        out[cfg.name] = (cfg, gafapel.build_manifest, gafapel.load_random_weights, gafapel.random_weights)
     from . import toy_int
 
     for lined in (False, True):
@@ -29,7 +51,14 @@ def families() -> dict:
 
 
 def resolve(name: str, **overrides):
-    """-> (config with overrides applied, builder, device loader, host weights maker)."""
+    """-> (config with overrides applied, builder, device loader, host weights maker). `name`: a family, or a checkpoint folder."""
+    if is_folder(name):
+        from .common import read_safetensors
+
+        cfg, build = from_folder(name, **overrides)
+        files = sorted(str(p) for p in Path(name).glob("*.safetensors"))
+        return cfg, build, lambda rt, cfg: rt.load_weights(files), \
+            lambda cfg: {k: t for f in files for k, t in read_safetensors(f).items()}
     fam = families()
     if name not in fam:
         raise KeyError(f"unknown model `{name}`; known: {', '.join(sorted(fam))}")
