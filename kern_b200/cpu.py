@@ -684,8 +684,8 @@ class CpuRuntime:
                 if fn is None:          # model families register their kernels' statements when imported
                     import importlib
 
-                    for mod in ("toy_int", "spec", "moe"):
-                        importlib.import_module(f"kern_b200.models.{mod}")
+                    for mod in ("models.toy_int", "models.spec", "models.moe", "ops.blocks"):
+                        importlib.import_module(f"kern_b200.{mod}")
                     fn = CPU_KERNELS.get(entry)
                 if fn is None:
                     raise NotImplementedError(f"no CPU statement of `{entry}` is registered")
