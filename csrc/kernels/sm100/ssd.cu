@@ -70,14 +70,14 @@ KERN_DEVICE float softplus(float v) { return v > 30.f ? v : log1pf(expf(v)); }
 template <typename T, int NL>
 KERN_DEVICE void rule_body(const T* xbc, const T* dt, float* y, uint8_t* state, const int* lines, const int* cu,
                            const __nv_bfloat16* A_log, const __nv_bfloat16* dt_bias, const __nv_bfloat16* D, int seqs, int H,
-                           int P, int N, int G, int dt_stride, long long line_bytes, int s_off, int tb) {
+                           int P, int N, int G, int dt_stride, long long line_bytes, int s_off, int tb, int max_rows) {
   extern __shared__ __align__(16) float ssd_sm[];
   const int parts = (P + 15) / 16;
   const int h = blockIdx.x / parts, p0 = (blockIdx.x % parts) * 16, s = blockIdx.y;
   if (s >= seqs) return;
   const int line = checked_line(state, lines[s], line_bytes);
   const int r0 = cu ? cu[s] : s, r1 = cu ? cu[s + 1] : s + 1;
-  if (r1 <= r0) return;
+  if (r1 <= r0 || r1 - r0 > max_rows) return;      // longer sequences belong to ssd_chunk.cu
   float* Bs = ssd_sm;
   float* Cs = Bs + (size_t)tb * N;
   float* xs = Cs + (size_t)tb * N;
@@ -176,10 +176,10 @@ KERN_DEVICE void gate_norm_body(const float* y, const T* z, const __nv_bfloat16*
       kern_ssd_rule_##SFX##_n##NL(const T* xbc, const T* dt, float* y, uint8_t* state, const int* lines, const int* cu,    \
                                   const __nv_bfloat16* A_log, const __nv_bfloat16* dt_bias, const __nv_bfloat16* D,        \
                                   int seqs, int H, int P, int N, int G, int dt_stride, long long line_bytes, int s_off,    \
-                                  int tb) {                                                                                \
+                                  int tb, int max_rows) {                                                                  \
     pdl_wait();                                                                                                            \
     rule_body<T, NL / 32>(xbc, dt, y, state, lines, cu, A_log, dt_bias, D, seqs, H, P, N, G, dt_stride, line_bytes, s_off, \
-                          tb);                                                                                             \
+                          tb, max_rows);                                                                                   \
     pdl_launch_dependents();                                                                                               \
   }
 // conv: grid [rows, ceil(channels / 256)]; conv_state: grid [seqs, ceil(channels / 256)]; rule: grid [H ceil(P / 16), seqs];

@@ -153,6 +153,9 @@ def short_conv_op(channels: int, taps: int, x_stride: int, line_bytes: int, ragg
     return _op(iface, conv, upd)
 
 
+SSD_CHUNK_MIN = 8       # rows of a call from which a sequence is computed in chunks
+
+
 def ssd_rule_op(heads: int, vdim: int, state: int, groups: int, dt_stride: int, line_bytes: int, s_off: int, ragged: bool,
                 act: str = "bf16") -> dict:
     """The recurrence. Interface [xbc, dt, y (f32), state, lines, (cu_seqlens,) A_log, dt_bias, D, seqs]."""
@@ -163,12 +166,20 @@ def ssd_rule_op(heads: int, vdim: int, state: int, groups: int, dt_stride: int, 
     iface += ["in buffer<bf16>"] * 3 + ["i32"]
     cu_t, cu_a = ("in buffer<i32>", P(5)) if ragged else NULL
     nl = next(n for n in (32, 64, 128, 256, 512) if state <= n)
-    tb = (32 if nl <= 128 else 8) if ragged else 1
-    return _op(iface, _launch(
-        "ssd", f"kern_ssd_rule_{act}_n{nl}", [256, 1, 1], [heads * -(-vdim // 16), "seqs", 1],
-        iface[:5] + [cu_t] + ["in buffer<bf16>"] * 3 + ["i32"] * 6 + ["i64", "i32", "i32"],
-        [*map(P, range(5)), cu_a, *map(P, range(w, w + 4)), I(heads), I(vdim), I(state), I(groups), I(dt_stride), L(line_bytes), I(s_off), I(tb)],
-        shared_mem=tb * (2 * state + 16 + 2) * 4))
+    lp = iface[:5] + [cu_t] + ["in buffer<bf16>"] * 3 + ["i32"] * 6 + ["i64", "i32"]
+    args = [*map(P, range(5)), cu_a, *map(P, range(w, w + 4)), I(heads), I(vdim), I(state), I(groups), I(dt_stride), L(line_bytes), I(s_off)]
+    chunked = ragged and act == "bf16" and state <= 256
+    tb = (32 if nl <= 128 else 8) if ragged and not chunked else (SSD_CHUNK_MIN if chunked else 1)
+    rule = _launch("ssd", f"kern_ssd_rule_{act}_n{nl}", [256, 1, 1], [heads * -(-vdim // 16), "seqs", 1], lp + ["i32", "i32"],
+                   args + [I(tb), I(SSD_CHUNK_MIN - 1 if chunked else C.I32_MAX)], shared_mem=tb * (2 * state + 16 + 2) * 4)
+    if not chunked:
+        return _op(iface, rule)
+    # a ragged call's long sequences in chunks on the tensor cores, its few-row ones (decode rows among prompts) row by row
+    np_, q = nl, 64
+    smem = 2 * (2 * q * (np_ + 8) + q * 40) * 2 + 3 * 32 * (np_ + 8) * 2 + q * 32 * 4 + 5 * q * 4
+    chunk = _launch("ssd_chunk", f"kern_ssd_chunk_n{np_}", [256, 1, 1], [heads * -(-vdim // 32), "seqs", 1], lp + ["i32"],
+                    args + [I(SSD_CHUNK_MIN)], shared_mem=smem)
+    return _op(iface, chunk, rule)
 
 
 def ssd_gate_norm_op(inner: int, parts: int, z_stride: int, eps: float, act: str = "bf16") -> dict:

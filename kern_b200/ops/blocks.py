@@ -135,12 +135,16 @@ def k_ssd_conv_state(g, x, state, lines, cu, seqs, ch, taps, xs, line_bytes):
         win.copy_(full[full.shape[0] - (taps - 1):].clone())
 
 
-def k_ssd_rule(g, xbc, dt, y, state, lines, cu, A_log, dt_bias, D, seqs, H, P, N, G, dts, line_bytes, s_off, tb):
+def k_ssd_chunk(g, xbc, dt, y, state, lines, cu, A_log, dt_bias, D, seqs, H, P, N, G, dts, line_bytes, s_off, min_rows):
+    k_ssd_rule(g, xbc, dt, y, state, lines, cu, A_log, dt_bias, D, seqs, H, P, N, G, dts, line_bytes, s_off, 0, 1 << 31, min_rows)
+
+
+def k_ssd_rule(g, xbc, dt, y, state, lines, cu, A_log, dt_bias, D, seqs, H, P, N, G, dts, line_bytes, s_off, tb, max_rows, min_rows=1):
     inner, ch, rep = H * P, H * P + 2 * G * N, H // G
     for s in range(g[1]):
         r0, r1 = _rows_of(cu, s)
         n = r1 - r0
-        if n <= 0:
+        if not min_rows <= n <= max_rows:
             continue
         ln = int(lines[s])
         Sb = state[ln * line_bytes + s_off: ln * line_bytes + s_off + H * P * N * 4].view(torch.float32).view(H, P, N)
@@ -218,4 +222,5 @@ for _a in ("bf16", "f32"):
     CPU_KERNELS.update({f"kern_latent_attn_{_a}_w{w}": k_latent_attn for w in (64, 128, 256, 512, 1024)})
 CPU_KERNELS.update({"kern_linear_bf16_f32": _k_linear(False), "kern_transpose_heads_bf16": k_transpose_heads,
                     "kern_moe_route_logits": k_route_logits})
+CPU_KERNELS.update({f"kern_ssd_chunk_n{n}": k_ssd_chunk for n in (32, 64, 128, 256)})
 CPU_KERNELS.update({f"kern_latent_decode_bf16_b{b}": k_latent_decode for b in range(1, 9)})
