@@ -119,18 +119,21 @@ struct EpArgs {
 // A tile's load may run into the next expert's rows; the epilogue stores only the tile's own rows.
 // FP8: A and B hold e4m3 bytes (a swizzle row is 128 elements, the instruction is kind::f8f6f4 with K = 32), the
 // accumulator is scaled by *scale_a * *scale_b (per-tensor scales) before the epilogue's conversion.
-template <int BN, int EPI, bool GROUPED = false, bool FP8 = false, bool MT2 = false, bool AG = false, int EP = 0>
+// HEADS: a batch of `heads` products over column ranges: C[:, h N ..] = A[:, h K ..] . W_h^T, W a 3-D map [K, N, heads]. A
+// head's last K block may reach into the next head's columns of A; the map fills W with zeros there.
+template <int BN, int EPI, bool GROUPED = false, bool FP8 = false, bool MT2 = false, bool AG = false, int EP = 0, bool HEADS = false>
 __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtensorMap* tma_b,
                                           void* Cv, const void* Rv,
                                           int M, int N, int K, int ldc, int* err,
                                           const int* tile_table = nullptr, const int* tile_count = nullptr,
                                           ScatterArgs sc = ScatterArgs(), const float* scale_a = nullptr,
-                                          const float* scale_b = nullptr, AgArgs ag = AgArgs(), EpArgs ep = EpArgs()) {
+                                          const float* scale_b = nullptr, AgArgs ag = AgArgs(), EpArgs ep = EpArgs(), int heads = 1) {
   using Cfg = GemmCfg<BN, MT2>;
   constexpr int kStages = Cfg::kStages;
   constexpr int BMT = Cfg::kRows;
   static_assert(!(MT2 && (GROUPED || EPI == 4 || BN != 256)), "the 256-row tile exists for the plain 256-wide GEMM");
   static_assert(!(AG && (FP8 || MT2)) && (!(AG && GROUPED) || EP == 1), "the all-gather form exists for the plain bf16 GEMM");
+  static_assert(!HEADS || (EPI == 0 && !GROUPED && !FP8 && !MT2 && !AG), "the batched form stores bf16");
   static_assert((EP != 1 || (AG && GROUPED)) && (EPI != 5 || GROUPED), "the expert-parallel forms are routed GEMMs");
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -175,7 +178,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtens
   }
   pdl_wait();  // everything above touched only this CTA's own state and the descriptors
   const int num_m = GROUPED ? *tile_count : (M + BMT - 1) / BMT;
-  const int num_tiles = num_m * num_n;
+  const int num_tiles = num_m * num_n * (HEADS ? heads : 1);
   // tile t -> (first row, row bound, n block, expert)
   // AG: blocks per rank, this rank's first block, and the counter value that says "every CTA's share of the block is in"
   const int ag_bpr = AG ? ((EP == 1 || ag.ready != nullptr) ? 0 : num_m_of(M, ag.nranks)) : 0;
@@ -191,6 +194,8 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtens
     __syncthreads();      // every thread has read this CTA's launch count before the gather warps can write the next one
   }
   auto tile_of = [&](int t, int& row0, int& row_end, int& n_blk, int& expert) {
+    const int head = HEADS ? t / (num_m * num_n) : 0;
+    if constexpr (HEADS) t -= head * num_m * num_n;
     int mt = t % num_m;
     n_blk = t / num_m;
     if constexpr (AG) {
@@ -207,7 +212,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtens
       const int4 e = reinterpret_cast<const int4*>(tile_table)[mt];
       expert = e.x; row0 = e.y; row_end = min(M, e.y + e.z);
     } else {
-      expert = 0; row0 = mt * BMT; row_end = M;
+      expert = head; row0 = mt * BMT; row_end = M;
     }
   };
 
@@ -246,9 +251,9 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtens
           uint8_t* sa = tiles + stage * Cfg::kStageBytes;
           uint8_t* sb = sa + Cfg::kStageBytesA;
           mbar_expect_tx(&full_bar[stage], Cfg::kStageBytes);
-          tma_load_2d(sa, tma_a, kb * BKE, row0, &full_bar[stage]);
+          tma_load_2d(sa, tma_a, (HEADS ? expert * K : 0) + kb * BKE, row0, &full_bar[stage]);
           auto load_b = [&](uint8_t* dst, int n_row) {
-            if constexpr (GROUPED) tma_load_3d(dst, tma_b, kb * BKE, n_row, expert, &full_bar[stage]);
+            if constexpr (GROUPED || HEADS) tma_load_3d(dst, tma_b, kb * BKE, n_row, expert, &full_bar[stage]);
             else tma_load_2d(dst, tma_b, kb * BKE, n_row, &full_bar[stage]);
           };
           if constexpr (EPI == 3) {
@@ -577,7 +582,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtens
         const int col = n_blk * BN + c * 32;
         if (row < row_end) {
           if constexpr (EPI == 0 || EPI == 2) {
-            __nv_bfloat16* C = reinterpret_cast<__nv_bfloat16*>(Cv) + (size_t)row * ldc + col;
+            __nv_bfloat16* C = reinterpret_cast<__nv_bfloat16*>(Cv) + (size_t)row * ldc + (HEADS ? expert * N : 0) + col;
             const __nv_bfloat16* R =
                 reinterpret_cast<const __nv_bfloat16*>(Rv) + (size_t)row * ldc + col;
 #pragma unroll
@@ -671,6 +676,18 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtens
     kern::gemm_body<256, EPI, false, false, true>(&tma_a, &tma_b, C, R, M, N, K, ldc, err);   \
   }
 
+#define KERN_GEMM_HEADS(name, BN)                                                                  \
+  extern "C" __global__ void __launch_bounds__(192, 1)                                             \
+      name(const __grid_constant__ CUtensorMap tma_a, const __grid_constant__ CUtensorMap tma_b,   \
+           void* C, int M, int N, int K, int ldc, int heads, int* err) {                           \
+    kern::gemm_body<BN, 0, false, false, false, false, 0, true>(                                   \
+        &tma_a, &tma_b, C, nullptr, M, N, K, ldc, err, nullptr, nullptr, kern::ScatterArgs(),      \
+        nullptr, nullptr, kern::AgArgs(), kern::EpArgs(), heads);                                  \
+  }
+
+KERN_GEMM_HEADS(kern_gemm_bf16_heads_n256, 256)
+KERN_GEMM_HEADS(kern_gemm_bf16_heads_n128, 128)
+KERN_GEMM_HEADS(kern_gemm_bf16_heads_n64, 64)
 KERN_GEMM_ENTRY_M256(kern_gemm_bf16_tn_m256_n256, 0)
 KERN_GEMM_ENTRY_M256(kern_gemm_bf16_tn_acc_m256_n256, 2)
 KERN_GEMM_ENTRY_M256(kern_gemm_bf16_tn_swiglu_m256_n256, 3)

@@ -52,10 +52,31 @@ def linear_op(n: int, k: int, *, act: str = "bf16", epilogue: str = "store", row
     return _op(iface, _generic(sfx, iface, cols, k, lda, ldc, rows_var))
 
 
+def head_tiles(n: int, k: int, lda: int, ldc: int, act: str) -> bool:
+    """Whether per-head products of this size run on the tensor-core tiles (which read weights as [n, k])."""
+    return act == "bf16" and tiles_fit(n, k, lda, ldc)
+
+
 def head_linear_op(heads: int, n: int, k: int, *, act: str = "bf16", rows_max: int, lda: int, ldc: int, transposed: bool = False) -> dict:
     """Per head h: C[:, h n : (h + 1) n] = A[:, h k : (h + 1) k] . W_h^T, with W_h [n, k] stacked by head, or [k, n] when
     `transposed`. Interface [a, w, c, rows, err]."""
     iface = [f"in buffer<{act}>", "in buffer<bf16>", f"out buffer<{act}>", "i32", "out buffer<i32>"]
+    if head_tiles(n, k, lda, ldc, act) and not transposed:
+        tmap = lambda param, dims, strides, box: {"pack": {"size": 128, "fields": [{"at": 0, "tensormap": {
+            "param": param, "dtype": "bf16", "dims": dims, "strides": strides, "box": box, "swizzle": 128, "l2_promotion": 256}}]}}
+        launches = []
+        # wide tiles once they give every SM one
+        wide = [(256, 4 * C.BM + 1, rows_max), (128, 1, min(4 * C.BM, rows_max))] if n >= 256 else [(128 if n >= 128 else 64, 1, rows_max)]
+        for bn, lo, hi in wide:
+            if lo > hi:
+                continue
+            when = {"var": "tokens", **({"min": lo} if lo > 1 else {}), **({"max": hi} if hi < rows_max else {})}
+            launches.append(_launch(
+                "gemm_bf16", f"kern_gemm_bf16_heads_n{bn}", [192, 1, 1], [C.SMS, 1, 1],
+                ["bytes<128>", "bytes<128>", iface[2]] + ["i32"] * 5 + ["out buffer<i32>"],
+                [tmap(0, [heads * k, 0], [lda * 2], [C.BK, C.BM]), tmap(1, [k, n, heads], [k * 2, n * k * 2], [C.BK, bn, 1]),
+                 P(2), P(3), I(n), I(k), I(ldc), I(heads), P(4)], shared_mem=C.gemm_smem(bn), **({"when": when} if len(when) > 1 else {})))
+        return _op(iface, *launches)
     return _op(iface, _generic(act, iface, n, k, lda, ldc, "tokens", heads, (1, n) if transposed else (k, 1), (k, n * k, n)))
 
 

@@ -231,7 +231,7 @@ def build_manifest(cfg: GafapelConfig) -> dict:
     es, layers = K.ACT_BYTES[A], cfg.depth
     if not layers:
         raise ValueError("a model without layers")
-    bufs, ops, states = {}, {}, {}
+    bufs, ops, states, once = {}, {}, {}, []
     B = lambda n, off=0: ({"buf": n, "offset": off} if off else {"buf": n})
     V = lambda n: {"var": n}
     err = B("error")
@@ -338,7 +338,12 @@ def build_manifest(cfg: GafapelConfig) -> dict:
         w_in = weight(f"w.{p}mix.qgc", (proj, d), p + "mix.q", p + "mix.g", p + "mix.dkv",
                       *([{"tensor": p + "mix.q", "rows": [0, proj - z["rows"]]}] if proj > z["rows"] else []))
         app = op(f"latent_append_{r}x{proj}", lambda: K.latent_append_op(r, proj, cfg.eps, A))
-        up = op(f"q_up_{H}x{dim}x{r}x{proj}", lambda: K.head_linear_op(H, r, dim, act=A, rows_max=T, lda=proj, ldc=z["lat"], transposed=True))
+        uk = same(p + "mix.uk", (z["q"], r))
+        tiles = K.head_tiles(r, dim, proj, z["lat"], A)
+        if tiles and prefill:      # the tensor-core form wants W_uk with a latent column per row: turned once, at load
+            bufs[f"ukt.l{i}"] = {"dtype": "bf16", "shape": [H, r, dim], "kind": "carry"}
+            once.append({"op": op(f"transpose_{H}x{dim}x{r}", lambda: K.transpose_heads_op(H, dim, r)), "label": p + "ukt", "args": [uk, B(f"ukt.l{i}")]})
+        up = op(f"q_up_{H}x{dim}x{r}x{proj}", lambda: K.head_linear_op(H, r, dim, act=A, rows_max=T, lda=proj, ldc=z["lat"], transposed=not tiles))
         down = op(f"v_up_{H}x{vdim}x{r}", lambda: K.head_linear_op(H, vdim, r, act=A, rows_max=T, lda=z["lat"], ldc=z["v"]))
         gate = op(f"gate_{z['v']}x{proj}", lambda: K.gate_mul_op(z["v"], proj, A))
         sfx = "_p" if prefill else "_d"
@@ -348,7 +353,7 @@ def build_manifest(cfg: GafapelConfig) -> dict:
             linear("lin", proj, d, B("xn"), w_in, B("proj"), label=p + "qgc"),
             {"op": app, "label": p + "append", "args": [B("proj", (z["q"] + z["v"]) * es), {"state": kv}, B("slot_mapping"),
                                                         same(p + "mix.dkv.norm", (r,))]},
-            {"op": up, "label": p + "q_up", "args": [B("proj"), same(p + "mix.uk", (z["q"], r)), B("qlat"), V("tokens"), err]},
+            {"op": up, "label": p + "q_up", "args": [B("proj"), B(f"ukt.l{i}") if tiles else uk, B("qlat"), V("tokens"), err]},
             {"op": attn, "label": p + "attn", "args": [B("qlat"), {"state": kv}, B("olat"), B("block_table"), *lens]},
             {"op": down, "label": p + "v_up", "args": [B("olat"), same(p + "mix.uv", (z["v"], r)), B("attn"), V("tokens"), err]},
             {"op": gate, "label": p + "gate", "args": [B("attn"), B("proj", z["q"] * es), B("attn"), V("tokens")]},
@@ -437,5 +442,8 @@ def build_manifest(cfg: GafapelConfig) -> dict:
             "logits": {"calls": logits},
         },
     }
-    doc["modules"] = C.modules_for(sorted({l["module"] for o in ops.values() for l in o["impl"]["launches"]}))
+    if once:
+        doc["programs"]["load"] = {"once": True, "calls": once}
+    used = {l["module"] for o in ops.values() for l in o["impl"]["launches"]}
+    doc["modules"] = {n: m for n, m in C.modules_for(sorted(used)).items() if n in used}
     return doc

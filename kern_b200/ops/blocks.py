@@ -82,6 +82,13 @@ def _k_linear(swiglu):
     return run
 
 
+def k_gemm_heads(g, a, w, c, m, n, k, ldc, heads, err):
+    lda = a._row_stride
+    for h in range(heads):
+        W = _f(w[h * n * k:(h + 1) * n * k].view(n, k))
+        _rows(c[h * n:], m, n, ldc).copy_(_f(_rows(a[h * k:], m, k, lda)) @ W.t())
+
+
 def _k_grouped(swiglu):
     def run(g, a, w, c, tiles, count, rows, n, k, wz, err):
         for e, r0, nr, _ in tiles.view(-1, 4)[: int(count[0])].tolist():
@@ -222,5 +229,6 @@ for _a in ("bf16", "f32"):
     CPU_KERNELS.update({f"kern_latent_attn_{_a}_w{w}": k_latent_attn for w in (64, 128, 256, 512, 1024)})
 CPU_KERNELS.update({"kern_linear_bf16_f32": _k_linear(False), "kern_transpose_heads_bf16": k_transpose_heads,
                     "kern_moe_route_logits": k_route_logits})
+CPU_KERNELS.update({f"kern_gemm_bf16_heads_n{n}": k_gemm_heads for n in (64, 128, 256)})
 CPU_KERNELS.update({f"kern_ssd_chunk_n{n}": k_ssd_chunk for n in (32, 64, 128, 256)})
 CPU_KERNELS.update({f"kern_latent_decode_bf16_b{b}": k_latent_decode for b in range(1, 9)})

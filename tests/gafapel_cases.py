@@ -40,6 +40,8 @@ CASES = {
         block(latent(3, 14, 10, 36, 0.5), moe(4, 4, 30)), block(mamba(3, 5, 7, 1, 5, 3), dense(30)),
         block(mamba(9, 7, 33, 3, 1, 7, "mamba2_2"), moe(5, 2, 11))]),
     "states_only": dict(width=64, vocab=96, streams=5, eps=1e-6, blocks=[block(mamba(4, 17, 130, 2, 3, 2)), block(mamba(2, 64, 16, 2, 4, 8), dense(48))]),
+    # ragged width, aligned latents: per-head products on the tiles, everything else generic
+    "ragged_width": dict(width=60, vocab=99, streams=2, eps=1e-6, blocks=[block(latent(3, 16, 24, 40, 0.3), dense(36)), block(mamba(2, 8, 20, 1, 3, 1))]),
     "cache_only": dict(width=96, vocab=160, streams=2, eps=1e-6, blocks=[block(latent(20, 8, 16, 200, 0.4), dense(64)), block(latent(17, 32, 8, 64, 0.2))]),
 }
 
@@ -173,7 +175,9 @@ def run_op(op, args, gpu: bool, vars_=None):
     vars_ = vars_ or {}
     doc = {"schema_version": 7, "model": "one-op", "vars": {n: {"max": v} for n, v in vars_.items()}, "states": {}, "buffers": {},
            "ops": {"op": op}, "programs": {"go": {"calls": [{"op": "op", "args": []}]}},
-           "modules": C.modules_for(sorted({l["module"] for l in op["impl"]["launches"]}))}
+           "modules": {}}
+    used = {l["module"] for l in op["impl"]["launches"]}
+    doc["modules"] = {n: m for n, m in C.modules_for(sorted(used)).items() if n in used}
     call, names = doc["programs"]["go"]["calls"][0]["args"], []
     for i, (a, p) in enumerate(zip(args, op["params"])):
         name = f"b{i}"
