@@ -66,6 +66,19 @@ KERN_DEVICE void tile_body(const AT* A, const __nv_bfloat16* W, OT* C, int m0, i
     }
 }
 
+// grid [columns / (256 V), rows]: a thread walks the rows blockIdx.y, + gridDim.y, .. of its columns
+template <typename T, int V>
+KERN_DEVICE void gate_mul_body(const T* x, const T* gate, T* out, int tokens, int d, int x_stride, int g_stride, int o_stride) {
+  for (int t = blockIdx.y; t < tokens; t += gridDim.y)
+    for (int c = (blockIdx.x * 256 + threadIdx.x) * V; c < d; c += gridDim.x * 256 * V) {
+      const Vec<V> a = ldv<V>(x + (size_t)t * x_stride + c), g = ldv<V>(gate + (size_t)t * g_stride + c);
+      Vec<V> o;
+#pragma unroll
+      for (int e = 0; e < V; ++e) o.v[e] = a.v[e] / (1.f + expf(-g.v[e]));
+      stv<V>(out + (size_t)t * o_stride + c, o);
+    }
+}
+
 }  // namespace
 
 // grid [ceil(N / 64), ceil(M / 64), batch], block 256. Batch z: A + z a_z, W + z w_z, C + z c_z (elements).
@@ -105,12 +118,10 @@ KERN_DEVICE void tile_body(const AT* A, const __nv_bfloat16* W, OT* C, int m0, i
   extern "C" __global__ void __launch_bounds__(256)                                                                         \
       kern_gate_mul_##SFX(const T* x, const T* gate, T* out, int tokens, int d, int x_stride, int g_stride, int o_stride) { \
     pdl_wait();                                                                                                             \
-    for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < (long long)tokens * d;                                \
-         i += (long long)gridDim.x * 256) {                                                                                 \
-      const int t = (int)(i / d), c = (int)(i % d);                                                                         \
-      const float g = ldf(gate + (size_t)t * g_stride + c);                                                                 \
-      stf(out + (size_t)t * o_stride + c, ldf(x + (size_t)t * x_stride + c) / (1.f + expf(-g)));                            \
-    }                                                                                                                       \
+    const bool vec = (d | x_stride | g_stride | o_stride) % 4 == 0 &&                                                       \
+                     ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & 15) == 0; \
+    if (vec) gate_mul_body<T, 4>(x, gate, out, tokens, d, x_stride, g_stride, o_stride);                                    \
+    else gate_mul_body<T, 1>(x, gate, out, tokens, d, x_stride, g_stride, o_stride);                                        \
   }
 
 LINEAR_ENTRY(kern_linear_bf16, __nv_bfloat16, __nv_bfloat16, false)

@@ -145,28 +145,38 @@ KERN_DEVICE void rule_body(const T* xbc, const T* dt, float* y, uint8_t* state, 
   }
 }
 
-template <typename T>
+template <typename T, int V>
 KERN_DEVICE void gate_norm_body(const float* y, const T* z, const __nv_bfloat16* w, T* out, int inner, int parts, int z_stride,
                                 float eps) {
   extern __shared__ __align__(16) float ssd_sm[];
   __shared__ float part[8];
-  const int t = blockIdx.x, width = inner / parts, c0 = blockIdx.y * width;
+  const int t = blockIdx.x, width = inner / parts, c0 = blockIdx.y * width, warps = blockDim.x >> 5;
+  const float* yr = y + (size_t)t * inner + c0;
+  const T* zr = z + (size_t)t * z_stride + c0;
   float ss = 0.f;
-  for (int i = threadIdx.x; i < width; i += 256) {
-    const float zv = ldf(z + (size_t)t * z_stride + c0 + i);
-    const float v = y[(size_t)t * inner + c0 + i] * (zv / (1.f + expf(-zv)));
-    ssd_sm[i] = v;
-    ss += v * v;
+  for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+    const Vec<V> g = ldv<V>(zr + i);
+    Vec<V> v = ldv<V>(yr + i);
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      v.v[e] *= g.v[e] / (1.f + expf(-g.v[e]));
+      ss += v.v[e] * v.v[e];
+    }
+    stv<V>(ssd_sm + i, v);
   }
   ss = warp_sum(ss);
   if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = ss;
   __syncthreads();
   ss = 0.f;
-#pragma unroll
-  for (int i = 0; i < 8; ++i) ss += part[i];
+  for (int i = 0; i < warps; ++i) ss += part[i];
   const float inv = 1.f / sqrtf(ss / (float)width + eps);
-  for (int i = threadIdx.x; i < width; i += 256)
-    stf(out + (size_t)t * inner + c0 + i, ssd_sm[i] * inv * __bfloat162float(w[c0 + i]));
+  for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+    const Vec<V> v = ldv<V>(ssd_sm + i), g = ldv<V>(w + c0 + i);
+    Vec<V> o;
+#pragma unroll
+    for (int e = 0; e < V; ++e) o.v[e] = v.v[e] * inv * g.v[e];
+    stv<V>(out + (size_t)t * inner + c0 + i, o);
+  }
 }
 
 }  // namespace
@@ -183,7 +193,7 @@ KERN_DEVICE void gate_norm_body(const float* y, const T* z, const __nv_bfloat16*
     pdl_launch_dependents();                                                                                               \
   }
 // conv: grid [rows, ceil(channels / 256)]; conv_state: grid [seqs, ceil(channels / 256)]; rule: grid [H ceil(P / 16), seqs];
-// gate_norm: grid [tokens, parts]; block 256 everywhere.
+// gate_norm: grid [tokens, parts], block a multiple of 32 up to 256; block 256 elsewhere.
 #define SSD_ENTRIES(T, SFX)                                                                                                \
   extern "C" __global__ void __launch_bounds__(256)                                                                        \
       kern_ssd_conv_##SFX(const T* x, T* y, const uint8_t* state, const int* lines, const int* cu, const __nv_bfloat16* w, \
@@ -207,7 +217,10 @@ KERN_DEVICE void gate_norm_body(const float* y, const T* z, const __nv_bfloat16*
       kern_ssd_gate_norm_##SFX(const float* y, const T* z, const __nv_bfloat16* w, T* out, int inner, int parts,           \
                                int z_stride, float eps) {                                                                  \
     pdl_wait();                                                                                                            \
-    gate_norm_body<T>(y, z, w, out, inner, parts, z_stride, eps);                                                          \
+    if ((inner / parts | z_stride) % 4 == 0 && (reinterpret_cast<uintptr_t>(z) & 15) == 0)                                 \
+      gate_norm_body<T, 4>(y, z, w, out, inner, parts, z_stride, eps);                                                     \
+    else                                                                                                                   \
+      gate_norm_body<T, 1>(y, z, w, out, inner, parts, z_stride, eps);                                                     \
     pdl_launch_dependents();                                                                                               \
   }
 

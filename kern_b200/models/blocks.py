@@ -83,7 +83,7 @@ def head_linear_op(heads: int, n: int, k: int, *, act: str = "bf16", rows_max: i
 def gate_mul_op(d: int, gate_stride: int, act: str = "bf16") -> dict:
     """out = x * sigmoid(gate). Interface [x, gate, out, tokens]."""
     iface = [f"in buffer<{act}>", f"in buffer<{act}>", f"out buffer<{act}>", "i32"]
-    return _op(iface, _launch("linear", f"kern_gate_mul_{act}", [256, 1, 1], [{"ceil_div": [{"mul": ["tokens", d]}, 1024]}, 1, 1],
+    return _op(iface, _launch("linear", f"kern_gate_mul_{act}", [256, 1, 1], [-(-d // 1024), {"clamp": ["tokens", 0, 4096]}, 1],
                               iface + ["i32"] * 4, [P(0), P(1), P(2), P(3), I(d), I(d), I(gate_stride), I(d)]))
 
 
@@ -208,7 +208,7 @@ def ssd_gate_norm_op(inner: int, parts: int, z_stride: int, eps: float, act: str
     if inner % parts:
         raise ValueError(f"{inner} columns do not split into {parts} norm groups")
     iface = ["in buffer<f32>", f"in buffer<{act}>", "in buffer<bf16>", f"out buffer<{act}>"]
-    return _op(iface, _launch("ssd", f"kern_ssd_gate_norm_{act}", [256, 1, 1], ["tokens", parts, 1], iface + ["i32", "i32", "i32", "f32"],
+    return _op(iface, _launch("ssd", f"kern_ssd_gate_norm_{act}", [min(256, -(-inner // parts // 128) * 32), 1, 1], ["tokens", parts, 1], iface + ["i32", "i32", "i32", "f32"],
                               [*map(P, range(4)), I(inner), I(parts), I(z_stride), {"f32": eps}], shared_mem=inner // parts * 4))
 
 
