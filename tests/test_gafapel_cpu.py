@@ -149,3 +149,28 @@ def test_replay_program_and_command_line(tmp_path):
                         "--steps", "4"], capture_output=True, text=True, cwd=ROOT)
     assert r.returncode == 0, r.stderr[-2000:]
     assert json.loads(r.stdout.splitlines()[-1])["tokens"] == greedy(truth, [4, 9, 1], 4)
+
+
+def test_pipeline_of_two_stages_emits_what_one_engine_does():
+    """Cut at a layer boundary: the streams, the normed input and the row plan cross; each state stays on its stage."""
+    from kern_b200.cpu import CpuRuntime
+    from kern_b200.serve import pp
+
+    cfg = A.config("mixed", "f32")
+    w = A.weights(cfg)
+    doc = G.build_manifest(cfg)
+    parts = pp.cut(doc, pp.layer_cuts(doc, 2))
+    assert sorted(s for d in parts for s in d["states"]) == ["kv.l1", "kv.l3", "ssd.l0", "ssd.l2"]
+    stages = [CpuRuntime(d, weights=w, tokens=cfg.page_size * 40, slots=4) for d in parts]
+    for rt in stages:
+        rt.once()
+    single = A.engine(cfg, w, False)
+    prompt, res = A.prompts_of(cfg, (22,))["r0"], []
+    for eng in (single, pp.PipelineEngine(stages, single.p)):
+        s = eng.open(40)
+        eng.step([(s, prompt[:10])])
+        out = [eng.step([(s, prompt[10:])])[0][0]]
+        for _ in range(4):
+            out.append(eng.step([(s, [out[-1]])])[0][0])
+        res.append(out)
+    assert res[0] == res[1]
