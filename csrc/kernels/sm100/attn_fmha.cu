@@ -81,10 +81,11 @@ struct FmhaArgs {
   int* err;
   int hq, hk, q_stride, out_stride, max_pages, page_size, pool_pages;
   float scale_log2;
+  AttnWindow win = {};
 };
 
 // `y`: the CTA's index into the work list (blockIdx.y unless the caller maps it)
-template <int D, int FN>
+template <int D, int FN, bool WIN = false>
 KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const int y) {
   using Cfg = FmhaCfg<D, FN>;
   constexpr int kStages = Cfg::kStages;
@@ -128,7 +129,9 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
   const int tok_n = min(toks_per_blk, R - tok_lo);
   const int valid_rows = tok_n * G;
   const int last_pos = L - R + tok_lo + tok_n - 1;
-  const int ntiles = last_pos / FN + 1;
+  // (WIN) the first tile that any row of this block sees; tile j of the walk starts at token tok_first + j FN
+  const int tok_first = WIN ? max(0, L - R + tok_lo - a.win.size + 1) / FN * FN : 0;
+  const int ntiles = (last_pos - tok_first) / FN + 1;
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < kStages; ++s) {
@@ -186,7 +189,7 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
         uint8_t* dst = kv_s + stage * 2 * Cfg::kTileBytes + which * Cfg::kTileBytes;
         mbar_expect_tx(full, Cfg::kTileBytes);
         for (int b = 0; b < boxes; ++b) {
-          const int tok = t * FN + b * box_rows;
+          const int tok = tok_first + t * FN + b * box_rows;
           int page = 0, in_page = 0;
           const int pidx = tok / a.page_size;
           if (tok < L && pidx < a.max_pages) {
@@ -268,7 +271,7 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
       if (!mbar_wait_ns(&s_full[j & 1], (j >> 1) & 1, abort_flag)) { set_error(a.err, ERR_WAIT_TMEM_FULL); *abort_flag = 1; ok = false; break; }
       tc_fence_after();
       const uint32_t s_tmem = tmem_base + lane_addr + (j & 1) * FN;
-      const int tok0 = j * FN;
+      const int tok0 = tok_first + j * FN;
       const bool diag = tok0 + FN - 1 > pos;                        // some column of the tile is above this row's limit
       // pass 1: the row maximum of the tile. With 64-token tiles the row's 64 scores stay in registers for pass 2 (one
       // read of S instead of two), and the S buffer is handed back to the MMA warp at once.
@@ -279,7 +282,16 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
 #pragma unroll
         for (int c = 0; c < FN / 32; ++c) tmem_ld_32x32(s_tmem + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&keep[c * 32]));
         tmem_ld_wait();
-        if (diag) {       // the causal limit, once, on the scores themselves (a per-row branch: no warp-wide instruction inside)
+        if constexpr (WIN) {      // capped scores in base-2 units, then both edges of the window
+          static_assert(!WIN || kKeep, "the windowed form keeps a tile's scores in registers");
+#pragma unroll
+          for (int i = 0; i < FN; ++i) keep[i] = __float_as_uint(capped_score(__uint_as_float(keep[i]), a.win));
+          if (diag || tok0 <= pos - a.win.size) {
+#pragma unroll
+            for (int i = 0; i < FN; ++i)
+              if (tok0 + i > pos || tok0 + i <= pos - a.win.size) keep[i] = 0xff800000u;
+          }
+        } else if (diag) {       // the causal limit, once, on the scores themselves (a per-row branch: no warp-wide instruction inside)
 #pragma unroll
           for (int i = 0; i < FN; ++i)
             if (tok0 + i > pos) keep[i] = 0xff800000u;      // -inf
@@ -303,7 +315,8 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
             if (!diag || tok0 + c * 32 + i <= pos) mx = fmaxf(mx, __uint_as_float(r[i]));
         }
       }
-      mx *= a.scale_log2;
+      if constexpr (!WIN) mx *= a.scale_log2;
+      const float sl = WIN ? 1.f : a.scale_log2;
       // lazy reference maximum: move it (and rescale O and l) only when the running maximum outgrew it by 2^8
       float alpha = 1.f;
       bool moved = false;
@@ -349,8 +362,8 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
         for (int i = 0; i < 16; ++i) {
           const int t = tok0 + c * 32 + 2 * i;
           // (kept scores carry the causal limit already: a masked one is -inf and its exponential 0)
-          const float p0 = (kKeep || !diag || t <= pos) ? exp2f(__uint_as_float(r[2 * i]) * a.scale_log2 - m_use) : 0.f;
-          const float p1 = (kKeep || !diag || t + 1 <= pos) ? exp2f(__uint_as_float(r[2 * i + 1]) * a.scale_log2 - m_use) : 0.f;
+          const float p0 = (kKeep || !diag || t <= pos) ? exp2f(__uint_as_float(r[2 * i]) * sl - m_use) : 0.f;
+          const float p1 = (kKeep || !diag || t + 1 <= pos) ? exp2f(__uint_as_float(r[2 * i + 1]) * sl - m_use) : 0.f;
           if (i & 1) sum_b += p0 + p1; else sum += p0 + p1;
           pk[i] = pack_bf16x2(p0, p1);
         }
@@ -373,7 +386,8 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
     if (ok) {
       tc_fence_after();
       const uint32_t o_tmem = tmem_base + lane_addr + 2 * FN;
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      if constexpr (WIN) inv = row < valid_rows ? sink_factor(m_ref, l_run, __bfloat162float(a.win.sink[kvh * G + row % G]), a.win.out_scale) : 0.f;
       __nv_bfloat16* dst = nullptr;
       if (row < valid_rows) {
         const int tk = row0_tok + tok_lo + row / G, head = kvh * G + row % G;
@@ -790,3 +804,14 @@ extern "C" __global__ void __launch_bounds__(192, 2)
 
 KERN_FMHA_CTX_ENTRY(kern_attn_fmha_ctx_qk192_v128, 2, 1)
 KERN_FMHA_CTX_ENTRY(kern_attn_fmha_ctx_qk192_v128_x2, 1, 2)
+
+// The 64-token form over a sliding window, with capped scores and a sink per query head (AttnWindow in attn_paged.cu).
+extern "C" __global__ void __launch_bounds__(192, 2)
+    kern_attn_window_fmha_d128(const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* q, __nv_bfloat16* out,
+                               const int* block_table, const int* seq_lens, const int* cu_q, const int* work,
+                               const int* work_count, int hq, int hk, int q_stride, int out_stride, int max_pages, int page_size,
+                               int pool_pages, int* err, const __nv_bfloat16* sink, int window, float c1, float c2, float out_scale) {
+  FmhaArgs a{q, out, block_table, seq_lens, cu_q, work, work_count, err, hq, hk, q_stride, out_stride, max_pages, page_size,
+             pool_pages, 1.f, {window, c1, c2, out_scale, sink}};
+  fmha_body<128, 64, true>(&kv_map, a, (int)blockIdx.y);
+}

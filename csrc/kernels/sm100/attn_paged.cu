@@ -59,6 +59,24 @@ struct AttnCfg {
   static constexpr int kSmem = 1024 + kStages * kStageBytes + kQBytes + 256;
 };
 
+// Attention in a sliding window with capped scores and a sink (the WIN forms): a row at position i sees the keys j with
+// 0 <= i - j < size; a score is cap tanh(score / cap), computed as c2 (1 - 2 / (1 + 2^(c1 q.k))) with c1 = 2 log2(e) scale / cap
+// and c2 = cap log2(e), in the base-2 units of the softmax; `sink` (bf16, one per query head) joins every row's denominator
+// once, as a score that is neither scaled nor capped. The finished rows are multiplied by out_scale.
+struct AttnWindow {
+  int size;
+  float c1, c2, out_scale;
+  const __nv_bfloat16* sink;
+};
+constexpr float kLog2e = 1.4426950408889634f;
+KERN_DEVICE float capped_score(float qk, const AttnWindow& w) { return w.c2 - __fdividef(2.f * w.c2, 1.f + exp2f(qk * w.c1)); }
+// (m, l): a finished row's maximum and sum in base-2 units -> the factor of its un-normalised output
+KERN_DEVICE float sink_factor(float m, float l, float sink, float out_scale) {
+  const float s = sink * kLog2e, top = fmaxf(m, s);
+  const float f = exp2f(m - top);          // 0 for a row that saw no key
+  return out_scale * f / (l * f + exp2f(s - top));
+}
+
 struct AttnArgs {
   const __nv_bfloat16* q;
   __nv_bfloat16* out;
@@ -72,11 +90,12 @@ struct AttnArgs {
   int* err;
   int seqs, hq, hk, q_stride, out_stride, max_pages, page_size, rows_per_seq, splits, pool_pages;
   float scale_log2;
+  AttnWindow win = {};
 };
 
 // PREFILL = false: decode/verify (warps split tokens); true: causal prefill (warps split rows)
 // `y`: the CTA's index into the work list (or its sequence), blockIdx.y unless the caller maps it
-template <int D, bool PREFILL, int ST = 0>
+template <int D, bool PREFILL, int ST = 0, bool WIN = false>
 KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const int y) {
   using Cfg = AttnCfg<D, PREFILL, ST>;
   constexpr int kStages = Cfg::kStages;
@@ -125,7 +144,9 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
   const int valid_rows = tok_n * G;
   // query token r (0-based among this step's R rows) sits at position L - R + r
   const int last_pos = L - R + tok_lo + tok_n - 1;
-  const int ntiles_all = last_pos / TK + 1;
+  // (WIN) no row of this block sees a key before `tile_first`
+  const int tile_first = WIN ? max(0, L - R + tok_lo - a.win.size + 1) / TK : 0;
+  const int ntiles_all = last_pos / TK + 1 - tile_first;
   // `splits` packs three numbers: bits 0-7 the KV splits of this launch, bits 8-15 the first partial slot it writes,
   // bits 16-31 the partial slots per (row, head) in the workspace (0: same as the splits). A context-parallel rank
   // writes its partials into its own run of slots of a workspace that holds every rank's; one merge covers them all.
@@ -139,6 +160,7 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
     if (tile_hi < tile_lo) tile_hi = tile_lo;
   }
   const int ntiles = tile_hi - tile_lo;
+  tile_lo += tile_first;
 
   // ---- q tile -> shared (all 5 warps help) ----
   for (int i = threadIdx.x; i < ROWS * (D / 8); i += kAttnThreads) {
@@ -225,7 +247,9 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
       const int wtok = PREFILL ? 0 : warp * 16;   // this warp's token offset inside the tile
       // a whole tile above the causal limit of this warp's rows contributes nothing
       const int warp_max_pos = L - R + tok_lo + min(valid_rows - 1, qrow_base + 15) / G;
-      const bool skip = PREFILL && (tok0 > warp_max_pos || qrow_base >= valid_rows);
+      bool skip = PREFILL && (tok0 > warp_max_pos || qrow_base >= valid_rows);
+      if constexpr (WIN)      // nor does one below the window of all of them
+        skip = skip || tok0 + TK - 1 <= L - R + tok_lo + qrow_base / G - a.win.size;
       if (!skip) {
         // ---- S = Q K^T ----
         float s[NT][4];
@@ -251,10 +275,17 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
           const int j = tok0 + wtok + n * 8 + 2 * (lane & 3);
-          s[n][0] = (j <= posA) ? s[n][0] * a.scale_log2 : -INFINITY;
-          s[n][1] = (j + 1 <= posA) ? s[n][1] * a.scale_log2 : -INFINITY;
-          s[n][2] = (j <= posB) ? s[n][2] * a.scale_log2 : -INFINITY;
-          s[n][3] = (j + 1 <= posB) ? s[n][3] * a.scale_log2 : -INFINITY;
+          if constexpr (WIN) {
+            s[n][0] = (j <= posA && j > posA - a.win.size) ? capped_score(s[n][0], a.win) : -INFINITY;
+            s[n][1] = (j + 1 <= posA && j + 1 > posA - a.win.size) ? capped_score(s[n][1], a.win) : -INFINITY;
+            s[n][2] = (j <= posB && j > posB - a.win.size) ? capped_score(s[n][2], a.win) : -INFINITY;
+            s[n][3] = (j + 1 <= posB && j + 1 > posB - a.win.size) ? capped_score(s[n][3], a.win) : -INFINITY;
+          } else {
+            s[n][0] = (j <= posA) ? s[n][0] * a.scale_log2 : -INFINITY;
+            s[n][1] = (j + 1 <= posA) ? s[n][1] * a.scale_log2 : -INFINITY;
+            s[n][2] = (j <= posB) ? s[n][2] * a.scale_log2 : -INFINITY;
+            s[n][3] = (j + 1 <= posB) ? s[n][3] * a.scale_log2 : -INFINITY;
+          }
           mxA = fmaxf(mxA, fmaxf(s[n][0], s[n][1]));
           mxB = fmaxf(mxB, fmaxf(s[n][2], s[n][3]));
         }
@@ -347,8 +378,10 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
       }
       const int tk = row0_tok + tok_lo + r / G, head = kvh * G + r % G;
       if (split_total == 1) {
-        a.out[(size_t)tk * a.out_stride + (size_t)head * D + c] =
-            __float2bfloat16(l > 0.f ? acc / l : 0.f);
+        float v;
+        if constexpr (WIN) v = acc * sink_factor(m, l, __bfloat162float(a.win.sink[head]), a.win.out_scale);
+        else v = l > 0.f ? acc / l : 0.f;
+        a.out[(size_t)tk * a.out_stride + (size_t)head * D + c] = __float2bfloat16(v);
       } else {
         const size_t base = ((size_t)tk * a.hq + head) * split_total + split_base + split;
         a.ws_o[base * D + c] = acc;
@@ -360,7 +393,11 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
     }
   } else if (warp < 4) {
     const int rA = warp * 16 + (lane >> 2), rB = rA + 8;
-    const float iA = l_run[0] > 0.f ? 1.f / l_run[0] : 0.f, iB = l_run[1] > 0.f ? 1.f / l_run[1] : 0.f;
+    float iA = l_run[0] > 0.f ? 1.f / l_run[0] : 0.f, iB = l_run[1] > 0.f ? 1.f / l_run[1] : 0.f;
+    if constexpr (WIN) {
+      if (rA < valid_rows) iA = sink_factor(m_run[0], l_run[0], __bfloat162float(a.win.sink[kvh * G + rA % G]), a.win.out_scale);
+      if (rB < valid_rows) iB = sink_factor(m_run[1], l_run[1], __bfloat162float(a.win.sink[kvh * G + rB % G]), a.win.out_scale);
+    }
 #pragma unroll
     for (int i = 0; i < D / 8; ++i) {
       const int c = i * 8 + 2 * (lane & 3);

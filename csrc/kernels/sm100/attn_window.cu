@@ -1,0 +1,244 @@
+// build: precise
+// Attention over a paged cache in a sliding window, with capped scores and a learned sink per query head:
+//     score = cap tanh(q.k scale / cap);  weight_j = exp(score_j) / (exp(sink_h) + sum over the window of exp(score))
+// and what prepares its rows.
+//   kern_qk_prep_<act>          per head: RMS norm of q and k with a weight of their own, rotary positions on the first
+//                               columns (pairs (2i, 2i + 1), or halves), k and v into their rows of the paged cache
+//   kern_window_attn_<act>_w*   one (row, query head) per block, any sizes, either activation type
+//   kern_attn_window_*_d*       bf16 with equal head dims 64 / 128 / 256: the bodies of attn_paged.cu (decode rows with split
+//                               keys, prompt rows, both lists of a ragged call in one launch)
+//   kern_attn_window_merge      the partials of split keys, where the sink joins the denominator
+// Cache of one layer: [page][k: head, offset, dim | v: head, offset, vdim]; with equal dims that is attn_prep.cu's layout.
+// Norms, angles, scores, weights and sums are f32.
+#define KERN_ATTN_NO_ENTRIES
+#include "attn_paged.cu"
+#include "act.cuh"
+
+using namespace kern;
+
+namespace {
+
+// grid = rows, block 256: a warp per head, heads dealt to the eight warps; 8 max(d, dv) floats of shared memory
+template <typename T>
+KERN_DEVICE void prep_body(T* qkv, uint8_t* cache, const long long* positions, const long long* slots, const float* cos_tab,
+                           const float* sin_tab, const __nv_bfloat16* q_norm, const __nv_bfloat16* k_norm, int hq, int hk, int d,
+                           int dv, int rot, int halves, int page_size, int row_stride, int max_pos, float eps, int* err) {
+  extern __shared__ __align__(16) float prep_sm[];
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* row = prep_sm + warp * max(d, dv);
+  long long pos = positions[t];
+  const long long slot = slots[t];
+  if (pos < 0 || pos >= max_pos) {
+    if (threadIdx.x == 0) set_error(err, ERR_BOUNDS);
+    pos = 0;
+  }
+  const int half = rot >> 1;
+  const float* cs = cos_tab + (size_t)pos * half;
+  const float* sn = sin_tab + (size_t)pos * half;
+  T* base = qkv + (size_t)t * row_stride;
+  T* page = reinterpret_cast<T*>(cache) + (size_t)(slot < 0 ? 0 : slot / page_size) * hk * page_size * (d + dv);
+  const int off = slot < 0 ? 0 : (int)(slot % page_size);
+  for (int h = warp; h < hq + 2 * hk; h += 8) {
+    const bool is_q = h < hq, is_v = h >= hq + hk;
+    if (!is_q && slot < 0) continue;
+    if (is_v) {
+      const int kh = h - hq - hk;
+      const T* src = base + (size_t)(hq + hk) * d + (size_t)kh * dv;
+      T* dst = page + (size_t)hk * page_size * d + ((size_t)kh * page_size + off) * dv;
+      if (!KERN_CHECK(dst, (size_t)dv * sizeof(T), SITE_KV_APPEND)) continue;
+      for (int i = lane; i < dv; i += 32) dst[i] = src[i];
+      continue;
+    }
+    T* src = base + (size_t)h * d;
+    T* dst = is_q ? src : page + ((size_t)(h - hq) * page_size + off) * d;
+    if (!is_q && !KERN_CHECK(dst, (size_t)d * sizeof(T), SITE_KV_APPEND)) continue;
+    const __nv_bfloat16* w = is_q ? q_norm : k_norm;
+    float ss = 0.f;
+    for (int i = lane; i < d; i += 32) {
+      const float v = ldf(src + i);
+      row[i] = v;
+      ss += v * v;
+    }
+    const float inv = w ? 1.f / sqrtf(warp_sum(ss) / (float)d + eps) : 1.f;
+    __syncwarp();
+    if (w)
+      for (int i = lane; i < d; i += 32) row[i] *= inv * __bfloat162float(w[i]);
+    __syncwarp();
+    for (int i = lane; i < d; i += 32) {
+      float o = row[i];
+      if (i < rot) {
+        const int j = halves ? (i < half ? i : i - half) : i >> 1;
+        const bool lo = halves ? i < half : !(i & 1);
+        const int other = halves ? (lo ? i + half : i - half) : i ^ 1;
+        o = lo ? o * cs[j] - row[other] * sn[j] : o * cs[j] + row[other] * sn[j];
+      }
+      stf(dst + i, o);
+    }
+    __syncwarp();
+  }
+}
+
+// Four warps walk the keys of the row's window (key j belongs to warp j % 4); a lane holds the columns i * 32 + lane of the
+// query and of the warp's running sum. RL = columns per lane.
+template <typename T, int RL>
+KERN_DEVICE void attn_any_body(const T* q, const uint8_t* cache, T* out, const int* table, const int* lens, const int* row_seq,
+                               const __nv_bfloat16* sink, int hq, int hk, int d, int dv, int q_stride, int out_stride, int max_pages,
+                               int page, int window, float scale, float cap, float out_scale, int* err) {
+  extern __shared__ __align__(16) float win_sm[];      // [4][dv] partial sums, then [4] maxima, [4] weights
+  const int h = blockIdx.x, r = blockIdx.y;
+  const int L = lens[r];
+  if (L <= 0) return;
+  if (L > max_pages * page && threadIdx.x == 0) set_error(err, ERR_BOUNDS);     // keys past the table row are left out
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kh = h / (hq / hk);
+  const int* pages = table + (size_t)(row_seq ? row_seq[r] : r) * max_pages;
+  const T* rows = reinterpret_cast<const T*>(cache);
+  const T* qr = q + (size_t)r * q_stride + (size_t)h * d;
+  float qv[RL], o[RL];
+#pragma unroll
+  for (int i = 0; i < RL; ++i) {
+    const int c = i * 32 + lane;
+    qv[i] = c < d ? ldf(qr + c) : 0.f;
+    o[i] = 0.f;
+  }
+  float m = -INFINITY, l = 0.f;
+  for (int j = max(0, L - window) + warp; j < L; j += 4) {
+    const int pi = j / page;
+    if (pi >= max_pages) break;
+    const T* pg = rows + (size_t)pages[pi] * hk * page * (d + dv);
+    const T* kr = pg + ((size_t)kh * page + j % page) * d;
+    const T* vr = pg + (size_t)hk * page * d + ((size_t)kh * page + j % page) * dv;
+    if (!KERN_CHECK(kr, (size_t)d * sizeof(T), SITE_KV_ROW) || !KERN_CHECK(vr, (size_t)dv * sizeof(T), SITE_KV_ROW)) continue;
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < RL; ++i) {
+      const int c = i * 32 + lane;
+      if (c < d) s += qv[i] * ldf(kr + c);
+    }
+    s = cap * tanhf(warp_sum(s) * scale / cap);
+    const float mn = fmaxf(m, s), f = expf(m - mn), e = expf(s - mn);
+    m = mn;
+    l = l * f + e;
+#pragma unroll
+    for (int i = 0; i < RL; ++i) {
+      const int c = i * 32 + lane;
+      o[i] = o[i] * f + e * (c < dv ? ldf(vr + c) : 0.f);
+    }
+  }
+  float* acc = win_sm;
+  float* ms = win_sm + 4 * dv;
+  float* ls = ms + 4;
+  if (lane == 0) { ms[warp] = m; ls[warp] = l; }
+#pragma unroll
+  for (int i = 0; i < RL; ++i)
+    if (i * 32 + lane < dv) acc[warp * dv + i * 32 + lane] = o[i];
+  __syncthreads();
+  const float sk = __bfloat162float(sink[h]);
+  const float mx = fmaxf(sk, fmaxf(fmaxf(ms[0], ms[1]), fmaxf(ms[2], ms[3])));
+  float f[4], den = expf(sk - mx);
+#pragma unroll
+  for (int w = 0; w < 4; ++w) { f[w] = expf(ms[w] - mx); den += f[w] * ls[w]; }
+  for (int c = threadIdx.x; c < dv; c += 128) {
+    float v = 0.f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) v += f[w] * acc[w * dv + c];
+    stf(out + (size_t)r * out_stride + (size_t)h * dv + c, v / den * out_scale);
+  }
+}
+
+}  // namespace
+
+// attn: grid [heads, rows], block 128, (4 dv + 8) floats of shared memory
+#define WINDOW_ATTN(T, SFX, W)                                                                                             \
+  extern "C" __global__ void __launch_bounds__(128)                                                                        \
+      kern_window_attn_##SFX##_w##W(const T* q, const uint8_t* cache, T* out, const int* table, const int* lens,           \
+                                    const int* row_seq, const __nv_bfloat16* sink, int hq, int hk, int d, int dv,          \
+                                    int q_stride, int out_stride, int max_pages, int page, int window, float scale,        \
+                                    float cap, float out_scale, int* err) {                                                \
+    pdl_wait();                                                                                                            \
+    attn_any_body<T, W / 32>(q, cache, out, table, lens, row_seq, sink, hq, hk, d, dv, q_stride, out_stride, max_pages,    \
+                             page, window, scale, cap, out_scale, err);                                                    \
+  }
+#define WINDOW_ENTRIES(T, SFX)                                                                                             \
+  extern "C" __global__ void __launch_bounds__(256)                                                                        \
+      kern_qk_prep_##SFX(T* qkv, uint8_t* cache, const long long* positions, const long long* slots, const float* cos_tab, \
+                         const float* sin_tab, const __nv_bfloat16* q_norm, const __nv_bfloat16* k_norm, int hq, int hk,   \
+                         int d, int dv, int rot, int halves, int page_size, int row_stride, int max_pos, float eps,        \
+                         int* err) {                                                                                       \
+    pdl_wait();                                                                                                            \
+    prep_body<T>(qkv, cache, positions, slots, cos_tab, sin_tab, q_norm, k_norm, hq, hk, d, dv, rot, halves, page_size,    \
+                 row_stride, max_pos, eps, err);                                                                           \
+    pdl_launch_dependents();                                                                                               \
+  }                                                                                                                        \
+  WINDOW_ATTN(T, SFX, 64)                                                                                                  \
+  WINDOW_ATTN(T, SFX, 128)                                                                                                 \
+  WINDOW_ATTN(T, SFX, 256)                                                                                                 \
+  WINDOW_ATTN(T, SFX, 512)
+
+WINDOW_ENTRIES(__nv_bfloat16, bf16)
+WINDOW_ENTRIES(float, f32)
+
+// ---- the tensor-core bodies ------------------------------------------------------------------------------------------
+#define WINDOW_TC(name, D, PREFILL)                                                                                        \
+  extern "C" __global__ void __launch_bounds__(160, (PREFILL && D <= 128) ? 2 : 1)                                         \
+      name(const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* q, __nv_bfloat16* out, float* ws_o,            \
+           float* ws_ml, const int* block_table, const int* seq_lens, const int* cu_q, const int* work,                    \
+           const int* work_count, int hq, int hk, int q_stride, int out_stride, int max_pages, int page_size, int splits,  \
+           int pool_pages, int* err, const __nv_bfloat16* sink, int window, float c1, float c2, float out_scale) {         \
+    AttnArgs a{q, out, ws_o, ws_ml, block_table, seq_lens, cu_q, work, work_count, err, 0x7fffffff, hq, hk, q_stride,      \
+               out_stride, max_pages, page_size, 1, splits, pool_pages, 1.f, {window, c1, c2, out_scale, sink}};           \
+    attn_body<D, PREFILL, 0, true>(&kv_map, a, (int)blockIdx.y);                                                           \
+  }
+WINDOW_TC(kern_attn_window_decode_d64, 64, false)
+WINDOW_TC(kern_attn_window_decode_d128, 128, false)
+WINDOW_TC(kern_attn_window_decode_d256, 256, false)
+WINDOW_TC(kern_attn_window_prefill_d64, 64, true)
+WINDOW_TC(kern_attn_window_prefill_d128, 128, true)
+WINDOW_TC(kern_attn_window_prefill_d256, 256, true)
+
+// Both lists of a ragged call in one launch, as in attn_paged.cu: two CTAs per SM with a two-stage ring each.
+#define WINDOW_RAGGED(name, D)                                                                                             \
+  extern "C" __global__ void __launch_bounds__(160, 2)                                                                     \
+      name(const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* q, __nv_bfloat16* out, const int* block_table, \
+           const int* seq_lens, const int* cu_q, const int* work_p, const int* count_p, const int* work_d,                 \
+           const int* count_d, int hq, int hk, int q_stride, int out_stride, int max_pages, int page_size, int pool_pages, \
+           int* err, const __nv_bfloat16* sink, int window, float c1, float c2, float out_scale) {                         \
+    const int np = *count_p, nd = *count_d, m = np < nd ? np : nd;                                                         \
+    const int y = blockIdx.y;                                                                                              \
+    if (y >= np + nd) return;                                                                                              \
+    const bool is_p = y < 2 * m ? !(y & 1) : np > nd;                                                                      \
+    AttnArgs a{q, out, nullptr, nullptr, block_table, seq_lens, cu_q, is_p ? work_p : work_d, is_p ? count_p : count_d,    \
+               err, 0x7fffffff, hq, hk, q_stride, out_stride, max_pages, page_size, 1, 1, pool_pages, 1.f,                 \
+               {window, c1, c2, out_scale, sink}};                                                                         \
+    const int idx = y < 2 * m ? (y >> 1) : y - m;                                                                          \
+    if (is_p) attn_body<D, true, 2, true>(&kv_map, a, idx);                                                                \
+    else attn_body<D, false, 2, true>(&kv_map, a, idx);                                                                    \
+  }
+WINDOW_RAGGED(kern_attn_window_ragged_d64, 64)
+WINDOW_RAGGED(kern_attn_window_ragged_d128, 128)
+
+// grid = rows x hq, block min(256, d)
+extern "C" __global__ void kern_attn_window_merge(const float* ws_o, const float* ws_ml, __nv_bfloat16* out,
+                                                  const __nv_bfloat16* sink, int rows, int hq, int d, int splits, int out_stride,
+                                                  float out_scale) {
+  pdl_wait();
+  const int row = blockIdx.x;  // row * hq + head
+  if (row >= rows) return;
+  const int tk = row / hq, head = row % hq;
+  float m = -INFINITY;
+  for (int s = 0; s < splits; ++s) m = fmaxf(m, ws_ml[((size_t)row * splits + s) * 2]);
+  const float m_use = m == -INFINITY ? 0.f : m;
+  float l = 0.f;
+  for (int s = 0; s < splits; ++s) {
+    const size_t b = (size_t)row * splits + s;
+    l += ws_ml[b * 2 + 1] * exp2f(ws_ml[b * 2] - m_use);
+  }
+  const float f = sink_factor(m, l, __bfloat162float(sink[head]), out_scale);
+  for (int c = threadIdx.x; c < d; c += blockDim.x) {
+    float acc = 0.f;
+    for (int s = 0; s < splits; ++s) {
+      const size_t b = (size_t)row * splits + s;
+      acc += ws_o[b * d + c] * exp2f(ws_ml[b * 2] - m_use);
+    }
+    out[(size_t)tk * out_stride + (size_t)head * d + c] = __float2bfloat16(acc * f);
+  }
+}

@@ -73,6 +73,7 @@ enum : int {
   SITE_EP_SLOT = 6,         // a result row stored into its (token, choice) slot
   SITE_STATE_SLOT = 7,      // a per-sequence recurrent state addressed by slot
   SITE_LATENT_ROW = 8,      // a latent cache row addressed through a page table
+  SITE_KV_ROW = 9,          // a key or value row addressed through a page table
 };
 
 // ---- address helpers ------------------------------------------------------------------------
@@ -290,6 +291,22 @@ KERN_DEVICE float2 unpack_bf16x2(uint32_t u) {
   return __bfloat1622float2(v);
 }
 KERN_DEVICE float silu(float x) { return x / (1.0f + __expf(-x)); }
+
+// Gated linear units over a gate and an up column. kGeglu: the tanh form of gelu, 0.5 g (1 + tanh(y)) = g sigmoid(2 y);
+// kClampedGlu: gate from above and up on both sides cut at `limit`, then g sigmoid(1.702 g) (u + 1).
+enum : int { kSwiglu = 0, kGeglu = 1, kClampedGlu = 2 };
+template <int ACT>
+KERN_DEVICE float glu(float g, float u, float limit) {
+  if constexpr (ACT == kGeglu) {
+    return g / (1.f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g))) * u;      // 2 sqrt(2 / pi)
+  } else if constexpr (ACT == kClampedGlu) {
+    g = fminf(g, limit);
+    u = fmaxf(-limit, fminf(u, limit));
+    return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
+  } else {
+    return silu(g) * u;
+  }
+}
 
 // system-scope acquire / release for flags that another GPU writes
 KERN_DEVICE void st_release_sys(uint32_t* p, uint32_t v) {

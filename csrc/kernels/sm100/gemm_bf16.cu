@@ -121,13 +121,18 @@ struct EpArgs {
 // accumulator is scaled by *scale_a * *scale_b (per-tensor scales) before the epilogue's conversion.
 // HEADS: a batch of `heads` products over column ranges: C[:, h N ..] = A[:, h K ..] . W_h^T, W a 3-D map [K, N, heads]. A
 // head's last K block may reach into the next head's columns of A; the map fills W with zeros there.
+// EPI 3, 6, 7: W = [gate rows ; up rows], stored as their gated unit (SwiGLU, GEGLU, the clamped form with its limit)
+__host__ __device__ constexpr bool is_glu(int epi) { return epi == 3 || epi == 6 || epi == 7; }
+__host__ __device__ constexpr int glu_of(int epi) { return epi == 6 ? kGeglu : (epi == 7 ? kClampedGlu : kSwiglu); }
+
 template <int BN, int EPI, bool GROUPED = false, bool FP8 = false, bool MT2 = false, bool AG = false, int EP = 0, bool HEADS = false>
 __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtensorMap* tma_b,
                                           void* Cv, const void* Rv,
                                           int M, int N, int K, int ldc, int* err,
                                           const int* tile_table = nullptr, const int* tile_count = nullptr,
                                           ScatterArgs sc = ScatterArgs(), const float* scale_a = nullptr,
-                                          const float* scale_b = nullptr, AgArgs ag = AgArgs(), EpArgs ep = EpArgs(), int heads = 1) {
+                                          const float* scale_b = nullptr, AgArgs ag = AgArgs(), EpArgs ep = EpArgs(), int heads = 1,
+                                          float glu_limit = 0.f) {
   using Cfg = GemmCfg<BN, MT2>;
   constexpr int kStages = Cfg::kStages;
   constexpr int BMT = Cfg::kRows;
@@ -256,7 +261,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtens
             if constexpr (GROUPED || HEADS) tma_load_3d(dst, tma_b, kb * BKE, n_row, expert, &full_bar[stage]);
             else tma_load_2d(dst, tma_b, kb * BKE, n_row, &full_bar[stage]);
           };
-          if constexpr (EPI == 3) {
+          if constexpr (is_glu(EPI)) {
             // W = [gate rows ; up rows]: this tile's B rows are BN/2 gate rows then the matching BN/2 up rows
             load_b(sb, n_blk * (BN / 2));
             load_b(sb + (BN / 2) * BK * 2, N / 2 + n_blk * (BN / 2));
@@ -474,8 +479,8 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtens
       for (int hh = 0; hh < (MT2 ? 2 : 1); ++hh) {     // the 256-row tile drains its two 128-row accumulators in turn
       const int row = row0 + hh * BM + quarter * 32 + lane;
       const uint32_t t_row = tmem_base + ((uint32_t)(quarter * 32) << 16) + (MT2 ? hh : acc) * BN;
-      if constexpr (EPI == 3) {
-        // SwiGLU: accumulator columns [0, BN/2) are gate, [BN/2, BN) the matching up columns
+      if constexpr (is_glu(EPI)) {
+        // gated unit: accumulator columns [0, BN/2) are gate, [BN/2, BN) the matching up columns
 #pragma unroll 1
         for (int c = 0; c < BN / 64; ++c) {
           uint32_t g[32], u[32];
@@ -491,7 +496,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtens
                 float f[8];
 #pragma unroll
                 for (int j = 0; j < 8; ++j)
-                  f[j] = silu(__uint_as_float(g[v * 8 + j])) * __uint_as_float(u[v * 8 + j]);
+                  f[j] = glu<glu_of(EPI)>(__uint_as_float(g[v * 8 + j]), __uint_as_float(u[v * 8 + j]), glu_limit);
                 uint4 o;
                 o.x = pack_bf16x2(f[0], f[1]); o.y = pack_bf16x2(f[2], f[3]);
                 o.z = pack_bf16x2(f[4], f[5]); o.w = pack_bf16x2(f[6], f[7]);
@@ -705,4 +710,8 @@ KERN_GEMM_ENTRY(kern_gemm_bf16_tn_acc_n32, 32, 2)
 KERN_GEMM_ENTRY(kern_gemm_bf16_tn_swiglu_n256, 256, 3)
 KERN_GEMM_ENTRY(kern_gemm_bf16_tn_swiglu_n128, 128, 3)
 KERN_GEMM_ENTRY(kern_gemm_bf16_tn_swiglu_n64, 64, 3)
+KERN_GEMM_ENTRY_M256(kern_gemm_bf16_tn_geglu_m256_n256, 6)
+KERN_GEMM_ENTRY(kern_gemm_bf16_tn_geglu_n256, 256, 6)
+KERN_GEMM_ENTRY(kern_gemm_bf16_tn_geglu_n128, 128, 6)
+KERN_GEMM_ENTRY(kern_gemm_bf16_tn_geglu_n64, 64, 6)
 #endif  // KERN_GEMM_NO_ENTRIES

@@ -6,7 +6,7 @@
 // A CTA owns four weight rows at a time (so A is fetched once per four outputs); its 256 threads stride over the K
 // vectors of those rows, partial sums meet through shuffles and shared memory. Persistent grid: CTAs take row groups
 // round-robin, eight or so resident per SM, so tens of kilobytes of loads are in flight on every SM.
-// Epilogues as in the tensor-core GEMM: 0 store bf16, 1 store f32, 2 accumulate into a bf16 residual, 3 SwiGLU over
+// Epilogues as in the tensor-core GEMM: 0 store bf16, 1 store f32, 2 accumulate into a bf16 residual, 3 SwiGLU / 6 GEGLU over
 // weights stacked [gate rows ; up rows] (two gate rows and their two up rows per group).
 // (The reference calls a library GEMM for every shape; this kernel has no counterpart there.)
 #include "common.cuh"
@@ -23,10 +23,11 @@ __device__ __forceinline__ void gemv_body(const __nv_bfloat16* A, const __nv_bfl
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int kv = K >> 3;
   const int half = N >> 1;
-  const int groups = EPI == 3 ? (half + 1) / 2 : (N + R - 1) / R;
+  constexpr bool kGlu = EPI == 3 || EPI == 6;      // SwiGLU, GEGLU
+  const int groups = kGlu ? (half + 1) / 2 : (N + R - 1) / R;
   for (int g = blockIdx.x; g < groups; g += gridDim.x) {
     int rows[R];
-    if constexpr (EPI == 3) {
+    if constexpr (kGlu) {
       rows[0] = 2 * g; rows[1] = 2 * g + 1; rows[2] = half + 2 * g; rows[3] = half + 2 * g + 1;
       if (rows[1] >= half) { rows[1] = rows[0]; rows[3] = rows[2]; }     // odd tail: duplicate, the store skips it
     } else {
@@ -86,11 +87,11 @@ __device__ __forceinline__ void gemv_body(const __nv_bfloat16* A, const __nv_bfl
     if (threadIdx.x < MT * R) {
       const int m = threadIdx.x / R, r = threadIdx.x % R;
       if (m < M) {
-        if constexpr (EPI == 3) {
+        if constexpr (kGlu) {
           // outputs 2g (r = 0) and 2g + 1 (r = 1): gate in columns 0..1, up in 2..3
           if (r < 2 && 2 * g + r < half)
             reinterpret_cast<__nv_bfloat16*>(Cv)[(size_t)m * ldc + 2 * g + r] =
-                __float2bfloat16(silu(part[0][m * R + r]) * part[0][m * R + 2 + r]);
+                __float2bfloat16(glu<EPI == 6 ? kGeglu : kSwiglu>(part[0][m * R + r], part[0][m * R + 2 + r], 0.f));
         } else {
           const int n = g * R + r;
           if (n < N) {
@@ -129,7 +130,8 @@ __device__ __forceinline__ void gemv_body(const __nv_bfloat16* A, const __nv_bfl
   KERN_GEMV_ENTRY(kern_gemv_bf16_tn_m##MT, MT, 0)                  \
   KERN_GEMV_ENTRY(kern_gemv_bf16_tn_f32_m##MT, MT, 1)              \
   KERN_GEMV_ENTRY(kern_gemv_bf16_tn_acc_m##MT, MT, 2)              \
-  KERN_GEMV_ENTRY(kern_gemv_bf16_tn_swiglu_m##MT, MT, 3)
+  KERN_GEMV_ENTRY(kern_gemv_bf16_tn_swiglu_m##MT, MT, 3)           \
+  KERN_GEMV_ENTRY(kern_gemv_bf16_tn_geglu_m##MT, MT, 6)
 
 KERN_GEMV_FAMILY(1)
 KERN_GEMV_FAMILY(2)

@@ -2,11 +2,12 @@
 // Matrix products for what the tensor-core tiles do not take: 32-bit activations (a model's exact form), and sizes whose
 // rows are not whole 16-byte vectors. C[M, N] = A[M, K] . W^T with W bf16 read through two strides (so a transposed view
 // needs no copy), one 64 x 64 tile per block, f32 products and sums.
-//   kern_linear_<act>[_f32 | _swiglu]          plain; blockIdx.z walks a batch (one weight, one column range of A and C per head)
-//   kern_linear_grouped_<act>[_swiglu]         rows sorted by expert, the planner's tile table (tiles of at most 64 rows)
+//   kern_linear_<act>[_f32 | _swiglu | _geglu | _clamped]   plain; blockIdx.z walks a batch (one weight, one column range of A and C per head)
+//   kern_linear_grouped_<act>[_<gated unit>]           rows sorted by expert, the planner's tile table (tiles of at most 64 rows)
 //   kern_rows_scatter_<act>                    x_perm[perm[i]] = x[i / k]
 //   kern_gate_mul_<act>                        out = x * sigmoid(gate)
 //   kern_transpose_heads_bf16                  [H][R][C] -> [H][C][R]
+//   kern_copy_cols_bf16                        [R][C] into columns of wider rows
 #include "act.cuh"
 
 using namespace kern;
@@ -15,10 +16,22 @@ namespace {
 
 constexpr int LB = 64, LK = 16;
 
-// rows [m0, m_end) of A, columns [n0, ..) of C; SWIGLU: W holds N gate rows, then N up rows
-template <typename AT, typename OT, bool SWIGLU>
+// the gated units of common.cuh without the fast exponential; ACT < 0: none
+template <int ACT>
+KERN_DEVICE float glu_exact(float g, float u, float limit) {
+  if constexpr (ACT == kGeglu) return g / (1.f + expf(-1.5957691216057308f * (g + 0.044715f * g * g * g))) * u;
+  if constexpr (ACT == kClampedGlu) {
+    g = fminf(g, limit);
+    return g / (1.f + expf(-1.702f * g)) * (fmaxf(-limit, fminf(u, limit)) + 1.f);
+  }
+  return g / (1.f + expf(-g)) * u;
+}
+
+// rows [m0, m_end) of A, columns [n0, ..) of C; with a gated unit W holds N gate rows, then N up rows
+template <typename AT, typename OT, int ACT>
 KERN_DEVICE void tile_body(const AT* A, const __nv_bfloat16* W, OT* C, int m0, int m_end, int n0, int N, int K, int lda,
-                           int ldc, long long wsn, long long wsk) {
+                           int ldc, long long wsn, long long wsk, float limit = 0.f) {
+  constexpr bool SWIGLU = ACT >= 0;
   __shared__ float as[LK][LB + 4], ws[LK][LB + 4], us[SWIGLU ? LK : 1][LB + 4];
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {}, acu[SWIGLU ? 4 : 1][4] = {};
@@ -61,7 +74,7 @@ KERN_DEVICE void tile_body(const AT* A, const __nv_bfloat16* W, OT* C, int m0, i
       const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
       if (m >= m_end || n >= N) continue;
       float v = acc[i][j];
-      if constexpr (SWIGLU) v = v / (1.f + expf(-v)) * acu[i][j];
+      if constexpr (SWIGLU) v = glu_exact<ACT>(v, acu[i][j], limit);
       stf(C + (size_t)m * ldc + n, v);
     }
 }
@@ -82,27 +95,27 @@ KERN_DEVICE void gate_mul_body(const T* x, const T* gate, T* out, int tokens, in
 }  // namespace
 
 // grid [ceil(N / 64), ceil(M / 64), batch], block 256. Batch z: A + z a_z, W + z w_z, C + z c_z (elements).
-#define LINEAR_ENTRY(NAME, AT, OT, SW)                                                                                      \
+#define LINEAR_ENTRY(NAME, AT, OT, ACT)                                                                                     \
   extern "C" __global__ void __launch_bounds__(256)                                                                         \
       NAME(const AT* A, const __nv_bfloat16* W, OT* C, int M, int N, int K, int lda, int ldc, long long wsn, long long wsk, \
-           long long a_z, long long w_z, long long c_z, int* err) {                                                         \
+           long long a_z, long long w_z, long long c_z, int* err, float limit) {                                            \
     pdl_wait();                                                                                                             \
     if (M > (int)gridDim.y * LB && threadIdx.x == 0) set_error(err, ERR_BOUNDS);   /* rows the grid does not cover */       \
     const int z = blockIdx.z;                                                                                               \
-    tile_body<AT, OT, SW>(A + z * a_z, W + z * w_z, C + z * c_z, blockIdx.y * LB, M, blockIdx.x * LB, N, K, lda, ldc, wsn,  \
-                          wsk);                                                                                             \
+    tile_body<AT, OT, ACT>(A + z * a_z, W + z * w_z, C + z * c_z, blockIdx.y * LB, M, blockIdx.x * LB, N, K, lda, ldc, wsn, \
+                           wsk, limit);                                                                                     \
   }
 // grid [ceil(N / 64), blocks], block 256; `tiles` int4 {expert, first row, rows, -}.
-#define LINEAR_GROUPED_ENTRY(NAME, T, SW)                                                                                   \
+#define LINEAR_GROUPED_ENTRY(NAME, T, ACT)                                                                                  \
   extern "C" __global__ void __launch_bounds__(256)                                                                         \
       NAME(const T* A, const __nv_bfloat16* W, T* C, const int* tiles, const int* tile_count, int rows, int N, int K,       \
-           long long w_z, int* err) {                                                                                       \
+           long long w_z, int* err, float limit) {                                                                          \
     pdl_wait();                                                                                                             \
     const int n = *tile_count;                                                                                              \
     for (int i = blockIdx.y; i < n; i += gridDim.y) {                                                                       \
       const int4 e = reinterpret_cast<const int4*>(tiles)[i];                                                               \
       if (e.y + e.z > rows || e.z > LB) { if (threadIdx.x == 0) set_error(err, ERR_BOUNDS); continue; }                     \
-      tile_body<T, T, SW>(A, W + e.x * w_z, C, e.y, e.y + e.z, blockIdx.x * LB, N, K, K, N, K, 1);                          \
+      tile_body<T, T, ACT>(A, W + e.x * w_z, C, e.y, e.y + e.z, blockIdx.x * LB, N, K, K, N, K, 1, limit);                  \
     }                                                                                                                       \
   }
 #define LINEAR_MISC(T, SFX)                                                                                                 \
@@ -124,15 +137,23 @@ KERN_DEVICE void gate_mul_body(const T* x, const T* gate, T* out, int tokens, in
     else gate_mul_body<T, 1>(x, gate, out, tokens, d, x_stride, g_stride, o_stride);                                        \
   }
 
-LINEAR_ENTRY(kern_linear_bf16, __nv_bfloat16, __nv_bfloat16, false)
-LINEAR_ENTRY(kern_linear_bf16_f32, __nv_bfloat16, float, false)
-LINEAR_ENTRY(kern_linear_bf16_swiglu, __nv_bfloat16, __nv_bfloat16, true)
-LINEAR_ENTRY(kern_linear_f32, float, float, false)
-LINEAR_ENTRY(kern_linear_f32_swiglu, float, float, true)
-LINEAR_GROUPED_ENTRY(kern_linear_grouped_bf16, __nv_bfloat16, false)
-LINEAR_GROUPED_ENTRY(kern_linear_grouped_bf16_swiglu, __nv_bfloat16, true)
-LINEAR_GROUPED_ENTRY(kern_linear_grouped_f32, float, false)
-LINEAR_GROUPED_ENTRY(kern_linear_grouped_f32_swiglu, float, true)
+LINEAR_ENTRY(kern_linear_bf16, __nv_bfloat16, __nv_bfloat16, -1)
+LINEAR_ENTRY(kern_linear_bf16_f32, __nv_bfloat16, float, -1)
+LINEAR_ENTRY(kern_linear_f32, float, float, -1)
+LINEAR_GROUPED_ENTRY(kern_linear_grouped_bf16, __nv_bfloat16, -1)
+LINEAR_GROUPED_ENTRY(kern_linear_grouped_f32, float, -1)
+#define LINEAR_GLU(SFX, ACT)                                                            \
+  LINEAR_ENTRY(kern_linear_bf16_##SFX, __nv_bfloat16, __nv_bfloat16, ACT)               \
+  LINEAR_ENTRY(kern_linear_f32_##SFX, float, float, ACT)
+LINEAR_GLU(swiglu, kSwiglu)
+LINEAR_GLU(geglu, kGeglu)
+LINEAR_GLU(clamped, kClampedGlu)
+LINEAR_GROUPED_ENTRY(kern_linear_grouped_bf16_swiglu, __nv_bfloat16, kSwiglu)
+LINEAR_GROUPED_ENTRY(kern_linear_grouped_f32_swiglu, float, kSwiglu)
+LINEAR_GROUPED_ENTRY(kern_linear_grouped_bf16_geglu, __nv_bfloat16, kGeglu)
+LINEAR_GROUPED_ENTRY(kern_linear_grouped_f32_geglu, float, kGeglu)
+LINEAR_GROUPED_ENTRY(kern_linear_grouped_bf16_clamped, __nv_bfloat16, kClampedGlu)
+LINEAR_GROUPED_ENTRY(kern_linear_grouped_f32_clamped, float, kClampedGlu)
 LINEAR_MISC(__nv_bfloat16, bf16)
 LINEAR_MISC(float, f32)
 
@@ -152,4 +173,11 @@ extern "C" __global__ void __launch_bounds__(256)
     const int c = blockIdx.x * 32 + j, r = blockIdx.y * 32 + tx;
     if (r < R && c < C) dst[base + (size_t)c * R + r] = tile[tx][j];
   }
+}
+
+// dst[r, 0 .. C) of rows `stride` elements apart. grid [rows], block 256.
+extern "C" __global__ void __launch_bounds__(256)
+    kern_copy_cols_bf16(const __nv_bfloat16* src, __nv_bfloat16* dst, int C, int stride) {
+  pdl_wait();
+  for (int c = threadIdx.x; c < C; c += 256) dst[(size_t)blockIdx.x * stride + c] = src[(size_t)blockIdx.x * C + c];
 }

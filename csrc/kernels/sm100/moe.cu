@@ -3,6 +3,7 @@
 //   kern_moe_route_f32      router scores -> top-k expert ids and weights per token (sigmoid or softmax scoring,
 //                           optional selection bias, renormalise, scale)
 //   kern_moe_route_logits   the same by the logits plus a bias: top-k largest, softmax over the chosen
+//   kern_moe_route_groups   sigmoid scores inside the best groups of neighbouring experts
 //   kern_moe_plan           counts per expert -> row offsets, the permuted row of every (token, choice), and the
 //                           M-tile table the grouped GEMM walks; experts outside [e_lo, e_hi) belong to another rank
 //   kern_moe_gather_bf16    x_perm[perm[t, j]] = x[t]
@@ -130,6 +131,69 @@ extern "C" __global__ void __launch_bounds__(128)
   if (lane < k) {
     topk_ids[(size_t)t * k + lane] = my_id;
     topk_w[(size_t)t * k + lane] = e / sum;
+  }
+}
+
+// Routing inside groups: s = sigmoid(logits); `groups` equal groups of neighbours, a group's score the sum of its two largest
+// (its one, in groups of one); the k largest of the best `keep` groups are chosen (ties: the lower group, the lower id) and
+// weigh s, divided by their sum when `renorm`. One warp per token; E <= 1024, k <= 32, at most 64 groups.
+extern "C" __global__ void __launch_bounds__(128)
+    kern_moe_route_groups(const float* logits, int* topk_ids, float* topk_w, int tokens, int experts, int k, int groups, int keep,
+                          int renorm, int ld) {
+  extern __shared__ float route_sm[];      // [4][experts] scores, then [4][groups] group scores
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * 4 + warp;
+  if (t >= tokens) return;
+  float* sc = route_sm + warp * experts;
+  float* gs = route_sm + 4 * experts + warp * groups;
+  const float* row = logits + (size_t)t * ld;
+  for (int e = lane; e < experts; e += 32) {
+    const float z = row[e], x = exp2f(-fabsf(z) * 1.4426950408889634f);
+    sc[e] = z >= 0.f ? 1.f / (1.f + x) : x / (1.f + x);
+  }
+  __syncwarp();
+  const int per = experts / groups;
+  for (int g = lane; g < groups; g += 32) {
+    float a = -INFINITY, b = -INFINITY;
+    for (int e = g * per; e < (g + 1) * per; ++e) {
+      const float v = sc[e];
+      if (v > a) { b = a; a = v; } else if (v > b) b = v;
+    }
+    gs[g] = per > 1 ? a + b : a;
+  }
+  __syncwarp();
+  // a group stays when fewer than `keep` groups come before it
+  unsigned long long kept = 0;
+  for (int g = lane; g < groups; g += 32) {
+    int before = 0;
+    for (int o = 0; o < groups; ++o) before += gs[o] > gs[g] || (gs[o] == gs[g] && o < g);
+    if (before < keep) kept |= 1ull << g;
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) kept |= __shfl_xor_sync(0xffffffffu, kept, o);
+  float my_w = 0.f, sum = 0.f;
+  int my_id = 0;
+  for (int j = 0; j < k; ++j) {
+    float best = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int e = lane; e < experts; e += 32)
+      if ((kept >> (e / per) & 1) && sc[e] > best) { best = sc[e]; bi = e; }
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+    }
+    if (bi >= experts) { bi = 0; best = 0.f; }      // no score is a number: still a valid row
+    __syncwarp();
+    if (lane == 0) sc[bi] = -INFINITY;
+    __syncwarp();
+    sum += best;
+    if (lane == j) { my_w = best; my_id = bi; }
+  }
+  if (lane < k) {
+    topk_ids[(size_t)t * k + lane] = my_id;
+    topk_w[(size_t)t * k + lane] = renorm ? my_w / (sum + 1e-20f) : my_w;
   }
 }
 
@@ -266,6 +330,18 @@ KERN_MOE_GEMM_ENTRY(kern_moe_gemm_bf16_n64, 64, 0)
 KERN_MOE_GEMM_ENTRY(kern_moe_gemm_bf16_swiglu_n256, 256, 3)
 KERN_MOE_GEMM_ENTRY(kern_moe_gemm_bf16_swiglu_n128, 128, 3)
 KERN_MOE_GEMM_ENTRY(kern_moe_gemm_bf16_swiglu_n64, 64, 3)
+KERN_MOE_GEMM_ENTRY(kern_moe_gemm_bf16_geglu_n128, 128, 6)
+KERN_MOE_GEMM_ENTRY(kern_moe_gemm_bf16_geglu_n64, 64, 6)
+
+#define KERN_MOE_GEMM_CLAMPED(name, BN)                                                                            \
+  extern "C" __global__ void __launch_bounds__(192, 1)                                                            \
+      name(const __grid_constant__ CUtensorMap tma_a, const __grid_constant__ CUtensorMap tma_b, void* C,          \
+           const int* tiles, const int* tile_count, int M, int N, int K, int ldc, int* err, float limit) {         \
+    kern::gemm_body<BN, 7, true>(&tma_a, &tma_b, C, nullptr, M, N, K, ldc, err, tiles, tile_count,                 \
+                                 kern::ScatterArgs(), nullptr, nullptr, kern::AgArgs(), kern::EpArgs(), 1, limit); \
+  }
+KERN_MOE_GEMM_CLAMPED(kern_moe_gemm_bf16_clamped_n128, 128)
+KERN_MOE_GEMM_CLAMPED(kern_moe_gemm_bf16_clamped_n64, 64)
 
 // ---- expert parallel over sharded tokens: dispatch by pull, combine by push -------------------------------------------
 // Tokens live on their home rank (rows_per_rank each, token t = home * rows_per_rank + local row); every rank knows

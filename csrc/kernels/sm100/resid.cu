@@ -1,0 +1,142 @@
+// build: precise
+// The residual of a decoder that norms a sublayer's result before adding it as well as the next sublayer's input:
+//     x <- x + rms(y) w_post;   xn = rms(x) w_next
+// x is f32 (one row per token), y the sublayer's result: a row of a plain buffer, or the weighted sum of a token's k
+// expert rows, summed here. Without `w_post` y is added as it is.
+// kern_resid_embed  token row into x, and the first sublayer's normed input
+// kern_resid_mix    as above; with `hidden` the sum goes there instead and nothing is normed (the last sublayer)
+// Residual, sums and norms are f32; activations are T (bf16, or f32 in the 32-bit form of a model).
+#include "act.cuh"
+
+using namespace kern;
+
+namespace {
+
+KERN_DEVICE float block_sum(float v) {      // block of 256
+  __shared__ float part[8];
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) s += part[i];
+  __syncthreads();
+  return s;
+}
+
+KERN_DEVICE float inv_rms(float ss, int width, float eps) { return 1.f / sqrtf(block_sum(ss) / (float)width + eps); }
+
+// u (shared, each thread reads what it wrote) -> xn = u inv w
+template <typename T, int V>
+KERN_DEVICE void norm_out(const float* u, float inv, const __nv_bfloat16* w, T* xn, int width) {
+  for (int i = threadIdx.x * V; i < width; i += 256 * V) {
+    const Vec<V> a = ldv<V>(u + i), b = ldv<V>(w + i);
+    Vec<V> o;
+#pragma unroll
+    for (int e = 0; e < V; ++e) o.v[e] = a.v[e] * inv * b.v[e];
+    stv<V>(xn + i, o);
+  }
+}
+
+template <typename T, int V>
+KERN_DEVICE void embed_body(const long long* ids, const __nv_bfloat16* table, const __nv_bfloat16* w_norm, float* x, T* xn,
+                            int width, int vocab, float eps, int* err) {
+  extern __shared__ __align__(16) float resid_sm[];
+  const int t = blockIdx.x;
+  long long id = ids[t];
+  if (id < 0 || id >= vocab) {
+    if (threadIdx.x == 0) set_error(err, ERR_BOUNDS);
+    id = 0;
+  }
+  const __nv_bfloat16* a = table + (size_t)id * width;
+  const bool ok = KERN_CHECK(a, (size_t)width * 2, SITE_EMBED_ROW);
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < width; i += 256 * V) {
+    Vec<V> v = {};
+    if (ok) v = ldv<V>(a + i);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += v.v[j] * v.v[j];
+    stv<V>(x + (size_t)t * width + i, v);
+    stv<V>(resid_sm + i, v);
+  }
+  norm_out<T, V>(resid_sm, inv_rms(ss, width, eps), w_norm, xn + (size_t)t * width, width);
+}
+
+template <typename T, int V>
+KERN_DEVICE void mix_body(float* x, const T* y, const int* perm, const float* topw, const __nv_bfloat16* w_post,
+                          const __nv_bfloat16* w_next, T* xn, float* hidden, int width, int k, float eps) {
+  extern __shared__ __align__(16) float resid_sm[];
+  __shared__ float tw[32];
+  __shared__ int tr[32];
+  const int t = blockIdx.x;
+  if (perm) {
+    if (threadIdx.x < k) {
+      const int r = perm[(size_t)t * k + threadIdx.x];
+      const bool ok = r >= 0 && KERN_CHECK(y + (size_t)r * width, (size_t)width * sizeof(T), SITE_MOE_COMBINE);
+      tr[threadIdx.x] = ok ? r : -1;
+      tw[threadIdx.x] = topw[(size_t)t * k + threadIdx.x];
+    }
+    __syncthreads();
+  }
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < width; i += 256 * V) {
+    Vec<V> v = {};
+    if (perm) {
+      for (int j = 0; j < k; ++j) {
+        if (tr[j] < 0) continue;
+        const Vec<V> r = ldv<V>(y + (size_t)tr[j] * width + i);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v.v[e] += tw[j] * r.v[e];
+      }
+    } else {
+      v = ldv<V>(y + (size_t)t * width + i);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss += v.v[e] * v.v[e];
+    stv<V>(resid_sm + i, v);
+  }
+  const float inv = w_post ? inv_rms(ss, width, eps) : 1.f;
+  float* xt = x + (size_t)t * width;
+  ss = 0.f;
+  for (int i = threadIdx.x * V; i < width; i += 256 * V) {
+    const Vec<V> v = ldv<V>(resid_sm + i);
+    Vec<V> s = ldv<V>(xt + i), w;
+    if (w_post) w = ldv<V>(w_post + i);
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      s.v[e] += w_post ? v.v[e] * inv * w.v[e] : v.v[e];
+      ss += s.v[e] * s.v[e];
+    }
+    if (hidden) {
+      stv<V>(hidden + (size_t)t * width + i, s);
+    } else {
+      stv<V>(xt + i, s);
+      stv<V>(resid_sm + i, s);
+    }
+  }
+  if (!hidden) norm_out<T, V>(resid_sm, inv_rms(ss, width, eps), w_next, xn + (size_t)t * width, width);
+}
+
+}  // namespace
+
+// grid = rows, block 256, `width` floats of shared memory
+#define RESID_ENTRIES(T, SFX)                                                                                             \
+  extern "C" __global__ void __launch_bounds__(256)                                                                       \
+      kern_resid_embed_##SFX(const long long* ids, const __nv_bfloat16* table, const __nv_bfloat16* w_norm, float* x,     \
+                             T* xn, int width, int vocab, float eps, int* err) {                                          \
+    pdl_wait();                                                                                                           \
+    if (width % 4 == 0) embed_body<T, 4>(ids, table, w_norm, x, xn, width, vocab, eps, err);                              \
+    else embed_body<T, 1>(ids, table, w_norm, x, xn, width, vocab, eps, err);                                             \
+    pdl_launch_dependents();                                                                                              \
+  }                                                                                                                       \
+  extern "C" __global__ void __launch_bounds__(256)                                                                       \
+      kern_resid_mix_##SFX(float* x, const T* y, const int* perm, const float* topw, const __nv_bfloat16* w_post,         \
+                           const __nv_bfloat16* w_next, T* xn, float* hidden, int width, int k, float eps) {              \
+    pdl_wait();                                                                                                           \
+    if (width % 4 == 0) mix_body<T, 4>(x, y, perm, topw, w_post, w_next, xn, hidden, width, k, eps);                      \
+    else mix_body<T, 1>(x, y, perm, topw, w_post, w_next, xn, hidden, width, k, eps);                                     \
+    pdl_launch_dependents();                                                                                              \
+  }
+
+RESID_ENTRIES(__nv_bfloat16, bf16)
+RESID_ENTRIES(float, f32)

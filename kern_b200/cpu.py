@@ -65,12 +65,15 @@ def k_fused_add_rms_norm(g, x, res, w, y, rows, n, eps, plus_one):
     k_rms_norm(g, res, w, y, rows, n, n, n, eps, plus_one)
 
 
+GLU_GATES = {"swiglu": torch.nn.functional.silu, "geglu": lambda g: torch.nn.functional.gelu(g, approximate="tanh")}
+
+
 def _gemm(epi):
     def run(g, a, w, c, r, m, n, k, ldc, err):
         av = torch.as_strided(a, (m, k), (a_stride(a, k), 1))
         acc = _f(av) @ _f(w[: n * k].view(n, k)).t()
-        if epi == "swiglu":
-            acc = torch.nn.functional.silu(acc[:, : n // 2]) * acc[:, n // 2:]
+        if epi in GLU_GATES:
+            acc = GLU_GATES[epi](acc[:, : n // 2]) * acc[:, n // 2:]
         cv = torch.as_strided(c, (m, acc.shape[1]), (ldc, 1))
         if epi == "acc":
             acc = acc + _f(torch.as_strided(r, (m, n), (ldc, 1)))
@@ -82,8 +85,8 @@ def _gemv(epi):
     def run(g, a, w, c, r, m, n, k, lda, ldc, err):
         av = torch.as_strided(a, (m, k), (lda, 1), a.storage_offset())
         acc = _f(av) @ _f(w[: n * k].view(n, k)).t()
-        if epi == "swiglu":
-            acc = torch.nn.functional.silu(acc[:, : n // 2]) * acc[:, n // 2:]
+        if epi in GLU_GATES:
+            acc = GLU_GATES[epi](acc[:, : n // 2]) * acc[:, n // 2:]
         cv = torch.as_strided(c, (m, acc.shape[1]), (ldc, 1), c.storage_offset())
         if epi == "acc":
             acc = acc + _f(torch.as_strided(r, (m, n), (ldc, 1), r.storage_offset()))
@@ -176,6 +179,18 @@ def _attention(prefill):
             o = torch.einsum("hrl,lhd->rhd", torch.softmax(sc, -1), vv.repeat_interleave(grp, 1))
             torch.as_strided(out, (R, hq * d), (out_stride, 1), out.storage_offset() + r0 * out_stride).copy_(o.reshape(R, hq * d).to(out.dtype))
     return run
+
+
+def k_attn_plan(g, cu, seqs, tpb_p, tpb_d, small_rows, work_p, count_p, max_p, work_d, count_d, max_d):
+    p, d = [], []
+    for s in range(seqs):
+        r = int(cu[s + 1] - cu[s])
+        tpb, to = (tpb_d, d) if r <= small_rows else (tpb_p, p)
+        to += [(s, b) for b in range(-(-r // tpb))]
+    for pairs, work, count, most in ((p, work_p, count_p, max_p), (d, work_d, count_d, max_d)):
+        n = min(len(pairs), most)
+        count[0] = n
+        work[: 2 * n] = torch.tensor(pairs[:n], dtype=work.dtype).reshape(-1)
 
 
 def k_noop(g, *a):
@@ -381,7 +396,7 @@ CPU_KERNELS = {
     "kern_rms_norm_bf16": k_rms_norm, "kern_rms_norm_wide_bf16": k_rms_norm,
     "kern_fused_add_rms_norm_bf16": k_fused_add_rms_norm,
     "kern_rope_kv_append_bf16": k_rope_append, "kern_rope_table_f32": k_rope_table,
-    "kern_attn_plan": k_noop, "kern_attn_merge_splits": k_noop,
+    "kern_attn_plan": k_attn_plan, "kern_attn_merge_splits": k_noop,
     "kern_last_row": k_last_row, "kern_argmax_partial_bf16": k_argmax_partial, "kern_argmax_partial_f32": k_argmax_partial,
     "kern_argmax_final_i64": k_argmax_final, "kern_sample_bf16": k_sample, "kern_sample_f32": k_sample,
     "kern_silu_mul_bf16": k_silu_mul, "kern_copy_rows": k_copy_rows, "kern_sigmoid_mul_bf16": k_sigmoid_mul,
@@ -394,7 +409,7 @@ CPU_KERNELS = {
     "kern_fill_f32": k_fill, "kern_fill_i32": k_fill, "kern_fill_i64": k_fill, "kern_fill_u8": k_fill,
 }
 for _bn in (256, 128, 64, 32):
-    for _epi, _sfx in (("store", ""), ("acc", "_acc"), ("f32", "_f32"), ("swiglu", "_swiglu")):
+    for _epi, _sfx in (("store", ""), ("acc", "_acc"), ("f32", "_f32"), ("swiglu", "_swiglu"), ("geglu", "_geglu")):
         CPU_KERNELS[f"kern_gemm_bf16_tn{_sfx}_n{_bn}"] = _gemm(_epi)
         for _mt in (1, 2, 4, 8):
             CPU_KERNELS[f"kern_gemv_bf16_tn{_sfx}_m{_mt}"] = _gemv(_epi)

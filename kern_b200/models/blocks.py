@@ -1,7 +1,8 @@
 """Op builders of the decoder blocks that take any size and either activation type (bf16, or f32 in a model's 32-bit
-form): matrix products, hyper-connections, the Mamba-2 mixer, latent attention without positions, routed experts. Where a
-bf16 size fits the tensor-core kernels the op is the one `common.py` builds; the rest runs the generic kernels of
-linear.cu / ssd.cu / latent.cu. Weights are bf16 in both forms.
+form): matrix products, hyper-connections, the residual with norms on both sides, the Mamba-2 mixer, linear attention with a
+decay per key channel, latent attention without positions, attention in a sliding window, routed experts. Where a bf16 size
+fits the tensor-core kernels the op is the one `common.py` builds or the tensor-core form of the mechanism; the rest runs
+generic kernels. Weights are bf16 in both forms.
 """
 from __future__ import annotations
 
@@ -30,26 +31,30 @@ def tiles_fit(*extents: int) -> bool:
 
 
 # ---- matrix products ----------------------------------------------------------------------------------
-def _generic(sfx: str, iface, n: int, k: int, lda: int, ldc: int, rows_var: str, batch: int = 1, w=None, strides=(0, 0, 0)) -> dict:
+def _generic(sfx: str, iface, n: int, k: int, lda: int, ldc: int, rows_var: str, batch: int = 1, w=None, strides=(0, 0, 0),
+             limit: float = 0.0) -> dict:
     """`w`: (row stride, column stride) of the weights in elements; `strides`: what a step of the batch adds to A, W, C."""
     wsn, wsk = w or (k, 1)
     return _launch("linear", f"kern_linear_{sfx}", [256, 1, 1], [-(-n // 64), {"ceil_div": [rows_var, 64]}, batch],
-                   iface[:3] + ["i32"] * 5 + ["i64"] * 5 + ["out buffer<i32>"],
-                   [P(0), P(1), P(2), P(3), I(n), I(k), I(lda), I(ldc), L(wsn), L(wsk), *map(L, strides), P(4)])
+                   iface[:3] + ["i32"] * 5 + ["i64"] * 5 + ["out buffer<i32>", "f32"],
+                   [P(0), P(1), P(2), P(3), I(n), I(k), I(lda), I(ldc), L(wsn), L(wsk), *map(L, strides), P(4), {"f32": limit}])
+
+
+GLUS = ("swiglu", "geglu", "clamped")      # gated units over [gate rows ; up rows]; `clamped` takes a limit
 
 
 def linear_op(n: int, k: int, *, act: str = "bf16", epilogue: str = "store", rows_var: str = "tokens", rows_max: int,
-              lda: int | None = None, ldc: int | None = None) -> dict:
-    """C[rows, n] = A[rows, k] . W[n, k]^T. Interface [a, w, c, rows, err]; epilogue store | f32 | swiglu as in `gemm_op`."""
+              lda: int | None = None, ldc: int | None = None, limit: float = 0.0) -> dict:
+    """C[rows, n] = A[rows, k] . W[n, k]^T. Interface [a, w, c, rows, err]; epilogue store | f32 | a gated unit as in `gemm_op`."""
     lda = k if lda is None else lda
-    cols = n // 2 if epilogue == "swiglu" else n
+    cols = n // 2 if epilogue in GLUS else n
     ldc = cols if ldc is None else ldc
-    if act == "bf16" and tiles_fit(cols, k, lda, ldc):
+    if act == "bf16" and epilogue != "clamped" and tiles_fit(cols, k, lda, ldc):
         return C.gemm_op(n, k, epilogue=epilogue, rows_var=rows_var, rows_max=rows_max, lda=lda, ldc=ldc)
     out = "f32" if epilogue == "f32" else act
-    sfx = act + {"store": "", "f32": "_f32" if act == "bf16" else "", "swiglu": "_swiglu"}[epilogue]
+    sfx = act + {"store": "", "f32": "_f32" if act == "bf16" else ""}.get(epilogue, "_" + epilogue)
     iface = [f"in buffer<{act}>", "in buffer<bf16>", f"out buffer<{out}>", "i32", "out buffer<i32>"]
-    return _op(iface, _generic(sfx, iface, cols, k, lda, ldc, rows_var))
+    return _op(iface, _generic(sfx, iface, cols, k, lda, ldc, rows_var, limit=limit))
 
 
 def head_tiles(n: int, k: int, lda: int, ldc: int, act: str) -> bool:
@@ -92,6 +97,12 @@ def transpose_heads_op(heads: int, rows: int, cols: int) -> dict:
     iface = ["in buffer<bf16>", "out buffer<bf16>"]
     return _op(iface, _launch("linear", "kern_transpose_heads_bf16", [256, 1, 1], [-(-cols // 32), -(-rows // 32), heads],
                               iface + ["i32", "i32"], [P(0), P(1), I(rows), I(cols)]))
+
+
+def copy_cols_op(rows: int, cols: int, stride: int) -> dict:
+    """A [rows, cols] matrix into columns of one whose rows are `stride` wide. Interface [src, dst]."""
+    iface = ["in buffer<bf16>", "inout buffer<bf16>"]
+    return _op(iface, _launch("linear", "kern_copy_cols_bf16", [256, 1, 1], [rows, 1, 1], iface + ["i32", "i32"], [P(0), P(1), I(cols), I(stride)]))
 
 
 # ---- hyper-connections ----------------------------------------------------------------------------------
@@ -238,6 +249,215 @@ def latent_attn_op(heads: int, rank: int, scale: float, page_size: int, table_wi
                                {"f32": scale}, P(5)], shared_mem=(4 * rank + 8) * 4))
 
 
+# ---- a residual with norms on both sides of a sublayer -----------------------------------------------------
+def resid_embed_op(width: int, vocab: int, eps: float, act: str = "bf16") -> dict:
+    """Token row into the f32 residual, and the first sublayer's normed input. Interface [ids, table, next norm w, x, xn, err]."""
+    iface = ["in buffer<i64>", "in buffer<bf16>", "in buffer<bf16>", "out buffer<f32>", f"out buffer<{act}>", "out buffer<i32>"]
+    return _op(iface, _launch("resid", f"kern_resid_embed_{act}", [256, 1, 1], ["tokens", 1, 1], iface[:5] + ["i32", "i32", "f32", "out buffer<i32>"],
+                              [*map(P, range(5)), I(width), I(vocab), {"f32": eps}, P(5)], shared_mem=width * 4))
+
+
+def resid_mix_op(width: int, eps: float, act: str = "bf16", routed: int = 0, last: bool = False) -> dict:
+    """x += rms(y) w_post, and the next sublayer's normed input. Interface [x, y, w_post, w_next, xn], with `routed` (experts per
+    token) also [perm, weights] at the end: y then holds expert-sorted rows. `last`: the sum goes to `hidden` and nothing is
+    normed; interface [x, y, w_post, hidden]."""
+    iface = ["in buffer<f32>" if last else "inout buffer<f32>", f"in buffer<{act}>", "in buffer<bf16>"]
+    iface += ["out buffer<f32>"] if last else ["in buffer<bf16>", f"out buffer<{act}>"]
+    n = len(iface)
+    iface += ["in buffer<i32>", "in buffer<f32>"] if routed else []
+    route = [(iface[n], P(n)), (iface[n + 1], P(n + 1))] if routed else [NULL, NULL]
+    tail = [NULL, NULL, (iface[3], P(3))] if last else [(iface[3], P(3)), (iface[4], P(4)), NULL]
+    parts = [(iface[0], P(0)), (iface[1], P(1)), *route, (iface[2], P(2)), *tail]
+    return _op(iface, _launch("resid", f"kern_resid_mix_{act}", [256, 1, 1], ["tokens", 1, 1], [t for t, _ in parts] + ["i32", "i32", "f32"],
+                              [a for _, a in parts] + [I(width), I(routed), {"f32": eps}], shared_mem=width * 4))
+
+
+# ---- linear attention with a decay per key channel -----------------------------------------------------------
+LIN_CHUNK_MIN = 8       # rows of a call from which a sequence is computed in chunks
+LIN_DIMS = 256          # most key channels of a head
+
+
+def lin_line_bytes(heads: int, dk: int, dv: int, shifted: int = 0) -> tuple[int, int]:
+    """(bytes of one per-sequence line, offset of S in it); `shifted`: columns of the kept previous row."""
+    s_off = (shifted * 4 + 255) // 256 * 256
+    return (s_off + heads * dk * dv * 4 + 255) // 256 * 256, s_off
+
+
+def token_shift_op(width: int, targets: int, line_bytes: int, ragged: bool, act: str = "bf16") -> dict:
+    """out[t, m] = h[t] + (h[t - 1] - h[t]) mu[m] for every target m; the row before a call's first is kept at the start of the
+    state line (f32). Interface [h, mu, out, state, lines, (cu_seqlens,) seqs]."""
+    iface = [f"in buffer<{act}>", "in buffer<bf16>", f"out buffer<{act}>", "inout state", "in buffer<i32>"] + (["in buffer<i32>"] if ragged else []) + ["i32"]
+    cu_t, cu_a = (iface[5], P(5)) if ragged else NULL
+    n = P(len(iface) - 1)
+    cols = -(-width // 1024)
+    shift = _launch("lin_attn", f"kern_token_shift_{act}", [256, 1, 1], ["tokens", cols, 1],
+                    [*iface[:3], "in state" if ragged else "inout state", iface[4], cu_t, "i32", "i32", "i32", "i64"],
+                    [*map(P, range(5)), cu_a, n, I(width), I(targets), L(line_bytes)])
+    if not ragged:
+        return _op(iface, shift)
+    keep = _launch("lin_attn", f"kern_shift_state_{act}", [256, 1, 1], ["seqs", cols, 1], [iface[0], "inout state", iface[4], cu_t, "i32", "i32", "i64"],
+                   [P(0), P(3), P(4), P(5), n, I(width), L(line_bytes)])
+    return _op(iface, shift, keep)
+
+
+def decay_op(n: int, rank: int, lda: int, kind: str, tau: float = 1.0, act: str = "f32") -> dict:
+    """alpha [tokens, n] (f32) from a low-rank row a [tokens, rank]: `root` sigmoid(W a + b)^(1 / tau), `double_exp`
+    exp(-exp(W tanh(a) + b)). Interface [a, w, bias, alpha, tokens]."""
+    iface = [f"in buffer<{act}>", "in buffer<bf16>", "in buffer<bf16>", "out buffer<f32>", "i32"]
+    return _op(iface, _launch("lin_attn", f"kern_decay_{act}", [256, 1, 1], [-(-n // 64), {"ceil_div": ["tokens", 64]}, 1], iface + ["i32"] * 4 + ["f32"],
+                              [*map(P, range(5)), I(n), I(rank), I(lda), I({"root": 0, "double_exp": 1}[kind]), {"f32": 1.0 / tau}]))
+
+
+def lin_fused(dv: int) -> bool:
+    """Whether the step of a one-row call also norms and gates (a block then owns a head's whole row)."""
+    return dv <= 128
+
+
+def lin_rule_op(heads: int, dk: int, dv: int, stride: int, line_bytes: int, s_off: int, ragged: bool, act: str = "bf16", *, bonus: bool,
+                q_scale: float = 1.0, fused: bool = False, norm_shared: bool = True, out_stride: int = 0, out_scale: float = 1.0,
+                eps: float = 0.0) -> dict:
+    """S = diag(alpha) S + k v^T and its read by q. Interface [q, k, v, alpha, (u,) out, state, lines, (cu_seqlens,) seqs]; `fused`
+    (out is then the normed, weighed and gated activation, else f32 rows) adds [gate, norm w] before the last. q, k, v and gate
+    share their row stride."""
+    if dk > LIN_DIMS:
+        raise ValueError(f"{dk} key channels per head (at most {LIN_DIMS})")
+    out_t = f"out buffer<{act if fused else 'f32'}>"
+    parts = [("q", f"in buffer<{act}>"), ("k", f"in buffer<{act}>"), ("v", f"in buffer<{act}>"), ("alpha", "in buffer<f32>")]
+    parts += [("u", "in buffer<bf16>")] if bonus else []
+    parts += [("out", out_t), ("state", "inout state"), ("lines", "in buffer<i32>")]
+    parts += [("cu", "in buffer<i32>")] if ragged else []
+    parts += [("gate", f"in buffer<{act}>"), ("norm", "in buffer<bf16>")] if fused else []
+    parts += [("seqs", "i32")]
+    at = {n: (t, P(i)) for i, (n, t) in enumerate(parts)}
+    pick = lambda *names: [at.get(n, NULL) for n in names]
+    rk = next(r for r in (4, 8, 16, 32) if dk <= 8 * r)
+    v = 1 if dv <= 32 else (2 if dv <= 64 else 4)
+    chunked = ragged and act == "bf16" and not fused
+    tb = 8 if ragged else 1
+    args = pick("q", "k", "v", "gate", "alpha", "u", "norm", "out", "state", "lines", "cu", "seqs")
+    rule = _launch("lin_attn", f"kern_lin_rule_{act}_r{rk}_v{v}", [256, 1, 1], [heads * -(-dv // (32 * v)), "seqs", 1],
+                   [t for t, _ in args] + ["i32"] * 6 + ["i64"] + ["i32"] * 4 + ["f32"] * 3,
+                   [a for _, a in args] + [I(heads), I(dk), I(dv), I(stride), I(0 if norm_shared else dv), I(out_stride), L(line_bytes), I(s_off), I(int(fused)),
+                                           I(tb), I(LIN_CHUNK_MIN - 1 if chunked else C.I32_MAX), {"f32": q_scale}, {"f32": out_scale}, {"f32": eps}],
+                   shared_mem=(3 * tb + 1) * dk * 4)
+    iface = [t for _, t in parts]
+    if not chunked:
+        return _op(iface, rule)
+    # a ragged call's long sequences in chunks on the tensor cores, its few-row ones (decode rows among prompts) row by row
+    np_ = next(n for n in (32, 64, 128, 256) if dk <= n)
+    prep = 5 * 16 * (np_ + 8) * 2 + 3 * 16 * 24 * 2 + np_ * 4
+    smem = 2 * prep + 2 * 16 * np_ * 8 + 3 * 16 * 72 * 2 + np_ * 4
+    args = pick("q", "k", "v", "alpha", "u", "out", "state", "lines", "cu", "seqs")
+    chunk = _launch("lin_attn_chunk", f"kern_lin_chunk_n{np_}", [256, 1, 1], [heads * -(-dv // 64), "seqs", 1],
+                    [t for t, _ in args] + ["i32"] * 4 + ["i64", "i32", "i32", "f32"],
+                    [a for _, a in args] + [I(heads), I(dk), I(dv), I(stride), L(line_bytes), I(s_off), I(LIN_CHUNK_MIN), {"f32": q_scale}], shared_mem=smem)
+    return _op(iface, chunk, rule)
+
+
+def lin_norm_gate_op(heads: int, dv: int, gate_stride: int, norm_shared: bool, out_stride: int, out_scale: float, eps: float, act: str = "bf16") -> dict:
+    """rms_norm per head of the f32 rows, times w (one per column, or shared by the heads), times silu(gate), times out_scale.
+    Interface [o, gate, w, out]."""
+    iface = ["in buffer<f32>", f"in buffer<{act}>", "in buffer<bf16>", f"out buffer<{act}>"]
+    return _op(iface, _launch("lin_attn", f"kern_lin_norm_gate_{act}", [256, 1, 1], ["tokens", -(-heads // 8), 1], iface + ["i32"] * 5 + ["f32", "f32"],
+                              [*map(P, range(4)), I(heads), I(dv), I(gate_stride), I(0 if norm_shared else dv), I(out_stride), {"f32": out_scale}, {"f32": eps}]))
+
+
+# ---- attention in a sliding window ---------------------------------------------------------------------------
+LOG2E = 1.4426950408889634
+
+
+def qk_prep_op(hq: int, hk: int, d: int, dv: int, rot: int, page_size: int, row_stride: int, max_pos: int, eps: float, act: str = "bf16",
+               halves: bool = False) -> dict:
+    """Norm of q and k per head, rotary positions on the first `rot` columns (pairs of neighbours, or `halves`), k and v into the
+    paged cache. Interface [qkv, state, positions, slots, cos, sin, q norm w, k norm w, err]."""
+    if rot % 2 or rot > d:
+        raise ValueError(f"rotary positions on {rot} of {d} columns")
+    iface = [f"inout buffer<{act}>", "inout state", "in buffer<i64>", "in buffer<i64>", "in buffer<f32>", "in buffer<f32>", "in buffer<bf16>",
+             "in buffer<bf16>", "out buffer<i32>"]
+    return _op(iface, _launch("attn_window", f"kern_qk_prep_{act}", [256, 1, 1], ["tokens", 1, 1], iface[:8] + ["i32"] * 9 + ["f32", "out buffer<i32>"],
+                              [*map(P, range(8)), I(hq), I(hk), I(d), I(dv), I(rot), I(int(halves)), I(page_size), I(row_stride), I(max_pos), {"f32": eps}, P(8)],
+                              shared_mem=8 * max(d, dv) * 4))
+
+
+def window_tiles(hq: int, hk: int, d: int, dv: int, page_size: int, act: str) -> bool:
+    """Whether windowed attention of this size runs on the tensor-core kernels."""
+    return act == "bf16" and d == dv and d in (64, 128, 256) and hq // hk <= 16 and (page_size % 64 == 0 or (page_size % 8 == 0 and 64 % page_size == 0))
+
+
+def window_attn_op(hq: int, hk: int, d: int, dv: int, window: int, scale: float, cap: float, page_size: int, table_width: int, q_stride: int,
+                   out_stride: int, out_scale: float, ragged: bool, act: str = "bf16", seqs_max: int = 0) -> dict:
+    """Attention over the last `window` positions, capped scores, a sink per query head; rows times out_scale into columns of
+    wider rows. Interface [q, state, out, block_table, lens, sink, err], then for ragged rows on the tensor cores (`window_tiles`)
+    [cu_seqlens, work_p, count_p, work_d, count_d] as `attn_plan_op` fills them (lens per sequence), else [row_seq] (lens per row)."""
+    if hq % hk:
+        raise ValueError(f"{hq} query heads over {hk} key heads")
+    iface = [f"in buffer<{act}>", "in state", f"out buffer<{act}>", "in buffer<i32>", "in buffer<i32>", "in buffer<bf16>", "out buffer<i32>"]
+    if not window_tiles(hq, hk, d, dv, page_size, act):
+        iface += ["in buffer<i32>"] if ragged else []
+        if max(d, dv) > 512:
+            raise ValueError(f"heads of {d} / {dv} columns (at most 512)")
+        w = next(n for n in (64, 128, 256, 512) if max(d, dv) <= n)
+        row_t, row_a = (iface[7], P(7)) if ragged else NULL
+        return _op(iface, _launch("attn_window", f"kern_window_attn_{act}_w{w}", [128, 1, 1], [hq, "tokens" if ragged else "seqs", 1],
+                                  [*iface[:5], row_t, iface[5]] + ["i32"] * 9 + ["f32"] * 3 + ["out buffer<i32>"],
+                                  [*map(P, range(5)), row_a, P(5), I(hq), I(hk), I(d), I(dv), I(q_stride), I(out_stride), I(table_width), I(page_size), I(window),
+                                   {"f32": scale}, {"f32": cap}, {"f32": out_scale}, P(6)], shared_mem=(4 * dv + 8) * 4))
+    g, kv = hq // hk, C._kv_map(d, page_size, 1)
+    win_t = ["out buffer<i32>", "in buffer<bf16>", "i32", "f32", "f32", "f32"]
+    win_a = [P(6), P(5), I(window), {"f32": 2 * LOG2E * scale / cap}, {"f32": cap * LOG2E}, {"f32": out_scale}]
+    lp = lambda ws, lists: ["bytes<128>", iface[0], iface[2]] + (["out buffer<f32>"] * 2 if ws else ["i64"] * 2) + ["in buffer<i32>"] * 2 \
+        + (["in buffer<i32>"] * 3 if lists else ["i64"] * 3) + ["i32"] * 8 + win_t
+    sizes = lambda splits: [I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(splits), I(C.I32_MAX)]
+    if not ragged:
+        ranges, hi = [], seqs_max
+        for splits in (1, 2, 4, 8):      # enough sequences that heads x sequences x splits cover the SMs; at least two tiles a split
+            if splits > 1 and splits * 128 > window + 64:
+                break
+            lo = max(1, -(-C.SMS // (hk * splits)))
+            if splits == 8 or 4 * splits * 64 > window + 64:
+                lo = 1
+            if lo <= hi:
+                ranges.append((splits, lo, hi))
+                hi = lo - 1
+        if hi >= 1:
+            s, lo, top = ranges.pop() if ranges else (1, 1, seqs_max)
+            ranges.append((s, 1, top))
+        launches, most = [], max(s for s, _, _ in ranges)
+        for splits, lo, hi in ranges:
+            when = {"var": "seqs", **({"min": lo} if lo > 1 else {}), **({"max": hi} if hi < seqs_max else {})}
+            kw = {"when": when} if len(when) > 1 else {}
+            ws = [{"scratch": "ws_o"}, {"scratch": "ws_ml"}] if splits > 1 else [L(0), L(0)]
+            launches.append(_launch("attn_window", f"kern_attn_window_decode_d{d}", [160, 1, 1], [hk, "seqs", splits], lp(splits > 1, False),
+                                    [kv, P(0), P(2), *ws, P(3), P(4), L(0), L(0), L(0), *sizes(splits), *win_a], shared_mem=C.attn_smem(d), **kw))
+            if splits > 1:
+                launches.append(_launch("attn_window", "kern_attn_window_merge", [min(256, d), 1, 1], [{"mul": ["seqs", hq]}, 1, 1],
+                                        ["in buffer<f32>", "in buffer<f32>", iface[2], "in buffer<bf16>"] + ["i32"] * 5 + ["f32"],
+                                        [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, P(2), P(5), I(C.I32_MAX), I(hq), I(d), I(splits), I(out_stride), {"f32": out_scale}], **kw))
+        scratch = {"scratch": {"ws_o": {"dtype": "f32", "shape": ["seqs", hq * most * d]}, "ws_ml": {"dtype": "f32", "shape": ["seqs", hq * most * 2]}}} if most > 1 else {}
+        return _op(iface, *launches, **scratch)
+    iface += ["in buffer<i32>"] * 5
+    mode = C.attn_mode(hq, hk, d)
+    few = {"var": "seqs", "max": C.FMHA_SEQS}
+    many = {"var": "seqs", "min": C.FMHA_SEQS + 1}
+    grid = lambda rows: [hk, {"add": [{"ceil_div": ["tokens", rows // g]}, "seqs"]}, 1]
+    causal = lambda **kw: _launch("attn_fmha", "kern_attn_window_fmha_d128", [192, 1, 1], grid(128), ["bytes<128>", iface[0], iface[2]] + ["in buffer<i32>"] * 5 + ["i32"] * 7 + win_t,
+                                  [kv, P(0), P(2), P(3), P(4), P(7), P(8), P(9), I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(C.I32_MAX), *win_a],
+                                  shared_mem=768 + 128 * d * 2 + 128 * 64 * 2 + 2 * 2 * (64 * d * 2) + 256, **kw)
+    listed = lambda kind, work, smem, g_, **kw: _launch("attn_window", f"kern_attn_window_{kind}_d{d}", [160, 1, 1], g_, lp(False, True),
+                                                        [kv, P(0), P(2), L(0), L(0), P(3), P(4), P(7), P(work), P(work + 1), *sizes(1), *win_a], shared_mem=smem, **kw)
+    one = lambda **kw: _launch("attn_window", f"kern_attn_window_ragged_d{d}", [160, 1, 1], grid(64), ["bytes<128>", iface[0], iface[2]] + ["in buffer<i32>"] * 7 + ["i32"] * 7 + win_t,
+                               [kv, P(0), P(2), P(3), P(4), P(7), P(8), P(9), P(10), P(11), I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(C.I32_MAX),
+                                *win_a], shared_mem=C.attn_smem(d, prefill=True), **kw)
+    rows = lambda **kw: listed("decode", 10, C.attn_smem(d), [hk, "seqs", 1], **kw)
+    if mode == "auto":
+        return _op(iface, causal(when=few), rows(when=few), one(when=many))
+    if mode in ("fmha", "fmha2"):
+        return _op(iface, causal(), rows())
+    if mode == "ragged":
+        return _op(iface, one())
+    return _op(iface, listed("prefill", 8, C.attn_smem(d, prefill=True), grid(64)), rows())
+
+
 # ---- routed experts ---------------------------------------------------------------------------------------
 def route_logits_op(experts: int, top: int, bias: bool = True) -> dict:
     """The `top` largest of logits + bias, weighed by the softmax over them. Interface [logits, (bias,) ids, weights, tokens]."""
@@ -251,17 +471,27 @@ def route_logits_op(experts: int, top: int, bias: bool = True) -> dict:
                               [P(0), b_a, P(o), P(o + 1), P(o + 2), I(experts), I(top), I(experts)]))
 
 
+def route_groups_op(experts: int, top: int, groups: int = 1, keep: int = 1, renorm: bool = False) -> dict:
+    """Sigmoid scores; the `top` largest inside the best `keep` of equal groups of neighbours (a group's score: the sum of its two
+    largest), weighing their scores. Interface [logits, ids, weights, tokens]."""
+    if not (1 <= top <= min(32, keep * (experts // groups)) and experts <= 1024 and experts % groups == 0 and 1 <= keep <= groups <= 64):
+        raise ValueError(f"{top} of {experts} experts per token in {keep} of {groups} groups (at most 32 of 1024, 64 groups)")
+    iface = ["in buffer<f32>", "out buffer<i32>", "out buffer<f32>", "i32"]
+    return _op(iface, _launch("moe", "kern_moe_route_groups", [128, 1, 1], [{"ceil_div": ["tokens", 4]}, 1, 1], iface + ["i32"] * 6,
+                              [*map(P, range(4)), I(experts), I(top), I(groups), I(keep), I(int(renorm)), I(experts)], shared_mem=4 * (experts + groups) * 4))
+
+
 def routed_tile_rows(act: str, width: int, ff: int) -> int:
     """Rows of a tile of the planner's table: 128 for the tensor-core kernels, 64 for the generic one."""
     return C.BM if act == "bf16" and tiles_fit(width, ff) else 64
 
 
-def routed_ops(width: int, ff: int, experts: int, top: int, tokens_max: int, act: str = "bf16") -> dict:
-    """plan / gather / fc1 / fc2 of routed SwiGLU experts under the interfaces of `moe._moe_ops`."""
+def routed_ops(width: int, ff: int, experts: int, top: int, tokens_max: int, act: str = "bf16", glu: str = "swiglu", limit: float = 0.0) -> dict:
+    """plan / gather / fc1 / fc2 of routed experts with a gated unit (GLUS), under the interfaces of `moe._moe_ops`."""
     from . import moe
 
     cfg = moe.MoeConfig(hidden=width, moe_intermediate=ff, experts=experts, top_k=top, max_tokens=tokens_max)
-    ops = moe._moe_ops(cfg, 0, experts)
+    ops = moe._moe_ops(cfg, 0, experts, glu=glu, limit=limit)
     if routed_tile_rows(act, width, ff) == C.BM:
         return {k: ops[k] for k in ("moe_plan", "moe_gather", "moe_fc1", "moe_fc2")}
     bm = routed_tile_rows(act, width, ff)
@@ -272,11 +502,11 @@ def routed_ops(width: int, ff: int, experts: int, top: int, tokens_max: int, act
                  _launch("linear", f"kern_rows_scatter_{act}", [256, 1, 1], [{"mul": ["tokens", top]}, 1, 1],
                          ["in " + b, "in buffer<i32>", "out " + b, "i32", "i32", "i32"], [P(0), P(1), P(2), P(3), I(top), I(width)]))
 
-    def routed(n, k, swiglu):
+    def routed(n, k, epi):
         return _op(["in " + b, "in buffer<bf16>", "out " + b, "in buffer<i32>", "in buffer<i32>", "i32", "out buffer<i32>"],
-                   _launch("linear", f"kern_linear_grouped_{act}" + ("_swiglu" if swiglu else ""), [256, 1, 1],
+                   _launch("linear", f"kern_linear_grouped_{act}" + (f"_{epi}" if epi else ""), [256, 1, 1],
                            [-(-n // 64), {"clamp": [{"add": [{"ceil_div": [{"mul": ["tokens", top]}, bm]}, experts]}, 0, 4096]}, 1],
-                           ["in " + b, "in buffer<bf16>", "out " + b, "in buffer<i32>", "in buffer<i32>", "i32", "i32", "i32", "i64", "out buffer<i32>"],
-                           [P(0), P(1), P(2), P(3), P(4), P(5), I(n), I(k), L((2 if swiglu else 1) * n * k), P(6)]))
+                           ["in " + b, "in buffer<bf16>", "out " + b, "in buffer<i32>", "in buffer<i32>", "i32", "i32", "i32", "i64", "out buffer<i32>", "f32"],
+                           [P(0), P(1), P(2), P(3), P(4), P(5), I(n), I(k), L((2 if epi else 1) * n * k), P(6), {"f32": limit}]))
 
-    return {"moe_plan": ops["moe_plan"], "moe_gather": gather, "moe_fc1": routed(ff, width, True), "moe_fc2": routed(width, ff, False)}
+    return {"moe_plan": ops["moe_plan"], "moe_gather": gather, "moe_fc1": routed(ff, width, glu), "moe_fc2": routed(width, ff, "")}

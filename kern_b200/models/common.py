@@ -81,6 +81,13 @@ def write_safetensors(path, tensors: dict[str, torch.Tensor], metadata: dict | N
             f.write(b)
 
 
+def safetensors_shapes(path) -> dict[str, tuple[int, ...]]:
+    """Tensor name -> shape, from the header alone."""
+    with open(path, "rb") as f:
+        (hlen,) = struct.unpack("<Q", f.read(8))
+        return {n: tuple(e["shape"]) for n, e in json.loads(f.read(hlen)).items() if n != "__metadata__"}
+
+
 def read_safetensors(path) -> dict[str, torch.Tensor]:
     inv = {v: k for k, v in _ST_DTYPES.items()}
     data = Path(path).read_bytes()
@@ -170,14 +177,15 @@ def gemm_op(n: int, k: int, *, epilogue: str = "store", rows_var: str = "tokens"
             lda: int | None = None, ldc: int | None = None) -> dict:
     """C[rows, n] = A[rows, k] · W[n, k]ᵀ through the tcgen05 GEMM, one launch per `when` range.
 
-    Interface: [a, w, c, rows, err]. epilogue store | acc (c += …, c is inout) | f32 | swiglu
+    Interface: [a, w, c, rows, err]. epilogue store | acc (c += …, c is inout) | f32 | swiglu | geglu
     (c is [rows, n/2] over weights stacked [gate rows ; up rows])."""
     lda = k if lda is None else lda
-    out_cols = n // 2 if epilogue == "swiglu" else n
+    glu = epilogue in ("swiglu", "geglu")
+    out_cols = n // 2 if glu else n
     ldc = out_cols if ldc is None else ldc
     cdt = "f32" if epilogue == "f32" else "bf16"
     cdir = "inout" if epilogue == "acc" else "out"
-    suffix = {"store": "", "acc": "_acc", "f32": "_f32", "swiglu": "_swiglu"}[epilogue]
+    suffix = {"store": "", "acc": "_acc", "f32": "_f32", "swiglu": "_swiglu", "geglu": "_geglu"}[epilogue]
     iface = ["in buffer<bf16>", "in buffer<bf16>", f"{cdir} buffer<{cdt}>", "i32", "out buffer<i32>"]
     lparams = ["bytes<128>", "bytes<128>", f"{cdir} buffer<{cdt}>", "in buffer<bf16>", "i32", "i32", "i32", "i32",
                "out buffer<i32>"]
@@ -203,7 +211,7 @@ def gemm_op(n: int, k: int, *, epilogue: str = "store", rows_var: str = "tokens"
     tiles = (256, 128, 64, 32) if epilogue in ("store", "acc") else (256, 128, 64)
     ranges = []
     for bn, lo, hi in gemm_ranges(n, rows_max, tiles):
-        if bn == 256 and epilogue in ("store", "acc", "swiglu") and M256_GAIN:
+        if bn == 256 and epilogue in ("store", "acc", "swiglu", "geglu") and M256_GAIN:
             ranges += [(bn, bm, a, b) for bm, a, b in m256_split(n, lo, hi)]
         else:
             ranges.append((bn, BM, lo, hi))
@@ -225,7 +233,7 @@ def gemm_op(n: int, k: int, *, epilogue: str = "store", rows_var: str = "tokens"
                     "swizzle": 128, "l2_promotion": 256}}]}},
                 {"pack": {"size": 128, "fields": [{"at": 0, "tensormap": {
                     "param": 1, "dtype": "bf16", "dims": [k, n], "strides": [k * 2],
-                    "box": [BK, bn // 2 if epilogue == "swiglu" else bn],
+                    "box": [BK, bn // 2 if glu else bn],
                     "swizzle": 128, "l2_promotion": 256}}]}},
                 {"param": 2}, {"param": 2 if epilogue == "acc" else 0}, {"param": 3}, {"i32": n}, {"i32": k},
                 {"i32": ldc}, {"param": 4}],

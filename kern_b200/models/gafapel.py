@@ -22,6 +22,8 @@ import torch
 
 from . import blocks as K
 from . import common as C
+from . import listed
+from .listed import Listed, load_random
 
 
 @dataclass
@@ -200,93 +202,26 @@ def random_weights(cfg: GafapelConfig, seed: int = 0, device: str = "cpu", std: 
 
 
 def load_random_weights(rt, cfg: GafapelConfig, seed: int = 0, std: float = 0.02) -> None:
-    """Fill the runtime's weights with the synthetic checkpoint, tensor by tensor on the runtime's device."""
-    shapes = weight_names(cfg)
-    order = {n: i for i, n in enumerate(shapes)}
-
-    def provider(name: str) -> torch.Tensor:
-        dev = rt.tensor("x").device
-        g = torch.Generator(device=dev).manual_seed(seed * 1000003 + order[name])
-        return _random(name, shapes[name], g, dev, std)
-
-    rt.load_tensors(provider)
+    load_random(rt, weight_names(cfg), _random, seed, std)
 
 
 def save_folder(path, cfg: GafapelConfig, weights: dict[str, torch.Tensor]) -> None:
-    """A checkpoint folder: config.json and model.safetensors."""
-    path = Path(path)
-    path.mkdir(parents=True, exist_ok=True)
-    (path / "config.json").write_text(json.dumps(to_config(cfg), indent=1))
-    C.write_safetensors(path / "model.safetensors", weights)
+    listed.save_folder(path, to_config(cfg), weights)
 
 
 # ---- the manifest -------------------------------------------------------------------------------------------
-WANTED = 512          # most rows one call of the `logits` program projects
-
-
 def build_manifest(cfg: GafapelConfig) -> dict:
     d, A, T, S, W = cfg.width, cfg.dtype, cfg.max_tokens, cfg.max_seqs, cfg.table_width
-    if A not in K.ACT_BYTES:
-        raise ValueError(f"dtype `{A}`: bf16 or f32")
-    es, layers = K.ACT_BYTES[A], cfg.depth
-    if not layers:
-        raise ValueError("a model without layers")
-    bufs, ops, states, once = {}, {}, {}, []
-    B = lambda n, off=0: ({"buf": n, "offset": off} if off else {"buf": n})
-    V = lambda n: {"var": n}
-    err = B("error")
-
-    def op(name: str, make) -> str:
-        """An op under a name that says its sizes, made once."""
-        if name not in ops:
-            ops[name] = make()
-        return name
-
-    def room(name: str, cols: int, dtype: str = A, kind: str = "workspace") -> None:
-        """A per-token buffer as wide as the widest layer that uses it."""
-        have = bufs.get(name, {"shape": ["tokens", 0]})["shape"][1]
-        bufs[name] = {"dtype": dtype, "shape": ["tokens", max(have, cols)], "kind": kind}
-
-    def weight(name: str, shape, *tensors) -> dict:
-        if name not in bufs:
-            bufs[name] = {"dtype": "bf16", "shape": list(shape), "kind": "weight",
-                          "bind": [t if isinstance(t, dict) else {"tensor": t} for t in tensors]}
-        return B(name)
-
-    def same(name: str, shape) -> dict:
-        return weight("w." + name, shape, name)
-
-    def linear(base: str, n: int, k: int, a, w, c, rows: str = "tokens", label: str = "", **kw) -> dict:
-        name = op(f"{base}_{n}x{k}", lambda: K.linear_op(n, k, act=A, rows_var=rows, rows_max=T if rows == "tokens" else
-                                                         (S if rows == "seqs" else WANTED), **kw))
-        return {"op": name, "label": label, "args": [a, w, c, V(rows), err]}
-
+    m_ = Listed(cfg)
+    layers, es, bufs, states, once, err = cfg.depth, m_.es, m_.bufs, m_.states, m_.once, m_.err
+    B, V, op, room, weight, same, linear = m_.B, m_.V, m_.op, m_.room, m_.weight, m_.same, m_.linear
     kinds = [kind_of(b) for b in layers]
     latents = [i for i, k in enumerate(kinds) if k == "latent_attention"]
     mambas = [i for i, k in enumerate(kinds) if k == "mamba2"]
-    inp = lambda dt, shape, **kw: {"dtype": dt, "shape": shape, "kind": "input", **kw}
-    bufs["token_ids"] = inp("i64", ["tokens"], fill="token", domain={"min": 0, "max": cfg.vocab - 1})
-    bufs["positions"] = inp("i64", ["tokens"], fill="position", domain={"min": 0, "max": cfg.context - 1})
-    bufs["cu_seqlens"] = inp("i32", [S + 1], fill="cu_seqlens")
-    if latents:
-        kv0 = f"kv.l{latents[0]}"
-        bufs["slot_mapping"] = inp("i64", ["tokens"], fill="slot", domain={"index_into": kv0})
-        bufs["seq_lens"] = inp("i32", ["seqs"], fill="seq_len")
-        bufs["block_table"] = inp("i32", ["seqs", W], domain={"index_into": kv0, "stride": cfg.page_size})
-        bufs["row_seq"] = {"dtype": "i32", "shape": ["tokens"], "kind": "workspace"}
-        bufs["row_len"] = {"dtype": "i32", "shape": ["tokens"], "kind": "workspace"}
-    if mambas:
-        bufs["lines"] = inp("i32", [1, "seqs"], domain={"index_into": f"ssd.l{mambas[0]}"})
-    bufs["next_token"] = {"dtype": "i64", "shape": ["seqs"], "kind": "output", "fill": "tokens"}
-    bufs["error"] = {"dtype": "i32", "shape": [1], "kind": "output", "fill": "error"}
+    m_.inputs(f"kv.l{latents[0]}" if latents else None, f"ssd.l{mambas[0]}" if mambas else None)
     room("x", cfg.streams * d, "f32")
     room("xn", d)
-    room("hidden", d, "f32", "carry")
-    bufs["last_n"] = {"dtype": A, "shape": ["seqs", d], "kind": "workspace"}
-    bufs["logits"] = {"dtype": "f32", "shape": ["seqs", cfg.vocab], "kind": "workspace"}
-    bufs["want_rows"] = inp("i32", ["wanted"])
-    bufs["want_n"] = {"dtype": A, "shape": ["wanted", d], "kind": "workspace"}
-    bufs["want_logits"] = {"dtype": "f32", "shape": ["wanted", cfg.vocab], "kind": "output"}
+    m_.outputs()
 
     # every sublayer in order: (its stream weights, its norm)
     subs = [(f"l{i}.hc{q}", f"l{i}.norm{q}") for i, b in enumerate(layers) for q in ((1, 2) if b["mlp"] is not None else (1,))]
@@ -361,44 +296,19 @@ def build_manifest(cfg: GafapelConfig) -> dict:
             finish(at, B("y"), p + "mix1"),
         ]
         if prefill and i == latents[0]:
-            calls.insert(0, {"op": op("rows", C.mla_rows_op), "label": p + "rows", "args": [B("positions"), B("cu_seqlens"), B("row_seq"), B("row_len"), V("seqs"), V("tokens")]})
+            calls.insert(0, m_.rows_call(p + "rows"))
         return calls
 
     def dense(i: int, at: int) -> list[dict]:
-        ff, p = layers[i]["mlp"]["ff"], f"l{i}."
-        room("act", ff); room("y", d)
-        return [
-            linear("glu", 2 * ff, d, B("xn"), weight(f"w.{p}mlp.gu", (2 * ff, d), p + "mlp.gate", p + "mlp.up"), B("act"), label=p + "gate_up", epilogue="swiglu"),
-            linear("lin", d, ff, B("act"), same(p + "mlp.down", (d, ff)), B("y"), label=p + "down"),
-            finish(at, B("y"), p + "mix2"),
-        ]
+        p = f"l{i}."
+        return m_.dense(p, layers[i]["mlp"]["ff"], "swiglu") + [finish(at, B("y"), p + "mix2")]
 
     def routed(i: int, at: int) -> list[dict]:
         f, p = layers[i]["mlp"], f"l{i}."
-        E, k, ff = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
-        room("moe.logits", E, "f32"); room("moe.ids", k, "i32"); room("moe.w", k, "f32"); room("moe.perm", k, "i32")
-        room("moe.x", k * d); room("moe.act", k * ff); room("moe.y", k * d)
-        tiles = T * k // K.routed_tile_rows(A, d, ff) + E
-        for name, shape in (("moe.offsets", [E + 1]), ("moe.tiles", [tiles, 4]), ("moe.tile_count", [1]), ("moe.rows", [1])):
-            have = bufs.get(name, {"shape": [0]})["shape"]
-            bufs[name] = {"dtype": "i32", "shape": [max(have[0], shape[0]), *shape[1:]], "kind": "workspace"}
-        tag = f"{d}x{ff}x{E}x{k}"
-        if f"moe_plan_{tag}" not in ops:
-            for n, o in K.routed_ops(d, ff, E, k, T, A).items():
-                ops[f"{n}_{tag}"] = o
+        E, k = f["router"]["experts"], f["router"]["top"]
         route = op(f"moe_route_{E}x{k}", lambda: K.route_logits_op(E, k))
-        n = {"expr": {"mul": ["tokens", k]}}
-        w1 = weight(f"w.{p}mlp.w1", (E, 2 * ff, d), *[f"{p}mlp.e{e}.{t}" for e in range(E) for t in ("gate", "up")])
-        w2 = weight(f"w.{p}mlp.w2", (E, d, ff), *[f"{p}mlp.e{e}.down" for e in range(E)])
-        return [
-            linear("router", E, d, B("xn"), same(p + "mlp.router", (E, d)), B("moe.logits"), label=p + "router", epilogue="f32"),
-            {"op": route, "label": p + "route", "args": [B("moe.logits"), same(p + "mlp.router.b", (E,)), B("moe.ids"), B("moe.w"), V("tokens")]},
-            {"op": f"moe_plan_{tag}", "label": p + "plan", "args": [B("moe.ids"), B("moe.perm"), B("moe.offsets"), B("moe.tiles"), B("moe.tile_count"), B("moe.rows"), n, err]},
-            {"op": f"moe_gather_{tag}", "label": p + "gather", "args": [B("xn"), B("moe.perm"), B("moe.x"), n]},
-            {"op": f"moe_fc1_{tag}", "label": p + "fc1", "args": [B("moe.x"), w1, B("moe.act"), B("moe.tiles"), B("moe.tile_count"), n, err]},
-            {"op": f"moe_fc2_{tag}", "label": p + "fc2", "args": [B("moe.act"), w2, B("moe.y"), B("moe.tiles"), B("moe.tile_count"), n, err]},
-            finish(at, B("moe.y"), p + "mix2", k, [B("moe.perm"), B("moe.w")]),
-        ]
+        pick = lambda logits, ids, w: {"op": route, "label": p + "route", "args": [logits, same(p + "mlp.router.b", (E,)), ids, w, V("tokens")]}
+        return m_.routed(p, E, k, f["expert"]["ff"], pick) + [finish(at, B("moe.y"), p + "mix2", k, [B("moe.perm"), B("moe.w")])]
 
     def forward(prefill: bool) -> list[dict]:
         embed = op("embed", lambda: K.hyper_embed_op(d, s, cfg.vocab, cfg.max_positions, cfg.eps, A))
@@ -412,38 +322,6 @@ def build_manifest(cfg: GafapelConfig) -> dict:
             if b["mlp"] is not None:
                 calls += (dense if b["mlp"]["kind"] == "dense" else routed)(i, at)
                 at += 1
-        pick = "last" if prefill else "each"
-        norm = op("final_norm_" + pick, lambda: K.row_norm_op(d, cfg.eps, T, A, pick))
-        calls += [{"op": norm, "label": "final_norm", "args": [B("hidden"), same("final.norm", (d,)), B("last_n"), *([B("cu_seqlens")] if prefill else [])]},
-                  linear("head", cfg.vocab, d, B("last_n"), same("head", (cfg.vocab, d)), B("logits"), rows="seqs", label="lm_head", epilogue="f32")]
-        if cfg.sampling:
-            pick_op = op("sample", lambda: C.sample_op(cfg.vocab, "f32"))
-            calls.append({"op": pick_op, "label": "sample", "args": [B("logits"), B("next_token"), *[B(n) for n in
-                          ("temperature", "top_k", "top_p", "min_p", "seed", "seq_lens")]]})
-        else:
-            calls.append({"op": op("pick", lambda: C.argmax_op(cfg.vocab, "f32")), "label": "argmax", "args": [B("logits"), B("next_token")]})
         return calls
 
-    if cfg.sampling:
-        bufs.setdefault("seq_lens", inp("i32", ["seqs"], fill="seq_len"))
-        for name, dt in (("temperature", "f32"), ("top_k", "i32"), ("top_p", "f32"), ("min_p", "f32"), ("seed", "i64")):
-            bufs[name] = inp(dt, ["seqs"], fill=name)
-    prefill, decode = forward(True), forward(False)
-    listed = op("final_norm_listed", lambda: K.row_norm_op(d, cfg.eps, T, A, "listed"))
-    logits = [{"op": listed, "label": "want_norm", "args": [B("hidden"), B("w.final.norm"), B("want_n"), B("want_rows")]},
-              linear("head_rows", cfg.vocab, d, B("want_n"), B("w.head"), B("want_logits"), rows="wanted", label="want_head", epilogue="f32")]
-    doc = {
-        "schema_version": 7, "model": cfg.name,
-        "vars": {"tokens": {"max": T, "axis": "rows"}, "seqs": {"max": S, "axis": "groups"}, "wanted": {"max": WANTED}},
-        "states": states, "buffers": bufs, "modules": {}, "ops": ops,
-        "programs": {
-            "prefill": {"batch": {"groups": S, "rows": "tokens"}, "calls": prefill},
-            "decode": {"batch": {"groups": S, "rows": 1}, "graph": True, "calls": decode},
-            "logits": {"calls": logits},
-        },
-    }
-    if once:
-        doc["programs"]["load"] = {"once": True, "calls": once}
-    used = {l["module"] for o in ops.values() for l in o["impl"]["launches"]}
-    doc["modules"] = {n: m for n, m in C.modules_for(sorted(used)).items() if n in used}
-    return doc
+    return m_.document(forward, "head")

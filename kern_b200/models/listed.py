@@ -1,0 +1,211 @@
+"""What the manifests of decoders with listed layers share: config.json names every layer with its mixer and feed-forward, a
+program walks the list, the residual is f32, and the last sublayer leaves its rows in `hidden` (a carry: the rows of the last
+call), from which `prefill` / `decode` norm and project each sequence's last row and the `logits` program any listed rows.
+
+`Listed` collects buffers, ops, states and load-time calls while a family writes its sublayers; every op and weight is made
+once, under a name that says its sizes.
+"""
+from __future__ import annotations
+
+import json
+from pathlib import Path
+
+import torch
+
+from . import blocks as K
+from . import common as C
+
+WANTED = 512          # most rows one call of the `logits` program projects
+
+
+class Listed:
+    def __init__(self, cfg):
+        """`cfg`: width, vocab, eps, dtype, max_tokens, max_seqs, context, table_width, page_size, sampling, name."""
+        if cfg.dtype not in K.ACT_BYTES:
+            raise ValueError(f"dtype `{cfg.dtype}`: bf16 or f32")
+        if not cfg.depth:
+            raise ValueError("a model without layers")
+        self.cfg, self.act, self.es = cfg, cfg.dtype, K.ACT_BYTES[cfg.dtype]
+        self.bufs, self.ops, self.states, self.once = {}, {}, {}, []
+        self.err = self.B("error")
+
+    # ---- names ----
+    @staticmethod
+    def B(name: str, offset: int = 0) -> dict:
+        return {"buf": name, "offset": offset} if offset else {"buf": name}
+
+    @staticmethod
+    def V(name: str) -> dict:
+        return {"var": name}
+
+    def op(self, name: str, make) -> str:
+        """An op under a name that says its sizes, made once."""
+        if name not in self.ops:
+            self.ops[name] = make()
+        return name
+
+    def room(self, name: str, cols: int, dtype: str | None = None, kind: str = "workspace") -> None:
+        """A per-token buffer as wide as the widest layer that uses it."""
+        have = self.bufs.get(name, {"shape": ["tokens", 0]})["shape"][1]
+        self.bufs[name] = {"dtype": dtype or self.act, "shape": ["tokens", max(have, cols)], "kind": kind}
+
+    def weight(self, name: str, shape, *tensors) -> dict:
+        if name not in self.bufs:
+            self.bufs[name] = {"dtype": "bf16", "shape": list(shape), "kind": "weight",
+                               "bind": [t if isinstance(t, dict) else {"tensor": t} for t in tensors]}
+        return self.B(name)
+
+    def same(self, name: str, shape) -> dict:
+        return self.weight("w." + name, shape, name)
+
+    def rows_weight(self, name: str, width: int, parts: list[tuple[str, int]]) -> tuple[dict, int]:
+        """Projections with one input as one matrix -> (the weight, its rows), filled up to whole 16-byte vectors of output with
+        copies of the first rows, which nobody reads. `parts`: (tensor, rows)."""
+        rows = sum(n for _, n in parts)
+        proj = -(-rows // 8) * 8
+        fill = [{"tensor": parts[0][0], "rows": [0, proj - rows]}] if proj > rows else []
+        return self.weight(name, (proj, width), *[t for t, _ in parts], *fill), proj
+
+    def linear(self, base: str, n: int, k: int, a, w, c, rows: str = "tokens", label: str = "", **kw) -> dict:
+        most = {"tokens": self.cfg.max_tokens, "seqs": self.cfg.max_seqs, "wanted": WANTED}[rows]
+        lda = kw.get("lda")
+        name = self.op(f"{base}_{n}x{k}" + (f"_of{lda}" if lda else ""), lambda: K.linear_op(n, k, act=self.act, rows_var=rows, rows_max=most, **kw))
+        return {"op": name, "label": label, "args": [a, w, c, self.V(rows), self.err]}
+
+    # ---- inputs and outputs ----
+    def inputs(self, paged: str | None, lined: str | None, row_plan: bool = True) -> None:
+        """The host's columns. `paged` / `lined`: a paged and a per-sequence state, when the model has them; `row_plan`: room for
+        every token's table row and reach (`rows_call`)."""
+        cfg, S = self.cfg, self.cfg.max_seqs
+        inp = lambda dt, shape, **kw: {"dtype": dt, "shape": shape, "kind": "input", **kw}
+        self.bufs["token_ids"] = inp("i64", ["tokens"], fill="token", domain={"min": 0, "max": cfg.vocab - 1})
+        self.bufs["positions"] = inp("i64", ["tokens"], fill="position", domain={"min": 0, "max": cfg.context - 1})
+        self.bufs["cu_seqlens"] = inp("i32", [S + 1], fill="cu_seqlens")
+        if paged:
+            self.bufs["slot_mapping"] = inp("i64", ["tokens"], fill="slot", domain={"index_into": paged})
+            self.bufs["seq_lens"] = inp("i32", ["seqs"], fill="seq_len")
+            self.bufs["block_table"] = inp("i32", ["seqs", cfg.table_width], domain={"index_into": paged, "stride": cfg.page_size})
+            if row_plan:
+                self.bufs["row_seq"] = {"dtype": "i32", "shape": ["tokens"], "kind": "workspace"}
+                self.bufs["row_len"] = {"dtype": "i32", "shape": ["tokens"], "kind": "workspace"}
+        if lined:
+            self.bufs["lines"] = inp("i32", [1, "seqs"], domain={"index_into": lined})
+        self.bufs["next_token"] = {"dtype": "i64", "shape": ["seqs"], "kind": "output", "fill": "tokens"}
+        self.bufs["error"] = {"dtype": "i32", "shape": [1], "kind": "output", "fill": "error"}
+
+    def outputs(self) -> None:
+        cfg, d = self.cfg, self.cfg.width
+        self.room("hidden", d, "f32", "carry")
+        self.bufs["last_n"] = {"dtype": self.act, "shape": ["seqs", d], "kind": "workspace"}
+        self.bufs["logits"] = {"dtype": "f32", "shape": ["seqs", cfg.vocab], "kind": "workspace"}
+        self.bufs["want_rows"] = {"dtype": "i32", "shape": ["wanted"], "kind": "input"}
+        self.bufs["want_n"] = {"dtype": self.act, "shape": ["wanted", d], "kind": "workspace"}
+        self.bufs["want_logits"] = {"dtype": "f32", "shape": ["wanted", cfg.vocab], "kind": "output"}
+
+    def rows_call(self, label: str) -> dict:
+        """The plan of a ragged call for kernels that take one attention row per token."""
+        B, V = self.B, self.V
+        return {"op": self.op("rows", C.mla_rows_op), "label": label,
+                "args": [B("positions"), B("cu_seqlens"), B("row_seq"), B("row_len"), V("seqs"), V("tokens")]}
+
+    # ---- feed-forward ----
+    def dense(self, p: str, ff: int, glu: str) -> list[dict]:
+        """Gate and up projections with their gated unit, and the projection back: xn -> y."""
+        d, B = self.cfg.width, self.B
+        self.room("act", ff); self.room("y", d)
+        base = "glu" if glu == "swiglu" else glu
+        return [
+            self.linear(base, 2 * ff, d, B("xn"), self.weight(f"w.{p}mlp.gu", (2 * ff, d), p + "mlp.gate", p + "mlp.up"), B("act"), label=p + "gate_up", epilogue=glu),
+            self.linear("lin", d, ff, B("act"), self.same(p + "mlp.down", (d, ff)), B("y"), label=p + "down"),
+        ]
+
+    def routed(self, p: str, experts: int, top: int, ff: int, route, glu: str = "swiglu", limit: float = 0.0) -> list[dict]:
+        """Routed experts up to their own rows: xn -> `moe.y` (expert-sorted), `moe.perm`, `moe.w`. `route(logits, ids, weights)` makes
+        the call that picks them."""
+        cfg, d, B, V = self.cfg, self.cfg.width, self.B, self.V
+        E, k, T, A, err = experts, top, cfg.max_tokens, self.act, self.err
+        self.room("moe.logits", E, "f32"); self.room("moe.ids", k, "i32"); self.room("moe.w", k, "f32"); self.room("moe.perm", k, "i32")
+        self.room("moe.x", k * d); self.room("moe.act", k * ff); self.room("moe.y", k * d)
+        tiles = T * k // K.routed_tile_rows(A, d, ff) + E
+        for name, shape in (("moe.offsets", [E + 1]), ("moe.tiles", [tiles, 4]), ("moe.tile_count", [1]), ("moe.rows", [1])):
+            have = self.bufs.get(name, {"shape": [0]})["shape"]
+            self.bufs[name] = {"dtype": "i32", "shape": [max(have[0], shape[0]), *shape[1:]], "kind": "workspace"}
+        tag = f"{d}x{ff}x{E}x{k}" + (f"_{glu}{limit:g}" if glu != "swiglu" else "")
+        if f"moe_plan_{tag}" not in self.ops:
+            for n, o in K.routed_ops(d, ff, E, k, T, A, glu, limit).items():
+                self.ops[f"{n}_{tag}"] = o
+        n = {"expr": {"mul": ["tokens", k]}}
+        w1 = self.weight(f"w.{p}mlp.w1", (E, 2 * ff, d), *[f"{p}mlp.e{e}.{t}" for e in range(E) for t in ("gate", "up")])
+        w2 = self.weight(f"w.{p}mlp.w2", (E, d, ff), *[f"{p}mlp.e{e}.down" for e in range(E)])
+        return [
+            self.linear("router", E, d, B("xn"), self.same(p + "mlp.router", (E, d)), B("moe.logits"), label=p + "router", epilogue="f32"),
+            route(B("moe.logits"), B("moe.ids"), B("moe.w")),
+            {"op": f"moe_plan_{tag}", "label": p + "plan", "args": [B("moe.ids"), B("moe.perm"), B("moe.offsets"), B("moe.tiles"), B("moe.tile_count"), B("moe.rows"), n, err]},
+            {"op": f"moe_gather_{tag}", "label": p + "gather", "args": [B("xn"), B("moe.perm"), B("moe.x"), n]},
+            {"op": f"moe_fc1_{tag}", "label": p + "fc1", "args": [B("moe.x"), w1, B("moe.act"), B("moe.tiles"), B("moe.tile_count"), n, err]},
+            {"op": f"moe_fc2_{tag}", "label": p + "fc2", "args": [B("moe.act"), w2, B("moe.y"), B("moe.tiles"), B("moe.tile_count"), n, err]},
+        ]
+
+    # ---- from `hidden` to tokens ----
+    def tail(self, head: str, prefill: bool) -> list[dict]:
+        """Final norm, the projection by tensor `head`, and the next token of every sequence."""
+        cfg, d, B = self.cfg, self.cfg.width, self.B
+        pick = "last" if prefill else "each"
+        norm = self.op("final_norm_" + pick, lambda: K.row_norm_op(d, cfg.eps, cfg.max_tokens, self.act, pick))
+        calls = [{"op": norm, "label": "final_norm", "args": [B("hidden"), self.same("final.norm", (d,)), B("last_n"), *([B("cu_seqlens")] if prefill else [])]},
+                 self.linear("head", cfg.vocab, d, B("last_n"), self.same(head, (cfg.vocab, d)), B("logits"), rows="seqs", label="lm_head", epilogue="f32")]
+        if cfg.sampling:
+            pick_op = self.op("sample", lambda: C.sample_op(cfg.vocab, "f32"))
+            calls.append({"op": pick_op, "label": "sample", "args": [B("logits"), B("next_token"), *[B(n) for n in
+                          ("temperature", "top_k", "top_p", "min_p", "seed", "seq_lens")]]})
+        else:
+            calls.append({"op": self.op("pick", lambda: C.argmax_op(cfg.vocab, "f32")), "label": "argmax", "args": [B("logits"), B("next_token")]})
+        return calls
+
+    def document(self, forward, head: str) -> dict:
+        """The manifest; `forward(prefill)` writes the calls from the embedding to `hidden`."""
+        cfg, d, B = self.cfg, self.cfg.width, self.B
+        if cfg.sampling:
+            self.bufs.setdefault("seq_lens", {"dtype": "i32", "shape": ["seqs"], "kind": "input", "fill": "seq_len"})
+            for name, dt in (("temperature", "f32"), ("top_k", "i32"), ("top_p", "f32"), ("min_p", "f32"), ("seed", "i64")):
+                self.bufs[name] = {"dtype": dt, "shape": ["seqs"], "kind": "input", "fill": name}
+        prefill, decode = (forward(p) + self.tail(head, p) for p in (True, False))
+        listed = self.op("final_norm_listed", lambda: K.row_norm_op(d, cfg.eps, cfg.max_tokens, self.act, "listed"))
+        logits = [{"op": listed, "label": "want_norm", "args": [B("hidden"), B("w.final.norm"), B("want_n"), B("want_rows")]},
+                  self.linear("head_rows", cfg.vocab, d, B("want_n"), B("w." + head), B("want_logits"), rows="wanted", label="want_head", epilogue="f32")]
+        doc = {
+            "schema_version": 7, "model": cfg.name,
+            "vars": {"tokens": {"max": cfg.max_tokens, "axis": "rows"}, "seqs": {"max": cfg.max_seqs, "axis": "groups"}, "wanted": {"max": WANTED}},
+            "states": self.states, "buffers": self.bufs, "modules": {}, "ops": self.ops,
+            "programs": {
+                "prefill": {"batch": {"groups": cfg.max_seqs, "rows": "tokens"}, "calls": prefill},
+                "decode": {"batch": {"groups": cfg.max_seqs, "rows": 1}, "graph": True, "calls": decode},
+                "logits": {"calls": logits},
+            },
+        }
+        if self.once:
+            doc["programs"]["load"] = {"once": True, "calls": self.once}
+        used = {l["module"] for o in self.ops.values() for l in o["impl"]["launches"]}
+        doc["modules"] = {n: m for n, m in C.modules_for(sorted(used)).items() if n in used}
+        return doc
+
+
+# ---- checkpoints -------------------------------------------------------------------------------------------
+def load_random(rt, shapes: dict, random, seed: int, std: float) -> None:
+    """Fill the runtime's weights with a family's synthetic checkpoint, tensor by tensor on the runtime's device."""
+    order = {n: i for i, n in enumerate(shapes)}
+
+    def provider(name: str) -> torch.Tensor:
+        dev = rt.tensor("x").device
+        g = torch.Generator(device=dev).manual_seed(seed * 1000003 + order[name])
+        return random(name, shapes[name], g, dev, std)
+
+    rt.load_tensors(provider)
+
+
+def save_folder(path, config: dict, weights: dict[str, torch.Tensor]) -> None:
+    """A checkpoint folder: config.json and model.safetensors."""
+    path = Path(path)
+    path.mkdir(parents=True, exist_ok=True)
+    (path / "config.json").write_text(json.dumps(config, indent=1))
+    C.write_safetensors(path / "model.safetensors", weights)

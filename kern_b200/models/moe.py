@@ -81,8 +81,9 @@ def load_random_weights(rt, cfg: MoeConfig, seed: int = 0, std: float = 0.02, sk
     rt.load_tensors(provider, skip=skip)
 
 
-def _moe_ops(cfg: MoeConfig, e_lo: int, e_n: int, ep_group: str | None = None, accumulate: bool = True) -> dict:
-    """`ep_group`: the rank of that group shifts the expert range by e_n per rank (expert parallel). `accumulate`: the
+def _moe_ops(cfg: MoeConfig, e_lo: int, e_n: int, ep_group: str | None = None, accumulate: bool = True,
+             glu: str = "swiglu", limit: float = 0.0) -> dict:
+    """`glu`: the experts' gated unit, swiglu | geglu | clamped (cut at `limit`). `ep_group`: the rank of that group shifts the expert range by e_n per rank (expert parallel). `accumulate`: the
     combine adds into its output (a residual) instead of overwriting it (a partial sum for an all-reduce)."""
     h, I, E, k, T = cfg.hidden, cfg.moe_intermediate, cfg.experts, cfg.top_k, cfg.max_tokens
     max_tiles = T * k // C.BM + e_n
@@ -111,21 +112,22 @@ def _moe_ops(cfg: MoeConfig, e_lo: int, e_n: int, ep_group: str | None = None, a
 
     def routed(n, kk, epi):
         bn = 128 if n >= 128 else 64
-        out_cols = n // 2 if epi == "swiglu" else n
+        out_cols = n if epi == "store" else n // 2
         a_map = {"pack": {"size": 128, "fields": [{"at": 0, "tensormap": {
             "param": 0, "dtype": "bf16", "dims": [kk, 0], "strides": [kk * 2], "box": [C.BK, C.BM], "swizzle": 128, "l2_promotion": 256}}]}}
         b_map = {"pack": {"size": 128, "fields": [{"at": 0, "tensormap": {
             "param": 1, "dtype": "bf16", "dims": [kk, n, e_n], "strides": [kk * 2, n * kk * 2],
-            "box": [C.BK, bn // 2 if epi == "swiglu" else bn, 1], "swizzle": 128, "l2_promotion": 256}}]}}
+            "box": [C.BK, bn if epi == "store" else bn // 2, 1], "swizzle": 128, "l2_promotion": 256}}]}}
+        extra_t, extra = (["f32"], [{"f32": limit}]) if epi == "clamped" else ([], [])
         return {"params": ["in buffer<bf16>", "in buffer<bf16>", "out buffer<bf16>", "in buffer<i32>", "in buffer<i32>", "i32",
                            "out buffer<i32>"], "impl": {"launches": [L(
-            "moe", f"kern_moe_gemm_bf16{'_swiglu' if epi == 'swiglu' else ''}_n{bn}", [192, 1, 1], [C.SMS, 1, 1],
+            "moe", f"kern_moe_gemm_bf16{'' if epi == 'store' else '_' + epi}_n{bn}", [192, 1, 1], [C.SMS, 1, 1],
             ["bytes<128>", "bytes<128>", "out buffer<bf16>", "in buffer<i32>", "in buffer<i32>", "i32", "i32", "i32", "i32",
-             "out buffer<i32>"],
+             "out buffer<i32>", *extra_t],
             [a_map, b_map, {"param": 2}, {"param": 3}, {"param": 4}, {"param": 5}, {"i32": n}, {"i32": kk}, {"i32": out_cols},
-             {"param": 6}], shared_mem=C.gemm_smem(bn))]}}
+             {"param": 6}, *extra], shared_mem=C.gemm_smem(bn))]}}
 
-    ops["moe_fc1"] = routed(2 * I, h, "swiglu")
+    ops["moe_fc1"] = routed(2 * I, h, glu)
     ops["moe_fc2"] = routed(h, I, "store")
     ops["moe_combine"] = {"params": ["in buffer<bf16>", "in buffer<i32>", "in buffer<f32>",
                                      ("inout" if accumulate else "out") + " buffer<bf16>"], "impl": {"launches": [L(

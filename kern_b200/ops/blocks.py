@@ -1,4 +1,5 @@
-"""CPU statements of the kernels in hyper.cu, linear.cu, ssd.cu, latent.cu (and the latent forms in mla_decode.cu / moe.cu):
+"""CPU statements of the kernels in hyper.cu, resid.cu, linear.cu, ssd.cu, lin_attn.cu, latent.cu, attn_window.cu (and the forms
+of the same mechanisms in mla_decode.cu / moe.cu / ssd_chunk.cu / lin_attn_chunk.cu / attn_fmha.cu / gemm_bf16.cu):
 what each launch computes, over the same arguments, for `kern_b200.cpu.CpuRuntime`. Rounding follows the buffers' types."""
 from __future__ import annotations
 
@@ -64,21 +65,51 @@ def k_row_norm(g, src, cu, rows, w, y, src_rows, d, eps):
     y[: n * d] = _norm(u, w[:d], eps).to(y.dtype).reshape(-1)
 
 
+# ---- the residual with norms on both sides ----
+def k_resid_embed(g, ids, table, w, x, xn, d, vocab, eps, err):
+    n = g[0]
+    tok = ids[:n].long()
+    if ((tok < 0) | (tok >= vocab)).any():
+        err[0] = 300
+    e = _f(table[: vocab * d].view(vocab, d)[torch.where((tok < 0) | (tok >= vocab), 0, tok)])
+    x[: n * d] = e.reshape(-1)
+    xn[: n * d] = _norm(e, w[:d], eps).to(xn.dtype).reshape(-1)
+
+
+def k_resid_mix(g, x, y, perm, topw, w_post, w_next, xn, hidden, d, k, eps):
+    n = g[0]
+    if isinstance(perm, T):
+        v = (_f(y.view(-1)[: n * k * d].view(-1, d)[perm[: n * k].long()]).view(n, k, d) * topw[: n * k].view(n, k, 1)).sum(1)
+    else:
+        v = _f(y[: n * d].view(n, d))
+    new = x[: n * d].view(n, d) + (_norm(v, w_post[:d], eps) if isinstance(w_post, T) else v)
+    if isinstance(hidden, T):
+        hidden[: n * d] = new.reshape(-1)
+    else:
+        x[: n * d] = new.reshape(-1)
+        xn[: n * d] = _norm(new, w_next[:d], eps).to(xn.dtype).reshape(-1)
+
+
 # ---- matrix products ----
-def _swiglu(v):
-    half = v.shape[1] // 2
-    return F.silu(v[:, :half]) * v[:, half:]
+def _glu(v, kind, limit=0.0):
+    g, u = v[:, :v.shape[1] // 2], v[:, v.shape[1] // 2:]
+    if kind == "geglu":
+        return F.gelu(g, approximate="tanh") * u
+    if kind == "clamped":
+        g = g.clamp(max=limit)
+        return g * torch.sigmoid(1.702 * g) * (u.clamp(-limit, limit) + 1)
+    return F.silu(g) * u
 
 
-def _k_linear(swiglu):
-    def run(g, a, w, c, m, n, k, lda, ldc, wsn, wsk, az, wz, cz, err):
+def _k_linear(glu):
+    def run(g, a, w, c, m, n, k, lda, ldc, wsn, wsk, az, wz, cz, err, limit):
         if m > g[1] * 64:
             err[0] = 300
         for z in range(g[2]):
             A = _f(_rows(a[z * az:], m, k, lda))
-            W = _f(torch.as_strided(w[z * wz:], ((2 if swiglu else 1) * n, k), (wsn, wsk)))
+            W = _f(torch.as_strided(w[z * wz:], ((2 if glu else 1) * n, k), (wsn, wsk)))
             v = A @ W.t()
-            _rows(c[z * cz:], m, n, ldc).copy_(_swiglu(v) if swiglu else v)
+            _rows(c[z * cz:], m, n, ldc).copy_(_glu(v, glu, limit) if glu else v)
     return run
 
 
@@ -89,13 +120,26 @@ def k_gemm_heads(g, a, w, c, m, n, k, ldc, heads, err):
         _rows(c[h * n:], m, n, ldc).copy_(_f(_rows(a[h * k:], m, k, lda)) @ W.t())
 
 
-def _k_grouped(swiglu):
-    def run(g, a, w, c, tiles, count, rows, n, k, wz, err):
+def _k_grouped(glu):
+    def run(g, a, w, c, tiles, count, rows, n, k, wz, err, limit):
         for e, r0, nr, _ in tiles.view(-1, 4)[: int(count[0])].tolist():
-            W = _f(w[e * wz: e * wz + (2 if swiglu else 1) * n * k].view(-1, k))
+            W = _f(w[e * wz: e * wz + (2 if glu else 1) * n * k].view(-1, k))
             v = _f(a[r0 * k:(r0 + nr) * k].view(nr, k)) @ W.t()
-            c[r0 * n:(r0 + nr) * n] = (_swiglu(v) if swiglu else v).to(c.dtype).reshape(-1)
+            c[r0 * n:(r0 + nr) * n] = (_glu(v, glu, limit) if glu else v).to(c.dtype).reshape(-1)
     return run
+
+
+def _k_moe_gemm(glu):
+    def run(g, a, w, c, tiles, count, rows, n, k, ldc, err, limit=0.0):
+        wz = n * k
+        for e, r0, nr, _ in tiles.view(-1, 4)[: int(count[0])].tolist():
+            v = _f(a[r0 * k:(r0 + nr) * k].view(nr, k)) @ _f(w[e * wz:(e + 1) * wz].view(n, k)).t()
+            _rows(c[r0 * ldc:], nr, ldc, ldc).copy_(_glu(v, glu, limit))
+    return run
+
+
+def k_copy_cols(g, src, dst, cols, stride):
+    _rows(dst, g[0], cols, stride).copy_(src[: g[0] * cols].view(g[0], cols))
 
 
 def k_rows_scatter(g, x, perm, out, entries, k, d):
@@ -179,6 +223,164 @@ def k_ssd_gate_norm(g, y, z, w, out, inner, parts, zs, eps):
     out[: n * inner] = v.to(out.dtype).reshape(-1)
 
 
+# ---- linear attention with a decay per key channel ----
+def _kept(state, line, line_bytes, width):
+    return state[line * line_bytes: line * line_bytes + width * 4].view(torch.float32)
+
+
+def k_token_shift(g, h, mu, out, state, lines, cu, seqs, d, targets, line_bytes):
+    m = _f(mu[: targets * d].view(targets, d))
+    for s in range(seqs):
+        r0, r1 = _rows_of(cu, s)
+        if r1 <= r0:
+            continue
+        ln = int(lines[s])
+        x = _f(h[r0 * d: r1 * d].view(-1, d))
+        last = _kept(state, ln, line_bytes, d) if ln > 0 else torch.zeros(d)
+        before = torch.cat([last[None], x[:-1]])
+        out[r0 * targets * d: r1 * targets * d] = (x[:, None] + (before - x)[:, None] * m).to(out.dtype).reshape(-1)
+        if not isinstance(cu, T) and ln > 0:
+            last.copy_(x[-1])
+
+
+def k_shift_state(g, h, state, lines, cu, seqs, d, line_bytes):
+    for s in range(seqs):
+        r0, r1 = _rows_of(cu, s)
+        if r1 > r0 and int(lines[s]) > 0:
+            _kept(state, int(lines[s]), line_bytes, d).copy_(_f(h[(r1 - 1) * d: r1 * d]))
+
+
+def k_decay(g, a, w, bias, alpha, rows, n, rank, lda, mode, inv_tau):
+    v = _f(_rows(a, rows, rank, lda))
+    z = (torch.tanh(v) if mode else v) @ _f(w[: n * rank].view(n, rank)).t() + _f(bias[:n])
+    alpha[: rows * n] = torch.exp(-torch.exp(z) if mode else F.logsigmoid(z) * inv_tau).reshape(-1)
+
+
+def k_lin_rule(g, q, k, v, gate, alpha, u, norm, out, state, lines, cu, seqs, H, dk, dv, stride, norm_step, out_stride, line_bytes, s_off, fused,
+               tb, max_rows, q_scale, out_scale, eps, min_rows=1):
+    for s in range(seqs):
+        r0, r1 = _rows_of(cu, s)
+        n = r1 - r0
+        if not min_rows <= n <= max_rows:
+            continue
+        ln = int(lines[s])
+        Sb = state[ln * line_bytes + s_off: ln * line_bytes + s_off + H * dk * dv * 4].view(torch.float32).view(H, dk, dv)
+        S = Sb.clone() if ln > 0 else torch.zeros(H, dk, dv)
+        part = lambda t, c: _f(_rows(t[r0 * stride:], n, H * c, stride)).view(n, H, c)
+        qq, kk, vv = part(q, dk) * q_scale, part(k, dk), part(v, dv)
+        al, o = alpha[r0 * H * dk: r1 * H * dk].view(n, H, dk), torch.empty(n, H, dv)
+        for t in range(n):
+            kv = kk[t][:, :, None] * vv[t][:, None, :]
+            if isinstance(u, T):
+                o[t] = torch.einsum("hkv,hk->hv", S + _f(u[: H * dk].view(H, dk, 1)) * kv, qq[t])
+            S = al[t][:, :, None] * S + kv
+            if not isinstance(u, T):
+                o[t] = torch.einsum("hkv,hk->hv", S, qq[t])
+        if fused:
+            k_lin_norm_gate((n,), o.reshape(-1), gate[r0 * stride:], norm, out[r0 * out_stride:], H, dv, stride, norm_step, out_stride, out_scale, eps)
+        else:
+            out[r0 * H * dv: r1 * H * dv] = o.reshape(-1)
+        if ln > 0:
+            Sb.copy_(S)
+
+
+def k_lin_chunk(g, q, k, v, alpha, u, out, state, lines, cu, seqs, H, dk, dv, stride, line_bytes, s_off, min_rows, q_scale):
+    k_lin_rule(g, q, k, v, 0, alpha, u, 0, out, state, lines, cu, seqs, H, dk, dv, stride, 0, 0, line_bytes, s_off, 0, 0, 1 << 31, q_scale, 1.0, 0.0, min_rows)
+
+
+def k_lin_norm_gate(g, o, gate, w, out, H, dv, gs, norm_step, os_, out_scale, eps):
+    n = g[0]
+    x = o[: n * H * dv].view(n, H, dv)
+    wt = _f(w[: H * dv].view(H, dv)) if norm_step else _f(w[:dv])
+    y = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * wt * out_scale
+    _rows(out, n, H * dv, os_).copy_(y.reshape(n, -1) * F.silu(_f(_rows(gate, n, H * dv, gs))))
+
+
+# ---- attention in a sliding window ----
+def _window_pool(cache, dt, hk, page, d, dv):
+    pool = cache.view(dt).view(-1, hk * page * (d + dv))
+    return pool[:, : hk * page * d].unflatten(1, (hk, page, d)), pool[:, hk * page * d:].unflatten(1, (hk, page, dv))
+
+
+def k_qk_prep(g, qkv, cache, positions, slots, cos, sin, qn, kn, hq, hk, d, dv, rot, halves, page, stride, max_pos, eps, err):
+    n = g[0]
+    rows, pos, sl = _rows(qkv, n, hq * d + hk * (d + dv), stride), positions[:n].long(), slots[:n].long()
+    if ((pos < 0) | (pos >= max_pos)).any():
+        err[0] = 300
+    pos = torch.where((pos < 0) | (pos >= max_pos), 0, pos)
+    c, s = (t.view(-1)[: max_pos * (rot // 2)].view(max_pos, rot // 2)[pos][:, None] for t in (cos, sin))
+
+    def turned(x, w):
+        x = _norm(x, w[:d], eps)
+        a, b = (x[..., : rot // 2], x[..., rot // 2: rot]) if halves else (x[..., :rot:2], x[..., 1:rot:2])
+        a, b = a * c - b * s, b * c + a * s
+        return torch.cat([a, b, x[..., rot:]] if halves else [torch.stack([a, b], -1).flatten(-2), x[..., rot:]], -1)
+
+    q = turned(_f(rows[:, : hq * d]).view(n, hq, d), qn)
+    k = turned(_f(rows[:, hq * d:(hq + hk) * d]).view(n, hk, d), kn).to(qkv.dtype)
+    v = rows[:, (hq + hk) * d:].reshape(n, hk, dv).clone()
+    rows[:, : hq * d] = q.reshape(n, -1).to(qkv.dtype)
+    ks, vs = _window_pool(cache, qkv.dtype, hk, page, d, dv)
+    ok = sl >= 0
+    ks[sl[ok] // page, :, sl[ok] % page] = k[ok]
+    vs[sl[ok] // page, :, sl[ok] % page] = v[ok]
+
+
+def _window_row(q, cache, out, pages, L, sink, hq, hk, d, dv, page, window, scale, cap, out_scale):
+    """One row at position L - 1: q [hq d] -> out [hq dv]."""
+    ks, vs = _window_pool(cache, q.dtype, hk, page, d, dv)
+    ids = pages[: -(-L // page)].long()
+    k, v = (_f(t[ids]).transpose(1, 2).reshape(-1, hk, t.shape[-1])[max(0, L - window):L].repeat_interleave(hq // hk, 1) for t in (ks, vs))
+    s = cap * torch.tanh(torch.einsum("hd,lhd->hl", _f(q).view(hq, d), k) * (scale / cap))
+    p = torch.softmax(torch.cat([s, _f(sink[:hq])[:, None]], 1), 1)[:, :-1]
+    out.copy_((torch.einsum("hl,lhv->hv", p, v) * out_scale).reshape(-1))
+
+
+def k_window_attn(g, q, cache, out, table, lens, row_seq, sink, hq, hk, d, dv, qs, os_, max_pages, page, window, scale, cap, out_scale, err):
+    tb = table.view(-1, max_pages)
+    for r in range(g[1]):
+        if int(lens[r]) > 0:
+            _window_row(q[r * qs: r * qs + hq * d], cache, out[r * os_: r * os_ + hq * dv], tb[int(row_seq[r]) if isinstance(row_seq, T) else r], int(lens[r]), sink,
+                        hq, hk, d, dv, page, window, scale, cap, out_scale)
+
+
+def _window_listed(q, cache, out, table, lens, cu, work, count, tokens, sink, hq, hk, d, qs, os_, max_pages, page, window, c1, c2, out_scale):
+    """The rows of a work list's (sequence, block) pairs, `tokens` to a block; without a list, one row per sequence."""
+    cap, tb = c2 / 1.4426950408889634, table.view(-1, max_pages)
+    scale = c1 * cap / (2 * 1.4426950408889634)
+    pairs = work.view(-1, 2)[: int(count[0])].tolist()
+    for s, b in pairs:
+        r0, r1 = int(cu[s]), int(cu[s + 1])
+        for t in range(b * tokens, min((b + 1) * tokens, r1 - r0)):
+            r = r0 + t
+            _window_row(q[r * qs: r * qs + hq * d], cache, out[r * os_: r * os_ + hq * d], tb[s], int(lens[s]) - (r1 - r0) + t + 1, sink, hq, hk, d, d, page, window,
+                        scale, cap, out_scale)
+
+
+def _k_window(prefill, d):
+    def run(g, kv, q, out, ws_o, ws_ml, table, lens, cu, work, count, hq, hk, qs, os_, max_pages, page, splits, pool_pages, err, sink, window, c1, c2, out_scale):
+        if isinstance(work, T):
+            _window_listed(q, kv, out, table, lens, cu, work, count, (64 if prefill else 16) // (hq // hk), sink, hq, hk, d, qs, os_, max_pages, page, window, c1, c2, out_scale)
+        else:      # a split launch is followed by the merge; here it writes the finished rows and the merge is a no-op
+            one = torch.arange(g[1] + 1, dtype=torch.int32)
+            pairs = torch.stack([one[:-1], torch.zeros(g[1], dtype=torch.int32)], 1)
+            live = [i for i in range(g[1]) if int(lens[i]) > 0]
+            _window_listed(q, kv, out, table, lens, one, pairs[live].contiguous(), torch.tensor([len(live)]), 1, sink, hq, hk, d, qs, os_, max_pages, page, window, c1, c2,
+                           out_scale)
+    return run
+
+
+def _k_window_ragged(d):
+    def run(g, kv, q, out, table, lens, cu, wp, cp, wd, cd, hq, hk, qs, os_, max_pages, page, pool_pages, err, sink, window, c1, c2, out_scale):
+        for w, c, rows in ((wp, cp, 64), (wd, cd, 16)):
+            _window_listed(q, kv, out, table, lens, cu, w, c, rows // (hq // hk), sink, hq, hk, d, qs, os_, max_pages, page, window, c1, c2, out_scale)
+    return run
+
+
+def k_window_fmha(g, kv, q, out, table, lens, cu, work, count, hq, hk, qs, os_, max_pages, page, pool_pages, err, sink, window, c1, c2, out_scale):
+    _window_listed(q, kv, out, table, lens, cu, work, count, 128 // (hq // hk), sink, hq, hk, 128, qs, os_, max_pages, page, window, c1, c2, out_scale)
+
+
 # ---- latent attention ----
 def k_latent_append(g, lat, cache, slots, w, rank, stride, eps):
     n = g[0]
@@ -217,18 +419,39 @@ def k_route_logits(g, logits, bias, ids, w, tokens, E, k, ld):
     w[: tokens * k] = torch.softmax(torch.gather(z, 1, order), -1).reshape(-1)
 
 
+def k_route_groups(g, logits, ids, w, tokens, E, k, groups, keep, renorm, ld):
+    s = torch.sigmoid(_rows(logits, tokens, E, ld))
+    of = s.view(tokens, groups, -1)
+    best = torch.argsort(of.topk(min(2, E // groups), -1).values.sum(-1), dim=-1, descending=True, stable=True)[:, :keep]
+    may = torch.zeros(tokens, groups, dtype=torch.bool).scatter_(1, best, True).repeat_interleave(E // groups, 1)
+    order = torch.argsort(s.masked_fill(~may, -1.0), dim=-1, descending=True, stable=True)[:, :k]
+    top = torch.gather(s, 1, order)
+    ids[: tokens * k] = order.to(ids.dtype).reshape(-1)
+    w[: tokens * k] = (top / top.sum(-1, keepdim=True) if renorm else top).reshape(-1)
+
+
 for _a in ("bf16", "f32"):
     CPU_KERNELS.update({f"kern_hyper_embed_{_a}": k_hyper_embed, f"kern_row_norm_f32_{_a}": k_row_norm,
                         f"kern_rows_scatter_{_a}": k_rows_scatter, f"kern_gate_mul_{_a}": k_gate_mul,
-                        f"kern_linear_{_a}": _k_linear(False), f"kern_linear_{_a}_swiglu": _k_linear(True),
-                        f"kern_linear_grouped_{_a}": _k_grouped(False), f"kern_linear_grouped_{_a}_swiglu": _k_grouped(True),
+                        f"kern_resid_embed_{_a}": k_resid_embed, f"kern_resid_mix_{_a}": k_resid_mix,
+                        f"kern_token_shift_{_a}": k_token_shift, f"kern_shift_state_{_a}": k_shift_state, f"kern_decay_{_a}": k_decay,
+                        f"kern_lin_norm_gate_{_a}": k_lin_norm_gate, f"kern_qk_prep_{_a}": k_qk_prep,
                         f"kern_ssd_conv_{_a}": k_ssd_conv, f"kern_ssd_conv_state_{_a}": k_ssd_conv_state,
                         f"kern_ssd_gate_norm_{_a}": k_ssd_gate_norm, f"kern_latent_append_{_a}": k_latent_append})
     CPU_KERNELS.update({f"kern_hyper_{k}_{_a}_s{s}": f for s in range(5) for k, f in (("mix", k_hyper_mix), ("last", k_hyper_last))})
     CPU_KERNELS.update({f"kern_ssd_rule_{_a}_n{n}": k_ssd_rule for n in (32, 64, 128, 256, 512)})
+    CPU_KERNELS.update({f"kern_{k}_{_a}{'_' + e if e else ''}": f(e) for k, f in (("linear", _k_linear), ("linear_grouped", _k_grouped))
+                        for e in ("", "swiglu", "geglu", "clamped")})
+    CPU_KERNELS.update({f"kern_lin_rule_{_a}_r{r}_v{v}": k_lin_rule for r in (4, 8, 16, 32) for v in (1, 2, 4)})
+    CPU_KERNELS.update({f"kern_window_attn_{_a}_w{w}": k_window_attn for w in (64, 128, 256, 512)})
     CPU_KERNELS.update({f"kern_latent_attn_{_a}_w{w}": k_latent_attn for w in (64, 128, 256, 512, 1024)})
-CPU_KERNELS.update({"kern_linear_bf16_f32": _k_linear(False), "kern_transpose_heads_bf16": k_transpose_heads,
-                    "kern_moe_route_logits": k_route_logits})
+CPU_KERNELS.update({"kern_linear_bf16_f32": _k_linear(""), "kern_transpose_heads_bf16": k_transpose_heads, "kern_copy_cols_bf16": k_copy_cols,
+                    "kern_moe_route_logits": k_route_logits, "kern_moe_route_groups": k_route_groups, "kern_attn_window_fmha_d128": k_window_fmha,
+                    "kern_attn_window_merge": lambda *a: None})
+CPU_KERNELS.update({f"kern_moe_gemm_bf16_{e}_n{n}": _k_moe_gemm(e) for e in ("geglu", "clamped") for n in (64, 128)})
+CPU_KERNELS.update({f"kern_lin_chunk_n{n}": k_lin_chunk for n in (32, 64, 128, 256)})
+CPU_KERNELS.update({f"kern_attn_window_{k}_d{d}": _k_window(k == "prefill", d) for k in ("decode", "prefill") for d in (64, 128, 256)})
+CPU_KERNELS.update({f"kern_attn_window_ragged_d{d}": _k_window_ragged(d) for d in (64, 128)})
 CPU_KERNELS.update({f"kern_gemm_bf16_heads_n{n}": k_gemm_heads for n in (64, 128, 256)})
 CPU_KERNELS.update({f"kern_ssd_chunk_n{n}": k_ssd_chunk for n in (32, 64, 128, 256)})
 CPU_KERNELS.update({f"kern_latent_decode_bf16_b{b}": k_latent_decode for b in range(1, 9)})

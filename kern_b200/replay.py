@@ -31,7 +31,7 @@ def open_engine(model, dtype: str, max_tokens: int, slots: int = 4, cpu: bool = 
 
     page = 64
     tokens = max(page, -(-max_tokens // page) * page)
-    cfg, build = registry.from_folder(model, dtype=DTYPES[dtype], page_size=page, max_tokens=min(ROWS, tokens), max_seqs=max(4, slots))
+    cfg, build = registry.from_folder(model, dtype=DTYPES[dtype], page_size=page, max_tokens=min(ROWS, tokens), max_seqs=max(4, slots), max_context=tokens)
     doc = build(cfg)
     stateful = any(s.get("bytes_per_seq") for s in doc["states"].values())
     if cpu:
