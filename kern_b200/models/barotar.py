@@ -220,7 +220,7 @@ def build_manifest(cfg: BarotarConfig) -> dict:
     windows = [i for i, b in enumerate(layers) if b["type"] == "parallel"]
     tiled = {i: K.window_tiles(*(layers[i]["mixer"]["left"][k] for k in ("heads", "kv_heads", "dim", "vdim")), page, A) for i in windows}
     untiled = [i for i in windows if not tiled[i]]
-    m_.inputs(f"kv.l{windows[0]}" if windows else None, "lin.l0", row_plan=bool(untiled))
+    m_.inputs(f"kv.l{windows[0]}" if windows else None, "lin.l0", positions=bool(windows), row_plan=bool(untiled))
     room("x", d, "f32")
     room("xn", d)
     m_.outputs()
@@ -242,18 +242,20 @@ def build_manifest(cfg: BarotarConfig) -> dict:
         """The recurrence from its projections (`ptrs`: q, k, v, gate) to the gated rows in `out`."""
         sfx, fused = "_p" if prefill else "_d", not prefill and K.lin_fused(dv)
         tag = f"{sfx}_{H}x{dk}x{dv}x{stride}x{out_stride}" + ("u" if u else "") + f"_{out_scale:g}"
-        rule = op(f"lin{tag}", lambda: K.lin_rule_op(H, dk, dv, stride, z["line"], z["s_off"], prefill, A, bonus=u is not None, q_scale=q_scale, fused=fused,
-                                                     norm_shared=norm_shared, out_stride=out_stride, out_scale=out_scale, eps=eps))
-        if not fused:
-            room("lin.o", H * dv, "f32")
-        cu = [B("cu_seqlens")] if prefill else []
+
+        def make():
+            rule = K.lin_rule_op(H, dk, dv, stride, z["line"], z["s_off"], prefill, A, bonus=u is not None, q_scale=q_scale, fused=fused, norm_shared=norm_shared,
+                                 out_stride=out_stride, out_scale=out_scale, eps=eps)
+            if fused:
+                return rule
+            ng = K.lin_norm_gate_op(H, dv, stride, norm_shared, out_stride, out_scale, eps, A)
+            return K.chain_ops(rule, ng, inner={(0, 5 if u else 4): "o", (1, 0): "o"}, scratch={"o": {"dtype": "f32", "shape": ["tokens", H * dv]}})
+
         q, k, v, gate = ptrs
-        calls = [{"op": rule, "label": p + "rule", "args": [q, k, v, B("alpha"), *([u] if u else []), out if fused else B("lin.o"), {"state": st}, B("lines"), *cu,
-                                                            *([gate, norm] if fused else []), V("seqs")]}]
-        if not fused:
-            ng = op(f"lin_norm_gate{tag}", lambda: K.lin_norm_gate_op(H, dv, stride, norm_shared, out_stride, out_scale, eps, A))
-            calls.append({"op": ng, "label": p + "norm", "args": [B("lin.o"), gate, norm, out]})
-        return calls
+        head, cu = [q, k, v, B("alpha"), *([u] if u else [])], [B("cu_seqlens")] if prefill else []
+        state = [{"state": st}, B("lines"), *cu]
+        args = [*head, out, *state, gate, norm, V("seqs")] if fused else [*head, *state, V("seqs"), gate, norm, out]
+        return [{"op": op(f"lin{tag}", make), "label": p + "rule", "args": args}]
 
     def gla(i: int, at: int, prefill: bool) -> list[dict]:
         m, p, rank = layers[i]["mixer"], f"l{i}.mix.", cfg.ranks[i]
@@ -282,26 +284,28 @@ def build_manifest(cfg: BarotarConfig) -> dict:
             m_.once.append({"op": op(f"rope_{dims}x{base:g}", lambda: C.rope_table_op(cfg.context, dims, base)), "label": name, "args": [B(name + ".cos"), B(name + ".sin")]})
         return [B(name + ".cos"), B(name + ".sin")]
 
-    def plan(i: int) -> tuple[list[dict], list[dict]]:
-        """-> (the work lists of a ragged call's tensor-core attention, the call that fills them, at their first layer); layers whose
-        blocks hold as many tokens share them."""
+    plans = {}      # name -> (work lists, op, args): the plans of a ragged call's attention, made with the embedding
+
+    def lists_of(i: int) -> list[dict]:
+        """The work lists of layer i's tensor-core attention; layers whose blocks hold as many tokens share them."""
         l = layers[i]["mixer"]["left"]
-        g = l["heads"] // l["kv_heads"]
-        name = f"plan.{g}" + (".128" if l["dim"] == 128 else "")
-        if name + ".work_p" not in bufs:
-            items = cfg.max_tokens // (64 // g) + S + 1
+        hq, hk, dim = l["heads"], l["kv_heads"], l["dim"]
+        name = f"plan.{hq // hk}" + (".128" if dim == 128 else "")
+        if name not in plans:
+            items = cfg.max_tokens // (64 // (hq // hk)) + S + 1
             for n, shape in ((".work_p", [items, 2]), (".count_p", [1]), (".work_d", [S, 2]), (".count_d", [1])):
                 bufs[name + n] = {"dtype": "i32", "shape": shape, "kind": "workspace"}
-        lists = [B(name + n) for n in (".work_p", ".count_p", ".work_d", ".count_d")]
-        if i == next(j for j in windows if tiled[j] and plan_key(j) == plan_key(i)):
-            make = op("attn_" + name, lambda: C.attn_plan_op(l["heads"], l["kv_heads"], S, l["dim"]))
-            items = {"expr": C.attn_plan_items(l["heads"], l["kv_heads"])}
-            return lists, [{"op": make, "label": f"l{i}.plan", "args": [B("cu_seqlens"), lists[0], lists[1], V("seqs"), items, lists[2], lists[3]]}]
-        return lists, []
+            lists = [B(name + n) for n in (".work_p", ".count_p", ".work_d", ".count_d")]
+            args = [B("cu_seqlens"), lists[0], lists[1], V("seqs"), {"expr": C.attn_plan_items(hq, hk)}, lists[2], lists[3]]
+            plans[name] = lists, C.attn_plan_op(hq, hk, S, dim), args
+        return plans[name][0]
 
-    def plan_key(i: int):
-        l = layers[i]["mixer"]["left"]
-        return l["heads"] // l["kv_heads"], l["dim"] == 128
+    def row_plan() -> list[dict]:
+        """The table row and reach of every token, for attention that takes a row per token."""
+        if "rows" not in plans:
+            c = m_.rows_call("")
+            plans["rows"] = [B("row_seq")], m_.ops.pop(c["op"]), c["args"]
+        return plans["rows"][0]
 
     def parallel(i: int, at: int, prefill: bool) -> list[dict]:
         m, p, rank = layers[i]["mixer"], f"l{i}.mix.", cfg.ranks[i]
@@ -316,15 +320,12 @@ def build_manifest(cfg: BarotarConfig) -> dict:
         prep = op(f"prep_{hq}x{hk}x{dim}x{vdim}x{l['rot']['dims']}", lambda: K.qk_prep_op(hq, hk, dim, vdim, l["rot"]["dims"], page, qkv, cfg.context, eps, A))
         attn = op(f"window_attn{sfx}_{hq}x{hk}x{dim}x{vdim}x{l['mask']['size']}x{both}_{l['scale']:.6g}_{l['softcap']:g}_{m['left_scale']:g}", lambda: K.window_attn_op(
             hq, hk, dim, vdim, l["mask"]["size"], l["scale"], l["softcap"], page, W, qkv, both, m["left_scale"], prefill, A, seqs_max=S))
-        calls, lens, lists = [], B("seq_lens"), []
+        lens, lists = B("seq_lens"), []
         if prefill and tiled[i]:
-            lists, calls = plan(i)
-            lists = [B("cu_seqlens"), *lists]
+            lists = [B("cu_seqlens"), *lists_of(i)]
         elif prefill:
-            lens, lists = B("row_len"), [B("row_seq")]
-            if i == untiled[0]:
-                calls = [m_.rows_call(p + "rows")]
-        calls += [
+            lens, lists = B("row_len"), row_plan()
+        calls = [
             linear("lin", qkv, d, B("xn"), w_in, B("qkv"), label=lp + "qkv"),
             {"op": prep, "label": lp + "prep", "args": [B("qkv"), {"state": kv}, B("positions"), B("slot_mapping"), *cos_sin, same(lp + "q.norm", (dim,)),
                                                         same(lp + "k.norm", (dim,)), err]},
@@ -366,15 +367,16 @@ def build_manifest(cfg: BarotarConfig) -> dict:
         return m_.routed(p, E, k, x["ff"], pick, "clamped", x["limit"]) + [finish(at, B("moe.y"), p + "mlp.out", k, [B("moe.perm"), B("moe.w")])]
 
     def forward(prefill: bool) -> list[dict]:
-        embed = op("embed", lambda: K.resid_embed_op(d, cfg.vocab, eps, A))
-        calls = [{"op": embed, "label": "embed", "args": [B("token_ids"), same("embed", (cfg.vocab, d)), same(subs[0][0], (d,)), B("x"), B("xn"), err]}]
-        at = 0
+        calls, at = [], 0
         for i, b in enumerate(layers):
             calls += (gla if b["type"] == "gla" else parallel)(i, at, prefill)
             at += 1
             if b["mlp"] is not None:
                 calls += (dense if b["mlp"]["kind"] == "dense" else routed)(i, at)
                 at += 1
-        return calls
+        args = [B("token_ids"), same("embed", (cfg.vocab, d)), same(subs[0][0], (d,)), B("x"), B("xn"), err]
+        first = plans.values() if prefill else ()      # in one call with the embedding: both programs have as many calls to every layer
+        name = op("embed" + ("_p" if prefill else "_d"), lambda: K.chain_ops(K.resid_embed_op(d, cfg.vocab, eps, A), *[o for _, o, _ in first]))
+        return [{"op": name, "label": "embed", "args": args + [a for _, _, more in first for a in more]}, *calls]
 
     return m_.document(forward, "embed")

@@ -25,6 +25,33 @@ L = lambda v: {"i64": v}
 NULL = ("i64", {"i64": 0})
 
 
+def chain_ops(*ops, inner: dict | None = None, scratch: dict | None = None) -> dict:
+    """Ops one after the other as one op (one call of a program): the interfaces in order, without the params that `inner` —
+    {(op, param): scratch name} — ties together through `scratch`."""
+    inner, iface, launches, room = inner or {}, [], [], dict(scratch or {})
+    for n, o in enumerate(ops):
+        at = {}
+        for i, t in enumerate(o["params"]):
+            if (n, i) not in inner:
+                at[i] = len(iface)
+                iface.append(t)
+
+        def sub(x):
+            if isinstance(x, list):
+                return [sub(v) for v in x]
+            if not isinstance(x, dict):
+                return x
+            if set(x) == {"param"} and (n, x["param"]) in inner:
+                return {"scratch": inner[n, x["param"]]}
+            if set(x) == {"scratch"}:
+                return {"scratch": f"{n}.{x['scratch']}"}
+            return {k: at[v] if k == "param" else (v if k == "when" else sub(v)) for k, v in x.items()}
+
+        launches += [sub(l) | {"params": l["params"]} for l in o["impl"]["launches"]]
+        room |= {f"{n}.{k}": v for k, v in o["impl"].get("scratch", {}).items()}
+    return _op(iface, *launches, **({"scratch": room} if room else {}))
+
+
 def tiles_fit(*extents: int) -> bool:
     """Whether rows of these lengths are whole 16-byte vectors of bf16, which the tensor-core tiles and TMA need."""
     return all(e % 8 == 0 for e in extents)

@@ -73,13 +73,14 @@ class Listed:
         return {"op": name, "label": label, "args": [a, w, c, self.V(rows), self.err]}
 
     # ---- inputs and outputs ----
-    def inputs(self, paged: str | None, lined: str | None, row_plan: bool = True) -> None:
-        """The host's columns. `paged` / `lined`: a paged and a per-sequence state, when the model has them; `row_plan`: room for
-        every token's table row and reach (`rows_call`)."""
+    def inputs(self, paged: str | None, lined: str | None, positions: bool = True, row_plan: bool = True) -> None:
+        """The host's columns. `paged` / `lined`: a paged and a per-sequence state, when the model has them; `positions`: whether
+        anything reads them; `row_plan`: room for every token's table row and reach (`rows_call`)."""
         cfg, S = self.cfg, self.cfg.max_seqs
         inp = lambda dt, shape, **kw: {"dtype": dt, "shape": shape, "kind": "input", **kw}
         self.bufs["token_ids"] = inp("i64", ["tokens"], fill="token", domain={"min": 0, "max": cfg.vocab - 1})
-        self.bufs["positions"] = inp("i64", ["tokens"], fill="position", domain={"min": 0, "max": cfg.context - 1})
+        if positions:
+            self.bufs["positions"] = inp("i64", ["tokens"], fill="position", domain={"min": 0, "max": cfg.context - 1})
         self.bufs["cu_seqlens"] = inp("i32", [S + 1], fill="cu_seqlens")
         if paged:
             self.bufs["slot_mapping"] = inp("i64", ["tokens"], fill="slot", domain={"index_into": paged})
