@@ -77,7 +77,7 @@ constexpr int DB = 64, DK = 16;
 template <typename T>
 KERN_DEVICE void decay_body(const T* a, const __nv_bfloat16* W, const __nv_bfloat16* bias, float* alpha, int rows, int n, int rank,
                             int lda, int mode, float inv_tau) {
-  __shared__ float as[DK][DB + 4], ws[DK][DB + 4];
+  __shared__ __align__(16) float as[DK][DB + 4], ws[DK][DB + 4];
   const int m0 = blockIdx.y * DB, n0 = blockIdx.x * DB;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {};
@@ -90,25 +90,36 @@ KERN_DEVICE void decay_body(const T* a, const __nv_bfloat16* W, const __nv_bfloa
     }
     __syncthreads();
 #pragma unroll
-    for (int k = 0; k < DK; ++k)
+    for (int k = 0; k < DK; ++k) {
+      const Vec<4> x = ldv<4>(&as[k][ty * 4]), w = ldv<4>(&ws[k][tx * 4]);
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] += as[k][ty * 4 + i] * ws[k][tx * 4 + j];
+        for (int j = 0; j < 4; ++j) acc[i][j] += x.v[i] * w.v[j];
+    }
     __syncthreads();
   }
+  const int c = n0 + tx * 4;
+  float b[4];
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    const int c = n0 + tx * 4 + j;
-    if (c >= n) continue;
-    const float b = __bfloat162float(bias[c]);
+  for (int j = 0; j < 4; ++j) b[j] = c + j < n ? __bfloat162float(bias[c + j]) : 0.f;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int r = m0 + ty * 4 + i;
-      if (r >= rows) continue;
-      const float z = acc[i][j] + b;
-      const float lg = mode ? -expf(z) : -(fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))) * inv_tau;
-      alpha[(size_t)r * n + c] = expf(lg);
+  for (int i = 0; i < 4; ++i) {
+    const int r = m0 + ty * 4 + i;
+    if (r >= rows) continue;
+    Vec<4> o;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float z = acc[i][j] + b[j];
+      o.v[j] = expf(mode ? -expf(z) : -(fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))) * inv_tau);
+    }
+    float* dst = alpha + (size_t)r * n + c;
+    if (n % 4 == 0) {
+      if (c < n) stv<4>(dst, o);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j < n) dst[j] = o.v[j];
     }
   }
 }

@@ -241,11 +241,11 @@ def build_manifest(cfg: BarotarConfig) -> dict:
                          out_scale) -> list[dict]:
         """The recurrence from its projections (`ptrs`: q, k, v, gate) to the gated rows in `out`."""
         sfx, fused = "_p" if prefill else "_d", not prefill and K.lin_fused(dv)
-        tag = f"{sfx}_{H}x{dk}x{dv}x{stride}x{out_stride}" + ("u" if u else "") + f"_{out_scale:g}"
+        tag = f"{sfx}_{H}x{dk}x{dv}x{stride}x{out_stride}" + ("u" if u else "") + f"_{out_scale!r}"
 
         def make():
             rule = K.lin_rule_op(H, dk, dv, stride, z["line"], z["s_off"], prefill, A, bonus=u is not None, q_scale=q_scale, fused=fused, norm_shared=norm_shared,
-                                 out_stride=out_stride, out_scale=out_scale, eps=eps)
+                                 out_stride=out_stride, out_scale=out_scale, eps=eps, rows_max=cfg.max_tokens, seqs_max=S)
             if fused:
                 return rule
             ng = K.lin_norm_gate_op(H, dv, stride, norm_shared, out_stride, out_scale, eps, A)
@@ -264,7 +264,7 @@ def build_manifest(cfg: BarotarConfig) -> dict:
         states[st] = {"bytes_per_seq": z["line"]}
         w_in, proj = m_.rows_weight(f"w.{p}qkvga", d, [(p + "q", q), (p + "k", q), (p + "v", v), (p + "g", v), (p + "a1", rank)])
         room("proj", proj); room("alpha", q, "f32"); room("mixed", v); room("y", d)
-        decay = op(f"decay_{q}x{rank}x{proj}_{m['tau']:g}", lambda: K.decay_op(q, rank, proj, "root", m["tau"], A))
+        decay = op(f"decay_{q}x{rank}x{proj}_{m['tau']!r}", lambda: K.decay_op(q, rank, proj, "root", m["tau"], A))
         col = lambda c: B("proj", c * es)
         return [
             linear("lin", proj, d, B("xn"), w_in, B("proj"), label=p + "in"),
@@ -277,11 +277,11 @@ def build_manifest(cfg: BarotarConfig) -> dict:
 
     def rotary(dims: int, base: float) -> list[dict]:
         """The cos and sin tables of one rotation, written when the model is loaded."""
-        name = f"rope.{dims}x{base:g}"
+        name = f"rope.{dims}x{base!r}"
         if name + ".cos" not in bufs:
             for n in (".cos", ".sin"):
                 bufs[name + n] = {"dtype": "f32", "shape": [cfg.context, dims // 2], "kind": "carry"}
-            m_.once.append({"op": op(f"rope_{dims}x{base:g}", lambda: C.rope_table_op(cfg.context, dims, base)), "label": name, "args": [B(name + ".cos"), B(name + ".sin")]})
+            m_.once.append({"op": op(f"rope_{dims}x{base!r}", lambda: C.rope_table_op(cfg.context, dims, base)), "label": name, "args": [B(name + ".cos"), B(name + ".sin")]})
         return [B(name + ".cos"), B(name + ".sin")]
 
     plans = {}      # name -> (work lists, op, args): the plans of a ragged call's attention, made with the embedding
@@ -318,7 +318,7 @@ def build_manifest(cfg: BarotarConfig) -> dict:
         # left: window attention into columns 0 .. o of `mixed`
         cos_sin = rotary(l["rot"]["dims"], l["rot"]["base"])
         prep = op(f"prep_{hq}x{hk}x{dim}x{vdim}x{l['rot']['dims']}", lambda: K.qk_prep_op(hq, hk, dim, vdim, l["rot"]["dims"], page, qkv, cfg.context, eps, A))
-        attn = op(f"window_attn{sfx}_{hq}x{hk}x{dim}x{vdim}x{l['mask']['size']}x{both}_{l['scale']:.6g}_{l['softcap']:g}_{m['left_scale']:g}", lambda: K.window_attn_op(
+        attn = op(f"window_attn{sfx}_{hq}x{hk}x{dim}x{vdim}x{l['mask']['size']}x{both}_{l['scale']!r}_{l['softcap']!r}_{m['left_scale']!r}", lambda: K.window_attn_op(
             hq, hk, dim, vdim, l["mask"]["size"], l["scale"], l["softcap"], page, W, qkv, both, m["left_scale"], prefill, A, seqs_max=S))
         lens, lists = B("seq_lens"), []
         if prefill and tiled[i]:

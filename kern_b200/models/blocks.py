@@ -342,10 +342,10 @@ def lin_fused(dv: int) -> bool:
 
 def lin_rule_op(heads: int, dk: int, dv: int, stride: int, line_bytes: int, s_off: int, ragged: bool, act: str = "bf16", *, bonus: bool,
                 q_scale: float = 1.0, fused: bool = False, norm_shared: bool = True, out_stride: int = 0, out_scale: float = 1.0,
-                eps: float = 0.0) -> dict:
+                eps: float = 0.0, rows_max: int = 0, seqs_max: int = 0) -> dict:
     """S = diag(alpha) S + k v^T and its read by q. Interface [q, k, v, alpha, (u,) out, state, lines, (cu_seqlens,) seqs]; `fused`
     (out is then the normed, weighed and gated activation, else f32 rows) adds [gate, norm w] before the last. q, k, v and gate
-    share their row stride."""
+    share their row stride. `rows_max`, `seqs_max`: the largest ragged call, which sizes what the chunks' preparation leaves behind."""
     if dk > LIN_DIMS:
         raise ValueError(f"{dk} key channels per head (at most {LIN_DIMS})")
     out_t = f"out buffer<{act if fused else 'f32'}>"
@@ -372,13 +372,16 @@ def lin_rule_op(heads: int, dk: int, dv: int, stride: int, line_bytes: int, s_of
         return _op(iface, rule)
     # a ragged call's long sequences in chunks on the tensor cores, its few-row ones (decode rows among prompts) row by row
     np_ = next(n for n in (32, 64, 128, 256) if dk <= n)
-    prep = 5 * 16 * (np_ + 8) * 2 + 3 * 16 * 24 * 2 + np_ * 4
-    smem = 2 * prep + 2 * 16 * np_ * 8 + 3 * 16 * 72 * 2 + np_ * 4
-    args = pick("q", "k", "v", "alpha", "u", "out", "state", "lines", "cu", "seqs")
-    chunk = _launch("lin_attn_chunk", f"kern_lin_chunk_n{np_}", [256, 1, 1], [heads * -(-dv // 64), "seqs", 1],
-                    [t for t, _ in args] + ["i32"] * 4 + ["i64", "i32", "i32", "f32"],
-                    [a for _, a in args] + [I(heads), I(dk), I(dv), I(stride), L(line_bytes), I(s_off), I(LIN_CHUNK_MIN), {"f32": q_scale}], shared_mem=smem)
-    return _op(iface, chunk, rule)
+    block = 5 * 16 * (np_ + 8) * 2 + 3 * 16 * 24 * 2 + np_ * 4
+    slots = rows_max // 16 + seqs_max + 1
+    pick_t = lambda args: ([t for t, _ in args], [a for _, a in args])
+    types, args = pick_t(pick("q", "k", "alpha", "u") + [("out buffer<u8>", {"scratch": "prep"})] + pick("cu", "seqs"))
+    prep = _launch("lin_attn_chunk", f"kern_lin_prep_n{np_}", [128, 1, 1], [{"add": [{"ceil_div": ["tokens", 16]}, "seqs"]}, heads, 1], types + ["i32"] * 5 + ["f32"],
+                   args + [I(heads), I(dk), I(stride), I(LIN_CHUNK_MIN), I(slots), {"f32": q_scale}], shared_mem=16 * np_ * 8 + np_ * 4)
+    types, args = pick_t(pick("v") + [("in buffer<u8>", {"scratch": "prep"})] + pick("out", "state", "lines", "cu", "seqs"))
+    chunk = _launch("lin_attn_chunk", f"kern_lin_chunk_n{np_}", [128, 1, 1], [heads * -(-dv // 64), "seqs", 1], types + ["i32"] * 4 + ["i64", "i32", "i32"],
+                    args + [I(heads), I(dk), I(dv), I(stride), L(line_bytes), I(s_off), I(LIN_CHUNK_MIN)], shared_mem=4 * (block + 16 * 72 * 2))
+    return _op(iface, prep, chunk, rule, scratch={"prep": {"dtype": "u8", "shape": [slots, heads * block]}})
 
 
 def lin_norm_gate_op(heads: int, dv: int, gate_stride: int, norm_shared: bool, out_stride: int, out_scale: float, eps: float, act: str = "bf16") -> dict:

@@ -131,7 +131,7 @@ class Listed:
         for name, shape in (("moe.offsets", [E + 1]), ("moe.tiles", [tiles, 4]), ("moe.tile_count", [1]), ("moe.rows", [1])):
             have = self.bufs.get(name, {"shape": [0]})["shape"]
             self.bufs[name] = {"dtype": "i32", "shape": [max(have[0], shape[0]), *shape[1:]], "kind": "workspace"}
-        tag = f"{d}x{ff}x{E}x{k}" + (f"_{glu}{limit:g}" if glu != "swiglu" else "")
+        tag = f"{d}x{ff}x{E}x{k}" + (f"_{glu}{limit!r}" if glu != "swiglu" else "")
         if f"moe_plan_{tag}" not in self.ops:
             for n, o in K.routed_ops(d, ff, E, k, T, A, glu, limit).items():
                 self.ops[f"{n}_{tag}"] = o

@@ -284,7 +284,13 @@ def k_lin_rule(g, q, k, v, gate, alpha, u, norm, out, state, lines, cu, seqs, H,
             Sb.copy_(S)
 
 
-def k_lin_chunk(g, q, k, v, alpha, u, out, state, lines, cu, seqs, H, dk, dv, stride, line_bytes, s_off, min_rows, q_scale):
+def k_lin_prep(g, q, k, alpha, u, prep, cu, seqs, H, dk, stride, min_rows, slots, q_scale):
+    """The real buffer holds scaled and split factors; here the chunk kernel's statement is handed the arguments themselves."""
+    prep._rows = (q, k, alpha, u, q_scale)
+
+
+def k_lin_chunk(g, v, prep, out, state, lines, cu, seqs, H, dk, dv, stride, line_bytes, s_off, min_rows):
+    q, k, alpha, u, q_scale = prep._rows
     k_lin_rule(g, q, k, v, 0, alpha, u, 0, out, state, lines, cu, seqs, H, dk, dv, stride, 0, 0, line_bytes, s_off, 0, 0, 1 << 31, q_scale, 1.0, 0.0, min_rows)
 
 
@@ -449,7 +455,7 @@ CPU_KERNELS.update({"kern_linear_bf16_f32": _k_linear(""), "kern_transpose_heads
                     "kern_moe_route_logits": k_route_logits, "kern_moe_route_groups": k_route_groups, "kern_attn_window_fmha_d128": k_window_fmha,
                     "kern_attn_window_merge": lambda *a: None})
 CPU_KERNELS.update({f"kern_moe_gemm_bf16_{e}_n{n}": _k_moe_gemm(e) for e in ("geglu", "clamped") for n in (64, 128)})
-CPU_KERNELS.update({f"kern_lin_chunk_n{n}": k_lin_chunk for n in (32, 64, 128, 256)})
+CPU_KERNELS.update({f"kern_lin_{k}_n{n}": f for k, f in (("prep", k_lin_prep), ("chunk", k_lin_chunk)) for n in (32, 64, 128, 256)})
 CPU_KERNELS.update({f"kern_attn_window_{k}_d{d}": _k_window(k == "prefill", d) for k in ("decode", "prefill") for d in (64, 128, 256)})
 CPU_KERNELS.update({f"kern_attn_window_ragged_d{d}": _k_window_ragged(d) for d in (64, 128)})
 CPU_KERNELS.update({f"kern_gemm_bf16_heads_n{n}": k_gemm_heads for n in (64, 128, 256)})

@@ -1,19 +1,20 @@
-"""Prefill and decode throughput of the Gafapel decoder beside the framework's closest model at equal size, with the time of
-every kind of kernel against its roofline: `python bench.py --config gafapel [--layers N]`.
+"""Prefill and decode throughput of a decoder with listed layers beside the framework's closest model at equal size, with the
+time of every kind of kernel against its roofline: `python bench.py --config gafapel|barotar [--layers N]`.
 
-Both decoders have the width, depth, vocabulary and routed experts of the 48B-A3B shape class and random weights; one has
-Mamba-2 and unrotated latent-attention layers over four residual streams, the other per-key-decay delta-rule layers and
-512 + 64 latent attention over one. A point is timed end to end (CUDA events around the call, captured graphs for decode,
+The decoders have the width, depth, vocabulary and routed experts of the 48B-A3B shape class and random weights. Gafapel has
+Mamba-2 and unrotated latent-attention layers over four residual streams, Barotar window attention beside time mixing and gated
+linear attention; the model beside them per-key-decay delta-rule layers and 512 + 64 latent attention. Beside Barotar there is
+also the routed decoder with grouped-query attention of the same head counts and dims, for its attention kernels. A point is timed end to end (CUDA events around the call, captured graphs for decode,
 L2 flushed before every sample) and once more call by call, where a call's roofline is the larger of its bytes over the
 measured copy rate and its flops over the measured tensor rate.
 """
 from __future__ import annotations
 
 import json
-import os
+import re
 from pathlib import Path
 
-MODELS = ("gafapel-48b-a3b", "latent-48b-a3b")
+MODELS = {"gafapel": ("gafapel-48b-a3b", "latent-48b-a3b"), "barotar": ("barotar-48b-a3b", "latent-48b-a3b", "moe-30b-a3b")}
 POINTS = ({"groups": 1, "chunk": 2048, "context": 2048}, {"groups": 4, "chunk": 512, "context": 2048},
           {"groups": 1, "rows": 1, "context": 1024}, {"groups": 16, "rows": 1, "context": 1024}, {"groups": 64, "rows": 1, "context": 1024})
 
@@ -31,7 +32,13 @@ def cost(doc: dict, call: dict, groups: int, rows: int, context: int) -> tuple[f
     """(bytes, flops) a call must at least move and do: weights once (routed experts: those the tokens can reach), every
     token-shaped argument once, the states it reads and writes, and the products it is made of."""
     op, n = call["op"], groups * rows
-    bufs = [(a, doc["buffers"][a["buf"]]) for a in call["args"] if "buf" in a]
+    seen, bufs = set(), []
+    for a in call["args"]:                                  # columns of one buffer bound several times are read once
+        if "buf" in a and a["buf"] not in seen and not a["buf"].startswith("rope."):
+            seen.add(a["buf"])
+            b = doc["buffers"][a["buf"]]
+            derived = b["kind"] == "carry" and isinstance(b["shape"][0], int) and b["dtype"] == "bf16"      # weights put together at load
+            bufs.append((a, b | {"kind": "weight"} if derived else b))
     es = {"bf16": 2, "f32": 4, "i32": 4, "i64": 8}
     wbytes = sum(2 * _prod(b["shape"]) for _, b in bufs if b["kind"] == "weight")
     w = [b["shape"] for _, b in bufs if b["kind"] == "weight"]
@@ -46,6 +53,23 @@ def cost(doc: dict, call: dict, groups: int, rows: int, context: int) -> tuple[f
     for s in st:
         if s.get("bytes_per_seq"):
             tok += 2 * groups * s["bytes_per_seq"]
+    if re.match(r"(window_)?attn_(prefill|decode|p_|d_)", op):
+        hq, hk, d, dv, window = _heads(doc, call)
+        seen_by = lambda p: min(p + 1, window)
+        flops = 2.0 * groups * hq * (d + dv) * sum(seen_by(p) for p in range(context - rows, context))
+        cols = groups * rows * (hq * (d + dv)) * 2.0
+        return cols + groups * min(context, window + rows - 1) * hk * (d + dv) * 2.0, flops
+    m = re.match(r"lin_[pd]_(\d+)x(\d+)x(\d+)", op)
+    if m:                                                   # a recurrence: its rows, its decays and its states
+        H, dk, dv = map(int, m.groups())
+        return n * H * (2 * dk + 3 * dv) * 2.0 + n * H * dk * 4.0 + 2.0 * groups * H * dk * dv * 4, 0.0
+    if op.startswith("shift_"):
+        width, targets = doc["buffers"][call["args"][1]["buf"]]["shape"][::-1]
+        return (n * (1 + targets) + targets) * width * 2.0 + 2.0 * groups * width * 4, 0.0
+    m = re.search(r"_(\d+)x(\d+)_of\d+$", op)
+    if m:                                                   # columns of wider rows
+        a, b = map(int, m.groups())
+        return a * b * 2.0 + n * (2.0 * b + 4.0 * a), 2.0 * n * a * b
     if "moe_fc" in op:
         E, a, b = w[0]
         k = next(x for _, x in bufs if x["shape"][0] == "tokens")["shape"]
@@ -53,13 +77,15 @@ def cost(doc: dict, call: dict, groups: int, rows: int, context: int) -> tuple[f
         hit = E * (1 - (1 - top / E) ** n)
         wbytes = wbytes * hit / E
         flops = 2.0 * n * top * a * b
-    elif w and len(w[0]) == 2 and op.split("_")[0] in ("lin", "glu", "head", "router", "q", "v", "qa", "o", "kda", "gate", "down", "lm", "moe"):
+    elif w and len(w[0]) == 3:
+        flops = 2.0 * n * _prod(w[0])
+    elif w and len(w[0]) == 2 and op.split("_")[0] in ("lin", "glu", "geglu", "qkv", "head", "router", "q", "v", "qa", "o", "kda", "gate", "down", "lm", "moe"):
         mats = [x for x in w if len(x) == 2]
         m = groups if doc["buffers"][call["args"][0]["buf"]]["shape"][0] == "seqs" else n
         flops = sum(2.0 * m * _prod(x) for x in mats)
         if op == "embed":
             flops = 0.0
-    elif op == "embed":
+    elif op.startswith("embed"):
         wbytes = n * 4 * w[0][1]
     elif "attn" in op and st:
         per = st[0]["bytes_per_token"] / 2                      # columns of a cached row
@@ -67,9 +93,22 @@ def cost(doc: dict, call: dict, groups: int, rows: int, context: int) -> tuple[f
         heads = _prod([doc["buffers"][call["args"][0]["buf"]]["shape"][1]]) / per
         tok += groups * context * per * 2
         flops = 4.0 * n * heads * per * reach
-    if op == "embed":
+    if op.startswith("embed_"):
+        wbytes = n * 2 * w[0][1]
+    elif op == "embed":
         wbytes = n * 4 * doc["buffers"][call["args"][7]["buf"]]["shape"][1] if len(call["args"]) > 7 else n * 2 * w[0][1]
     return wbytes + tok, flops
+
+
+def _heads(doc: dict, call: dict) -> tuple[int, int, int, int, int]:
+    """(query heads, key heads, key columns, value columns, window) of a grouped-query attention call."""
+    m = re.match(r"window_attn_._(\d+)x(\d+)x(\d+)x(\d+)x(\d+)", call["op"])
+    if m:
+        return tuple(map(int, m.groups()))
+    args = doc["ops"][call["op"]]["impl"]["launches"][0]
+    d = int(re.search(r"_d(\d+)", args["entry"]).group(1))
+    hk = doc["states"][next(a["state"] for a in call["args"] if "state" in a)]["bytes_per_token"] // (4 * d)
+    return doc["buffers"][call["args"][2]["buf"]]["shape"][1] // d, hk, d, d, 1 << 30
 
 
 def _prod(v) -> float:
@@ -130,7 +169,7 @@ def run(model: str, layers: int, points, samples: int, by_call: bool = True) -> 
 def main(args) -> int:
     layers = args.layers if args.layers != 36 else 8
     hbm, tf, src = peaks()
-    for model in MODELS:
+    for model in MODELS[args.config]:
         for rec in run(model, layers, POINTS, max(12, min(args.steps, 24))):
             rec["peaks"] = {"copy_tb_s": round(hbm / 1e12, 2), "bf16_pflop_s": round(tf / 1e15, 2), "source": src}
             rec["data"] = "synthetic (random-init weights, random token ids)"

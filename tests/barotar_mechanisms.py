@@ -148,7 +148,8 @@ def rule(gpu, act, H, dk, dv, chunks, ragged, bonus):
     s_off, os_ = 256, H * dv + 5
     line = 256 + (H * dk * dv * 4 + 255) // 256 * 256
     state, lines, at = torch.zeros(4 * line, dtype=torch.uint8), ints([3, 1]), [0, 0]
-    op = K.lin_rule_op(H, dk, dv, stride, line, s_off, ragged, act, bonus=bonus, q_scale=scale, fused=fused, norm_shared=not bonus, out_stride=os_, out_scale=out_scale, eps=eps)
+    op = K.lin_rule_op(H, dk, dv, stride, line, s_off, ragged, act, bonus=bonus, q_scale=scale, fused=fused, norm_shared=not bonus, out_stride=os_, out_scale=out_scale, eps=eps,
+                       rows_max=140, seqs_max=2)
     ng = K.lin_norm_gate_op(H, dv, stride, not bonus, os_, out_scale, eps, act)
     for step in zip(*chunks):
         n = sum(step)
