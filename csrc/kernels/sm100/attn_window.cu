@@ -18,8 +18,9 @@ using namespace kern;
 
 namespace {
 
-// grid = rows, block 256: a warp per head, heads dealt to the eight warps; 8 max(d, dv) floats of shared memory
-template <typename T>
+// grid = rows, block 256: a warp per head, heads dealt to the eight warps; 8 max(d, dv) floats of shared memory. N > 0: pairs of
+// neighbours, heads of up to 128 N whole vectors, norms on both.
+template <typename T, int N>
 KERN_DEVICE void prep_body(T* qkv, uint8_t* cache, const long long* positions, const long long* slots, const float* cos_tab,
                            const float* sin_tab, const __nv_bfloat16* q_norm, const __nv_bfloat16* k_norm, int hq, int hk, int d,
                            int dv, int rot, int halves, int page_size, int row_stride, int max_pos, float eps, int* err) {
@@ -38,7 +39,54 @@ KERN_DEVICE void prep_body(T* qkv, uint8_t* cache, const long long* positions, c
   T* base = qkv + (size_t)t * row_stride;
   T* page = reinterpret_cast<T*>(cache) + (size_t)(slot < 0 ? 0 : slot / page_size) * hk * page_size * (d + dv);
   const int off = slot < 0 ? 0 : (int)(slot % page_size);
-  for (int h = warp; h < hq + 2 * hk; h += 8) {
+  if constexpr (N > 0) {
+    // four neighbouring columns per lane and step, both columns of a pair in the lane: nothing leaves the registers
+    Vec<4> w[2][N], c2[N];
+    bool turned[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int c = (i * 32 + lane) * 4;
+      turned[i] = c < rot;
+      if (c < d) { w[0][i] = ldv<4>(q_norm + c); w[1][i] = ldv<4>(k_norm + c); }
+      if (turned[i]) {
+        const float2 a = *reinterpret_cast<const float2*>(cs + c / 2), b = *reinterpret_cast<const float2*>(sn + c / 2);
+        c2[i].v[0] = a.x; c2[i].v[1] = b.x; c2[i].v[2] = a.y; c2[i].v[3] = b.y;
+      }
+    }
+#pragma unroll 4
+    for (int h = warp; h < hq + hk; h += 8) {
+      const bool is_q = h < hq;
+      T* src = base + (size_t)h * d;
+      T* dst = is_q ? src : page + ((size_t)(h - hq) * page_size + off) * d;
+      const bool store = is_q || (slot >= 0 && KERN_CHECK(dst, (size_t)d * sizeof(T), SITE_KV_APPEND));
+      Vec<4> x[N];
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const int c = (i * 32 + lane) * 4;
+        if (c >= d) continue;
+        x[i] = ldv<4>(src + c);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) ss += x[i].v[e] * x[i].v[e];
+      }
+      const float inv = 1.f / sqrtf(warp_sum(ss) / (float)d + eps);
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const int c = (i * 32 + lane) * 4;
+        if (c >= d || !store) continue;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[i].v[e] *= inv * (is_q ? w[0][i].v[e] : w[1][i].v[e]);
+        if (turned[i]) {
+          Vec<4> o;
+          o.v[0] = x[i].v[0] * c2[i].v[0] - x[i].v[1] * c2[i].v[1]; o.v[1] = x[i].v[1] * c2[i].v[0] + x[i].v[0] * c2[i].v[1];
+          o.v[2] = x[i].v[2] * c2[i].v[2] - x[i].v[3] * c2[i].v[3]; o.v[3] = x[i].v[3] * c2[i].v[2] + x[i].v[2] * c2[i].v[3];
+          x[i] = o;
+        }
+        stv<4>(dst + c, x[i]);
+      }
+    }
+  }
+  for (int h = (N > 0 ? hq + hk : 0) + warp; h < hq + 2 * hk; h += 8) {
     const bool is_q = h < hq, is_v = h >= hq + hk;
     if (!is_q && slot < 0) continue;
     if (is_v) {
@@ -165,8 +213,18 @@ KERN_DEVICE void attn_any_body(const T* q, const uint8_t* cache, T* out, const i
                          int d, int dv, int rot, int halves, int page_size, int row_stride, int max_pos, float eps,        \
                          int* err) {                                                                                       \
     pdl_wait();                                                                                                            \
-    prep_body<T>(qkv, cache, positions, slots, cos_tab, sin_tab, q_norm, k_norm, hq, hk, d, dv, rot, halves, page_size,    \
-                 row_stride, max_pos, eps, err);                                                                           \
+    const bool vec = !halves && (d | dv | rot | row_stride) % 4 == 0 && q_norm && k_norm &&                                \
+                     ((reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(q_norm) | \
+                       reinterpret_cast<uintptr_t>(k_norm)) & 15) == 0;                                                    \
+    if (vec && d <= 128)                                                                                                   \
+      prep_body<T, 1>(qkv, cache, positions, slots, cos_tab, sin_tab, q_norm, k_norm, hq, hk, d, dv, rot, halves,          \
+                      page_size, row_stride, max_pos, eps, err);                                                           \
+    else if (vec && d <= 256)                                                                                              \
+      prep_body<T, 2>(qkv, cache, positions, slots, cos_tab, sin_tab, q_norm, k_norm, hq, hk, d, dv, rot, halves,          \
+                      page_size, row_stride, max_pos, eps, err);                                                           \
+    else                                                                                                                   \
+      prep_body<T, 0>(qkv, cache, positions, slots, cos_tab, sin_tab, q_norm, k_norm, hq, hk, d, dv, rot, halves,          \
+                      page_size, row_stride, max_pos, eps, err);                                                           \
     pdl_launch_dependents();                                                                                               \
   }                                                                                                                        \
   WINDOW_ATTN(T, SFX, 64)                                                                                                  \

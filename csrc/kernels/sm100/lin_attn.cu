@@ -73,7 +73,7 @@ KERN_DEVICE void shift_state_body(const T* h, uint8_t* state, const int* lines, 
 // ---- the decays ---------------------------------------------------------------------------------------------------
 // One 64 x 64 tile of alpha [rows, n] per block: z = act(a) . W^T + bias in f32, then the decay. mode 0: act(a) = a,
 // alpha = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau); mode 1: act = tanh, alpha = exp(-exp(z)).
-constexpr int DB = 64, DK = 16;
+constexpr int DB = 64, DK = 64;
 template <typename T>
 KERN_DEVICE void decay_body(const T* a, const __nv_bfloat16* W, const __nv_bfloat16* bias, float* alpha, int rows, int n, int rank,
                             int lda, int mode, float inv_tau) {
@@ -82,15 +82,17 @@ KERN_DEVICE void decay_body(const T* a, const __nv_bfloat16* W, const __nv_bfloa
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < rank; k0 += DK) {
+#pragma unroll 8
     for (int i = threadIdx.x; i < DB * DK; i += 256) {
       const int r = i / DK, k = i % DK;
       float v = (k0 + k < rank && m0 + r < rows) ? ldf(a + (size_t)(m0 + r) * lda + k0 + k) : 0.f;
-      as[k][r] = mode ? tanhf(v) : v;
+      as[k][r] = mode && v != 0.f ? tanhf(v) : v;
       ws[k][r] = (k0 + k < rank && n0 + r < n) ? __bfloat162float(W[(size_t)(n0 + r) * rank + k0 + k]) : 0.f;
     }
     __syncthreads();
-#pragma unroll
-    for (int k = 0; k < DK; ++k) {
+    const int kn = min(DK, (rank - k0 + 3) & ~3);      // what is past the rank is zero
+#pragma unroll 4
+    for (int k = 0; k < kn; ++k) {
       const Vec<4> x = ldv<4>(&as[k][ty * 4]), w = ldv<4>(&ws[k][tx * 4]);
 #pragma unroll
       for (int i = 0; i < 4; ++i)
@@ -330,7 +332,7 @@ KERN_DEVICE bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(
   }
 // rule: grid [H ceil(dv / (32 V)), seqs], block 256, (3 tb + 1) dk floats of shared memory; RK >= ceil(dk / 8)
 #define LIN_RULE(T, SFX, RK, V)                                                                                           \
-  extern "C" __global__ void __launch_bounds__(256)                                                                       \
+  extern "C" __global__ void __launch_bounds__(256, RK <= 8 ? (V <= 2 ? 5 : 3) : (RK == 16 ? 2 : 1))                      \
       kern_lin_rule_##SFX##_r##RK##_v##V(const T* q, const T* k, const T* v, const T* gate, const float* alpha,           \
                                          const __nv_bfloat16* u, const __nv_bfloat16* norm, void* out, uint8_t* state,    \
                                          const int* lines, const int* cu, int seqs, int H, int dk, int dv, int stride,    \

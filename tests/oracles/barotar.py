@@ -39,22 +39,20 @@ def rwkv_decay(z):
 
 def gla_rule(q, k, v, alpha, S):
     """q, k, alpha [T, H, dk], v [T, H, dv], S [H, dk, dv] -> (o [T, H, dv], S after the last token)."""
-    S, out = S.clone(), torch.zeros_like(v)
+    out = torch.zeros_like(v)
     for t in range(q.shape[0]):
-        for h in range(q.shape[1]):
-            S[h] = alpha[t, h][:, None] * S[h] + torch.outer(k[t, h], v[t, h])
-            out[t, h] = S[h].t() @ q[t, h]
+        S = alpha[t][:, :, None] * S + k[t][:, :, None] * v[t][:, None, :]
+        out[t] = torch.einsum("hkv,hk->hv", S, q[t])
     return out, S
 
 
 def rwkv_rule(r, k, v, w, u, S):
     """As above with a read before the update and `u` [H, dk] weighing the current token in that read."""
-    S, out = S.clone(), torch.zeros_like(v)
+    out = torch.zeros_like(v)
     for t in range(r.shape[0]):
-        for h in range(r.shape[1]):
-            kv = torch.outer(k[t, h], v[t, h])
-            out[t, h] = (S[h] + u[h][:, None] * kv).t() @ r[t, h]
-            S[h] = w[t, h][:, None] * S[h] + kv
+        kv = k[t][:, :, None] * v[t][:, None, :]
+        out[t] = torch.einsum("hkv,hk->hv", S + u[:, :, None] * kv, r[t])
+        S = w[t][:, :, None] * S + kv
     return out, S
 
 
@@ -86,15 +84,15 @@ def rotate(x, positions, dims, base):
 def window_attend(q, k, v, scale, cap, size, sink):
     """q [T, H, d] of the last T positions, k [L, G, d] / v [L, G, e] of all; a row at a time."""
     T, H, L = q.shape[0], q.shape[1], k.shape[0]
-    per, out = H // k.shape[1], torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    of = torch.arange(H) // (H // k.shape[1])                # the key head of every query head
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
     for t in range(T):
         i = L - T + t
         lo = max(0, i - size + 1)
-        for h in range(H):
-            s = cap * torch.tanh((k[lo:i + 1, h // per] @ q[t, h]) * scale / cap)
-            top = torch.maximum(s.max(), sink[h])
-            e = torch.exp(s - top)
-            out[t, h] = (e / (e.sum() + torch.exp(sink[h] - top))) @ v[lo:i + 1, h // per]
+        s = cap * torch.tanh(torch.einsum("hd,lhd->hl", q[t], k[lo:i + 1, of]) * scale / cap)
+        top = torch.maximum(s.max(-1).values, sink)
+        e = torch.exp(s - top[:, None])
+        out[t] = torch.einsum("hl,lhe->he", e / (e.sum(-1) + torch.exp(sink - top))[:, None], v[lo:i + 1, of])
     return out
 
 
