@@ -284,8 +284,25 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
         tmem_ld_wait();
         if constexpr (WIN) {      // capped scores in base-2 units, then both edges of the window
           static_assert(!WIN || kKeep, "the windowed form keeps a tile's scores in registers");
+          float ab[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-          for (int i = 0; i < FN; ++i) keep[i] = __float_as_uint(capped_score(__uint_as_float(keep[i]), a.win));
+          for (int i = 0; i < FN; ++i) ab[i & 3] = fmaxf(ab[i & 3], fabsf(__uint_as_float(keep[i])));
+          const bool far = fmaxf(fmaxf(ab[0], ab[1]), fmaxf(ab[2], ab[3])) * a.win.c1 > 0.72f;      // some |score / cap| above 1/4
+          if (__any_sync(0xffffffffu, far)) {
+#pragma unroll
+            for (int i = 0; i < FN; ++i) keep[i] = __float_as_uint(capped_score(__uint_as_float(keep[i]), a.win));
+          } else {
+            // the Taylor series of tanh to x^9: below a quarter what is left out is under 1e-8 of x, and there are no
+            // special functions in it
+            const float u = a.win.c1 * 0.34657359f, uu = u * u, k0 = a.win.c2 * u;      // x = score / cap = q.k u
+            const float k1 = k0 * uu * (-1.f / 3.f), k2 = k0 * uu * uu * (2.f / 15.f), k3 = k0 * uu * uu * uu * (-17.f / 315.f),
+                        k4 = k0 * uu * uu * uu * uu * (62.f / 2835.f);
+#pragma unroll
+            for (int i = 0; i < FN; ++i) {
+              const float v = __uint_as_float(keep[i]), y = v * v;
+              keep[i] = __float_as_uint(v * (k0 + y * (k1 + y * (k2 + y * (k3 + y * k4)))));
+            }
+          }
           if (diag || tok0 <= pos - a.win.size) {
 #pragma unroll
             for (int i = 0; i < FN; ++i)

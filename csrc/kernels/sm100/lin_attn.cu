@@ -82,10 +82,12 @@ KERN_DEVICE void decay_body(const T* a, const __nv_bfloat16* W, const __nv_bfloa
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < rank; k0 += DK) {
-#pragma unroll 8
-    for (int i = threadIdx.x; i < DB * DK; i += 256) {
-      const int r = i / DK, k = i % DK;
-      float v = (k0 + k < rank && m0 + r < rows) ? ldf(a + (size_t)(m0 + r) * lda + k0 + k) : 0.f;
+    // a warp moves 8 columns of 4 rows at a time: whole sectors in, no two lanes on one bank
+    const int kb = threadIdx.x & 7, rb = (threadIdx.x >> 3) & 3, warp = threadIdx.x >> 5;
+#pragma unroll 4
+    for (int i = warp; i < (DB / 4) * (DK / 8); i += 8) {
+      const int r = (i / (DK / 8)) * 4 + rb, k = (i % (DK / 8)) * 8 + kb;
+      const float v = (k0 + k < rank && m0 + r < rows) ? ldf(a + (size_t)(m0 + r) * lda + k0 + k) : 0.f;
       as[k][r] = mode && v != 0.f ? tanhf(v) : v;
       ws[k][r] = (k0 + k < rank && n0 + r < n) ? __bfloat162float(W[(size_t)(n0 + r) * rank + k0 + k]) : 0.f;
     }
@@ -313,7 +315,7 @@ KERN_DEVICE bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(
     shift_state_body<T>(h, state, lines, cu, seqs, width, line_bytes);                                                    \
     pdl_launch_dependents();                                                                                              \
   }                                                                                                                       \
-  extern "C" __global__ void __launch_bounds__(256)                                                                       \
+  extern "C" __global__ void __launch_bounds__(256, 4)                                                                    \
       kern_decay_##SFX(const T* a, const __nv_bfloat16* W, const __nv_bfloat16* bias, float* alpha, int rows, int n,      \
                        int rank, int lda, int mode, float inv_tau) {                                                      \
     pdl_wait();                                                                                                           \
