@@ -29,7 +29,7 @@ CASES = {
     "mixed": dict(width=72, vocab=200, eps=1e-5, ranks=[8, 16, 24, 8], blocks=[
         block(parallel((4, 2, 64, 64, 21, 32, 1e4, 0.15, 9.0), (3, 24), 0.7, 1.2), moe(12, 3, 24, 3, 2, 1.5)),
         block(gla(3, 40, 24, 4.0), dense(88)),
-        block(parallel((8, 1, 128, 128, 50, 128, 5e5, 0.1, 30.0), (2, 64), 1.3, 0.4)),
+        block(parallel((4, 1, 128, 128, 50, 128, 5e5, 0.1, 28.0), (2, 64), 1.3, 0.4)),
         block(gla(2, 16, 72, 16.0), moe(8, 2, 32, 2, 1, 0.8))]),
     # nothing is a multiple of eight, keys and values of different sizes, one group per expert
     "odd": dict(width=50, vocab=101, eps=1e-6, ranks=[5, 3, 7], blocks=[

@@ -5,7 +5,7 @@ CHUNKS2 = [(5, 1, 70, 3, 16), (1, 2, 33, 66, 8)]
 MANY = tuple((20 + 7 * i, r) for i, r in enumerate((1, 1, 5, 20, 1, 2, 33, 1, 1, 27)))      # more sequences than the few-sequence form takes
 SIZES = (      # hq, hk, d, dv, window, page, sequences
     (4, 2, 64, 64, 21, 16, ((1, 1), (60, 60), (90, 3))),
-    (8, 1, 128, 128, 50, 16, ((150, 150), (33, 2), (70, 1))),
+    (16, 2, 128, 128, 50, 16, ((150, 150), (33, 2), (70, 1))),
     (6, 2, 128, 128, 70, 64, MANY),
     (16, 1, 64, 64, 9, 64, MANY),
     (3, 3, 256, 256, 33, 16, ((80, 70), (20, 1))),
@@ -16,7 +16,7 @@ SIZES = (      # hq, hk, d, dv, window, page, sequences
 )
 DECODE = (
     (4, 2, 64, 64, 21, 16, ((1, 1), (21, 1), (22, 1), (90, 1))),
-    (8, 1, 128, 128, 300, 64, ((299, 1), (300, 1), (301, 1), (570, 1))),      # split keys
+    (16, 2, 128, 128, 300, 64, ((299, 1), (300, 1), (301, 1), (570, 1))),      # split keys
     (8, 4, 128, 128, 65, 16, ((64, 1), (65, 1), (66, 1), (200, 1), (129, 1))),
     (3, 3, 256, 256, 33, 16, ((80, 1), (20, 1))),
     (6, 2, 18, 11, 9, 16, ((40, 1), (9, 1), (10, 1))),
