@@ -85,9 +85,10 @@ struct FmhaArgs {
 };
 
 // `y`: the CTA's index into the work list (blockIdx.y unless the caller maps it)
-template <int D, int FN, bool WIN = false>
+template <int D, int FN, int FORM = kAttnPlain>
 KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const int y) {
   using Cfg = FmhaCfg<D, FN>;
+  constexpr bool WIN = FORM == kAttnWindow;
   constexpr int kStages = Cfg::kStages;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -404,11 +405,14 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
       tc_fence_after();
       const uint32_t o_tmem = tmem_base + lane_addr + 2 * FN;
       float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-      if constexpr (WIN) inv = row < valid_rows ? sink_factor(m_ref, l_run, __bfloat162float(a.win.sink[kvh * G + row % G]), a.win.out_scale) : 0.f;
+      if constexpr (FORM != kAttnPlain) inv = row < valid_rows ? sink_factor(m_ref, l_run, sink_of(a.win, kvh * G + row % G), a.win.out_scale) : 0.f;
       __nv_bfloat16* dst = nullptr;
+      const __nv_bfloat16* gate = nullptr;
       if (row < valid_rows) {
         const int tk = row0_tok + tok_lo + row / G, head = kvh * G + row % G;
         dst = a.out + (size_t)tk * a.out_stride + (size_t)head * D;
+        if constexpr (FORM == kAttnSink)
+          if (a.win.gate) gate = a.win.gate + (size_t)tk * a.win.gate_stride + (size_t)head * D;
       }
 #pragma unroll 1
       for (int c = 0; c < D / 32; ++c) {
@@ -416,6 +420,21 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
         tmem_ld_32x32(o_tmem + c * 32, r);
         tmem_ld_wait();
         if (dst != nullptr) {
+          if constexpr (FORM == kAttnSink) {
+            if (gate != nullptr) {
+#pragma unroll
+              for (int v = 0; v < 4; ++v) {
+                const uint4 gv = *reinterpret_cast<const uint4*>(gate + c * 32 + v * 8);
+                const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                  const float2 g = unpack_bf16x2(gw[e]);
+                  r[v * 8 + 2 * e] = __float_as_uint(__uint_as_float(r[v * 8 + 2 * e]) * gate_factor(g.x));
+                  r[v * 8 + 2 * e + 1] = __float_as_uint(__uint_as_float(r[v * 8 + 2 * e + 1]) * gate_factor(g.y));
+                }
+              }
+            }
+          }
 #pragma unroll
           for (int v = 0; v < 4; ++v) {
             uint4 o;
@@ -830,5 +849,16 @@ extern "C" __global__ void __launch_bounds__(192, 2)
                                int pool_pages, int* err, const __nv_bfloat16* sink, int window, float c1, float c2, float out_scale) {
   FmhaArgs a{q, out, block_table, seq_lens, cu_q, work, work_count, err, hq, hk, q_stride, out_stride, max_pages, page_size,
              pool_pages, 1.f, {window, c1, c2, out_scale, sink}};
-  fmha_body<128, 64, true>(&kv_map, a, (int)blockIdx.y);
+  fmha_body<128, 64, kAttnWindow>(&kv_map, a, (int)blockIdx.y);
+}
+
+// The 64-token form over the whole causal reach, with a sink and an output gate.
+extern "C" __global__ void __launch_bounds__(192, 2)
+    kern_attn_sink_fmha_d128(const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* q, __nv_bfloat16* out,
+                             const int* block_table, const int* seq_lens, const int* cu_q, const int* work, const int* work_count,
+                             int hq, int hk, int q_stride, int out_stride, int max_pages, int page_size, int pool_pages, int* err,
+                             const __nv_bfloat16* sink, const __nv_bfloat16* gate, int gate_stride, float scale_log2) {
+  FmhaArgs a{q, out, block_table, seq_lens, cu_q, work, work_count, err, hq, hk, q_stride, out_stride, max_pages, page_size,
+             pool_pages, scale_log2, {0, 0.f, 0.f, 1.f, sink, gate, gate_stride}};
+  fmha_body<128, 64, kAttnSink>(&kv_map, a, (int)blockIdx.y);
 }

@@ -59,22 +59,44 @@ struct AttnCfg {
   static constexpr int kSmem = 1024 + kStages * kStageBytes + kQBytes + 256;
 };
 
-// Attention in a sliding window with capped scores and a sink (the WIN forms): a row at position i sees the keys j with
+// The forms of the bodies here and in attn_fmha.cu: plain softmax; in a sliding window with capped scores and a sink; causal
+// with a sink.
+enum AttnForm : int { kAttnPlain = 0, kAttnWindow = 1, kAttnSink = 2 };
+
+// Attention in a sliding window with capped scores and a sink (kAttnWindow): a row at position i sees the keys j with
 // 0 <= i - j < size; a score is cap tanh(score / cap), computed as c2 (1 - 2 / (1 + 2^(c1 q.k))) with c1 = 2 log2(e) scale / cap
 // and c2 = cap log2(e), in the base-2 units of the softmax; `sink` (bf16, one per query head) joins every row's denominator
-// once, as a score that is neither scaled nor capped. The finished rows are multiplied by out_scale.
+// once, as a score that is neither scaled nor capped. The finished rows are multiplied by out_scale. kAttnSink has the sink only
+// (no pointer: a score of 0 for every head), and multiplies the finished rows by sigmoid(gate), [token][gate_stride] with a
+// column per output column, where there is one.
 struct AttnWindow {
-  int size;
-  float c1, c2, out_scale;
-  const __nv_bfloat16* sink;
+  int size = 0;
+  float c1 = 0.f, c2 = 0.f, out_scale = 1.f;
+  const __nv_bfloat16* sink = nullptr;
+  const __nv_bfloat16* gate = nullptr;
+  int gate_stride = 0;
 };
 constexpr float kLog2e = 1.4426950408889634f;
 KERN_DEVICE float capped_score(float qk, const AttnWindow& w) { return w.c2 - __fdividef(2.f * w.c2, 1.f + exp2f(qk * w.c1)); }
+KERN_DEVICE float sink_of(const AttnWindow& w, int head) { return w.sink ? __bfloat162float(w.sink[head]) : 0.f; }
+KERN_DEVICE float gate_factor(float g) { return __fdividef(1.f, 1.f + __expf(-g)); }
 // (m, l): a finished row's maximum and sum in base-2 units -> the factor of its un-normalised output
 KERN_DEVICE float sink_factor(float m, float l, float sink, float out_scale) {
   const float s = sink * kLog2e, top = fmaxf(m, s);
   const float f = exp2f(m - top);          // 0 for a row that saw no key
   return out_scale * f / (l * f + exp2f(s - top));
+}
+
+// the factors of two neighbouring output columns
+template <int FORM>
+KERN_DEVICE float2 gate_pair(const AttnWindow& w, int row, int col) {
+  if constexpr (FORM == kAttnSink) {
+    if (w.gate) {
+      const float2 g = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(w.gate + (size_t)row * w.gate_stride + col));
+      return make_float2(gate_factor(g.x), gate_factor(g.y));
+    }
+  }
+  return make_float2(1.f, 1.f);
 }
 
 struct AttnArgs {
@@ -95,9 +117,10 @@ struct AttnArgs {
 
 // PREFILL = false: decode/verify (warps split tokens); true: causal prefill (warps split rows)
 // `y`: the CTA's index into the work list (or its sequence), blockIdx.y unless the caller maps it
-template <int D, bool PREFILL, int ST = 0, bool WIN = false>
+template <int D, bool PREFILL, int ST = 0, int FORM = kAttnPlain>
 KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const int y) {
   using Cfg = AttnCfg<D, PREFILL, ST>;
+  constexpr bool WIN = FORM == kAttnWindow;
   constexpr int kStages = Cfg::kStages;
   constexpr int NT = PREFILL ? 8 : 2;        // 8-token n-tiles of S per warp per KV tile
   constexpr int ROWS = PREFILL ? 64 : 16;    // query rows per CTA
@@ -379,8 +402,10 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
       const int tk = row0_tok + tok_lo + r / G, head = kvh * G + r % G;
       if (split_total == 1) {
         float v;
-        if constexpr (WIN) v = acc * sink_factor(m, l, __bfloat162float(a.win.sink[head]), a.win.out_scale);
+        if constexpr (FORM != kAttnPlain) v = acc * sink_factor(m, l, sink_of(a.win, head), a.win.out_scale);
         else v = l > 0.f ? acc / l : 0.f;
+        if constexpr (FORM == kAttnSink)
+          if (a.win.gate) v *= gate_factor(__bfloat162float(a.win.gate[(size_t)tk * a.win.gate_stride + (size_t)head * D + c]));
         a.out[(size_t)tk * a.out_stride + (size_t)head * D + c] = __float2bfloat16(v);
       } else {
         const size_t base = ((size_t)tk * a.hq + head) * split_total + split_base + split;
@@ -394,22 +419,24 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
   } else if (warp < 4) {
     const int rA = warp * 16 + (lane >> 2), rB = rA + 8;
     float iA = l_run[0] > 0.f ? 1.f / l_run[0] : 0.f, iB = l_run[1] > 0.f ? 1.f / l_run[1] : 0.f;
-    if constexpr (WIN) {
-      if (rA < valid_rows) iA = sink_factor(m_run[0], l_run[0], __bfloat162float(a.win.sink[kvh * G + rA % G]), a.win.out_scale);
-      if (rB < valid_rows) iB = sink_factor(m_run[1], l_run[1], __bfloat162float(a.win.sink[kvh * G + rB % G]), a.win.out_scale);
+    if constexpr (FORM != kAttnPlain) {
+      if (rA < valid_rows) iA = sink_factor(m_run[0], l_run[0], sink_of(a.win, kvh * G + rA % G), a.win.out_scale);
+      if (rB < valid_rows) iB = sink_factor(m_run[1], l_run[1], sink_of(a.win, kvh * G + rB % G), a.win.out_scale);
     }
 #pragma unroll
     for (int i = 0; i < D / 8; ++i) {
       const int c = i * 8 + 2 * (lane & 3);
       if (rA < valid_rows) {
         const int tk = row0_tok + tok_lo + rA / G, head = kvh * G + rA % G;
+        const float2 g = gate_pair<FORM>(a.win, tk, head * D + c);
         *reinterpret_cast<uint32_t*>(a.out + (size_t)tk * a.out_stride + (size_t)head * D + c) =
-            pack_bf16x2(o[i][0] * iA, o[i][1] * iA);
+            pack_bf16x2(o[i][0] * iA * g.x, o[i][1] * iA * g.y);
       }
       if (rB < valid_rows) {
         const int tk = row0_tok + tok_lo + rB / G, head = kvh * G + rB % G;
+        const float2 g = gate_pair<FORM>(a.win, tk, head * D + c);
         *reinterpret_cast<uint32_t*>(a.out + (size_t)tk * a.out_stride + (size_t)head * D + c) =
-            pack_bf16x2(o[i][2] * iB, o[i][3] * iB);
+            pack_bf16x2(o[i][2] * iB * g.x, o[i][3] * iB * g.y);
       }
     }
   }

@@ -103,18 +103,26 @@ extern "C" __global__ void __launch_bounds__(128)
 }
 
 // cos/sin tables [max_pos][rot/2] in f32, angles evaluated in double so large positions stay exact.
-extern "C" __global__ void kern_rope_table_f32(float* cos_tab, float* sin_tab, int max_pos, int rot,
-                                               double theta) {
+KERN_DEVICE void rope_table(float* cos_tab, float* sin_tab, int max_pos, int rot, double theta, double factor) {
   const int half = rot >> 1;
   const long long n = (long long)max_pos * half;
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n;
        i += (long long)gridDim.x * blockDim.x) {
     const int j = (int)(i % half);
     const long long p = i / half;
-    const double inv_freq = pow(theta, -2.0 * (double)j / (double)rot);
+    const double inv_freq = pow(theta, -2.0 * (double)j / (double)rot) / factor;
     double s, c;
     sincos((double)p * inv_freq, &s, &c);
     cos_tab[i] = (float)c;
     sin_tab[i] = (float)s;
   }
+}
+extern "C" __global__ void kern_rope_table_f32(float* cos_tab, float* sin_tab, int max_pos, int rot,
+                                               double theta) {
+  rope_table(cos_tab, sin_tab, max_pos, rot, theta, 1.0);
+}
+// linear scaling: every frequency divided by `factor`
+extern "C" __global__ void kern_rope_table_scaled_f32(float* cos_tab, float* sin_tab, int max_pos, int rot,
+                                                      double theta, double factor) {
+  rope_table(cos_tab, sin_tab, max_pos, rot, theta, factor);
 }

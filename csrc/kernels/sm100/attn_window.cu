@@ -1,12 +1,15 @@
 // build: precise
 // Attention over a paged cache in a sliding window, with capped scores and a learned sink per query head:
 //     score = cap tanh(q.k scale / cap);  weight_j = exp(score_j) / (exp(sink_h) + sum over the window of exp(score))
-// and what prepares its rows.
+// and attention over the whole causal reach with a sink (learned, or a score of 0) and an output gate, and what prepares their rows.
 //   kern_qk_prep_<act>          per head: RMS norm of q and k with a weight of their own, rotary positions on the first
 //                               columns (pairs (2i, 2i + 1), or halves), k and v into their rows of the paged cache
+//   kern_qk_prep_whole_<act>    the same with a norm over all heads' columns at once, and values from any columns of the row (the
+//                               keys' own, as projected, in a mixer whose keys are its values)
 //   kern_window_attn_<act>_w*   one (row, query head) per block, any sizes, either activation type
 //   kern_attn_window_*_d*       bf16 with equal head dims 64 / 128 / 256: the bodies of attn_paged.cu (decode rows with split
 //                               keys, prompt rows, both lists of a ragged call in one launch)
+//   kern_attn_sink_*_d*         the same bodies without window and cap
 //   kern_attn_window_merge      the partials of split keys, where the sink joins the denominator
 // Cache of one layer: [page][k: head, offset, dim | v: head, offset, vdim]; with equal dims that is attn_prep.cu's layout.
 // Norms, angles, scores, weights and sums are f32.
@@ -126,12 +129,84 @@ KERN_DEVICE void prep_body(T* qkv, uint8_t* cache, const long long* positions, c
   }
 }
 
+// grid = rows, block 256; (hq + hk) d floats of shared memory. V columns per thread and step.
+template <typename T, int V>
+KERN_DEVICE void prep_whole_body(T* qkv, uint8_t* cache, const long long* positions, const long long* slots, const float* cos_tab,
+                                 const float* sin_tab, const __nv_bfloat16* q_norm, const __nv_bfloat16* k_norm, int hq, int hk,
+                                 int d, int dv, int v_col, int rot, int halves, int page_size, int row_stride, int max_pos,
+                                 float eps, int* err) {
+  extern __shared__ __align__(16) float prep_sm[];      // q and k as projected
+  __shared__ float part[2][8];
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nq = hq * d, n = (hq + hk) * d;
+  long long pos = positions[t];
+  const long long slot = slots[t];
+  if (pos < 0 || pos >= max_pos) {
+    if (threadIdx.x == 0) set_error(err, ERR_BOUNDS);
+    pos = 0;
+  }
+  const int half = rot >> 1;
+  const float* cs = cos_tab + (size_t)pos * half;
+  const float* sn = sin_tab + (size_t)pos * half;
+  T* row = qkv + (size_t)t * row_stride;
+  float ssq = 0.f, ssk = 0.f;
+  for (int c = threadIdx.x * V; c < n; c += 256 * V) {
+    const Vec<V> a = ldv<V>(row + c);
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < V; ++e) s += a.v[e] * a.v[e];
+    if (c < nq) ssq += s; else ssk += s;
+    stv<V>(prep_sm + c, a);
+  }
+  ssq = warp_sum(ssq);
+  ssk = warp_sum(ssk);
+  if (lane == 0) { part[0][warp] = ssq; part[1][warp] = ssk; }
+  __syncthreads();
+  ssq = ssk = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { ssq += part[0][i]; ssk += part[1][i]; }
+  const float inv_q = 1.f / sqrtf(ssq / (float)nq + eps), inv_k = 1.f / sqrtf(ssk / (float)(n - nq) + eps);
+  T* page = reinterpret_cast<T*>(cache) + (size_t)(slot < 0 ? 0 : slot / page_size) * hk * page_size * (d + dv);
+  const int off = slot < 0 ? 0 : (int)(slot % page_size);
+  for (int c = threadIdx.x * V; c < n; c += 256 * V) {
+    const bool is_q = c < nq;
+    if (!is_q && slot < 0) break;
+    const __nv_bfloat16* w = is_q ? q_norm : k_norm - nq;
+    const float inv = is_q ? inv_q : inv_k;
+    const int h = c / d, i = c - h * d;
+    T* dst = is_q ? row + c : page + ((size_t)(h - hq) * page_size + off) * d + i;
+    if (!is_q && !KERN_CHECK(dst, V * sizeof(T), SITE_KV_APPEND)) continue;
+    const Vec<V> a = ldv<V>(prep_sm + c), b = ldv<V>(w + c);
+    Vec<V> o;
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      o.v[e] = a.v[e] * inv * b.v[e];
+      if (i + e < rot) {
+        const int j = halves ? (i + e < half ? i + e : i + e - half) : (i + e) >> 1;
+        const bool lo = halves ? i + e < half : !((i + e) & 1);
+        const int other = c + e + (halves ? (lo ? half : -half) : (lo ? 1 : -1));
+        const float x = prep_sm[other] * inv * __bfloat162float(w[other]);
+        o.v[e] = lo ? o.v[e] * cs[j] - x * sn[j] : o.v[e] * cs[j] + x * sn[j];
+      }
+    }
+    stv<V>(dst, o);
+  }
+  if (slot < 0) return;
+  // the values, as they are: k above went to the cache only, so these may be its columns
+  for (int c = threadIdx.x * V; c < hk * dv; c += 256 * V) {
+    const int h = c / dv, i = c - h * dv;
+    T* dst = page + (size_t)hk * page_size * d + ((size_t)h * page_size + off) * dv + i;
+    if (!KERN_CHECK(dst, V * sizeof(T), SITE_KV_APPEND)) continue;
+    stv<V>(dst, ldv<V>(row + v_col + c));
+  }
+}
+
 // Four warps walk the keys of the row's window (key j belongs to warp j % 4); a lane holds the columns i * 32 + lane of the
-// query and of the warp's running sum. RL = columns per lane.
+// query and of the warp's running sum. RL = columns per lane. cap 0: scores as they are; no sink pointer: a score of 0; gate:
+// sigmoid of it multiplies the finished row.
 template <typename T, int RL>
 KERN_DEVICE void attn_any_body(const T* q, const uint8_t* cache, T* out, const int* table, const int* lens, const int* row_seq,
-                               const __nv_bfloat16* sink, int hq, int hk, int d, int dv, int q_stride, int out_stride, int max_pages,
-                               int page, int window, float scale, float cap, float out_scale, int* err) {
+                               const __nv_bfloat16* sink, const T* gate, int hq, int hk, int d, int dv, int q_stride, int out_stride,
+                               int gate_stride, int max_pages, int page, int window, float scale, float cap, float out_scale, int* err) {
   extern __shared__ __align__(16) float win_sm[];      // [4][dv] partial sums, then [4] maxima, [4] weights
   const int h = blockIdx.x, r = blockIdx.y;
   const int L = lens[r];
@@ -162,7 +237,8 @@ KERN_DEVICE void attn_any_body(const T* q, const uint8_t* cache, T* out, const i
       const int c = i * 32 + lane;
       if (c < d) s += qv[i] * ldf(kr + c);
     }
-    s = cap * tanhf(warp_sum(s) * scale / cap);
+    s = warp_sum(s) * scale;
+    if (cap > 0.f) s = cap * tanhf(s / cap);
     const float mn = fmaxf(m, s), f = expf(m - mn), e = expf(s - mn);
     m = mn;
     l = l * f + e;
@@ -180,7 +256,7 @@ KERN_DEVICE void attn_any_body(const T* q, const uint8_t* cache, T* out, const i
   for (int i = 0; i < RL; ++i)
     if (i * 32 + lane < dv) acc[warp * dv + i * 32 + lane] = o[i];
   __syncthreads();
-  const float sk = __bfloat162float(sink[h]);
+  const float sk = sink ? __bfloat162float(sink[h]) : 0.f;
   const float mx = fmaxf(sk, fmaxf(fmaxf(ms[0], ms[1]), fmaxf(ms[2], ms[3])));
   float f[4], den = expf(sk - mx);
 #pragma unroll
@@ -189,7 +265,9 @@ KERN_DEVICE void attn_any_body(const T* q, const uint8_t* cache, T* out, const i
     float v = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) v += f[w] * acc[w * dv + c];
-    stf(out + (size_t)r * out_stride + (size_t)h * dv + c, v / den * out_scale);
+    v = v / den * out_scale;
+    if (gate) v /= 1.f + expf(-ldf(gate + (size_t)r * gate_stride + (size_t)h * dv + c));
+    stf(out + (size_t)r * out_stride + (size_t)h * dv + c, v);
   }
 }
 
@@ -199,12 +277,12 @@ KERN_DEVICE void attn_any_body(const T* q, const uint8_t* cache, T* out, const i
 #define WINDOW_ATTN(T, SFX, W)                                                                                             \
   extern "C" __global__ void __launch_bounds__(128)                                                                        \
       kern_window_attn_##SFX##_w##W(const T* q, const uint8_t* cache, T* out, const int* table, const int* lens,           \
-                                    const int* row_seq, const __nv_bfloat16* sink, int hq, int hk, int d, int dv,          \
-                                    int q_stride, int out_stride, int max_pages, int page, int window, float scale,        \
-                                    float cap, float out_scale, int* err) {                                                \
+                                    const int* row_seq, const __nv_bfloat16* sink, const T* gate, int hq, int hk, int d,   \
+                                    int dv, int q_stride, int out_stride, int gate_stride, int max_pages, int page,        \
+                                    int window, float scale, float cap, float out_scale, int* err) {                       \
     pdl_wait();                                                                                                            \
-    attn_any_body<T, W / 32>(q, cache, out, table, lens, row_seq, sink, hq, hk, d, dv, q_stride, out_stride, max_pages,    \
-                             page, window, scale, cap, out_scale, err);                                                    \
+    attn_any_body<T, W / 32>(q, cache, out, table, lens, row_seq, sink, gate, hq, hk, d, dv, q_stride, out_stride,         \
+                             gate_stride, max_pages, page, window, scale, cap, out_scale, err);                            \
   }
 #define WINDOW_ENTRIES(T, SFX)                                                                                             \
   extern "C" __global__ void __launch_bounds__(256)                                                                        \
@@ -227,6 +305,23 @@ KERN_DEVICE void attn_any_body(const T* q, const uint8_t* cache, T* out, const i
                       page_size, row_stride, max_pos, eps, err);                                                           \
     pdl_launch_dependents();                                                                                               \
   }                                                                                                                        \
+  extern "C" __global__ void __launch_bounds__(256)                                                                        \
+      kern_qk_prep_whole_##SFX(T* qkv, uint8_t* cache, const long long* positions, const long long* slots,                 \
+                               const float* cos_tab, const float* sin_tab, const __nv_bfloat16* q_norm,                    \
+                               const __nv_bfloat16* k_norm, int hq, int hk, int d, int dv, int v_col, int rot, int halves, \
+                               int page_size, int row_stride, int max_pos, float eps, int* err) {                          \
+    pdl_wait();                                                                                                            \
+    const bool vec = (d | dv | v_col | row_stride) % 4 == 0 &&                                                             \
+                     ((reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(q_norm) | \
+                       reinterpret_cast<uintptr_t>(k_norm)) & 15) == 0;                                                    \
+    if (vec)                                                                                                               \
+      prep_whole_body<T, 4>(qkv, cache, positions, slots, cos_tab, sin_tab, q_norm, k_norm, hq, hk, d, dv, v_col, rot,     \
+                            halves, page_size, row_stride, max_pos, eps, err);                                             \
+    else                                                                                                                   \
+      prep_whole_body<T, 1>(qkv, cache, positions, slots, cos_tab, sin_tab, q_norm, k_norm, hq, hk, d, dv, v_col, rot,     \
+                            halves, page_size, row_stride, max_pos, eps, err);                                             \
+    pdl_launch_dependents();                                                                                               \
+  }                                                                                                                        \
   WINDOW_ATTN(T, SFX, 64)                                                                                                  \
   WINDOW_ATTN(T, SFX, 128)                                                                                                 \
   WINDOW_ATTN(T, SFX, 256)                                                                                                 \
@@ -244,7 +339,7 @@ WINDOW_ENTRIES(float, f32)
            int pool_pages, int* err, const __nv_bfloat16* sink, int window, float c1, float c2, float out_scale) {         \
     AttnArgs a{q, out, ws_o, ws_ml, block_table, seq_lens, cu_q, work, work_count, err, 0x7fffffff, hq, hk, q_stride,      \
                out_stride, max_pages, page_size, 1, splits, pool_pages, 1.f, {window, c1, c2, out_scale, sink}};           \
-    attn_body<D, PREFILL, 0, true>(&kv_map, a, (int)blockIdx.y);                                                           \
+    attn_body<D, PREFILL, 0, kAttnWindow>(&kv_map, a, (int)blockIdx.y);                                                           \
   }
 WINDOW_TC(kern_attn_window_decode_d64, 64, false)
 WINDOW_TC(kern_attn_window_decode_d128, 128, false)
@@ -268,16 +363,55 @@ WINDOW_TC(kern_attn_window_prefill_d256, 256, true)
                err, 0x7fffffff, hq, hk, q_stride, out_stride, max_pages, page_size, 1, 1, pool_pages, 1.f,                 \
                {window, c1, c2, out_scale, sink}};                                                                         \
     const int idx = y < 2 * m ? (y >> 1) : y - m;                                                                          \
-    if (is_p) attn_body<D, true, 2, true>(&kv_map, a, idx);                                                                \
-    else attn_body<D, false, 2, true>(&kv_map, a, idx);                                                                    \
+    if (is_p) attn_body<D, true, 2, kAttnWindow>(&kv_map, a, idx);                                                                \
+    else attn_body<D, false, 2, kAttnWindow>(&kv_map, a, idx);                                                                    \
   }
 WINDOW_RAGGED(kern_attn_window_ragged_d64, 64)
 WINDOW_RAGGED(kern_attn_window_ragged_d128, 128)
 
-// grid = rows x hq, block min(256, d)
+// ---- the same over the whole causal reach ------------------------------------------------------------------------------
+#define SINK_TC(name, D, PREFILL)                                                                                          \
+  extern "C" __global__ void __launch_bounds__(160, (PREFILL && D <= 128) ? 2 : 1)                                         \
+      name(const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* q, __nv_bfloat16* out, float* ws_o,            \
+           float* ws_ml, const int* block_table, const int* seq_lens, const int* cu_q, const int* work,                    \
+           const int* work_count, int hq, int hk, int q_stride, int out_stride, int max_pages, int page_size, int splits,  \
+           int pool_pages, int* err, const __nv_bfloat16* sink, const __nv_bfloat16* gate, int gate_stride,                \
+           float scale_log2) {                                                                                             \
+    AttnArgs a{q, out, ws_o, ws_ml, block_table, seq_lens, cu_q, work, work_count, err, 0x7fffffff, hq, hk, q_stride,      \
+               out_stride, max_pages, page_size, 1, splits, pool_pages, scale_log2, {0, 0.f, 0.f, 1.f, sink, gate, gate_stride}}; \
+    attn_body<D, PREFILL, 0, kAttnSink>(&kv_map, a, (int)blockIdx.y);                                                      \
+  }
+SINK_TC(kern_attn_sink_decode_d64, 64, false)
+SINK_TC(kern_attn_sink_decode_d128, 128, false)
+SINK_TC(kern_attn_sink_decode_d256, 256, false)
+SINK_TC(kern_attn_sink_prefill_d64, 64, true)
+SINK_TC(kern_attn_sink_prefill_d128, 128, true)
+SINK_TC(kern_attn_sink_prefill_d256, 256, true)
+
+#define SINK_RAGGED(name, D)                                                                                               \
+  extern "C" __global__ void __launch_bounds__(160, 2)                                                                     \
+      name(const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* q, __nv_bfloat16* out, const int* block_table, \
+           const int* seq_lens, const int* cu_q, const int* work_p, const int* count_p, const int* work_d,                 \
+           const int* count_d, int hq, int hk, int q_stride, int out_stride, int max_pages, int page_size, int pool_pages, \
+           int* err, const __nv_bfloat16* sink, const __nv_bfloat16* gate, int gate_stride, float scale_log2) {            \
+    const int np = *count_p, nd = *count_d, m = np < nd ? np : nd;                                                         \
+    const int y = blockIdx.y;                                                                                              \
+    if (y >= np + nd) return;                                                                                              \
+    const bool is_p = y < 2 * m ? !(y & 1) : np > nd;                                                                      \
+    AttnArgs a{q, out, nullptr, nullptr, block_table, seq_lens, cu_q, is_p ? work_p : work_d, is_p ? count_p : count_d,    \
+               err, 0x7fffffff, hq, hk, q_stride, out_stride, max_pages, page_size, 1, 1, pool_pages, scale_log2,          \
+               {0, 0.f, 0.f, 1.f, sink, gate, gate_stride}};                                                               \
+    const int idx = y < 2 * m ? (y >> 1) : y - m;                                                                          \
+    if (is_p) attn_body<D, true, 2, kAttnSink>(&kv_map, a, idx);                                                           \
+    else attn_body<D, false, 2, kAttnSink>(&kv_map, a, idx);                                                               \
+  }
+SINK_RAGGED(kern_attn_sink_ragged_d64, 64)
+SINK_RAGGED(kern_attn_sink_ragged_d128, 128)
+
+// grid = rows x hq, block min(256, d); sink and gate as in AttnWindow
 extern "C" __global__ void kern_attn_window_merge(const float* ws_o, const float* ws_ml, __nv_bfloat16* out,
-                                                  const __nv_bfloat16* sink, int rows, int hq, int d, int splits, int out_stride,
-                                                  float out_scale) {
+                                                  const __nv_bfloat16* sink, const __nv_bfloat16* gate, int gate_stride, int rows,
+                                                  int hq, int d, int splits, int out_stride, float out_scale) {
   pdl_wait();
   const int row = blockIdx.x;  // row * hq + head
   if (row >= rows) return;
@@ -290,13 +424,15 @@ extern "C" __global__ void kern_attn_window_merge(const float* ws_o, const float
     const size_t b = (size_t)row * splits + s;
     l += ws_ml[b * 2 + 1] * exp2f(ws_ml[b * 2] - m_use);
   }
-  const float f = sink_factor(m, l, __bfloat162float(sink[head]), out_scale);
+  const float f = sink_factor(m, l, sink ? __bfloat162float(sink[head]) : 0.f, out_scale);
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < splits; ++s) {
       const size_t b = (size_t)row * splits + s;
       acc += ws_o[b * d + c] * exp2f(ws_ml[b * 2] - m_use);
     }
-    out[(size_t)tk * out_stride + (size_t)head * d + c] = __float2bfloat16(acc * f);
+    acc *= f;
+    if (gate) acc *= gate_factor(__bfloat162float(gate[(size_t)tk * gate_stride + (size_t)head * d + c]));
+    out[(size_t)tk * out_stride + (size_t)head * d + c] = __float2bfloat16(acc);
   }
 }

@@ -121,8 +121,9 @@ struct EpArgs {
 // accumulator is scaled by *scale_a * *scale_b (per-tensor scales) before the epilogue's conversion.
 // HEADS: a batch of `heads` products over column ranges: C[:, h N ..] = A[:, h K ..] . W_h^T, W a 3-D map [K, N, heads]. A
 // head's last K block may reach into the next head's columns of A; the map fills W with zeros there.
-// EPI 3, 6, 7: W = [gate rows ; up rows], stored as their gated unit (SwiGLU, GEGLU, the clamped form with its limit)
-__host__ __device__ constexpr bool is_glu(int epi) { return epi == 3 || epi == 6 || epi == 7; }
+// EPI 3, 6, 7: W = [gate rows ; up rows], stored as their gated unit (SwiGLU, GEGLU, the clamped form with its limit). EPI 8: SwiGLU
+// with a bias per row of W, which R then holds
+__host__ __device__ constexpr bool is_glu(int epi) { return epi == 3 || epi == 6 || epi == 7 || epi == 8; }
 __host__ __device__ constexpr int glu_of(int epi) { return epi == 6 ? kGeglu : (epi == 7 ? kClampedGlu : kSwiglu); }
 
 template <int BN, int EPI, bool GROUPED = false, bool FP8 = false, bool MT2 = false, bool AG = false, int EP = 0, bool HEADS = false>
@@ -494,6 +495,17 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tma_a, const CUtens
             for (int v = 0; v < 4; ++v) {
               if (col + v * 8 < N / 2) {
                 float f[8];
+                if constexpr (EPI == 8) {
+                  const __nv_bfloat16* bias = reinterpret_cast<const __nv_bfloat16*>(Rv) + col + v * 8;
+                  const uint4 bg = *reinterpret_cast<const uint4*>(bias), bu = *reinterpret_cast<const uint4*>(bias + N / 2);
+                  const uint32_t wg[4] = {bg.x, bg.y, bg.z, bg.w}, wu[4] = {bu.x, bu.y, bu.z, bu.w};
+#pragma unroll
+                  for (int j = 0; j < 8; ++j) {
+                    const float2 a = unpack_bf16x2(wg[j >> 1]), b = unpack_bf16x2(wu[j >> 1]);
+                    g[v * 8 + j] = __float_as_uint(__uint_as_float(g[v * 8 + j]) + ((j & 1) ? a.y : a.x));
+                    u[v * 8 + j] = __float_as_uint(__uint_as_float(u[v * 8 + j]) + ((j & 1) ? b.y : b.x));
+                  }
+                }
 #pragma unroll
                 for (int j = 0; j < 8; ++j)
                   f[j] = glu<glu_of(EPI)>(__uint_as_float(g[v * 8 + j]), __uint_as_float(u[v * 8 + j]), glu_limit);
@@ -714,4 +726,8 @@ KERN_GEMM_ENTRY_M256(kern_gemm_bf16_tn_geglu_m256_n256, 6)
 KERN_GEMM_ENTRY(kern_gemm_bf16_tn_geglu_n256, 256, 6)
 KERN_GEMM_ENTRY(kern_gemm_bf16_tn_geglu_n128, 128, 6)
 KERN_GEMM_ENTRY(kern_gemm_bf16_tn_geglu_n64, 64, 6)
+KERN_GEMM_ENTRY_M256(kern_gemm_bf16_tn_swiglu_bias_m256_n256, 8)
+KERN_GEMM_ENTRY(kern_gemm_bf16_tn_swiglu_bias_n256, 256, 8)
+KERN_GEMM_ENTRY(kern_gemm_bf16_tn_swiglu_bias_n128, 128, 8)
+KERN_GEMM_ENTRY(kern_gemm_bf16_tn_swiglu_bias_n64, 64, 8)
 #endif  // KERN_GEMM_NO_ENTRIES

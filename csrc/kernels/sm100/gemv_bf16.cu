@@ -7,7 +7,7 @@
 // vectors of those rows, partial sums meet through shuffles and shared memory. Persistent grid: CTAs take row groups
 // round-robin, eight or so resident per SM, so tens of kilobytes of loads are in flight on every SM.
 // Epilogues as in the tensor-core GEMM: 0 store bf16, 1 store f32, 2 accumulate into a bf16 residual, 3 SwiGLU / 6 GEGLU over
-// weights stacked [gate rows ; up rows] (two gate rows and their two up rows per group).
+// weights stacked [gate rows ; up rows] (two gate rows and their two up rows per group), 8 SwiGLU with a bias per weight row.
 // (The reference calls a library GEMM for every shape; this kernel has no counterpart there.)
 #include "common.cuh"
 
@@ -23,7 +23,7 @@ __device__ __forceinline__ void gemv_body(const __nv_bfloat16* A, const __nv_bfl
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int kv = K >> 3;
   const int half = N >> 1;
-  constexpr bool kGlu = EPI == 3 || EPI == 6;      // SwiGLU, GEGLU
+  constexpr bool kGlu = EPI == 3 || EPI == 6 || EPI == 8;      // SwiGLU, GEGLU, SwiGLU with biases
   const int groups = kGlu ? (half + 1) / 2 : (N + R - 1) / R;
   for (int g = blockIdx.x; g < groups; g += gridDim.x) {
     int rows[R];
@@ -89,9 +89,14 @@ __device__ __forceinline__ void gemv_body(const __nv_bfloat16* A, const __nv_bfl
       if (m < M) {
         if constexpr (kGlu) {
           // outputs 2g (r = 0) and 2g + 1 (r = 1): gate in columns 0..1, up in 2..3
-          if (r < 2 && 2 * g + r < half)
-            reinterpret_cast<__nv_bfloat16*>(Cv)[(size_t)m * ldc + 2 * g + r] =
-                __float2bfloat16(glu<EPI == 6 ? kGeglu : kSwiglu>(part[0][m * R + r], part[0][m * R + 2 + r], 0.f));
+          if (r < 2 && 2 * g + r < half) {
+            float a = part[0][m * R + r], b = part[0][m * R + 2 + r];
+            if constexpr (EPI == 8) {
+              a += __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(Rv)[2 * g + r]);
+              b += __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(Rv)[half + 2 * g + r]);
+            }
+            reinterpret_cast<__nv_bfloat16*>(Cv)[(size_t)m * ldc + 2 * g + r] = __float2bfloat16(glu<EPI == 6 ? kGeglu : kSwiglu>(a, b, 0.f));
+          }
         } else {
           const int n = g * R + r;
           if (n < N) {
@@ -131,7 +136,8 @@ __device__ __forceinline__ void gemv_body(const __nv_bfloat16* A, const __nv_bfl
   KERN_GEMV_ENTRY(kern_gemv_bf16_tn_f32_m##MT, MT, 1)              \
   KERN_GEMV_ENTRY(kern_gemv_bf16_tn_acc_m##MT, MT, 2)              \
   KERN_GEMV_ENTRY(kern_gemv_bf16_tn_swiglu_m##MT, MT, 3)           \
-  KERN_GEMV_ENTRY(kern_gemv_bf16_tn_geglu_m##MT, MT, 6)
+  KERN_GEMV_ENTRY(kern_gemv_bf16_tn_geglu_m##MT, MT, 6)            \
+  KERN_GEMV_ENTRY(kern_gemv_bf16_tn_swiglu_bias_m##MT, MT, 8)
 
 KERN_GEMV_FAMILY(1)
 KERN_GEMV_FAMILY(2)

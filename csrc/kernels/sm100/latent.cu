@@ -1,40 +1,73 @@
 // build: precise
-// Latent attention whose keys and values are both linear maps of one cached row per token (no rotated part), in the
-// absorbed form: per head, score = (W_uk^T q) . c, and the weighted sum of the rows c goes through W_uv afterwards. These
-// kernels take any latent width and either activation type; mla_decode.cu holds the tensor-core form.
+// Latent attention whose keys and values are both linear maps of one cached row per token, in the absorbed form: per head,
+// score = (W_uk^T q) . c, and the weighted sum of the rows c goes through W_uv afterwards. A row may hold rotated key columns
+// behind the latent, one part for all heads, and a sink per head may join the denominator. These kernels take any latent width
+// and either activation type; mla_decode.cu holds the tensor-core form.
 //   kern_latent_append_<act>   RMS norm of a token's latent, written to its row of the paged cache
+//   kern_latent_prep_<act>     the same with the rotated columns behind it, and the RMS norm of a low-rank query row
 //   kern_latent_attn_<act>     one (row, head) per block: softmax over the row's causal reach, f32 throughout
+//   kern_latent_rot_attn_<act> the same with rotated columns (turning the query's) and a sink
 #include "act.cuh"
 
 using namespace kern;
 
 namespace {
 
+// x [n] -> out = x / rms w, by a block of 128
+template <typename T>
+KERN_DEVICE void norm_row(const T* x, const __nv_bfloat16* w, T* out, int n, float eps) {
+  __shared__ float part[4];
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < n; i += 128) { const float v = ldf(x + i); ss += v * v; }
+  ss = warp_sum(ss);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  const float inv = 1.f / sqrtf((part[0] + part[1] + part[2] + part[3]) / (float)n + eps);
+  for (int i = threadIdx.x; i < n; i += 128) stf(out + i, ldf(x + i) * inv * __bfloat162float(w[i]));
+}
+
+// the latent, then `rot` columns behind it turned by the token's position (pairs i, i + rot / 2)
 template <typename T>
 KERN_DEVICE void append_body(const T* lat, uint8_t* cache, const long long* slots, const __nv_bfloat16* w, int rank, int stride,
-                             float eps) {
-  __shared__ float part[4];
+                             float eps, const long long* positions = nullptr, const float* cos_tab = nullptr,
+                             const float* sin_tab = nullptr, int rot = 0, int max_pos = 0, int* err = nullptr) {
   const int t = blockIdx.x;
   const long long slot = slots[t];
   if (slot < 0) return;
   const T* x = lat + (size_t)t * stride;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < rank; i += 128) { const float v = ldf(x + i); ss += v * v; }
-  ss = warp_sum(ss);
-  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = ss;
-  __syncthreads();
-  const float inv = 1.f / sqrtf((part[0] + part[1] + part[2] + part[3]) / (float)rank + eps);
-  T* dst = reinterpret_cast<T*>(cache) + (size_t)slot * rank;
-  if (!KERN_CHECK(dst, (size_t)rank * sizeof(T), SITE_KV_APPEND)) return;
-  for (int i = threadIdx.x; i < rank; i += 128) stf(dst + i, ldf(x + i) * inv * __bfloat162float(w[i]));
+  T* dst = reinterpret_cast<T*>(cache) + (size_t)slot * (rank + rot);
+  if (!KERN_CHECK(dst, (size_t)(rank + rot) * sizeof(T), SITE_KV_APPEND)) return;
+  norm_row(x, w, dst, rank, eps);
+  if (rot == 0) return;
+  long long pos = positions[t];
+  if (pos < 0 || pos >= max_pos) {
+    if (threadIdx.x == 0) set_error(err, ERR_BOUNDS);
+    pos = 0;
+  }
+  const int half = rot >> 1;
+  for (int i = threadIdx.x; i < half; i += 128) {
+    const float a = ldf(x + rank + i), b = ldf(x + rank + half + i), c = cos_tab[pos * half + i], s = sin_tab[pos * half + i];
+    stf(dst + rank + i, a * c - b * s);
+    stf(dst + rank + half + i, b * c + a * s);
+  }
 }
 
+template <typename T>
+struct RotArgs {      // as LatentExtra in mla_decode.cu
+  const T* q_rot = nullptr;
+  int stride = 0, rot = 0, max_pos = 0;
+  const float* cos_tab = nullptr;
+  const float* sin_tab = nullptr;
+  const __nv_bfloat16* sink = nullptr;
+};
+
 // Four warps walk the keys (key j belongs to warp j % 4); a lane holds the columns i * 32 + lane of the query and of the
-// warp's running sum. RL = columns per lane.
-template <typename T, int RL>
+// warp's running sum. RL = columns per lane. The rotated columns of the query are turned into shared memory first (ROT).
+template <typename T, int RL, bool ROT = false>
 KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* table, const int* lens, const int* row_seq,
-                           int heads, int rank, int max_pages, int page, float scale, int* err) {
-  extern __shared__ __align__(16) float lat_sm[];      // [4][rank] partial sums, then [4] maxima, [4] weights
+                           int heads, int rank, int max_pages, int page, float scale, int* err, const RotArgs<T>& ex = RotArgs<T>()) {
+  extern __shared__ __align__(16) float lat_sm[];      // [4][rank] partial sums, then [4] maxima, [4] weights, [rot] turned query
   const int h = blockIdx.x, r = blockIdx.y;
   const int L = lens[r];
   if (L <= 0) return;
@@ -43,6 +76,19 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
   const int* pages = table + (size_t)(row_seq ? row_seq[r] : r) * max_pages;
   const T* rows = reinterpret_cast<const T*>(cache);
   const T* qr = q + ((size_t)r * heads + h) * rank;
+  const int cols = rank + (ROT ? ex.rot : 0);
+  float* turned = lat_sm + 4 * rank + 8;
+  if constexpr (ROT) {
+    if (L > ex.max_pos && threadIdx.x == 0) set_error(err, ERR_BOUNDS);
+    const int half = ex.rot >> 1, pos = min(L, ex.max_pos) - 1;
+    const T* x = ex.q_rot + (size_t)r * ex.stride + (size_t)h * ex.rot;
+    for (int i = threadIdx.x; i < half; i += 128) {
+      const float a = ldf(x + i), b = ldf(x + half + i), c = ex.cos_tab[(size_t)pos * half + i], s = ex.sin_tab[(size_t)pos * half + i];
+      turned[i] = a * c - b * s;
+      turned[half + i] = b * c + a * s;
+    }
+    __syncthreads();
+  }
   float qv[RL], o[RL];
 #pragma unroll
   for (int i = 0; i < RL; ++i) {
@@ -54,8 +100,8 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
   for (int j = warp; j < L; j += 4) {
     const int pi = j / page;
     if (pi >= max_pages) break;
-    const T* row = rows + ((size_t)pages[pi] * page + j % page) * rank;
-    if (!KERN_CHECK(row, (size_t)rank * sizeof(T), SITE_LATENT_ROW)) continue;
+    const T* row = rows + ((size_t)pages[pi] * page + j % page) * cols;
+    if (!KERN_CHECK(row, (size_t)cols * sizeof(T), SITE_LATENT_ROW)) continue;
     float c[RL], s = 0.f;
 #pragma unroll
     for (int i = 0; i < RL; ++i) {
@@ -63,6 +109,8 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
       c[i] = k < rank ? ldf(row + k) : 0.f;
       s += qv[i] * c[i];
     }
+    if constexpr (ROT)
+      for (int k = lane; k < ex.rot; k += 32) s += turned[k] * ldf(row + rank + k);
     s = warp_sum(s) * scale;
     const float mn = fmaxf(m, s), f = expf(m - mn), e = expf(s - mn);
     m = mn;
@@ -78,8 +126,15 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
   for (int i = 0; i < RL; ++i)
     if (i * 32 + lane < rank) acc[warp * rank + i * 32 + lane] = o[i];
   __syncthreads();
-  const float mx = fmaxf(fmaxf(ms[0], ms[1]), fmaxf(ms[2], ms[3]));
+  float mx = fmaxf(fmaxf(ms[0], ms[1]), fmaxf(ms[2], ms[3]));
   float f[4], den = 0.f;
+  if constexpr (ROT) {
+    if (ex.sink) {
+      const float sk = __bfloat162float(ex.sink[h]);
+      mx = fmaxf(mx, sk);
+      den = expf(sk - mx);
+    }
+  }
 #pragma unroll
   for (int w = 0; w < 4; ++w) { f[w] = expf(ms[w] - mx); den += f[w] * ls[w]; }
   for (int c = threadIdx.x; c < rank; c += 128) {
@@ -92,7 +147,7 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
 
 }  // namespace
 
-// append: grid = tokens, block 128. attn: grid [heads, rows], block 128, (4 rank + 8) floats of shared memory.
+// append, prep: grid = tokens, block 128. attn: grid [heads, rows], block 128, (4 rank + 8 + rot) floats of shared memory.
 #define LATENT_ATTN(T, SFX, W)                                                                                            \
   extern "C" __global__ void __launch_bounds__(128)                                                                       \
       kern_latent_attn_##SFX##_w##W(const T* q, const uint8_t* cache, T* out, const int* table, const int* lens,          \
@@ -101,6 +156,16 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
     pdl_wait();                                                                                                           \
     attn_body<T, W / 32>(q, cache, out, table, lens, row_seq, heads, rank, max_pages, page, scale, err);                  \
   }
+#define LATENT_ROT_ATTN(T, SFX, W)                                                                                        \
+  extern "C" __global__ void __launch_bounds__(128)                                                                       \
+      kern_latent_rot_attn_##SFX##_w##W(const T* q, const uint8_t* cache, T* out, const int* table, const int* lens,      \
+                                        const int* row_seq, int heads, int rank, int max_pages, int page, float scale,    \
+                                        int* err, const T* q_rot, const float* cos_tab, const float* sin_tab,             \
+                                        const __nv_bfloat16* sink, int rot_stride, int rot, int max_pos) {                \
+    pdl_wait();                                                                                                           \
+    const RotArgs<T> ex{q_rot, rot_stride, rot, max_pos, cos_tab, sin_tab, sink};                                         \
+    attn_body<T, W / 32, true>(q, cache, out, table, lens, row_seq, heads, rank, max_pages, page, scale, err, ex);        \
+  }
 #define LATENT_ENTRIES(T, SFX)                                                                                            \
   extern "C" __global__ void __launch_bounds__(128)                                                                       \
       kern_latent_append_##SFX(const T* lat, uint8_t* cache, const long long* slots, const __nv_bfloat16* w, int rank,    \
@@ -108,11 +173,25 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
     pdl_wait();                                                                                                           \
     append_body<T>(lat, cache, slots, w, rank, stride, eps);                                                              \
   }                                                                                                                       \
+  extern "C" __global__ void __launch_bounds__(128)                                                                       \
+      kern_latent_prep_##SFX(const T* rows, uint8_t* cache, T* q_low, const long long* positions, const long long* slots, \
+                             const float* cos_tab, const float* sin_tab, const __nv_bfloat16* w, const __nv_bfloat16* wq, \
+                             int rank, int rot, int q_rank, int stride, int q_stride, int max_pos, float eps, int* err) { \
+    pdl_wait();                                                                                                           \
+    norm_row(rows + (size_t)blockIdx.x * stride, wq, q_low + (size_t)blockIdx.x * q_stride, q_rank, eps);                 \
+    append_body<T>(rows + q_rank, cache, slots, w, rank, stride, eps, positions, cos_tab, sin_tab, rot, max_pos, err);    \
+    pdl_launch_dependents();                                                                                              \
+  }                                                                                                                       \
   LATENT_ATTN(T, SFX, 64)                                                                                                 \
   LATENT_ATTN(T, SFX, 128)                                                                                                \
   LATENT_ATTN(T, SFX, 256)                                                                                                \
   LATENT_ATTN(T, SFX, 512)                                                                                                \
-  LATENT_ATTN(T, SFX, 1024)
+  LATENT_ATTN(T, SFX, 1024)                                                                                               \
+  LATENT_ROT_ATTN(T, SFX, 64)                                                                                             \
+  LATENT_ROT_ATTN(T, SFX, 128)                                                                                            \
+  LATENT_ROT_ATTN(T, SFX, 256)                                                                                            \
+  LATENT_ROT_ATTN(T, SFX, 512)                                                                                            \
+  LATENT_ROT_ATTN(T, SFX, 1024)
 
 LATENT_ENTRIES(__nv_bfloat16, bf16)
 LATENT_ENTRIES(float, f32)

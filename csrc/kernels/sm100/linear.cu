@@ -27,10 +27,10 @@ KERN_DEVICE float glu_exact(float g, float u, float limit) {
   return g / (1.f + expf(-g)) * u;
 }
 
-// rows [m0, m_end) of A, columns [n0, ..) of C; with a gated unit W holds N gate rows, then N up rows
+// rows [m0, m_end) of A, columns [n0, ..) of C; with a gated unit W holds N gate rows, then N up rows. `bias`: one per row of W
 template <typename AT, typename OT, int ACT>
 KERN_DEVICE void tile_body(const AT* A, const __nv_bfloat16* W, OT* C, int m0, int m_end, int n0, int N, int K, int lda,
-                           int ldc, long long wsn, long long wsk, float limit = 0.f) {
+                           int ldc, long long wsn, long long wsk, float limit = 0.f, const __nv_bfloat16* bias = nullptr) {
   constexpr bool SWIGLU = ACT >= 0;
   __shared__ float as[LK][LB + 4], ws[LK][LB + 4], us[SWIGLU ? LK : 1][LB + 4];
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -74,7 +74,8 @@ KERN_DEVICE void tile_body(const AT* A, const __nv_bfloat16* W, OT* C, int m0, i
       const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
       if (m >= m_end || n >= N) continue;
       float v = acc[i][j];
-      if constexpr (SWIGLU) v = glu_exact<ACT>(v, acu[i][j], limit);
+      if (bias) v += __bfloat162float(bias[n]);
+      if constexpr (SWIGLU) v = glu_exact<ACT>(v, acu[i][j] + (bias ? __bfloat162float(bias[N + n]) : 0.f), limit);
       stf(C + (size_t)m * ldc + n, v);
     }
 }
@@ -98,12 +99,12 @@ KERN_DEVICE void gate_mul_body(const T* x, const T* gate, T* out, int tokens, in
 #define LINEAR_ENTRY(NAME, AT, OT, ACT)                                                                                     \
   extern "C" __global__ void __launch_bounds__(256)                                                                         \
       NAME(const AT* A, const __nv_bfloat16* W, OT* C, int M, int N, int K, int lda, int ldc, long long wsn, long long wsk, \
-           long long a_z, long long w_z, long long c_z, int* err, float limit) {                                            \
+           long long a_z, long long w_z, long long c_z, int* err, float limit, const __nv_bfloat16* bias) {                 \
     pdl_wait();                                                                                                             \
     if (M > (int)gridDim.y * LB && threadIdx.x == 0) set_error(err, ERR_BOUNDS);   /* rows the grid does not cover */       \
     const int z = blockIdx.z;                                                                                               \
     tile_body<AT, OT, ACT>(A + z * a_z, W + z * w_z, C + z * c_z, blockIdx.y * LB, M, blockIdx.x * LB, N, K, lda, ldc, wsn, \
-                           wsk, limit);                                                                                     \
+                           wsk, limit, bias);                                                                               \
   }
 // grid [ceil(N / 64), blocks], block 256; `tiles` int4 {expert, first row, rows, -}.
 #define LINEAR_GROUPED_ENTRY(NAME, T, ACT)                                                                                  \

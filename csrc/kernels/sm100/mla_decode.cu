@@ -31,8 +31,20 @@ constexpr int HM = 16;                   // heads per CTA
 constexpr int kPStride = TKM + 8, kPBytes = HM * kPStride * 2;
 constexpr int DQK = 576;                 // row of the 512 + 64 form
 
+// What a mixer with a rotated part and a sink adds: a head's rotated query columns are in a row of their own, not yet turned
+// (pairs i, i + rot / 2; a row's position is its length - 1), and `sink` (one per head) joins the denominator once, unscaled.
+struct LatentExtra {
+  const __nv_bfloat16* q_rot = nullptr;      // [rows][stride], head h at column h * rot
+  int stride = 0, rot = 0, max_pos = 0;
+  const float* cos_tab = nullptr;            // [max_pos][rot / 2]
+  const float* sin_tab = nullptr;
+  const __nv_bfloat16* sink = nullptr;
+};
+constexpr float kLog2eM = 1.4426950408889634f;
+
 // QB / VB: 64-column blocks of a cached row that serve as key / value. The 512 + 64 form is <9, 8>; a latent without
-// rotary columns is <B, B>, its last block filled up with zeros by the copy when the width is not a multiple of 64.
+// rotary columns is <B, B>, its last block filled up with zeros by the copy when the width is not a multiple of 64. Latents with
+// rotary columns behind them are <B, B> or <B + 1, B>, whichever their columns fill.
 template <int QB, int VB>
 struct MlaCfg {
   static constexpr int kQ = QB * 64;
@@ -70,7 +82,8 @@ template <int QB, int VB>
 __device__ __forceinline__ void mla_body(const CUtensorMap* lat_map, const __nv_bfloat16* q, __nv_bfloat16* out, float* ws_o,
                                          float* ws_ml, const int* block_table, const int* seq_lens, int seqs, int heads,
                                          int q_stride, int out_stride, int max_pages, int page_size, int splits, int pool_pages,
-                                         float scale_log2, int* err, const int* row_seq, int q_cols, int v_cols) {
+                                         float scale_log2, int* err, const int* row_seq, int q_cols, int v_cols,
+                                         const LatentExtra& ex = LatentExtra()) {
   using Cfg = MlaCfg<QB, VB>;
   constexpr int kStagesM = Cfg::kStages, kTileBytes = Cfg::kTileBytes, kQBytes = Cfg::kQBytes, kQStride = Cfg::kQStride;
   constexpr int ON = Cfg::kON;
@@ -105,6 +118,7 @@ __device__ __forceinline__ void mla_body(const CUtensorMap* lat_map, const __nv_
   const int nsplit = splits & 0xff, split_base = (splits >> 8) & 0xff;
   const int split_total = (splits >> 16) ? (splits >> 16) : nsplit;
   if (L <= 0 || valid_rows <= 0) return;       // uniform per CTA
+  if (ex.rot > 0 && L > ex.max_pos && threadIdx.x == 0) set_error(err, ERR_BOUNDS);
   const int ntiles_all = (L + TKM - 1) / TKM;
   int tile_lo = 0, tile_hi = ntiles_all;
   if (nsplit > 1) {
@@ -121,6 +135,20 @@ __device__ __forceinline__ void mla_body(const CUtensorMap* lat_map, const __nv_
     uint4 v = make_uint4(0, 0, 0, 0);
     if (r < valid_rows && c * 8 < q_cols)
       v = *reinterpret_cast<const uint4*>(q + (size_t)seq * q_stride + (size_t)(head0 + r) * q_cols + c * 8);
+    if (ex.rot > 0 && r < valid_rows && c * 8 >= q_cols && c * 8 < q_cols + ex.rot) {
+      const int half = ex.rot >> 1, pos = min(L - 1, ex.max_pos - 1);
+      const __nv_bfloat16* x = ex.q_rot + (size_t)seq * ex.stride + (size_t)(head0 + r) * ex.rot;
+      const float* cs = ex.cos_tab + (size_t)pos * half;
+      const float* sn = ex.sin_tab + (size_t)pos * half;
+      float f[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const int i = c * 8 - q_cols + e, j = i < half ? i : i - half;
+        const float a = __bfloat162float(x[i]), b = __bfloat162float(x[i < half ? i + half : j]);
+        f[e] = i < half ? a * cs[j] - b * sn[j] : a * cs[j] + b * sn[j];
+      }
+      v = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+    }
     *reinterpret_cast<uint4*>(qs + r * kQStride + c * 8) = v;
   }
   __syncthreads();
@@ -281,7 +309,16 @@ __device__ __forceinline__ void mla_body(const CUtensorMap* lat_map, const __nv_
 #pragma unroll
     for (int w = 0; w < MW; ++w) { lA += sm_l[w * HM + rA]; lB += sm_l[w * HM + rB]; }
     if (split_total == 1) {
-      const float iA = lA > 0.f ? 1.f / lA : 0.f, iB = lB > 0.f ? 1.f / lB : 0.f;
+      float iA = lA > 0.f ? 1.f / lA : 0.f, iB = lB > 0.f ? 1.f / lB : 0.f;
+      if (ex.sink != nullptr) {
+        auto factor = [&](float m, float l, int r) {
+          if (r >= valid_rows) return 0.f;
+          const float sk = __bfloat162float(ex.sink[head0 + r]) * kLog2eM, top = fmaxf(m, sk), f = exp2f(m - top);
+          return f / (l * f + exp2f(sk - top));
+        };
+        iA = factor(m_run[0], lA, rA);
+        iB = factor(m_run[1], lB, rB);
+      }
 #pragma unroll
       for (int i = 0; i < ON; ++i) {
         const int c = warp * (ON * 8) + i * 8 + 2 * (lane & 3);
@@ -339,6 +376,36 @@ KERN_LATENT_DECODE(5)
 KERN_LATENT_DECODE(6)
 KERN_LATENT_DECODE(7)
 KERN_LATENT_DECODE(8)
+
+// latents of `rank` columns with `rot` rotated ones behind them, B blocks of 64 as values; keys in as many or one more
+#define KERN_LATENT_ROT_DECODE(Q, B)                                                                                         \
+  extern "C" __global__ void __launch_bounds__(MW * 32 + 32, 1)                                                              \
+      kern_latent_rot_decode_bf16_q##Q##_b##B(                                                                               \
+          const __grid_constant__ CUtensorMap lat_map, const __nv_bfloat16* q, __nv_bfloat16* out, float* ws_o,              \
+          float* ws_ml, const int* block_table, const int* seq_lens, int seqs, int heads, int q_stride, int out_stride,      \
+          int max_pages, int page_size, int splits, int pool_pages, float scale_log2, int* err, const int* row_seq,          \
+          int rank, const __nv_bfloat16* q_rot, const float* cos_tab, const float* sin_tab, const __nv_bfloat16* sink,       \
+          int rot_stride, int rot, int max_pos) {                                                                            \
+    const LatentExtra ex{q_rot, rot_stride, rot, max_pos, cos_tab, sin_tab, sink};                                           \
+    mla_body<Q, B>(&lat_map, q, out, ws_o, ws_ml, block_table, seq_lens, seqs, heads, q_stride, out_stride, max_pages,       \
+                   page_size, splits, pool_pages, scale_log2, err, row_seq, rank, rank, ex);                                 \
+  }
+KERN_LATENT_ROT_DECODE(1, 1)
+KERN_LATENT_ROT_DECODE(2, 2)
+KERN_LATENT_ROT_DECODE(3, 3)
+KERN_LATENT_ROT_DECODE(4, 4)
+KERN_LATENT_ROT_DECODE(5, 5)
+KERN_LATENT_ROT_DECODE(6, 6)
+KERN_LATENT_ROT_DECODE(7, 7)
+KERN_LATENT_ROT_DECODE(8, 8)
+KERN_LATENT_ROT_DECODE(2, 1)
+KERN_LATENT_ROT_DECODE(3, 2)
+KERN_LATENT_ROT_DECODE(4, 3)
+KERN_LATENT_ROT_DECODE(5, 4)
+KERN_LATENT_ROT_DECODE(6, 5)
+KERN_LATENT_ROT_DECODE(7, 6)
+KERN_LATENT_ROT_DECODE(8, 7)
+KERN_LATENT_ROT_DECODE(9, 8)
 
 // ---- the steps around the attention of a latent-attention layer ----------------------------------------------------
 // kern_mla_rope_append_bf16: grid = tokens, block 128. Per token: RMS-norm of the 512 compressed columns (weight w),

@@ -3,7 +3,7 @@
 //   kern_moe_route_f32      router scores -> top-k expert ids and weights per token (sigmoid or softmax scoring,
 //                           optional selection bias, renormalise, scale)
 //   kern_moe_route_logits   the same by the logits plus a bias: top-k largest, softmax over the chosen
-//   kern_moe_route_groups   sigmoid scores inside the best groups of neighbouring experts
+//   kern_moe_route_groups   sigmoid or softmax scores, choices inside the best groups of neighbouring experts
 //   kern_moe_plan           counts per expert -> row offsets, the permuted row of every (token, choice), and the
 //                           M-tile table the grouped GEMM walks; experts outside [e_lo, e_hi) belong to another rank
 //   kern_moe_gather_bf16    x_perm[perm[t, j]] = x[t]
@@ -134,13 +134,14 @@ extern "C" __global__ void __launch_bounds__(128)
   }
 }
 
-// Routing inside groups: s = sigmoid(logits); `groups` equal groups of neighbours, a group's score the sum of its two largest
-// (its one, in groups of one); the k largest of the best `keep` groups are chosen (ties: the lower group, the lower id) and
-// weigh s, divided by their sum when `renorm`. One warp per token; E <= 1024, k <= 32, at most 64 groups.
+// Routing inside groups: s = sigmoid(logits), or their softmax; choices go by c = s + bias (one per expert, may be null), which
+// may be negative. `groups` equal groups of neighbours, a group's score the sum of its `group_top` largest c (1 or 2; its one, in
+// groups of one); the k largest c of the best `keep` groups are chosen (ties: the lower group, the lower id) and weigh s,
+// divided by their sum when `renorm`, times `scale`. One warp per token; E <= 1024, k <= 32, at most 64 groups.
 extern "C" __global__ void __launch_bounds__(128)
-    kern_moe_route_groups(const float* logits, int* topk_ids, float* topk_w, int tokens, int experts, int k, int groups, int keep,
-                          int renorm, int ld) {
-  extern __shared__ float route_sm[];      // [4][experts] scores, then [4][groups] group scores
+    kern_moe_route_groups(const float* logits, const __nv_bfloat16* bias, int* topk_ids, float* topk_w, int tokens, int experts, int k,
+                          int groups, int keep, int softmax, int group_top, int renorm, float scale, int ld) {
+  extern __shared__ float route_sm[];      // [4][experts] choice scores, then [4][groups] group scores
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp;
@@ -148,10 +149,21 @@ extern "C" __global__ void __launch_bounds__(128)
   float* sc = route_sm + warp * experts;
   float* gs = route_sm + 4 * experts + warp * groups;
   const float* row = logits + (size_t)t * ld;
-  for (int e = lane; e < experts; e += 32) {
-    const float z = row[e], x = exp2f(-fabsf(z) * 1.4426950408889634f);
-    sc[e] = z >= 0.f ? 1.f / (1.f + x) : x / (1.f + x);
+  float mx = -INFINITY, over = 1.f;
+  if (softmax) {
+    for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, row[e]);
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < experts; e += 32) sum += exp2f((row[e] - mx) * 1.4426950408889634f);
+    over = 1.f / warp_sum(sum);
   }
+  auto score = [&](int e) {
+    const float z = row[e];
+    if (softmax) return exp2f((z - mx) * 1.4426950408889634f) * over;
+    const float x = exp2f(-fabsf(z) * 1.4426950408889634f);
+    return z >= 0.f ? 1.f / (1.f + x) : x / (1.f + x);
+  };
+  for (int e = lane; e < experts; e += 32) sc[e] = score(e) + (bias ? __bfloat162float(bias[e]) : 0.f);
   __syncwarp();
   const int per = experts / groups;
   for (int g = lane; g < groups; g += 32) {
@@ -160,7 +172,7 @@ extern "C" __global__ void __launch_bounds__(128)
       const float v = sc[e];
       if (v > a) { b = a; a = v; } else if (v > b) b = v;
     }
-    gs[g] = per > 1 ? a + b : a;
+    gs[g] = per > 1 && group_top > 1 ? a + b : a;
   }
   __syncwarp();
   // a group stays when fewer than `keep` groups come before it
@@ -184,16 +196,17 @@ extern "C" __global__ void __launch_bounds__(128)
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
     }
-    if (bi >= experts) { bi = 0; best = 0.f; }      // no score is a number: still a valid row
+    const bool none = bi >= experts;      // no score is a number: still a valid row
+    if (none) bi = 0;
     __syncwarp();
     if (lane == 0) sc[bi] = -INFINITY;
     __syncwarp();
-    sum += best;
-    if (lane == j) { my_w = best; my_id = bi; }
+    if (lane == j) { my_w = none ? 0.f : (bias ? score(bi) : best); my_id = bi; }
   }
+  sum = warp_sum(my_w);
   if (lane < k) {
     topk_ids[(size_t)t * k + lane] = my_id;
-    topk_w[(size_t)t * k + lane] = renorm ? my_w / (sum + 1e-20f) : my_w;
+    topk_w[(size_t)t * k + lane] = (renorm ? my_w / (sum + 1e-20f) : my_w) * scale;
   }
 }
 

@@ -3,8 +3,11 @@
 //     x <- x + rms(y) w_post;   xn = rms(x) w_next
 // x is f32 (one row per token), y the sublayer's result: a row of a plain buffer, or the weighted sum of a token's k
 // expert rows, summed here. Without `w_post` y is added as it is.
+// or, in a decoder that only scales a sublayer's result, element by element:
+//     x <- x + s (y + bias + w_id h + sigmoid(gate) shared);   xn = rms(x) w_next
+// where h is the sublayer's own input, w_id the weight of the experts that hand it back, and `shared` an expert for every token.
 // kern_resid_embed  token row into x, and the first sublayer's normed input
-// kern_resid_mix    as above; with `hidden` the sum goes there instead and nothing is normed (the last sublayer)
+// kern_resid_scale  the second form; kern_resid_mix the first; with `hidden` the sum goes there instead and nothing is normed (the last sublayer)
 // Residual, sums and norms are f32; activations are T (bf16, or f32 in the 32-bit form of a model).
 #include "act.cuh"
 
@@ -117,6 +120,77 @@ KERN_DEVICE void mix_body(float* x, const T* y, const int* perm, const float* to
   if (!hidden) norm_out<T, V>(resid_sm, inv_rms(ss, width, eps), w_next, xn + (size_t)t * width, width);
 }
 
+// A sublayer's result: y, or with `perm` the weighted sum of a token's expert rows; choices without a row (perm < 0) are the
+// experts that hand back the input, xn as it is on entry. `shared` [rows][width] is weighed by sigmoid(gate[t gate_stride]).
+template <typename T, int V>
+KERN_DEVICE void scale_body(float* x, const T* y, const int* perm, const float* topw, const T* shared, const float* gate,
+                            const __nv_bfloat16* bias, const __nv_bfloat16* scale, const __nv_bfloat16* w_next, T* xn, float* hidden,
+                            int width, int k, int gate_stride, float eps) {
+  extern __shared__ __align__(16) float resid_sm[];
+  __shared__ float tw[32];
+  __shared__ int tr[32];
+  const int t = blockIdx.x;
+  if (perm) {
+    if (threadIdx.x < k) {
+      const int r = perm[(size_t)t * k + threadIdx.x];
+      const bool ok = r >= 0 && KERN_CHECK(y + (size_t)r * width, (size_t)width * sizeof(T), SITE_MOE_COMBINE);
+      tr[threadIdx.x] = ok ? r : -1;
+      tw[threadIdx.x] = topw[(size_t)t * k + threadIdx.x];
+    }
+    __syncthreads();
+  }
+  float self = 0.f;
+  if (perm)
+    for (int j = 0; j < k; ++j)
+      if (tr[j] < 0) self += tw[j];
+  const float g = shared ? 1.f / (1.f + expf(-gate[(size_t)t * gate_stride])) : 0.f;
+  float* xt = x + (size_t)t * width;
+  T* xnt = xn + (size_t)t * width;
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < width; i += 256 * V) {
+    Vec<V> v = {};
+    if (perm) {
+      for (int j = 0; j < k; ++j) {
+        if (tr[j] < 0) continue;
+        const Vec<V> r = ldv<V>(y + (size_t)tr[j] * width + i);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v.v[e] += tw[j] * r.v[e];
+      }
+      if (self != 0.f) {
+        const Vec<V> h = ldv<V>(xnt + i);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v.v[e] += self * h.v[e];
+      }
+    } else {
+      v = ldv<V>(y + (size_t)t * width + i);
+    }
+    if (shared) {
+      const Vec<V> r = ldv<V>(shared + (size_t)t * width + i);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v.v[e] += g * r.v[e];
+    }
+    if (bias) {
+      const Vec<V> r = ldv<V>(bias + i);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v.v[e] += r.v[e];
+    }
+    Vec<V> s = ldv<V>(xt + i);
+    const Vec<V> w = ldv<V>(scale + i);
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      s.v[e] += v.v[e] * w.v[e];
+      ss += s.v[e] * s.v[e];
+    }
+    if (hidden) {
+      stv<V>(hidden + (size_t)t * width + i, s);
+    } else {
+      stv<V>(xt + i, s);
+      stv<V>(resid_sm + i, s);
+    }
+  }
+  if (!hidden) norm_out<T, V>(resid_sm, inv_rms(ss, width, eps), w_next, xnt, width);
+}
+
 }  // namespace
 
 // grid = rows, block 256, `width` floats of shared memory
@@ -135,6 +209,17 @@ KERN_DEVICE void mix_body(float* x, const T* y, const int* perm, const float* to
     pdl_wait();                                                                                                           \
     if (width % 4 == 0) mix_body<T, 4>(x, y, perm, topw, w_post, w_next, xn, hidden, width, k, eps);                      \
     else mix_body<T, 1>(x, y, perm, topw, w_post, w_next, xn, hidden, width, k, eps);                                     \
+    pdl_launch_dependents();                                                                                              \
+  }                                                                                                                       \
+  extern "C" __global__ void __launch_bounds__(256)                                                                       \
+      kern_resid_scale_##SFX(float* x, const T* y, const int* perm, const float* topw, const T* shared, const float* gate, \
+                             const __nv_bfloat16* bias, const __nv_bfloat16* scale, const __nv_bfloat16* w_next, T* xn,   \
+                             float* hidden, int width, int k, int gate_stride, float eps) {                               \
+    pdl_wait();                                                                                                           \
+    if (width % 4 == 0)                                                                                                   \
+      scale_body<T, 4>(x, y, perm, topw, shared, gate, bias, scale, w_next, xn, hidden, width, k, gate_stride, eps);      \
+    else                                                                                                                  \
+      scale_body<T, 1>(x, y, perm, topw, shared, gate, bias, scale, w_next, xn, hidden, width, k, gate_stride, eps);      \
     pdl_launch_dependents();                                                                                              \
   }
 

@@ -227,10 +227,11 @@ def k_sample(g, logits, probs, out, temperature, top_k, top_p, min_p, seeds, off
     out[:r] = sample_rows(lv, temperature[:r], top_k[:r], top_p[:r], min_p[:r], seeds[:r], offsets[:r])
 
 
-def k_rope_table(g, cos, sin, max_pos, rot, theta_bits):
-    theta = struct.unpack("<d", struct.pack("<q", theta_bits))[0]
+def k_rope_table(g, cos, sin, max_pos, rot, theta_bits, factor_bits=None):
+    factor_bits = struct.unpack("<q", struct.pack("<d", 1.0))[0] if factor_bits is None else factor_bits
+    theta, factor = (struct.unpack("<d", struct.pack("<q", b))[0] for b in (theta_bits, factor_bits))
     half = rot // 2
-    inv = theta ** (-torch.arange(0, half, dtype=torch.float64) * 2.0 / rot)
+    inv = theta ** (-torch.arange(0, half, dtype=torch.float64) * 2.0 / rot) / factor
     ang = torch.arange(max_pos, dtype=torch.float64)[:, None] * inv[None]
     cos.view(-1)[: max_pos * half] = ang.cos().float().reshape(-1)
     sin.view(-1)[: max_pos * half] = ang.sin().float().reshape(-1)
@@ -395,7 +396,7 @@ CPU_KERNELS = {
     "kern_embedding_i64_bf16": k_embedding, "kern_embedding_i32_bf16": k_embedding,
     "kern_rms_norm_bf16": k_rms_norm, "kern_rms_norm_wide_bf16": k_rms_norm,
     "kern_fused_add_rms_norm_bf16": k_fused_add_rms_norm,
-    "kern_rope_kv_append_bf16": k_rope_append, "kern_rope_table_f32": k_rope_table,
+    "kern_rope_kv_append_bf16": k_rope_append, "kern_rope_table_f32": k_rope_table, "kern_rope_table_scaled_f32": k_rope_table,
     "kern_attn_plan": k_attn_plan, "kern_attn_merge_splits": k_noop,
     "kern_last_row": k_last_row, "kern_argmax_partial_bf16": k_argmax_partial, "kern_argmax_partial_f32": k_argmax_partial,
     "kern_argmax_final_i64": k_argmax_final, "kern_sample_bf16": k_sample, "kern_sample_f32": k_sample,

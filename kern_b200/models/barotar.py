@@ -23,7 +23,7 @@ import torch
 from . import blocks as K
 from . import common as C
 from . import listed
-from .listed import Listed, load_random
+from .listed import Listed, gla_sizes, load_random
 
 
 @dataclass
@@ -130,12 +130,6 @@ BAROTAR_LARGE = BarotarConfig(
 
 
 # ---- sizes of a layer ---------------------------------------------------------------------------------------
-def gla_sizes(m: dict) -> dict:
-    q, v = m["heads"] * m["dim"], m["heads"] * m["vdim"]
-    line, s_off = K.lin_line_bytes(m["heads"], m["dim"], m["vdim"])
-    return {"q": q, "v": v, "line": line, "s_off": s_off}
-
-
 def parallel_sizes(m: dict, width: int) -> dict:
     l, r = m["left"], m["right"]
     inner = r["heads"] * r["dim"]
@@ -237,75 +231,9 @@ def build_manifest(cfg: BarotarConfig) -> dict:
         name = op(f"resid_mix_{routed}", lambda: K.resid_mix_op(d, eps, A, routed))
         return {"op": name, "label": label, "args": [B("x"), y, post, same(subs[at + 1][0], (d,)), B("xn"), *extra]}
 
-    def linear_attention(p: str, st: str, H: int, dk: int, dv: int, stride: int, ptrs, z, prefill: bool, norm, norm_shared: bool, u, q_scale, out, out_stride,
-                         out_scale) -> list[dict]:
-        """The recurrence from its projections (`ptrs`: q, k, v, gate) to the gated rows in `out`."""
-        sfx, fused = "_p" if prefill else "_d", not prefill and K.lin_fused(dv)
-        tag = f"{sfx}_{H}x{dk}x{dv}x{stride}x{out_stride}" + ("u" if u else "") + f"_{out_scale!r}"
-
-        def make():
-            rule = K.lin_rule_op(H, dk, dv, stride, z["line"], z["s_off"], prefill, A, bonus=u is not None, q_scale=q_scale, fused=fused, norm_shared=norm_shared,
-                                 out_stride=out_stride, out_scale=out_scale, eps=eps, rows_max=cfg.max_tokens, seqs_max=S)
-            if fused:
-                return rule
-            ng = K.lin_norm_gate_op(H, dv, stride, norm_shared, out_stride, out_scale, eps, A)
-            return K.chain_ops(rule, ng, inner={(0, 5 if u else 4): "o", (1, 0): "o"}, scratch={"o": {"dtype": "f32", "shape": ["tokens", H * dv]}})
-
-        q, k, v, gate = ptrs
-        head, cu = [q, k, v, B("alpha"), *([u] if u else [])], [B("cu_seqlens")] if prefill else []
-        state = [{"state": st}, B("lines"), *cu]
-        args = [*head, out, *state, gate, norm, V("seqs")] if fused else [*head, *state, V("seqs"), gate, norm, out]
-        return [{"op": op(f"lin{tag}", make), "label": p + "rule", "args": args}]
-
     def gla(i: int, at: int, prefill: bool) -> list[dict]:
-        m, p, rank = layers[i]["mixer"], f"l{i}.mix.", cfg.ranks[i]
-        z = gla_sizes(m)
-        H, dk, dv, q, v, st = m["heads"], m["dim"], m["vdim"], z["q"], z["v"], f"lin.l{i}"
-        states[st] = {"bytes_per_seq": z["line"]}
-        w_in, proj = m_.rows_weight(f"w.{p}qkvga", d, [(p + "q", q), (p + "k", q), (p + "v", v), (p + "g", v), (p + "a1", rank)])
-        room("proj", proj); room("alpha", q, "f32"); room("mixed", v); room("y", d)
-        decay = op(f"decay_{q}x{rank}x{proj}_{m['tau']!r}", lambda: K.decay_op(q, rank, proj, "root", m["tau"], A))
-        col = lambda c: B("proj", c * es)
-        return [
-            linear("lin", proj, d, B("xn"), w_in, B("proj"), label=p + "in"),
-            {"op": decay, "label": p + "decay", "args": [col(2 * q + 2 * v), same(p + "a2", (q, rank)), same(p + "a2.b", (q,)), B("alpha"), V("tokens")]},
-            *linear_attention(p, st, H, dk, dv, proj, (col(0), col(q), col(2 * q), col(2 * q + v)), z, prefill, same(p + "norm", (dv,)), True, None,
-                              dk ** -0.5, B("mixed"), v, 1.0),
-            linear("lin", d, v, B("mixed"), same(p + "o", (d, v)), B("y"), label=p + "o"),
-            finish(at, B("y"), p + "out"),
-        ]
-
-    def rotary(dims: int, base: float) -> list[dict]:
-        """The cos and sin tables of one rotation, written when the model is loaded."""
-        name = f"rope.{dims}x{base!r}"
-        if name + ".cos" not in bufs:
-            for n in (".cos", ".sin"):
-                bufs[name + n] = {"dtype": "f32", "shape": [cfg.context, dims // 2], "kind": "carry"}
-            m_.once.append({"op": op(f"rope_{dims}x{base!r}", lambda: C.rope_table_op(cfg.context, dims, base)), "label": name, "args": [B(name + ".cos"), B(name + ".sin")]})
-        return [B(name + ".cos"), B(name + ".sin")]
-
-    plans = {}      # name -> (work lists, op, args): the plans of a ragged call's attention, made with the embedding
-
-    def lists_of(i: int) -> list[dict]:
-        """The work lists of layer i's tensor-core attention; layers whose blocks hold as many tokens share them."""
-        l = layers[i]["mixer"]["left"]
-        hq, hk, dim = l["heads"], l["kv_heads"], l["dim"]
-        name = f"plan.{hq // hk}" + (".128" if dim == 128 else "")
-        if name not in plans:
-            items = cfg.max_tokens // (64 // (hq // hk)) + S + 1
-            for n, shape in ((".work_p", [items, 2]), (".count_p", [1]), (".work_d", [S, 2]), (".count_d", [1])):
-                bufs[name + n] = {"dtype": "i32", "shape": shape, "kind": "workspace"}
-            lists = [B(name + n) for n in (".work_p", ".count_p", ".work_d", ".count_d")]
-            args = [B("cu_seqlens"), lists[0], lists[1], V("seqs"), {"expr": C.attn_plan_items(hq, hk)}, lists[2], lists[3]]
-            plans[name] = lists, C.attn_plan_op(hq, hk, S, dim), args
-        return plans[name][0]
-
-    def row_plan() -> list[dict]:
-        """The table row and reach of every token, for attention that takes a row per token."""
-        if "rows" not in plans:
-            c = m_.rows_call("")
-            plans["rows"] = [B("row_seq")], m_.ops.pop(c["op"]), c["args"]
-        return plans["rows"][0]
+        p = f"l{i}.mix."
+        return m_.gla(p, f"lin.l{i}", layers[i]["mixer"], cfg.ranks[i], prefill) + [finish(at, B("y"), p + "out")]
 
     def parallel(i: int, at: int, prefill: bool) -> list[dict]:
         m, p, rank = layers[i]["mixer"], f"l{i}.mix.", cfg.ranks[i]
@@ -316,15 +244,15 @@ def build_manifest(cfg: BarotarConfig) -> dict:
         w_in, qkv = m_.rows_weight(f"w.{lp}qkv", d, [(lp + "q", z["q"]), (lp + "k", z["k"]), (lp + "v", z["v"])])
         room("qkv", qkv); room("shifted", len(MU) * d); room("rkvg", 4 * n); room("low", rank, "f32"); room("alpha", n, "f32"); room("mixed", both); room("y", d)
         # left: window attention into columns 0 .. o of `mixed`
-        cos_sin = rotary(l["rot"]["dims"], l["rot"]["base"])
+        cos_sin = m_.rotary(l["rot"]["dims"], l["rot"]["base"])
         prep = op(f"prep_{hq}x{hk}x{dim}x{vdim}x{l['rot']['dims']}", lambda: K.qk_prep_op(hq, hk, dim, vdim, l["rot"]["dims"], page, qkv, cfg.context, eps, A))
         attn = op(f"window_attn{sfx}_{hq}x{hk}x{dim}x{vdim}x{l['mask']['size']}x{both}_{l['scale']!r}_{l['softcap']!r}_{m['left_scale']!r}", lambda: K.window_attn_op(
             hq, hk, dim, vdim, l["mask"]["size"], l["scale"], l["softcap"], page, W, qkv, both, m["left_scale"], prefill, A, seqs_max=S))
         lens, lists = B("seq_lens"), []
         if prefill and tiled[i]:
-            lists = [B("cu_seqlens"), *lists_of(i)]
+            lists = [B("cu_seqlens"), *m_.lists_of(hq, hk, dim)]
         elif prefill:
-            lens, lists = B("row_len"), row_plan()
+            lens, lists = B("row_len"), m_.row_plan()
         calls = [
             linear("lin", qkv, d, B("xn"), w_in, B("qkv"), label=lp + "qkv"),
             {"op": prep, "label": lp + "prep", "args": [B("qkv"), {"state": kv}, B("positions"), B("slot_mapping"), *cos_sin, same(lp + "q.norm", (dim,)),
@@ -343,7 +271,7 @@ def build_manifest(cfg: BarotarConfig) -> dict:
             {"op": heads, "label": rp + "rkvg", "args": [B("shifted"), weight(f"w.{rp}rkvg", (4, n, d), *[rp + s for s in "rkvg"]), B("rkvg"), V("tokens"), err]},
             linear("low", rank, d, B("shifted", 4 * d * es), same(rp + "w1", (rank, d)), B("low"), label=rp + "w1", epilogue="f32", lda=len(MU) * d),
             {"op": decay, "label": rp + "decay", "args": [B("low"), same(rp + "w2", (n, rank)), same(rp + "w0", (n,)), B("alpha"), V("tokens")]},
-            *linear_attention(rp, st, H, dk, dk, 4 * n, [col(c) for c in range(4)], z, prefill, same(rp + "norm", (n,)), False, same(rp + "u", (H, dk)), 1.0,
+            *m_.linear_attention(rp, st, H, dk, dk, 4 * n, [col(c) for c in range(4)], z, prefill, same(rp + "norm", (n,)), False, same(rp + "u", (H, dk)), 1.0,
                               B("mixed", z["o"] * es), both, m["right_scale"]),
         ]
         # both output projections next to each other, so one product adds the halves up
@@ -374,9 +302,6 @@ def build_manifest(cfg: BarotarConfig) -> dict:
             if b["mlp"] is not None:
                 calls += (dense if b["mlp"]["kind"] == "dense" else routed)(i, at)
                 at += 1
-        args = [B("token_ids"), same("embed", (cfg.vocab, d)), same(subs[0][0], (d,)), B("x"), B("xn"), err]
-        first = plans.values() if prefill else ()      # in one call with the embedding: both programs have as many calls to every layer
-        name = op("embed" + ("_p" if prefill else "_d"), lambda: K.chain_ops(K.resid_embed_op(d, cfg.vocab, eps, A), *[o for _, o, _ in first]))
-        return [{"op": name, "label": "embed", "args": args + [a for _, _, more in first for a in more]}, *calls]
+        return [m_.embed(subs[0][0], prefill), *calls]
 
     return m_.document(forward, "embed")

@@ -1,8 +1,8 @@
 """Op builders of the decoder blocks that take any size and either activation type (bf16, or f32 in a model's 32-bit
 form): matrix products, hyper-connections, the residual with norms on both sides, the Mamba-2 mixer, linear attention with a
-decay per key channel, latent attention without positions, attention in a sliding window, routed experts. Where a bf16 size
-fits the tensor-core kernels the op is the one `common.py` builds or the tensor-core form of the mechanism; the rest runs
-generic kernels. Weights are bf16 in both forms.
+decay per key channel, latent attention with or without rotated columns, attention in a sliding window or with a sink and an
+output gate, routed experts. Where a bf16 size fits the tensor-core kernels the op is the one `common.py` builds or the
+tensor-core form of the mechanism; the rest runs generic kernels. Weights are bf16 in both forms.
 """
 from __future__ import annotations
 
@@ -59,29 +59,32 @@ def tiles_fit(*extents: int) -> bool:
 
 # ---- matrix products ----------------------------------------------------------------------------------
 def _generic(sfx: str, iface, n: int, k: int, lda: int, ldc: int, rows_var: str, batch: int = 1, w=None, strides=(0, 0, 0),
-             limit: float = 0.0) -> dict:
+             limit: float = 0.0, bias=NULL) -> dict:
     """`w`: (row stride, column stride) of the weights in elements; `strides`: what a step of the batch adds to A, W, C."""
     wsn, wsk = w or (k, 1)
     return _launch("linear", f"kern_linear_{sfx}", [256, 1, 1], [-(-n // 64), {"ceil_div": [rows_var, 64]}, batch],
-                   iface[:3] + ["i32"] * 5 + ["i64"] * 5 + ["out buffer<i32>", "f32"],
-                   [P(0), P(1), P(2), P(3), I(n), I(k), I(lda), I(ldc), L(wsn), L(wsk), *map(L, strides), P(4), {"f32": limit}])
+                   iface[:3] + ["i32"] * 5 + ["i64"] * 5 + ["out buffer<i32>", "f32", bias[0]],
+                   [P(0), P(1), P(2), P(3), I(n), I(k), I(lda), I(ldc), L(wsn), L(wsk), *map(L, strides), P(4), {"f32": limit}, bias[1]])
 
 
 GLUS = ("swiglu", "geglu", "clamped")      # gated units over [gate rows ; up rows]; `clamped` takes a limit
 
 
 def linear_op(n: int, k: int, *, act: str = "bf16", epilogue: str = "store", rows_var: str = "tokens", rows_max: int,
-              lda: int | None = None, ldc: int | None = None, limit: float = 0.0) -> dict:
-    """C[rows, n] = A[rows, k] . W[n, k]^T. Interface [a, w, c, rows, err]; epilogue store | f32 | a gated unit as in `gemm_op`."""
+              lda: int | None = None, ldc: int | None = None, limit: float = 0.0, bias: bool = False) -> dict:
+    """C[rows, n] = A[rows, k] . W[n, k]^T. Interface [a, w, c, rows, err]; epilogue store | f32 | a gated unit as in `gemm_op`.
+    `bias` (swiglu): one per row of W, at the end of the interface."""
+    if bias and epilogue != "swiglu":
+        raise ValueError(f"biases in a product with epilogue `{epilogue}`")
     lda = k if lda is None else lda
     cols = n // 2 if epilogue in GLUS else n
     ldc = cols if ldc is None else ldc
     if act == "bf16" and epilogue != "clamped" and tiles_fit(cols, k, lda, ldc):
-        return C.gemm_op(n, k, epilogue=epilogue, rows_var=rows_var, rows_max=rows_max, lda=lda, ldc=ldc)
+        return C.gemm_op(n, k, epilogue=epilogue + ("_bias" if bias else ""), rows_var=rows_var, rows_max=rows_max, lda=lda, ldc=ldc)
     out = "f32" if epilogue == "f32" else act
     sfx = act + {"store": "", "f32": "_f32" if act == "bf16" else ""}.get(epilogue, "_" + epilogue)
-    iface = [f"in buffer<{act}>", "in buffer<bf16>", f"out buffer<{out}>", "i32", "out buffer<i32>"]
-    return _op(iface, _generic(sfx, iface, cols, k, lda, ldc, rows_var, limit=limit))
+    iface = [f"in buffer<{act}>", "in buffer<bf16>", f"out buffer<{out}>", "i32", "out buffer<i32>"] + (["in buffer<bf16>"] if bias else [])
+    return _op(iface, _generic(sfx, iface, cols, k, lda, ldc, rows_var, limit=limit, bias=(iface[5], P(5)) if bias else NULL))
 
 
 def head_tiles(n: int, k: int, lda: int, ldc: int, act: str) -> bool:
@@ -276,6 +279,38 @@ def latent_attn_op(heads: int, rank: int, scale: float, page_size: int, table_wi
                                {"f32": scale}, P(5)], shared_mem=(4 * rank + 8) * 4))
 
 
+# ---- latent attention with a rotated part and a sink ------------------------------------------------------------
+def latent_prep_op(rank: int, rot: int, q_rank: int, stride: int, q_stride: int, max_pos: int, eps: float, act: str = "bf16") -> dict:
+    """Of a projected row [query latent | latent | rotated key part]: the query latent normed into rows of its own, the latent
+    normed and the key part turned (pairs i, i + rot / 2) into a row of the paged cache.
+    Interface [rows, state, q latent, positions, slots, cos, sin, latent norm w, query norm w, err]."""
+    if rot % 2 or not rot:
+        raise ValueError(f"a rotated key part of {rot} columns")
+    iface = [f"in buffer<{act}>", "inout state", f"out buffer<{act}>", "in buffer<i64>", "in buffer<i64>", "in buffer<f32>", "in buffer<f32>", "in buffer<bf16>",
+             "in buffer<bf16>", "out buffer<i32>"]
+    return _op(iface, _launch("latent", f"kern_latent_prep_{act}", [128, 1, 1], ["tokens", 1, 1], iface[:9] + ["i32"] * 6 + ["f32", "out buffer<i32>"],
+                              [*map(P, range(9)), I(rank), I(rot), I(q_rank), I(stride), I(q_stride), I(max_pos), {"f32": eps}, P(9)]))
+
+
+def latent_rot_attn_op(heads: int, rank: int, rot: int, scale: float, page_size: int, table_width: int, max_pos: int, rot_stride: int, ragged: bool,
+                       act: str = "bf16", seqs_max: int = 0) -> dict:
+    """`latent_attn_op` over rows with `rot` rotated key columns behind the latent, and a sink per head.
+    Interface [q, state, out, block_table, lens, err] (+ [row_seq] for ragged rows), then [q_rot, cos, sin, sink]."""
+    if act == "bf16" and tiles_fit(rank, rot) and rank <= 512 and rot <= 64 and (page_size % 64 == 0 or 64 % page_size == 0):
+        return C.mla_attn_op(heads, page_size, table_width, ragged, seqs_max=seqs_max, rank=rank, scale=scale, rot=rot, max_pos=max_pos, rot_stride=rot_stride)
+    if rank > 1024:
+        raise ValueError(f"latent rows of {rank} columns (at most 1024)")
+    iface = [f"in buffer<{act}>", "in state", f"out buffer<{act}>", "in buffer<i32>", "in buffer<i32>", "out buffer<i32>"]
+    iface += ["in buffer<i32>"] if ragged else []
+    o = len(iface)
+    iface += [f"in buffer<{act}>", "in buffer<f32>", "in buffer<f32>", "in buffer<bf16>"]
+    w = next(n for n in (64, 128, 256, 512, 1024) if rank <= n)
+    return _op(iface, _launch("latent", f"kern_latent_rot_attn_{act}_w{w}", [128, 1, 1], [heads, "tokens" if ragged else "seqs", 1],
+                              [*iface[:5], iface[6] if ragged else NULL[0], "i32", "i32", "i32", "i32", "f32", "out buffer<i32>", *iface[o:], "i32", "i32", "i32"],
+                              [*map(P, range(5)), P(6) if ragged else NULL[1], I(heads), I(rank), I(table_width), I(page_size), {"f32": scale}, P(5),
+                               *map(P, range(o, o + 4)), I(rot_stride), I(rot), I(max_pos)], shared_mem=(4 * rank + 8 + rot) * 4))
+
+
 # ---- a residual with norms on both sides of a sublayer -----------------------------------------------------
 def resid_embed_op(width: int, vocab: int, eps: float, act: str = "bf16") -> dict:
     """Token row into the f32 residual, and the first sublayer's normed input. Interface [ids, table, next norm w, x, xn, err]."""
@@ -297,6 +332,32 @@ def resid_mix_op(width: int, eps: float, act: str = "bf16", routed: int = 0, las
     parts = [(iface[0], P(0)), (iface[1], P(1)), *route, (iface[2], P(2)), *tail]
     return _op(iface, _launch("resid", f"kern_resid_mix_{act}", [256, 1, 1], ["tokens", 1, 1], [t for t, _ in parts] + ["i32", "i32", "f32"],
                               [a for _, a in parts] + [I(width), I(routed), {"f32": eps}], shared_mem=width * 4))
+
+
+def resid_scale_op(width: int, eps: float, act: str = "bf16", *, routed: int = 0, bias: bool = False, shared_gate: int | None = None,
+                   last: bool = False) -> dict:
+    """x += s y element by element, and the next sublayer's normed input. Interface [x, y, s, w_next, xn] (`last`: [x, y, s, hidden],
+    plus xn at the end of the list below when experts may hand back the input), then with `bias` [bias], with `routed` (experts
+    per token) [perm, weights] — y holds expert-sorted rows, and a choice without a row stands for xn itself — and with
+    `shared_gate` (the row stride of the gate's buffer) [shared rows, gate]: sigmoid(gate) weighs an expert of every token."""
+    iface = ["in buffer<f32>" if last else "inout buffer<f32>", f"in buffer<{act}>", "in buffer<bf16>"]
+    iface += ["out buffer<f32>"] if last else ["in buffer<bf16>", f"inout buffer<{act}>"]
+
+    def more(*types):
+        at = len(iface)
+        iface.extend(types)
+        return [(t, P(at + i)) for i, t in enumerate(types)]
+
+    b = more("in buffer<bf16>") if bias else [NULL]
+    route = more("in buffer<i32>", "in buffer<f32>") if routed else [NULL, NULL]
+    sh = more(f"in buffer<{act}>", "in buffer<f32>") if shared_gate is not None else [NULL, NULL]
+    if last:
+        tail = [NULL, *(more(f"in buffer<{act}>") if routed else [NULL]), (iface[3], P(3))]
+    else:
+        tail = [(iface[3], P(3)), (iface[4], P(4)), NULL]
+    parts = [(iface[0], P(0)), (iface[1], P(1)), *route, *sh, *b, (iface[2], P(2)), *tail]
+    return _op(iface, _launch("resid", f"kern_resid_scale_{act}", [256, 1, 1], ["tokens", 1, 1], [t for t, _ in parts] + ["i32", "i32", "i32", "f32"],
+                              [a for _, a in parts] + [I(width), I(routed), I(shared_gate or 0), {"f32": eps}], shared_mem=width * 4))
 
 
 # ---- linear attention with a decay per key channel -----------------------------------------------------------
@@ -409,6 +470,21 @@ def qk_prep_op(hq: int, hk: int, d: int, dv: int, rot: int, page_size: int, row_
                               shared_mem=8 * max(d, dv) * 4))
 
 
+def qk_prep_whole_op(hq: int, hk: int, d: int, dv: int, v_col: int, rot: int, page_size: int, row_stride: int, max_pos: int, eps: float, act: str = "bf16",
+                     halves: bool = False) -> dict:
+    """As `qk_prep_op` with norms over all columns of q and of k at once, and values from column `v_col` of the row, which may be
+    the keys' own. Interface [qkv, state, positions, slots, cos, sin, q norm w, k norm w, err]."""
+    if rot % 2 or rot > d:
+        raise ValueError(f"rotary positions on {rot} of {d} columns")
+    if (hq + hk) * d > 50000:
+        raise ValueError(f"{hq} + {hk} heads of {d} columns (at most 50000 together)")
+    iface = [f"inout buffer<{act}>", "inout state", "in buffer<i64>", "in buffer<i64>", "in buffer<f32>", "in buffer<f32>", "in buffer<bf16>",
+             "in buffer<bf16>", "out buffer<i32>"]
+    return _op(iface, _launch("attn_window", f"kern_qk_prep_whole_{act}", [256, 1, 1], ["tokens", 1, 1], iface[:8] + ["i32"] * 10 + ["f32", "out buffer<i32>"],
+                              [*map(P, range(8)), I(hq), I(hk), I(d), I(dv), I(v_col), I(rot), I(int(halves)), I(page_size), I(row_stride), I(max_pos), {"f32": eps}, P(8)],
+                              shared_mem=(hq + hk) * d * 4))
+
+
 def window_tiles(hq: int, hk: int, d: int, dv: int, page_size: int, act: str) -> bool:
     """Whether windowed attention of this size runs on the tensor-core kernels."""
     return act == "bf16" and d == dv and d in (64, 128, 256) and hq // hk <= 16 and (page_size % 64 == 0 or (page_size % 8 == 0 and 64 % page_size == 0))
@@ -429,9 +505,9 @@ def window_attn_op(hq: int, hk: int, d: int, dv: int, window: int, scale: float,
         w = next(n for n in (64, 128, 256, 512) if max(d, dv) <= n)
         row_t, row_a = (iface[7], P(7)) if ragged else NULL
         return _op(iface, _launch("attn_window", f"kern_window_attn_{act}_w{w}", [128, 1, 1], [hq, "tokens" if ragged else "seqs", 1],
-                                  [*iface[:5], row_t, iface[5]] + ["i32"] * 9 + ["f32"] * 3 + ["out buffer<i32>"],
-                                  [*map(P, range(5)), row_a, P(5), I(hq), I(hk), I(d), I(dv), I(q_stride), I(out_stride), I(table_width), I(page_size), I(window),
-                                   {"f32": scale}, {"f32": cap}, {"f32": out_scale}, P(6)], shared_mem=(4 * dv + 8) * 4))
+                                  [*iface[:5], row_t, iface[5], NULL[0]] + ["i32"] * 10 + ["f32"] * 3 + ["out buffer<i32>"],
+                                  [*map(P, range(5)), row_a, P(5), NULL[1], I(hq), I(hk), I(d), I(dv), I(q_stride), I(out_stride), I(0), I(table_width), I(page_size),
+                                   I(window), {"f32": scale}, {"f32": cap}, {"f32": out_scale}, P(6)], shared_mem=(4 * dv + 8) * 4))
     g, kv = hq // hk, C._kv_map(d, page_size, 1)
     win_t = ["out buffer<i32>", "in buffer<bf16>", "i32", "f32", "f32", "f32"]
     win_a = [P(6), P(5), I(window), {"f32": 2 * LOG2E * scale / cap}, {"f32": cap * LOG2E}, {"f32": out_scale}]
@@ -461,8 +537,8 @@ def window_attn_op(hq: int, hk: int, d: int, dv: int, window: int, scale: float,
                                     [kv, P(0), P(2), *ws, P(3), P(4), L(0), L(0), L(0), *sizes(splits), *win_a], shared_mem=C.attn_smem(d), **kw))
             if splits > 1:
                 launches.append(_launch("attn_window", "kern_attn_window_merge", [min(256, d), 1, 1], [{"mul": ["seqs", hq]}, 1, 1],
-                                        ["in buffer<f32>", "in buffer<f32>", iface[2], "in buffer<bf16>"] + ["i32"] * 5 + ["f32"],
-                                        [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, P(2), P(5), I(C.I32_MAX), I(hq), I(d), I(splits), I(out_stride), {"f32": out_scale}], **kw))
+                                        ["in buffer<f32>", "in buffer<f32>", iface[2], "in buffer<bf16>", NULL[0]] + ["i32"] * 6 + ["f32"],
+                                        [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, P(2), P(5), NULL[1], I(0), I(C.I32_MAX), I(hq), I(d), I(splits), I(out_stride), {"f32": out_scale}], **kw))
         scratch = {"scratch": {"ws_o": {"dtype": "f32", "shape": ["seqs", hq * most * d]}, "ws_ml": {"dtype": "f32", "shape": ["seqs", hq * most * 2]}}} if most > 1 else {}
         return _op(iface, *launches, **scratch)
     iface += ["in buffer<i32>"] * 5
@@ -488,6 +564,80 @@ def window_attn_op(hq: int, hk: int, d: int, dv: int, window: int, scale: float,
     return _op(iface, listed("prefill", 8, C.attn_smem(d, prefill=True), grid(64)), rows())
 
 
+# ---- attention with a sink and an output gate --------------------------------------------------------------------
+def sink_attn_op(hq: int, hk: int, d: int, dv: int, scale: float, page_size: int, table_width: int, q_stride: int, out_stride: int, gate_stride: int,
+                 ragged: bool, act: str = "bf16", *, sink: bool = False, seqs_max: int = 0) -> dict:
+    """Causal attention whose softmax has one more score per query head in the denominator (`sink`: learned; else a score of 0),
+    rows times sigmoid(gate). Interface [q, state, out, block_table, lens, gate, err, (sink)], then for ragged rows on the tensor
+    cores (`window_tiles`) [cu_seqlens, work_p, count_p, work_d, count_d] as `attn_plan_op` fills them (lens per sequence), else
+    [row_seq] (lens per row)."""
+    if hq % hk:
+        raise ValueError(f"{hq} query heads over {hk} key heads")
+    iface = [f"in buffer<{act}>", "in state", f"out buffer<{act}>", "in buffer<i32>", "in buffer<i32>", f"in buffer<{act}>", "out buffer<i32>"]
+    iface += ["in buffer<bf16>"] if sink else []
+    sk, o = (("in buffer<bf16>", P(7)) if sink else NULL), len(iface)
+    if not window_tiles(hq, hk, d, dv, page_size, act):
+        iface += ["in buffer<i32>"] if ragged else []
+        if max(d, dv) > 512:
+            raise ValueError(f"heads of {d} / {dv} columns (at most 512)")
+        w = next(n for n in (64, 128, 256, 512) if max(d, dv) <= n)
+        row_t, row_a = (iface[o], P(o)) if ragged else NULL
+        return _op(iface, _launch("attn_window", f"kern_window_attn_{act}_w{w}", [128, 1, 1], [hq, "tokens" if ragged else "seqs", 1],
+                                  [*iface[:5], row_t, sk[0], iface[5]] + ["i32"] * 10 + ["f32"] * 3 + ["out buffer<i32>"],
+                                  [*map(P, range(5)), row_a, sk[1], P(5), I(hq), I(hk), I(d), I(dv), I(q_stride), I(out_stride), I(gate_stride), I(table_width),
+                                   I(page_size), I(C.I32_MAX), {"f32": scale}, {"f32": 0.0}, {"f32": 1.0}, P(6)], shared_mem=(4 * dv + 8) * 4))
+    g, kv = hq // hk, C._kv_map(d, page_size, 1)
+    form_t, form_a = ["out buffer<i32>", sk[0], iface[5], "i32", "f32"], [P(6), sk[1], P(5), I(gate_stride), {"f32": scale * LOG2E}]
+    lp = lambda ws, lists: ["bytes<128>", iface[0], iface[2]] + (["out buffer<f32>"] * 2 if ws else ["i64"] * 2) + ["in buffer<i32>"] * 2 \
+        + (["in buffer<i32>"] * 3 if lists else ["i64"] * 3) + ["i32"] * 8 + form_t
+    sizes = lambda splits: [I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(splits), I(C.I32_MAX)]
+    if not ragged:
+        ranges, hi = [], seqs_max
+        for splits in (1, 2, 4, 8, 16, 32):      # enough sequences that heads x sequences x splits cover the SMs
+            lo = 1 if splits == 32 else max(1, -(-C.SMS // (hk * splits)))
+            if lo <= hi:
+                ranges.append((splits, lo, hi))
+                hi = lo - 1
+            if hi < 1:
+                break
+        launches, most = [], max(s for s, _, _ in ranges)
+        for splits, lo, hi in ranges:
+            when = {"var": "seqs", **({"min": lo} if lo > 1 else {}), **({"max": hi} if hi < seqs_max else {})}
+            kw = {"when": when} if len(when) > 1 else {}
+            ws = [{"scratch": "ws_o"}, {"scratch": "ws_ml"}] if splits > 1 else [L(0), L(0)]
+            launches.append(_launch("attn_window", f"kern_attn_sink_decode_d{d}", [160, 1, 1], [hk, "seqs", splits], lp(splits > 1, False),
+                                    [kv, P(0), P(2), *ws, P(3), P(4), L(0), L(0), L(0), *sizes(splits), *form_a], shared_mem=C.attn_smem(d), **kw))
+            if splits > 1:
+                launches.append(_launch("attn_window", "kern_attn_window_merge", [min(256, d), 1, 1], [{"mul": ["seqs", hq]}, 1, 1],
+                                        ["in buffer<f32>", "in buffer<f32>", iface[2], sk[0], iface[5]] + ["i32"] * 6 + ["f32"],
+                                        [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, P(2), sk[1], P(5), I(gate_stride), I(C.I32_MAX), I(hq), I(d), I(splits), I(out_stride),
+                                         {"f32": 1.0}], **kw))
+        scratch = {"scratch": {"ws_o": {"dtype": "f32", "shape": ["seqs", hq * most * d]}, "ws_ml": {"dtype": "f32", "shape": ["seqs", hq * most * 2]}}} if most > 1 else {}
+        return _op(iface, *launches, **scratch)
+    iface += ["in buffer<i32>"] * 5
+    lists = [P(o + i) for i in range(5)]
+    mode = C.attn_mode(hq, hk, d)
+    few = {"var": "seqs", "max": C.FMHA_SEQS}
+    many = {"var": "seqs", "min": C.FMHA_SEQS + 1}
+    grid = lambda rows: [hk, {"add": [{"ceil_div": ["tokens", rows // g]}, "seqs"]}, 1]
+    tail = [I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(C.I32_MAX), *form_a]
+    causal = lambda **kw: _launch("attn_fmha", "kern_attn_sink_fmha_d128", [192, 1, 1], grid(128), ["bytes<128>", iface[0], iface[2]] + ["in buffer<i32>"] * 5 + ["i32"] * 7 + form_t,
+                                  [kv, P(0), P(2), P(3), P(4), *lists[:3], *tail], shared_mem=768 + 128 * d * 2 + 128 * 64 * 2 + 2 * 2 * (64 * d * 2) + 256, **kw)
+    listed = lambda kind, work, smem, g_, **kw: _launch("attn_window", f"kern_attn_sink_{kind}_d{d}", [160, 1, 1], g_, lp(False, True),
+                                                        [kv, P(0), P(2), L(0), L(0), P(3), P(4), lists[0], lists[work], lists[work + 1], *sizes(1), *form_a],
+                                                        shared_mem=smem, **kw)
+    one = lambda **kw: _launch("attn_window", f"kern_attn_sink_ragged_d{d}", [160, 1, 1], grid(64), ["bytes<128>", iface[0], iface[2]] + ["in buffer<i32>"] * 7 + ["i32"] * 7 + form_t,
+                               [kv, P(0), P(2), P(3), P(4), *lists, *tail], shared_mem=C.attn_smem(d, prefill=True), **kw)
+    rows = lambda **kw: listed("decode", 3, C.attn_smem(d), [hk, "seqs", 1], **kw)
+    if mode == "auto":
+        return _op(iface, causal(when=few), rows(when=few), one(when=many))
+    if mode in ("fmha", "fmha2"):
+        return _op(iface, causal(), rows())
+    if mode == "ragged":
+        return _op(iface, one())
+    return _op(iface, listed("prefill", 1, C.attn_smem(d, prefill=True), grid(64)), rows())
+
+
 # ---- routed experts ---------------------------------------------------------------------------------------
 def route_logits_op(experts: int, top: int, bias: bool = True) -> dict:
     """The `top` largest of logits + bias, weighed by the softmax over them. Interface [logits, (bias,) ids, weights, tokens]."""
@@ -501,14 +651,21 @@ def route_logits_op(experts: int, top: int, bias: bool = True) -> dict:
                               [P(0), b_a, P(o), P(o + 1), P(o + 2), I(experts), I(top), I(experts)]))
 
 
-def route_groups_op(experts: int, top: int, groups: int = 1, keep: int = 1, renorm: bool = False) -> dict:
-    """Sigmoid scores; the `top` largest inside the best `keep` of equal groups of neighbours (a group's score: the sum of its two
-    largest), weighing their scores. Interface [logits, ids, weights, tokens]."""
+def route_groups_op(experts: int, top: int, groups: int = 1, keep: int = 1, renorm: bool = False, *, softmax: bool = False,
+                    correction: bool = False, group_top: int = 2, scale: float = 1.0, ld: int | None = None) -> dict:
+    """Sigmoid scores, or their softmax; choices by the score plus a `correction` per expert: the `top` largest inside the best `keep`
+    of equal groups of neighbours (a group's score: the sum of its `group_top` largest choices, two or one), weighing their
+    scores, `renorm` divided by their sum, times `scale`. `ld`: row stride of the logits.
+    Interface [logits, (correction,) ids, weights, tokens]."""
     if not (1 <= top <= min(32, keep * (experts // groups)) and experts <= 1024 and experts % groups == 0 and 1 <= keep <= groups <= 64):
         raise ValueError(f"{top} of {experts} experts per token in {keep} of {groups} groups (at most 32 of 1024, 64 groups)")
-    iface = ["in buffer<f32>", "out buffer<i32>", "out buffer<f32>", "i32"]
-    return _op(iface, _launch("moe", "kern_moe_route_groups", [128, 1, 1], [{"ceil_div": ["tokens", 4]}, 1, 1], iface + ["i32"] * 6,
-                              [*map(P, range(4)), I(experts), I(top), I(groups), I(keep), I(int(renorm)), I(experts)], shared_mem=4 * (experts + groups) * 4))
+    iface = ["in buffer<f32>"] + (["in buffer<bf16>"] if correction else []) + ["out buffer<i32>", "out buffer<f32>", "i32"]
+    b_t, b_a = (iface[1], P(1)) if correction else NULL
+    o = 2 if correction else 1
+    return _op(iface, _launch("moe", "kern_moe_route_groups", [128, 1, 1], [{"ceil_div": ["tokens", 4]}, 1, 1],
+                              [iface[0], b_t, *iface[o:]] + ["i32"] * 7 + ["f32", "i32"],
+                              [P(0), b_a, P(o), P(o + 1), P(o + 2), I(experts), I(top), I(groups), I(keep), I(int(softmax)), I(group_top), I(int(renorm)),
+                               {"f32": scale}, I(ld or experts)], shared_mem=4 * (experts + groups) * 4))
 
 
 def routed_tile_rows(act: str, width: int, ff: int) -> int:

@@ -177,16 +177,18 @@ def gemm_op(n: int, k: int, *, epilogue: str = "store", rows_var: str = "tokens"
             lda: int | None = None, ldc: int | None = None) -> dict:
     """C[rows, n] = A[rows, k] · W[n, k]ᵀ through the tcgen05 GEMM, one launch per `when` range.
 
-    Interface: [a, w, c, rows, err]. epilogue store | acc (c += …, c is inout) | f32 | swiglu | geglu
-    (c is [rows, n/2] over weights stacked [gate rows ; up rows])."""
+    Interface: [a, w, c, rows, err]. epilogue store | acc (c += …, c is inout) | f32 | swiglu | geglu | swiglu_bias
+    (c is [rows, n/2] over weights stacked [gate rows ; up rows]; swiglu_bias takes one bias per weight row at the end)."""
     lda = k if lda is None else lda
-    glu = epilogue in ("swiglu", "geglu")
+    bias = epilogue == "swiglu_bias"
+    glu = epilogue in ("swiglu", "geglu") or bias
     out_cols = n // 2 if glu else n
     ldc = out_cols if ldc is None else ldc
     cdt = "f32" if epilogue == "f32" else "bf16"
     cdir = "inout" if epilogue == "acc" else "out"
-    suffix = {"store": "", "acc": "_acc", "f32": "_f32", "swiglu": "_swiglu", "geglu": "_geglu"}[epilogue]
-    iface = ["in buffer<bf16>", "in buffer<bf16>", f"{cdir} buffer<{cdt}>", "i32", "out buffer<i32>"]
+    suffix = {"store": "", "acc": "_acc", "f32": "_f32", "swiglu": "_swiglu", "geglu": "_geglu", "swiglu_bias": "_swiglu_bias"}[epilogue]
+    iface = ["in buffer<bf16>", "in buffer<bf16>", f"{cdir} buffer<{cdt}>", "i32", "out buffer<i32>"] + (["in buffer<bf16>"] if bias else [])
+    extra = {"param": 5 if bias else 2}      # the residual of `acc`, the biases
     lparams = ["bytes<128>", "bytes<128>", f"{cdir} buffer<{cdt}>", "in buffer<bf16>", "i32", "i32", "i32", "i32",
                "out buffer<i32>"]
     launches = []
@@ -201,9 +203,9 @@ def gemm_op(n: int, k: int, *, epilogue: str = "store", rows_var: str = "tokens"
         if hi < rows_max:
             when["max"] = hi
         launch = {"module": "gemv_bf16", "entry": f"kern_gemv_bf16_tn{suffix}_m{mt}", "block": [256, 1, 1], "grid": [8 * SMS, 1, 1],
-                  "params": ["in buffer<bf16>", "in buffer<bf16>", f"{cdir} buffer<{cdt}>", "in buffer<bf16>" if epilogue == "acc" else "i64",
+                  "params": ["in buffer<bf16>", "in buffer<bf16>", f"{cdir} buffer<{cdt}>", "in buffer<bf16>" if epilogue == "acc" or bias else "i64",
                              "i32", "i32", "i32", "i32", "i32", "out buffer<i32>"],
-                  "args": [{"param": 0}, {"param": 1}, {"param": 2}, {"param": 2} if epilogue == "acc" else {"i64": 0}, {"param": 3},
+                  "args": [{"param": 0}, {"param": 1}, {"param": 2}, extra if epilogue == "acc" or bias else {"i64": 0}, {"param": 3},
                            {"i32": n}, {"i32": k}, {"i32": lda}, {"i32": ldc}, {"param": 4}]}
         if len(when) > 1:
             launch["when"] = when
@@ -211,7 +213,7 @@ def gemm_op(n: int, k: int, *, epilogue: str = "store", rows_var: str = "tokens"
     tiles = (256, 128, 64, 32) if epilogue in ("store", "acc") else (256, 128, 64)
     ranges = []
     for bn, lo, hi in gemm_ranges(n, rows_max, tiles):
-        if bn == 256 and epilogue in ("store", "acc", "swiglu", "geglu") and M256_GAIN:
+        if bn == 256 and epilogue != "f32" and M256_GAIN:
             ranges += [(bn, bm, a, b) for bm, a, b in m256_split(n, lo, hi)]
         else:
             ranges.append((bn, BM, lo, hi))
@@ -235,7 +237,7 @@ def gemm_op(n: int, k: int, *, epilogue: str = "store", rows_var: str = "tokens"
                     "param": 1, "dtype": "bf16", "dims": [k, n], "strides": [k * 2],
                     "box": [BK, bn // 2 if glu else bn],
                     "swizzle": 128, "l2_promotion": 256}}]}},
-                {"param": 2}, {"param": 2 if epilogue == "acc" else 0}, {"param": 3}, {"i32": n}, {"i32": k},
+                {"param": 2}, extra if epilogue == "acc" or bias else {"param": 0}, {"param": 3}, {"i32": n}, {"i32": k},
                 {"i32": ldc}, {"param": 4}],
         }
         if len(when) > 1:
@@ -636,13 +638,14 @@ def sample_op(vocab: int, dtype: str = "bf16") -> dict:
                                             {"i32": vocab}, {"i32": vocab}]}]}}
 
 
-def rope_table_op(max_pos: int, rot: int, theta: float) -> dict:
-    """Interface [cos, sin]: the `once` program's table of angles."""
+def rope_table_op(max_pos: int, rot: int, theta: float, factor: float = 1.0) -> dict:
+    """Interface [cos, sin]: the `once` program's table of angles, position * theta^(-2i / rot) / factor."""
+    scaled = factor != 1.0
     return {"params": ["out buffer<f32>", "out buffer<f32>"], "impl": {"launches": [{
-        "module": "attn_prep", "entry": "kern_rope_table_f32", "block": [256, 1, 1],
+        "module": "attn_prep", "entry": "kern_rope_table_scaled_f32" if scaled else "kern_rope_table_f32", "block": [256, 1, 1],
         "grid": [min(1024, -(-max_pos * (rot // 2) // 256)), 1, 1],
-        "params": ["out buffer<f32>", "out buffer<f32>", "i32", "i32", "i64"],
-        "args": [{"param": 0}, {"param": 1}, {"i32": max_pos}, {"i32": rot}, {"i64": f64_bits(theta)}]}]}}
+        "params": ["out buffer<f32>", "out buffer<f32>", "i32", "i32", "i64"] + ["i64"] * scaled,
+        "args": [{"param": 0}, {"param": 1}, {"i32": max_pos}, {"i32": rot}, {"i64": f64_bits(theta)}] + [{"i64": f64_bits(factor)}] * scaled}]}}
 
 
 # ---- tensor-parallel ops ---------------------------------------------------------------------------
@@ -1131,20 +1134,26 @@ def latent_smem(blocks: int) -> int:
 
 
 def mla_attn_op(heads: int, page_size: int, table_width: int, ragged: bool, head_width: int = 192, seqs_max: int = 0,
-                sms: int = SMS, rank: int = 0, scale: float | None = None) -> dict:
+                sms: int = SMS, rank: int = 0, scale: float | None = None, rot: int = 0, max_pos: int = 0, rot_stride: int = 0) -> dict:
     """Absorbed latent attention: every head attends over the shared 576-wide latent rows, values their first 512
     columns. One row per sequence: interface [q, latent state, out, block_table, seq_lens, err], the context split over
     CTAs by `when` ranges of the batch (partials merged by a second launch) so that a few long sequences still fill
     the machine; ragged rows bring [.., row_len, err, row_seq] — a row reads its sequence's table row and attends over
     its own causal reach. `rank`: latent rows of that many columns (no rotary part), keys and values alike, scores times
-    `scale`; 0 is the 512 + 64 form."""
-    dq, dv = (rank, rank) if rank else (MLA_DQK, MLA_DV)
+    `scale`; 0 is the 512 + 64 form. `rot`: as many rotated columns behind them; [q_rot, cos, sin, sink] then come at the end:
+    the heads' rotated query columns, not yet turned, in rows of their own `rot_stride` apart, tables of `max_pos` positions, and
+    a score per head that joins the denominator."""
+    dq, dv = (rank + rot, rank) if rank else (MLA_DQK, MLA_DV)
     scale = head_width ** -0.5 if scale is None else scale
     assert page_size % 64 == 0 or 64 % page_size == 0
     iface = ["in buffer<bf16>", "in state", "out buffer<bf16>", "in buffer<i32>", "in buffer<i32>", "out buffer<i32>"]
     if ragged:
         iface.append("in buffer<i32>")
+    o = len(iface)
+    if rot:
+        iface += ["in buffer<bf16>", "in buffer<f32>", "in buffer<f32>", "in buffer<bf16>"]
     blocks = -(-heads // 16)
+    qb, vb = -(-(rank + rot) // 64), -(-rank // 64)
     ranges, hi = [], seqs_max
     if ragged or not seqs_max:
         ranges = [(1, 1, seqs_max)]
@@ -1170,19 +1179,28 @@ def mla_attn_op(heads: int, page_size: int, table_width: int, ragged: bool, head
              ["f32", "out buffer<i32>", "in buffer<i32>" if ragged else "i64"]
         ws = [{"scratch": "ws_o"}, {"scratch": "ws_ml"}] if part else [{"i64": 0}, {"i64": 0}]
         args = [_kv_map(dq, page_size, 1), {"param": 0}, {"param": 2}, *ws, {"param": 3}, {"param": 4},
-                {"i32": I32_MAX}, {"i32": heads}, {"i32": heads * dq}, {"i32": heads * dv}, {"i32": table_width},
+                {"i32": I32_MAX}, {"i32": heads}, {"i32": heads * (rank or dq)}, {"i32": heads * dv}, {"i32": table_width},
                 {"i32": page_size}, {"i32": splits}, {"i32": I32_MAX}, {"f32": scale * 1.4426950408889634},
                 {"param": 5}, {"param": 6} if ragged else {"i64": 0}]
         if rank:
             lp, args = lp + ["i32"], args + [{"i32": rank}]
-        launch = {"module": "mla_decode", "entry": f"kern_latent_decode_bf16_b{-(-rank // 64)}" if rank else "kern_mla_decode_bf16",
+        if rot:
+            lp = lp + iface[o:o + 4] + ["i32"] * 3
+            args = args + [{"param": o + i} for i in range(4)] + [{"i32": rot_stride}, {"i32": rot}, {"i32": max_pos}]
+        entry = f"kern_latent_rot_decode_bf16_q{qb}_b{vb}" if rot else (f"kern_latent_decode_bf16_b{vb}" if rank else "kern_mla_decode_bf16")
+        launch = {"module": "mla_decode", "entry": entry,
                   "block": [288, 1, 1], "grid": [blocks, "tokens" if ragged else "seqs", splits],
-                  "shared_mem": latent_smem(-(-rank // 64)) if rank else MLA_SMEM, "params": lp, "args": args}
+                  "shared_mem": latent_smem(qb) if rank else MLA_SMEM, "params": lp, "args": args}
         merge = {"module": "attn_paged", "entry": "kern_attn_merge_splits", "block": [256, 1, 1],
                  "grid": [{"mul": ["tokens", heads]}, 1, 1],
                  "params": ["in buffer<f32>", "in buffer<f32>", "out buffer<bf16>", "i32", "i32", "i32", "i32", "i32"],
                  "args": [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, {"param": 2}, {"i32": I32_MAX}, {"i32": heads},
                           {"i32": dv}, {"i32": splits}, {"i32": heads * dv}]}
+        if rot:
+            merge = {"module": "attn_window", "entry": "kern_attn_window_merge", "block": [256, 1, 1], "grid": [{"mul": ["tokens", heads]}, 1, 1],
+                     "params": ["in buffer<f32>", "in buffer<f32>", "out buffer<bf16>", "in buffer<bf16>", "i64"] + ["i32"] * 6 + ["f32"],
+                     "args": [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, {"param": 2}, {"param": o + 3}, {"i64": 0}, {"i32": 0}, {"i32": I32_MAX},
+                              {"i32": heads}, {"i32": dv}, {"i32": splits}, {"i32": heads * dv}, {"f32": 1.0}]}
         for l in ([launch, merge] if part else [launch]):
             if len(when) > 1:
                 l["when"] = when

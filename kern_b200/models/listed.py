@@ -27,6 +27,7 @@ class Listed:
             raise ValueError("a model without layers")
         self.cfg, self.act, self.es = cfg, cfg.dtype, K.ACT_BYTES[cfg.dtype]
         self.bufs, self.ops, self.states, self.once = {}, {}, {}, []
+        self.plans = {}      # name -> (buffers, op, args): what a ragged call's attention needs, made with the embedding
         self.err = self.B("error")
 
     # ---- names ----
@@ -63,14 +64,18 @@ class Listed:
         copies of the first rows, which nobody reads. `parts`: (tensor, rows)."""
         rows = sum(n for _, n in parts)
         proj = -(-rows // 8) * 8
-        fill = [{"tensor": parts[0][0], "rows": [0, proj - rows]}] if proj > rows else []
+        (first, n), fill, left = parts[0], [], proj - rows
+        while left > 0:
+            fill.append({"tensor": first, "rows": [0, min(n, left)]})
+            left -= n
         return self.weight(name, (proj, width), *[t for t, _ in parts], *fill), proj
 
-    def linear(self, base: str, n: int, k: int, a, w, c, rows: str = "tokens", label: str = "", **kw) -> dict:
+    def linear(self, base: str, n: int, k: int, a, w, c, rows: str = "tokens", label: str = "", bias: dict | None = None, **kw) -> dict:
+        kw |= {"bias": True} if bias else {}
         most = {"tokens": self.cfg.max_tokens, "seqs": self.cfg.max_seqs, "wanted": WANTED}[rows]
         lda = kw.get("lda")
         name = self.op(f"{base}_{n}x{k}" + (f"_of{lda}" if lda else ""), lambda: K.linear_op(n, k, act=self.act, rows_var=rows, rows_max=most, **kw))
-        return {"op": name, "label": label, "args": [a, w, c, self.V(rows), self.err]}
+        return {"op": name, "label": label, "args": [a, w, c, self.V(rows), self.err, *([bias] if bias else [])]}
 
     # ---- inputs and outputs ----
     def inputs(self, paged: str | None, lined: str | None, positions: bool = True, row_plan: bool = True) -> None:
@@ -109,23 +114,119 @@ class Listed:
         return {"op": self.op("rows", C.mla_rows_op), "label": label,
                 "args": [B("positions"), B("cu_seqlens"), B("row_seq"), B("row_len"), V("seqs"), V("tokens")]}
 
+    # ---- the first call, and what rides with it ----
+    def rotary(self, dims: int, base: float, factor: float = 1.0) -> list[dict]:
+        """The cos and sin tables of one rotation, written when the model is loaded."""
+        context, B = self.cfg.context, self.B
+        tag = f"{dims}x{base!r}" + (f"x{factor!r}" if factor != 1.0 else "")
+        name = "rope." + tag
+        if name + ".cos" not in self.bufs:
+            for n in (".cos", ".sin"):
+                self.bufs[name + n] = {"dtype": "f32", "shape": [context, dims // 2], "kind": "carry"}
+            op = self.op("rope_" + tag, lambda: C.rope_table_op(context, dims, base, factor))
+            self.once.append({"op": op, "label": name, "args": [B(name + ".cos"), B(name + ".sin")]})
+        return [B(name + ".cos"), B(name + ".sin")]
+
+    def lists_of(self, hq: int, hk: int, dim: int) -> list[dict]:
+        """The work lists of a tensor-core attention; layers whose blocks hold as many tokens share them."""
+        cfg, B = self.cfg, self.B
+        name = f"plan.{hq // hk}" + (".128" if dim == 128 else "")
+        if name not in self.plans:
+            items = cfg.max_tokens // (64 // (hq // hk)) + cfg.max_seqs + 1
+            for n, shape in ((".work_p", [items, 2]), (".count_p", [1]), (".work_d", [cfg.max_seqs, 2]), (".count_d", [1])):
+                self.bufs[name + n] = {"dtype": "i32", "shape": shape, "kind": "workspace"}
+            lists = [B(name + n) for n in (".work_p", ".count_p", ".work_d", ".count_d")]
+            args = [B("cu_seqlens"), lists[0], lists[1], self.V("seqs"), {"expr": C.attn_plan_items(hq, hk)}, lists[2], lists[3]]
+            self.plans[name] = lists, C.attn_plan_op(hq, hk, cfg.max_seqs, dim), args
+        return self.plans[name][0]
+
+    def row_plan(self) -> list[dict]:
+        """The table row and reach of every token, for attention that takes a row per token."""
+        if "rows" not in self.plans:
+            c = self.rows_call("")
+            self.plans["rows"] = [self.B("row_seq")], self.ops.pop(c["op"]), c["args"]
+        return self.plans["rows"][0]
+
+    def embed(self, next_norm: str, prefill: bool) -> dict:
+        """Token rows into the residual and the first sublayer's normed input; the plans in the same call, so that both programs
+        have as many calls to every layer."""
+        cfg, B, d = self.cfg, self.B, self.cfg.width
+        args = [B("token_ids"), self.same("embed", (cfg.vocab, d)), self.same(next_norm, (d,)), B("x"), B("xn"), self.err]
+        first = self.plans.values() if prefill else ()
+        name = self.op("embed" + ("_p" if prefill else "_d"), lambda: K.chain_ops(K.resid_embed_op(d, cfg.vocab, cfg.eps, self.act), *[o for _, o, _ in first]))
+        return {"op": name, "label": "embed", "args": args + [a for _, _, more in first for a in more]}
+
+    # ---- linear attention with a decay per key channel ----
+    def linear_attention(self, p: str, st: str, H: int, dk: int, dv: int, stride: int, ptrs, z, prefill: bool, norm, norm_shared: bool, u, q_scale, out, out_stride,
+                         out_scale) -> list[dict]:
+        """The recurrence from its projections (`ptrs`: q, k, v, gate) to the gated rows in `out`."""
+        cfg, A, eps, B, V = self.cfg, self.act, self.cfg.eps, self.B, self.V
+        sfx, fused = "_p" if prefill else "_d", not prefill and K.lin_fused(dv)
+        tag = f"{sfx}_{H}x{dk}x{dv}x{stride}x{out_stride}" + ("u" if u else "") + f"_{out_scale!r}"
+
+        def make():
+            rule = K.lin_rule_op(H, dk, dv, stride, z["line"], z["s_off"], prefill, A, bonus=u is not None, q_scale=q_scale, fused=fused, norm_shared=norm_shared,
+                                 out_stride=out_stride, out_scale=out_scale, eps=eps, rows_max=cfg.max_tokens, seqs_max=cfg.max_seqs)
+            if fused:
+                return rule
+            ng = K.lin_norm_gate_op(H, dv, stride, norm_shared, out_stride, out_scale, eps, A)
+            return K.chain_ops(rule, ng, inner={(0, 5 if u else 4): "o", (1, 0): "o"}, scratch={"o": {"dtype": "f32", "shape": ["tokens", H * dv]}})
+
+        q, k, v, gate = ptrs
+        head, cu = [q, k, v, B("alpha"), *([u] if u else [])], [B("cu_seqlens")] if prefill else []
+        state = [{"state": st}, B("lines"), *cu]
+        args = [*head, out, *state, gate, norm, V("seqs")] if fused else [*head, *state, V("seqs"), gate, norm, out]
+        return [{"op": self.op(f"lin{tag}", make), "label": p + "rule", "args": args}]
+
+    def gla(self, p: str, st: str, m: dict, rank: int, prefill: bool) -> list[dict]:
+        """Gated linear attention of tensors `p`, its state in lines `st`, its decays through `rank` columns: xn -> y."""
+        d, A, es, B = self.cfg.width, self.act, self.es, self.B
+        z = gla_sizes(m)
+        H, dk, dv, q, v = m["heads"], m["dim"], m["vdim"], z["q"], z["v"]
+        self.states[st] = {"bytes_per_seq": z["line"]}
+        w_in, proj = self.rows_weight(f"w.{p}qkvga", d, [(p + "q", q), (p + "k", q), (p + "v", v), (p + "g", v), (p + "a1", rank)])
+        self.room("proj", proj); self.room("alpha", q, "f32"); self.room("mixed", v); self.room("y", d)
+        decay = self.op(f"decay_{q}x{rank}x{proj}_{m['tau']!r}", lambda: K.decay_op(q, rank, proj, "root", m["tau"], A))
+        col = lambda c: B("proj", c * es)
+        return [
+            self.linear("lin", proj, d, B("xn"), w_in, B("proj"), label=p + "in"),
+            {"op": decay, "label": p + "decay", "args": [col(2 * q + 2 * v), self.same(p + "a2", (q, rank)), self.same(p + "a2.b", (q,)), B("alpha"), self.V("tokens")]},
+            *self.linear_attention(p, st, H, dk, dv, proj, (col(0), col(q), col(2 * q), col(2 * q + v)), z, prefill, self.same(p + "norm", (dv,)), True, None,
+                                   dk ** -0.5, B("mixed"), v, 1.0),
+            self.linear("lin", d, v, B("mixed"), self.same(p + "o", (d, v)), B("y"), label=p + "o"),
+        ]
+
     # ---- feed-forward ----
-    def dense(self, p: str, ff: int, glu: str) -> list[dict]:
-        """Gate and up projections with their gated unit, and the projection back: xn -> y."""
+    def dense(self, p: str, ff: int, glu: str, bias: bool = False) -> list[dict]:
+        """Gate and up projections with their gated unit, and the projection back: xn -> y. `bias`: gate and up have one each (the
+        way back's is left to whoever adds y to the residual)."""
         d, B = self.cfg.width, self.B
         self.room("act", ff); self.room("y", d)
-        base = "glu" if glu == "swiglu" else glu
+        base = ("glu" if glu == "swiglu" else glu) + ("_bias" if bias else "")
+        b = self.weight(f"w.{p}mlp.gu.b", (2 * ff,), p + "mlp.gate.b", p + "mlp.up.b") if bias else None
         return [
-            self.linear(base, 2 * ff, d, B("xn"), self.weight(f"w.{p}mlp.gu", (2 * ff, d), p + "mlp.gate", p + "mlp.up"), B("act"), label=p + "gate_up", epilogue=glu),
+            self.linear(base, 2 * ff, d, B("xn"), self.weight(f"w.{p}mlp.gu", (2 * ff, d), p + "mlp.gate", p + "mlp.up"), B("act"), label=p + "gate_up", bias=b, epilogue=glu),
             self.linear("lin", d, ff, B("act"), self.same(p + "mlp.down", (d, ff)), B("y"), label=p + "down"),
         ]
 
-    def routed(self, p: str, experts: int, top: int, ff: int, route, glu: str = "swiglu", limit: float = 0.0) -> list[dict]:
+    def shared(self, p: str, ff: int) -> list[dict]:
+        """An expert of every token: xn -> `shared.y`."""
+        d, B = self.cfg.width, self.B
+        self.room("shared.act", ff); self.room("shared.y", d)
+        return [
+            self.linear("glu", 2 * ff, d, B("xn"), self.weight(f"w.{p}mlp.shared.gu", (2 * ff, d), p + "mlp.shared.gate", p + "mlp.shared.up"), B("shared.act"),
+                        label=p + "shared_gate_up", epilogue="swiglu"),
+            self.linear("lin", d, ff, B("shared.act"), self.same(p + "mlp.shared.down", (d, ff)), B("shared.y"), label=p + "shared_down"),
+        ]
+
+    def routed(self, p: str, experts: int, top: int, ff: int, route, glu: str = "swiglu", limit: float = 0.0, router: tuple[dict, int] | None = None) -> list[dict]:
         """Routed experts up to their own rows: xn -> `moe.y` (expert-sorted), `moe.perm`, `moe.w`. `route(logits, ids, weights)` makes
-        the call that picks them."""
+        the call that picks them; an id from `experts` on has no row (`moe.perm` -1). `router`: a matrix of more rows than experts,
+        and their number."""
         cfg, d, B, V = self.cfg, self.cfg.width, self.B, self.V
         E, k, T, A, err = experts, top, cfg.max_tokens, self.act, self.err
-        self.room("moe.logits", E, "f32"); self.room("moe.ids", k, "i32"); self.room("moe.w", k, "f32"); self.room("moe.perm", k, "i32")
+        w_router, outputs = router or (self.same(p + "mlp.router", (E, d)), E)
+        self.room("moe.logits", outputs, "f32"); self.room("moe.ids", k, "i32"); self.room("moe.w", k, "f32"); self.room("moe.perm", k, "i32")
         self.room("moe.x", k * d); self.room("moe.act", k * ff); self.room("moe.y", k * d)
         tiles = T * k // K.routed_tile_rows(A, d, ff) + E
         for name, shape in (("moe.offsets", [E + 1]), ("moe.tiles", [tiles, 4]), ("moe.tile_count", [1]), ("moe.rows", [1])):
@@ -139,7 +240,7 @@ class Listed:
         w1 = self.weight(f"w.{p}mlp.w1", (E, 2 * ff, d), *[f"{p}mlp.e{e}.{t}" for e in range(E) for t in ("gate", "up")])
         w2 = self.weight(f"w.{p}mlp.w2", (E, d, ff), *[f"{p}mlp.e{e}.down" for e in range(E)])
         return [
-            self.linear("router", E, d, B("xn"), self.same(p + "mlp.router", (E, d)), B("moe.logits"), label=p + "router", epilogue="f32"),
+            self.linear("router", outputs, d, B("xn"), w_router, B("moe.logits"), label=p + "router", epilogue="f32"),
             route(B("moe.logits"), B("moe.ids"), B("moe.w")),
             {"op": f"moe_plan_{tag}", "label": p + "plan", "args": [B("moe.ids"), B("moe.perm"), B("moe.offsets"), B("moe.tiles"), B("moe.tile_count"), B("moe.rows"), n, err]},
             {"op": f"moe_gather_{tag}", "label": p + "gather", "args": [B("xn"), B("moe.perm"), B("moe.x"), n]},
@@ -189,6 +290,12 @@ class Listed:
         used = {l["module"] for o in self.ops.values() for l in o["impl"]["launches"]}
         doc["modules"] = {n: m for n, m in C.modules_for(sorted(used)).items() if n in used}
         return doc
+
+
+def gla_sizes(m: dict) -> dict:
+    q, v = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+    line, s_off = K.lin_line_bytes(m["heads"], m["dim"], m["vdim"])
+    return {"q": q, "v": v, "line": line, "s_off": s_off}
 
 
 # ---- checkpoints -------------------------------------------------------------------------------------------
