@@ -65,13 +65,16 @@ def k_fused_add_rms_norm(g, x, res, w, y, rows, n, eps, plus_one):
     k_rms_norm(g, res, w, y, rows, n, n, n, eps, plus_one)
 
 
-GLU_GATES = {"swiglu": torch.nn.functional.silu, "geglu": lambda g: torch.nn.functional.gelu(g, approximate="tanh")}
+GLU_GATES = {"swiglu": torch.nn.functional.silu, "geglu": lambda g: torch.nn.functional.gelu(g, approximate="tanh"),
+             "swiglu_bias": torch.nn.functional.silu}
 
 
 def _gemm(epi):
     def run(g, a, w, c, r, m, n, k, ldc, err):
         av = torch.as_strided(a, (m, k), (a_stride(a, k), 1))
         acc = _f(av) @ _f(w[: n * k].view(n, k)).t()
+        if epi == "swiglu_bias":
+            acc = acc + _f(r[:n])
         if epi in GLU_GATES:
             acc = GLU_GATES[epi](acc[:, : n // 2]) * acc[:, n // 2:]
         cv = torch.as_strided(c, (m, acc.shape[1]), (ldc, 1))
@@ -85,6 +88,8 @@ def _gemv(epi):
     def run(g, a, w, c, r, m, n, k, lda, ldc, err):
         av = torch.as_strided(a, (m, k), (lda, 1), a.storage_offset())
         acc = _f(av) @ _f(w[: n * k].view(n, k)).t()
+        if epi == "swiglu_bias":
+            acc = acc + _f(r[:n])
         if epi in GLU_GATES:
             acc = GLU_GATES[epi](acc[:, : n // 2]) * acc[:, n // 2:]
         cv = torch.as_strided(c, (m, acc.shape[1]), (ldc, 1), c.storage_offset())
@@ -410,7 +415,7 @@ CPU_KERNELS = {
     "kern_fill_f32": k_fill, "kern_fill_i32": k_fill, "kern_fill_i64": k_fill, "kern_fill_u8": k_fill,
 }
 for _bn in (256, 128, 64, 32):
-    for _epi, _sfx in (("store", ""), ("acc", "_acc"), ("f32", "_f32"), ("swiglu", "_swiglu"), ("geglu", "_geglu")):
+    for _epi, _sfx in (("store", ""), ("acc", "_acc"), ("f32", "_f32"), ("swiglu", "_swiglu"), ("geglu", "_geglu"), ("swiglu_bias", "_swiglu_bias")):
         CPU_KERNELS[f"kern_gemm_bf16_tn{_sfx}_n{_bn}"] = _gemm(_epi)
         for _mt in (1, 2, 4, 8):
             CPU_KERNELS[f"kern_gemv_bf16_tn{_sfx}_m{_mt}"] = _gemv(_epi)

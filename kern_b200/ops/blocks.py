@@ -90,6 +90,27 @@ def k_resid_mix(g, x, y, perm, topw, w_post, w_next, xn, hidden, d, k, eps):
         xn[: n * d] = _norm(new, w_next[:d], eps).to(xn.dtype).reshape(-1)
 
 
+def k_resid_scale(g, x, y, perm, topw, shared, gate, bias, scale, w_next, xn, hidden, d, k, gs, eps):
+    n = g[0]
+    if isinstance(perm, T):
+        p, w = perm[: n * k].view(n, k).long(), topw[: n * k].view(n, k, 1)
+        rows = _f(y.view(-1)[: n * k * d].view(-1, d)[p.clamp_min(0)])
+        own = _f(xn[: n * d].view(n, 1, d)) if isinstance(xn, T) else torch.zeros(n, 1, d)
+        v = (torch.where((p < 0)[..., None], own, rows) * w).sum(1)
+    else:
+        v = _f(y[: n * d].view(n, d))
+    if isinstance(shared, T):
+        v = v + torch.sigmoid(_rows(gate, n, 1, gs)) * _f(shared[: n * d].view(n, d))
+    if isinstance(bias, T):
+        v = v + _f(bias[:d])
+    new = x[: n * d].view(n, d) + v * _f(scale[:d])
+    if isinstance(hidden, T):
+        hidden[: n * d] = new.reshape(-1)
+    else:
+        x[: n * d] = new.reshape(-1)
+        xn[: n * d] = _norm(new, w_next[:d], eps).to(xn.dtype).reshape(-1)
+
+
 # ---- matrix products ----
 def _glu(v, kind, limit=0.0):
     g, u = v[:, :v.shape[1] // 2], v[:, v.shape[1] // 2:]
@@ -102,13 +123,15 @@ def _glu(v, kind, limit=0.0):
 
 
 def _k_linear(glu):
-    def run(g, a, w, c, m, n, k, lda, ldc, wsn, wsk, az, wz, cz, err, limit):
+    def run(g, a, w, c, m, n, k, lda, ldc, wsn, wsk, az, wz, cz, err, limit, bias):
         if m > g[1] * 64:
             err[0] = 300
         for z in range(g[2]):
             A = _f(_rows(a[z * az:], m, k, lda))
             W = _f(torch.as_strided(w[z * wz:], ((2 if glu else 1) * n, k), (wsn, wsk)))
             v = A @ W.t()
+            if isinstance(bias, T):
+                v = v + _f(bias[: v.shape[1]])
             _rows(c[z * cz:], m, n, ldc).copy_(_glu(v, glu, limit) if glu else v)
     return run
 
@@ -332,35 +355,66 @@ def k_qk_prep(g, qkv, cache, positions, slots, cos, sin, qn, kn, hq, hk, d, dv, 
     vs[sl[ok] // page, :, sl[ok] % page] = v[ok]
 
 
-def _window_row(q, cache, out, pages, L, sink, hq, hk, d, dv, page, window, scale, cap, out_scale):
-    """One row at position L - 1: q [hq d] -> out [hq dv]."""
+def k_qk_prep_whole(g, qkv, cache, positions, slots, cos, sin, qn, kn, hq, hk, d, dv, v_col, rot, halves, page, stride, max_pos, eps, err):
+    n = g[0]
+    rows, pos, sl = _rows(qkv, n, max((hq + hk) * d, v_col + hk * dv), stride), positions[:n].long(), slots[:n].long()
+    if ((pos < 0) | (pos >= max_pos)).any():
+        err[0] = 300
+    pos = torch.where((pos < 0) | (pos >= max_pos), 0, pos)
+    c, s = (t.view(-1)[: max_pos * (rot // 2)].view(max_pos, rot // 2)[pos][:, None] for t in (cos, sin))
+
+    def turned(x, w, heads):
+        x = _norm(_f(x), w[: heads * d], eps).view(n, heads, d)
+        a, b = (x[..., : rot // 2], x[..., rot // 2: rot]) if halves else (x[..., :rot:2], x[..., 1:rot:2])
+        a, b = a * c - b * s, b * c + a * s
+        return torch.cat([a, b, x[..., rot:]] if halves else [torch.stack([a, b], -1).flatten(-2), x[..., rot:]], -1).to(qkv.dtype)
+
+    q, k = turned(rows[:, : hq * d], qn, hq), turned(rows[:, hq * d:(hq + hk) * d], kn, hk)
+    v = rows[:, v_col: v_col + hk * dv].reshape(n, hk, dv).clone()
+    rows[:, : hq * d] = q.reshape(n, -1)
+    ks, vs = _window_pool(cache, qkv.dtype, hk, page, d, dv)
+    ok = sl >= 0
+    ks[sl[ok] // page, :, sl[ok] % page] = k[ok]
+    vs[sl[ok] // page, :, sl[ok] % page] = v[ok]
+
+
+def _window_row(q, cache, out, pages, L, sink, hq, hk, d, dv, page, window, scale, cap, out_scale, gate=None):
+    """One row at position L - 1: q [hq d] -> out [hq dv]. No cap (0), no sink (a score of 0) and no gate are forms too."""
     ks, vs = _window_pool(cache, q.dtype, hk, page, d, dv)
     ids = pages[: -(-L // page)].long()
     k, v = (_f(t[ids]).transpose(1, 2).reshape(-1, hk, t.shape[-1])[max(0, L - window):L].repeat_interleave(hq // hk, 1) for t in (ks, vs))
-    s = cap * torch.tanh(torch.einsum("hd,lhd->hl", _f(q).view(hq, d), k) * (scale / cap))
-    p = torch.softmax(torch.cat([s, _f(sink[:hq])[:, None]], 1), 1)[:, :-1]
-    out.copy_((torch.einsum("hl,lhv->hv", p, v) * out_scale).reshape(-1))
+    s = torch.einsum("hd,lhd->hl", _f(q).view(hq, d), k) * scale
+    s = cap * torch.tanh(s / cap) if cap > 0 else s
+    sk = _f(sink[:hq]) if isinstance(sink, T) else torch.zeros(hq)
+    p = torch.softmax(torch.cat([s, sk[:, None]], 1), 1)[:, :-1]
+    o = (torch.einsum("hl,lhv->hv", p, v) * out_scale).reshape(-1)
+    out.copy_(o * torch.sigmoid(_f(gate)) if gate is not None else o)
 
 
-def k_window_attn(g, q, cache, out, table, lens, row_seq, sink, hq, hk, d, dv, qs, os_, max_pages, page, window, scale, cap, out_scale, err):
+def _gate_row(gate, r, gs, cols):
+    return gate[r * gs: r * gs + cols] if isinstance(gate, T) else None
+
+
+def k_window_attn(g, q, cache, out, table, lens, row_seq, sink, gate, hq, hk, d, dv, qs, os_, gs, max_pages, page, window, scale, cap, out_scale, err):
     tb = table.view(-1, max_pages)
     for r in range(g[1]):
         if int(lens[r]) > 0:
             _window_row(q[r * qs: r * qs + hq * d], cache, out[r * os_: r * os_ + hq * dv], tb[int(row_seq[r]) if isinstance(row_seq, T) else r], int(lens[r]), sink,
-                        hq, hk, d, dv, page, window, scale, cap, out_scale)
+                        hq, hk, d, dv, page, window, scale, cap, out_scale, _gate_row(gate, r, gs, hq * dv))
 
 
-def _window_listed(q, cache, out, table, lens, cu, work, count, tokens, sink, hq, hk, d, qs, os_, max_pages, page, window, c1, c2, out_scale):
-    """The rows of a work list's (sequence, block) pairs, `tokens` to a block; without a list, one row per sequence."""
+def _window_listed(q, cache, out, table, lens, cu, work, count, tokens, sink, hq, hk, d, qs, os_, max_pages, page, window, c1, c2, out_scale, gate=0, gs=0):
+    """The rows of a work list's (sequence, block) pairs, `tokens` to a block; without a list, one row per sequence. c2 0: no cap,
+    and c1 is the scale in base-2 units."""
     cap, tb = c2 / 1.4426950408889634, table.view(-1, max_pages)
-    scale = c1 * cap / (2 * 1.4426950408889634)
+    scale = c1 * cap / (2 * 1.4426950408889634) if cap else c1 / 1.4426950408889634
     pairs = work.view(-1, 2)[: int(count[0])].tolist()
     for s, b in pairs:
         r0, r1 = int(cu[s]), int(cu[s + 1])
         for t in range(b * tokens, min((b + 1) * tokens, r1 - r0)):
             r = r0 + t
             _window_row(q[r * qs: r * qs + hq * d], cache, out[r * os_: r * os_ + hq * d], tb[s], int(lens[s]) - (r1 - r0) + t + 1, sink, hq, hk, d, d, page, window,
-                        scale, cap, out_scale)
+                        scale, cap, out_scale, _gate_row(gate, r, gs, hq * d))
 
 
 def _k_window(prefill, d):
@@ -368,12 +422,39 @@ def _k_window(prefill, d):
         if isinstance(work, T):
             _window_listed(q, kv, out, table, lens, cu, work, count, (64 if prefill else 16) // (hq // hk), sink, hq, hk, d, qs, os_, max_pages, page, window, c1, c2, out_scale)
         else:      # a split launch is followed by the merge; here it writes the finished rows and the merge is a no-op
-            one = torch.arange(g[1] + 1, dtype=torch.int32)
-            pairs = torch.stack([one[:-1], torch.zeros(g[1], dtype=torch.int32)], 1)
-            live = [i for i in range(g[1]) if int(lens[i]) > 0]
-            _window_listed(q, kv, out, table, lens, one, pairs[live].contiguous(), torch.tensor([len(live)]), 1, sink, hq, hk, d, qs, os_, max_pages, page, window, c1, c2,
-                           out_scale)
+            _window_listed(q, kv, out, table, lens, *_one_each(g[1], lens), 1, sink, hq, hk, d, qs, os_, max_pages, page, window, c1, c2, out_scale)
     return run
+
+
+def _one_each(n, lens):
+    """(row starts, list, count) of one row per sequence."""
+    one = torch.arange(n + 1, dtype=torch.int32)
+    live = [i for i in range(n) if int(lens[i]) > 0]
+    return one, torch.stack([one[:-1], torch.zeros(n, dtype=torch.int32)], 1)[live].contiguous(), torch.tensor([len(live)])
+
+
+WHOLE = 1 << 30
+
+
+def _k_sink(prefill, d):
+    def run(g, kv, q, out, ws_o, ws_ml, table, lens, cu, work, count, hq, hk, qs, os_, max_pages, page, splits, pool_pages, err, sink, gate, gs, scale_log2):
+        if isinstance(work, T):
+            rows = (cu, work, count, (64 if prefill else 16) // (hq // hk))
+        else:
+            rows = (*_one_each(g[1], lens), 1)
+        _window_listed(q, kv, out, table, lens, *rows, sink, hq, hk, d, qs, os_, max_pages, page, WHOLE, scale_log2, 0.0, 1.0, gate, gs)
+    return run
+
+
+def _k_sink_ragged(d):
+    def run(g, kv, q, out, table, lens, cu, wp, cp, wd, cd, hq, hk, qs, os_, max_pages, page, pool_pages, err, sink, gate, gs, scale_log2):
+        for w, c, rows in ((wp, cp, 64), (wd, cd, 16)):
+            _window_listed(q, kv, out, table, lens, cu, w, c, rows // (hq // hk), sink, hq, hk, d, qs, os_, max_pages, page, WHOLE, scale_log2, 0.0, 1.0, gate, gs)
+    return run
+
+
+def k_sink_fmha(g, kv, q, out, table, lens, cu, work, count, hq, hk, qs, os_, max_pages, page, pool_pages, err, sink, gate, gs, scale_log2):
+    _window_listed(q, kv, out, table, lens, cu, work, count, 128 // (hq // hk), sink, hq, hk, 128, qs, os_, max_pages, page, WHOLE, scale_log2, 0.0, 1.0, gate, gs)
 
 
 def _k_window_ragged(d):
@@ -418,6 +499,51 @@ def k_latent_decode(g, kv, q, out, ws_o, ws_ml, table, lens, seqs, heads, qs, os
     _attend(q, kv, out, table, lens, row_seq, g[1], heads, rank, max_pages, page, scale_log2 / 1.4426950408889634)
 
 
+def _turn_halves(x, pos, cos, sin, max_pos, rot):
+    """x [n, heads, rot], pairs (i, i + rot / 2), by the tables' rows `pos` [n]."""
+    c, s = (t.view(-1)[: max_pos * (rot // 2)].view(max_pos, rot // 2)[pos][:, None] for t in (cos, sin))
+    a, b = x[..., : rot // 2], x[..., rot // 2:]
+    return torch.cat([a * c - b * s, b * c + a * s], -1)
+
+
+def k_latent_prep(g, rows, cache, q_low, positions, slots, cos, sin, w, wq, rank, rot, q_rank, stride, qs, max_pos, eps, err):
+    n = g[0]
+    x, pos, sl = _f(_rows(rows, n, q_rank + rank + rot, stride)), positions[:n].long(), slots[:n].long()
+    if ((pos < 0) | (pos >= max_pos)).any():
+        err[0] = 300
+    pos = torch.where((pos < 0) | (pos >= max_pos), 0, pos)
+    _rows(q_low, n, q_rank, qs).copy_(_norm(x[:, :q_rank], wq[:q_rank], eps))
+    key = _turn_halves(x[:, None, q_rank + rank:], pos, cos, sin, max_pos, rot)[:, 0]
+    new = torch.cat([_norm(x[:, q_rank: q_rank + rank], w[:rank], eps), key], -1).to(rows.dtype)
+    cache.view(rows.dtype).view(-1, rank + rot)[sl[sl >= 0]] = new[sl >= 0]
+
+
+def _attend_rot(q, cache, out, table, lens, row_seq, n, heads, rank, rot, max_pages, page, scale, q_rot, cos, sin, sink, rs, max_pos, err):
+    pool = cache.view(q.dtype).view(-1, page, rank + rot)
+    tb = table.view(-1, max_pages)
+    for r in range(n):
+        L = int(lens[r])
+        if L <= 0:
+            continue
+        if L > max_pos:
+            err[0] = 300
+        c = _f(pool[tb[int(row_seq[r]) if isinstance(row_seq, T) else r, : -(-L // page)].long()]).reshape(-1, rank + rot)[:L]
+        turned = _turn_halves(_f(q_rot[r * rs: r * rs + heads * rot].view(1, heads, rot)), torch.tensor([min(L, max_pos) - 1]), cos, sin, max_pos, rot)[0]
+        qq = torch.cat([_f(q[r * heads * rank:(r + 1) * heads * rank].view(heads, rank)), turned.to(q.dtype).float()], -1)
+        p = torch.softmax(torch.cat([qq @ c.t() * scale, _f(sink[:heads])[:, None]], 1), -1)[:, :-1]
+        out[r * heads * rank:(r + 1) * heads * rank] = (p @ c[:, :rank]).to(out.dtype).reshape(-1)
+
+
+def k_latent_rot_attn(g, q, cache, out, table, lens, row_seq, heads, rank, max_pages, page, scale, err, q_rot, cos, sin, sink, rs, rot, max_pos):
+    _attend_rot(q, cache, out, table, lens, row_seq, g[1], heads, rank, rot, max_pages, page, scale, q_rot, cos, sin, sink, rs, max_pos, err)
+
+
+def k_latent_rot_decode(g, kv, q, out, ws_o, ws_ml, table, lens, seqs, heads, qs, os_, max_pages, page, splits, pool_pages, scale_log2, err, row_seq, rank,
+                        q_rot, cos, sin, sink, rs, rot, max_pos):
+    # a split launch is followed by the merge; here the first writes the finished rows and the merge is a no-op
+    _attend_rot(q, kv, out, table, lens, row_seq, g[1], heads, rank, rot, max_pages, page, scale_log2 / 1.4426950408889634, q_rot, cos, sin, sink, rs, max_pos, err)
+
+
 def k_route_logits(g, logits, bias, ids, w, tokens, E, k, ld):
     z = _rows(logits, tokens, E, ld) + (_f(bias[:E]) if isinstance(bias, T) else 0.0)
     order = torch.argsort(z, dim=-1, descending=True, stable=True)[:, :k]
@@ -425,21 +551,24 @@ def k_route_logits(g, logits, bias, ids, w, tokens, E, k, ld):
     w[: tokens * k] = torch.softmax(torch.gather(z, 1, order), -1).reshape(-1)
 
 
-def k_route_groups(g, logits, ids, w, tokens, E, k, groups, keep, renorm, ld):
-    s = torch.sigmoid(_rows(logits, tokens, E, ld))
-    of = s.view(tokens, groups, -1)
-    best = torch.argsort(of.topk(min(2, E // groups), -1).values.sum(-1), dim=-1, descending=True, stable=True)[:, :keep]
+def k_route_groups(g, logits, bias, ids, w, tokens, E, k, groups, keep, softmax, group_top, renorm, scale, ld):
+    z = _rows(logits, tokens, E, ld)
+    s = torch.softmax(z, -1) if softmax else torch.sigmoid(z)
+    choice = s + _f(bias[:E]) if isinstance(bias, T) else s
+    of = choice.view(tokens, groups, -1)
+    best = torch.argsort(of.topk(min(group_top, E // groups), -1).values.sum(-1), dim=-1, descending=True, stable=True)[:, :keep]
     may = torch.zeros(tokens, groups, dtype=torch.bool).scatter_(1, best, True).repeat_interleave(E // groups, 1)
-    order = torch.argsort(s.masked_fill(~may, -1.0), dim=-1, descending=True, stable=True)[:, :k]
+    order = torch.argsort(choice.masked_fill(~may, -torch.inf), dim=-1, descending=True, stable=True)[:, :k]
     top = torch.gather(s, 1, order)
     ids[: tokens * k] = order.to(ids.dtype).reshape(-1)
-    w[: tokens * k] = (top / top.sum(-1, keepdim=True) if renorm else top).reshape(-1)
+    w[: tokens * k] = ((top / (top.sum(-1, keepdim=True) + 1e-20) if renorm else top) * scale).reshape(-1)
 
 
 for _a in ("bf16", "f32"):
     CPU_KERNELS.update({f"kern_hyper_embed_{_a}": k_hyper_embed, f"kern_row_norm_f32_{_a}": k_row_norm,
                         f"kern_rows_scatter_{_a}": k_rows_scatter, f"kern_gate_mul_{_a}": k_gate_mul,
                         f"kern_resid_embed_{_a}": k_resid_embed, f"kern_resid_mix_{_a}": k_resid_mix,
+                        f"kern_resid_scale_{_a}": k_resid_scale, f"kern_qk_prep_whole_{_a}": k_qk_prep_whole, f"kern_latent_prep_{_a}": k_latent_prep,
                         f"kern_token_shift_{_a}": k_token_shift, f"kern_shift_state_{_a}": k_shift_state, f"kern_decay_{_a}": k_decay,
                         f"kern_lin_norm_gate_{_a}": k_lin_norm_gate, f"kern_qk_prep_{_a}": k_qk_prep,
                         f"kern_ssd_conv_{_a}": k_ssd_conv, f"kern_ssd_conv_state_{_a}": k_ssd_conv_state,
@@ -450,14 +579,18 @@ for _a in ("bf16", "f32"):
                         for e in ("", "swiglu", "geglu", "clamped")})
     CPU_KERNELS.update({f"kern_lin_rule_{_a}_r{r}_v{v}": k_lin_rule for r in (4, 8, 16, 32) for v in (1, 2, 4)})
     CPU_KERNELS.update({f"kern_window_attn_{_a}_w{w}": k_window_attn for w in (64, 128, 256, 512)})
-    CPU_KERNELS.update({f"kern_latent_attn_{_a}_w{w}": k_latent_attn for w in (64, 128, 256, 512, 1024)})
+    CPU_KERNELS.update({f"kern_latent_{n}_{_a}_w{w}": f for n, f in (("attn", k_latent_attn), ("rot_attn", k_latent_rot_attn)) for w in (64, 128, 256, 512, 1024)})
 CPU_KERNELS.update({"kern_linear_bf16_f32": _k_linear(""), "kern_transpose_heads_bf16": k_transpose_heads, "kern_copy_cols_bf16": k_copy_cols,
                     "kern_moe_route_logits": k_route_logits, "kern_moe_route_groups": k_route_groups, "kern_attn_window_fmha_d128": k_window_fmha,
+                    "kern_attn_sink_fmha_d128": k_sink_fmha,
                     "kern_attn_window_merge": lambda *a: None})
 CPU_KERNELS.update({f"kern_moe_gemm_bf16_{e}_n{n}": _k_moe_gemm(e) for e in ("geglu", "clamped") for n in (64, 128)})
 CPU_KERNELS.update({f"kern_lin_{k}_n{n}": f for k, f in (("prep", k_lin_prep), ("chunk", k_lin_chunk)) for n in (32, 64, 128, 256)})
 CPU_KERNELS.update({f"kern_attn_window_{k}_d{d}": _k_window(k == "prefill", d) for k in ("decode", "prefill") for d in (64, 128, 256)})
 CPU_KERNELS.update({f"kern_attn_window_ragged_d{d}": _k_window_ragged(d) for d in (64, 128)})
+CPU_KERNELS.update({f"kern_attn_sink_{k}_d{d}": _k_sink(k == "prefill", d) for k in ("decode", "prefill") for d in (64, 128, 256)})
+CPU_KERNELS.update({f"kern_attn_sink_ragged_d{d}": _k_sink_ragged(d) for d in (64, 128)})
 CPU_KERNELS.update({f"kern_gemm_bf16_heads_n{n}": k_gemm_heads for n in (64, 128, 256)})
 CPU_KERNELS.update({f"kern_ssd_chunk_n{n}": k_ssd_chunk for n in (32, 64, 128, 256)})
 CPU_KERNELS.update({f"kern_latent_decode_bf16_b{b}": k_latent_decode for b in range(1, 9)})
+CPU_KERNELS.update({f"kern_latent_rot_decode_bf16_q{b + more}_b{b}": k_latent_rot_decode for b in range(1, 9) for more in (0, 1)})
