@@ -167,12 +167,16 @@ def _far_key(r, p, page):
 
 
 def attention(gpu, act, hq, hk, d, dv, page, seqs, ragged, learned):
-    """`seqs`: (context, new rows) of every sequence, over scattered pages."""
+    """`seqs`: (context, new rows) of every sequence, over scattered pages. Most rows have a key that stands far out; every fifth
+    turns away from all of them, so that the sink takes nearly everything."""
     dt, scale = DT[act], 0.35
     rows = [(s, L - R + i) for s, (L, R) in enumerate(seqs) for i in range(R)]
     n, gs, os_ = len(rows), hq * dv + 24, hq * dv + 8
     qs = hq * d + 16
-    ks, table, flat = _paged(seqs, page, (hk, d), dt, 4, .5)
+    ks, table, flat = _paged(seqs, page, (hk, d), torch.float32, 4, .5)
+    u = rnd(hk, d, seed=9)
+    u = u / u.pow(2).sum(-1, keepdim=True).sqrt()
+    ks = (ks + 2 * u[:, None]).to(dt)
     vs, _, _ = _paged(seqs, page, (hk, dv), dt, 5)
     sink = bf(2 + rnd(hq, seed=6, scale=2)) if learned else torch.zeros(hq)
     q = rnd(n, hq, d, seed=7, scale=.3)
@@ -181,6 +185,8 @@ def attention(gpu, act, hq, hk, d, dv, page, seqs, ragged, learned):
         for h in range(hq):
             c = kf[s][min(_far_key(r + h, p, page), seqs[s][0] - 1), h // (hq // hk)].float()
             q[r, h] += 12 * c / c.pow(2).sum() ** 0.5
+            if (r + h) % 5 == 1:
+                q[r, h] = -6 / scale * u[h // (hq // hk)]
     q = q.to(dt)
     buf, gate = torch.zeros(n, qs, dtype=dt), rnd(n, gs, seed=8, scale=2).to(dt)
     buf[:, : hq * d] = q.view(n, -1)
@@ -232,7 +238,12 @@ def latent(gpu, act, H, rank, rot, page, seqs, ragged):
     dt, scale, base, pos_max = DT[act], 0.3, 200.0, 1200
     rows = [(s, L - R + i) for s, (L, R) in enumerate(seqs) for i in range(R)]
     n, rs = len(rows), H * rot + 8
-    pool, table, flat = _paged(seqs, page, (rank + rot,), dt, 4, .5)
+    pool, table, flat = _paged(seqs, page, (rank + rot,), torch.float32, 4, .5)
+    u = rnd(rank, seed=9)
+    u = u / u.pow(2).sum().sqrt()
+    pool[..., :rank] += 2 * u
+    pool[..., rank:] *= (rank / rot) ** 0.5          # the turned part weighs as much as the latent
+    pool = pool.to(dt)
     cf = [flat(pool, s).double() for s in range(len(seqs))]
     sink = bf(2 + rnd(H, seed=6, scale=2))
     ql, qr, pos = rnd(n, H, rank, seed=7, scale=.2), rnd(n, H, rot, seed=8, scale=.4), torch.tensor([p for _, p in rows])
@@ -243,6 +254,8 @@ def latent(gpu, act, H, rank, rot, page, seqs, ragged):
             ql[r, h] += 13 * c[:rank] / size
             turned = c[None, None, rank:].double()
             qr[r, h] += 13 * O.rotate(turned, torch.tensor([-p]), rot, base)[0, 0].float() / size      # the row's turn brings it onto the key
+            if (r + h) % 5 == 1:      # away from every key: the sink takes nearly everything
+                ql[r, h], qr[r, h] = -6 / scale * u, 0
     ql, qr = ql.to(dt), qr.to(dt)
     tabs = run_op(C.rope_table_op(pos_max, rot, base), [torch.zeros(pos_max, rot // 2), torch.zeros(pos_max, rot // 2)], gpu)
     buf = torch.zeros(n, rs, dtype=dt)
@@ -262,5 +275,6 @@ def latent(gpu, act, H, rank, rot, page, seqs, ragged):
     close(out[2], want, act, 1.5)
     assert int(out[5]) == 0
     # without the sink, or the query's turn, some row is far away
-    for other in ([wanted(r, sink - 1e4) for r in range(min(n, 6))], [wanted(r, sink, qr.double()) for r in range(min(n, 6))]):
+    some = range(min(n, 12))
+    for other in ([wanted(r, sink - 1e4) for r in some], [wanted(r, sink, qr.double()) for r in some]):
         assert float((torch.stack(other) - want[:len(other)]).abs().max() / want.abs().max()) > 0.06
