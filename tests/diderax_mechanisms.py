@@ -239,9 +239,9 @@ def latent(gpu, act, H, rank, rot, page, seqs, ragged):
     rows = [(s, L - R + i) for s, (L, R) in enumerate(seqs) for i in range(R)]
     n, rs = len(rows), H * rot + 8
     pool, table, flat = _paged(seqs, page, (rank + rot,), torch.float32, 4, .5)
-    u = rnd(rank, seed=9)
+    u, length = rnd(rank, seed=9), 2 * max(1.0, rank / 72) ** 0.5
     u = u / u.pow(2).sum().sqrt()
-    pool[..., :rank] += 2 * u
+    pool[..., :rank] += length * u
     pool[..., rank:] *= (rank / rot) ** 0.5          # the turned part weighs as much as the latent
     pool = pool.to(dt)
     cf = [flat(pool, s).double() for s in range(len(seqs))]
@@ -251,11 +251,11 @@ def latent(gpu, act, H, rank, rot, page, seqs, ragged):
         for h in range(H):
             c = cf[s][min(_far_key(r + h, p, page), seqs[s][0] - 1)].float()
             size = c.pow(2).sum() ** 0.5
-            ql[r, h] += 13 * c[:rank] / size
+            ql[r, h] += (13 if (r + h) % 5 != 3 else 0) * c[:rank] / size      # some find their key by the turned part alone
             turned = c[None, None, rank:].double()
             qr[r, h] += 13 * O.rotate(turned, torch.tensor([-p]), rot, base)[0, 0].float() / size      # the row's turn brings it onto the key
             if (r + h) % 5 == 1:      # away from every key: the sink takes nearly everything
-                ql[r, h], qr[r, h] = -6 / scale * u, 0
+                ql[r, h], qr[r, h] = -12 / scale / length * u, 0
     ql, qr = ql.to(dt), qr.to(dt)
     tabs = run_op(C.rope_table_op(pos_max, rot, base), [torch.zeros(pos_max, rot // 2), torch.zeros(pos_max, rot // 2)], gpu)
     buf = torch.zeros(n, rs, dtype=dt)
