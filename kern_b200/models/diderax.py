@@ -272,7 +272,7 @@ def build_manifest(cfg: DideraxConfig) -> dict:
         w_in, qkg = m_.rows_weight(f"w.{p}qkg", d, [(p + "q", q), (p + "k", k), (p + "g", q)])
         room("qkg", qkg); room("attn", q); room("y", d)
         cos_sin = m_.rotary(r["dims"], r["base"], r.get("scaling", {}).get("factor", 1.0))
-        prep = op(f"prep_{hq}x{hk}x{dim}x{r['dims']}x{qkg}", lambda: K.qk_prep_whole_op(hq, hk, dim, dim, q, r["dims"], page, qkg, cfg.context, eps, A, halves=True))
+        prep = op(f"prep_whole_{hq}x{hk}x{dim}x{r['dims']}x{qkg}", lambda: K.qk_prep_whole_op(hq, hk, dim, dim, q, r["dims"], page, qkg, cfg.context, eps, A, halves=True))
         attn = op(f"sink_attn{sfx}_{hq}x{hk}x{dim}x{qkg}_{m['scale']!r}", lambda: K.sink_attn_op(hq, hk, dim, dim, m["scale"], page, W, qkg, q, qkg, prefill, A, seqs_max=S))
         lens, lists = B("seq_lens"), []
         if prefill and tiled[i]:

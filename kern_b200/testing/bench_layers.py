@@ -1,10 +1,11 @@
 """Prefill and decode throughput of a decoder with listed layers beside the framework's closest model at equal size, with the
-time of every kind of kernel against its roofline: `python bench.py --config gafapel|barotar [--layers N]`.
+time of every kind of kernel against its roofline: `python bench.py --config gafapel|barotar|diderax [--layers N]`.
 
 The decoders have the width, depth, vocabulary and routed experts of the 48B-A3B shape class and random weights. Gafapel has
 Mamba-2 and unrotated latent-attention layers over four residual streams, Barotar window attention beside time mixing and gated
-linear attention; the model beside them per-key-decay delta-rule layers and 512 + 64 latent attention. Beside Barotar there is
-also the routed decoder with grouped-query attention of the same head counts and dims, for its attention kernels. A point is timed end to end (CUDA events around the call, captured graphs for decode,
+linear attention, Diderax gated linear attention, grouped-query attention and 512 + 64 latent attention with sinks; the model beside
+them per-key-decay delta-rule layers and 512 + 64 latent attention. Beside Barotar and Diderax there is also the routed decoder
+with grouped-query attention of the same head counts and dims, for its attention kernels. A point is timed end to end (CUDA events around the call, captured graphs for decode,
 L2 flushed before every sample) and once more call by call, where a call's roofline is the larger of its bytes over the
 measured copy rate and its flops over the measured tensor rate.
 """
@@ -14,7 +15,8 @@ import json
 import re
 from pathlib import Path
 
-MODELS = {"gafapel": ("gafapel-48b-a3b", "latent-48b-a3b"), "barotar": ("barotar-48b-a3b", "latent-48b-a3b", "moe-30b-a3b")}
+MODELS = {"gafapel": ("gafapel-48b-a3b", "latent-48b-a3b"), "barotar": ("barotar-48b-a3b", "latent-48b-a3b", "moe-30b-a3b"),
+          "diderax": ("diderax-48b-a3b", "latent-48b-a3b", "moe-30b-a3b")}
 POINTS = ({"groups": 1, "chunk": 2048, "context": 2048}, {"groups": 4, "chunk": 512, "context": 2048},
           {"groups": 1, "rows": 1, "context": 1024}, {"groups": 16, "rows": 1, "context": 1024}, {"groups": 64, "rows": 1, "context": 1024})
 
@@ -53,11 +55,20 @@ def cost(doc: dict, call: dict, groups: int, rows: int, context: int) -> tuple[f
     for s in st:
         if s.get("bytes_per_seq"):
             tok += 2 * groups * s["bytes_per_seq"]
-    if re.match(r"(window_)?attn_(prefill|decode|p_|d_)", op):
+    m = re.match(r"latent_attn_[pd]_(\d+)x(\d+)x(\d+)x", op)
+    if m:                                                   # heads, latent columns, rotated columns behind them
+        H, rank, rot = map(int, m.groups())
+        flops = 2.0 * n * H * (2 * rank + rot) * (context if rows == 1 else context - (rows - 1) / 2)
+        return n * H * (2 * rank + rot) * 2.0 + groups * context * (rank + rot) * 2.0, flops
+    m = re.match(r"prep_whole_(\d+)x(\d+)x(\d+)x", op)
+    if m:                                                   # q read and written, k read, keys and values written
+        hq, hk, d = map(int, m.groups())
+        return n * (2 * hq + 3 * hk) * d * 2.0, 0.0
+    if re.match(r"(window_|sink_)?attn_(prefill|decode|p_|d_)", op):
         hq, hk, d, dv, window = _heads(doc, call)
         seen_by = lambda p: min(p + 1, window)
         flops = 2.0 * groups * hq * (d + dv) * sum(seen_by(p) for p in range(context - rows, context))
-        cols = groups * rows * (hq * (d + dv)) * 2.0
+        cols = groups * rows * (hq * (d + dv + (dv if op.startswith("sink_") else 0))) * 2.0      # with the gate's columns
         return cols + groups * min(context, window + rows - 1) * hk * (d + dv) * 2.0, flops
     m = re.match(r"lin_[pd]_(\d+)x(\d+)x(\d+)", op)
     if m:                                                   # a recurrence: its rows, its decays and its states
@@ -105,6 +116,10 @@ def _heads(doc: dict, call: dict) -> tuple[int, int, int, int, int]:
     m = re.match(r"window_attn_._(\d+)x(\d+)x(\d+)x(\d+)x(\d+)", call["op"])
     if m:
         return tuple(map(int, m.groups()))
+    m = re.match(r"sink_attn_._(\d+)x(\d+)x(\d+)x", call["op"])
+    if m:
+        hq, hk, d = map(int, m.groups())
+        return hq, hk, d, d, 1 << 30
     args = doc["ops"][call["op"]]["impl"]["launches"][0]
     d = int(re.search(r"_d(\d+)", args["entry"]).group(1))
     hk = doc["states"][next(a["state"] for a in call["args"] if "state" in a)]["bytes_per_token"] // (4 * d)
