@@ -20,37 +20,76 @@ KERN_DEVICE void norm_row(const T* x, const __nv_bfloat16* w, T* out, int n, flo
   float ss = 0.f;
   for (int i = threadIdx.x; i < n; i += 128) { const float v = ldf(x + i); ss += v * v; }
   ss = warp_sum(ss);
-  __syncthreads();
   if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = ss;
   __syncthreads();
   const float inv = 1.f / sqrtf((part[0] + part[1] + part[2] + part[3]) / (float)n + eps);
   for (int i = threadIdx.x; i < n; i += 128) stf(out + i, ldf(x + i) * inv * __bfloat162float(w[i]));
 }
 
-// the latent, then `rot` columns behind it turned by the token's position (pairs i, i + rot / 2)
 template <typename T>
 KERN_DEVICE void append_body(const T* lat, uint8_t* cache, const long long* slots, const __nv_bfloat16* w, int rank, int stride,
-                             float eps, const long long* positions = nullptr, const float* cos_tab = nullptr,
-                             const float* sin_tab = nullptr, int rot = 0, int max_pos = 0, int* err = nullptr) {
+                             float eps) {
   const int t = blockIdx.x;
   const long long slot = slots[t];
   if (slot < 0) return;
-  const T* x = lat + (size_t)t * stride;
-  T* dst = reinterpret_cast<T*>(cache) + (size_t)slot * (rank + rot);
-  if (!KERN_CHECK(dst, (size_t)(rank + rot) * sizeof(T), SITE_KV_APPEND)) return;
-  norm_row(x, w, dst, rank, eps);
-  if (rot == 0) return;
+  T* dst = reinterpret_cast<T*>(cache) + (size_t)slot * rank;
+  if (!KERN_CHECK(dst, (size_t)rank * sizeof(T), SITE_KV_APPEND)) return;
+  norm_row(lat + (size_t)t * stride, w, dst, rank, eps);
+}
+
+// Row [query latent | latent | rot columns]: the first normed to q_low, the second normed and the third turned by the token's
+// position (pairs i, i + rot / 2) to the token's cached row. Block 256, (q_rank + rank) floats of shared memory, V columns per
+// thread and step.
+template <typename T, int V>
+KERN_DEVICE void prep_body(const T* rows, uint8_t* cache, T* q_low, const long long* positions, const long long* slots,
+                           const float* cos_tab, const float* sin_tab, const __nv_bfloat16* w, const __nv_bfloat16* wq, int rank,
+                           int rot, int q_rank, int stride, int q_stride, int max_pos, float eps, int* err) {
+  extern __shared__ __align__(16) float lat_sm[];
+  __shared__ float part[2][8];
+  const int t = blockIdx.x, n = q_rank + rank, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* x = rows + (size_t)t * stride;
+  const long long slot = slots[t];
   long long pos = positions[t];
+  float sq = 0.f, sc = 0.f;
+  for (int c = threadIdx.x * V; c < n; c += 256 * V) {
+    const Vec<V> a = ldv<V>(x + c);
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < V; ++e) s += a.v[e] * a.v[e];
+    if (c < q_rank) sq += s; else sc += s;
+    stv<V>(lat_sm + c, a);
+  }
+  sq = warp_sum(sq);
+  sc = warp_sum(sc);
+  if (lane == 0) { part[0][warp] = sq; part[1][warp] = sc; }
+  __syncthreads();
+  sq = sc = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { sq += part[0][i]; sc += part[1][i]; }
+  const float inv_q = 1.f / sqrtf(sq / (float)q_rank + eps), inv_c = 1.f / sqrtf(sc / (float)rank + eps);
+  T* dst = reinterpret_cast<T*>(cache) + (size_t)(slot < 0 ? 0 : slot) * (rank + rot);
+  const bool store = slot >= 0 && KERN_CHECK(dst, (size_t)(rank + rot) * sizeof(T), SITE_KV_APPEND);
+  for (int c = threadIdx.x * V; c < n; c += 256 * V) {
+    const bool is_q = c < q_rank;
+    if (!is_q && !store) break;
+    const Vec<V> a = ldv<V>(lat_sm + c), b = ldv<V>(is_q ? wq + c : w + (c - q_rank));
+    const float inv = is_q ? inv_q : inv_c;
+    Vec<V> o;
+#pragma unroll
+    for (int e = 0; e < V; ++e) o.v[e] = a.v[e] * inv * b.v[e];
+    stv<V>(is_q ? q_low + (size_t)t * q_stride + c : dst + (c - q_rank), o);
+  }
   if (pos < 0 || pos >= max_pos) {
     if (threadIdx.x == 0) set_error(err, ERR_BOUNDS);
     pos = 0;
   }
   const int half = rot >> 1;
-  for (int i = threadIdx.x; i < half; i += 128) {
-    const float a = ldf(x + rank + i), b = ldf(x + rank + half + i), c = cos_tab[pos * half + i], s = sin_tab[pos * half + i];
-    stf(dst + rank + i, a * c - b * s);
-    stf(dst + rank + half + i, b * c + a * s);
-  }
+  if (store)
+    for (int i = threadIdx.x; i < half; i += 256) {
+      const float a = ldf(x + n + i), b = ldf(x + n + half + i), c = cos_tab[pos * half + i], s = sin_tab[pos * half + i];
+      stf(dst + rank + i, a * c - b * s);
+      stf(dst + rank + half + i, b * c + a * s);
+    }
 }
 
 template <typename T>
@@ -147,7 +186,7 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
 
 }  // namespace
 
-// append, prep: grid = tokens, block 128. attn: grid [heads, rows], block 128, (4 rank + 8 + rot) floats of shared memory.
+// append: grid = tokens, block 128. prep: grid = tokens. attn: grid [heads, rows], block 128, (4 rank + 8 + rot) floats of shared memory.
 #define LATENT_ATTN(T, SFX, W)                                                                                            \
   extern "C" __global__ void __launch_bounds__(128)                                                                       \
       kern_latent_attn_##SFX##_w##W(const T* q, const uint8_t* cache, T* out, const int* table, const int* lens,          \
@@ -173,13 +212,20 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
     pdl_wait();                                                                                                           \
     append_body<T>(lat, cache, slots, w, rank, stride, eps);                                                              \
   }                                                                                                                       \
-  extern "C" __global__ void __launch_bounds__(128)                                                                       \
+  extern "C" __global__ void __launch_bounds__(256)                                                                       \
       kern_latent_prep_##SFX(const T* rows, uint8_t* cache, T* q_low, const long long* positions, const long long* slots, \
                              const float* cos_tab, const float* sin_tab, const __nv_bfloat16* w, const __nv_bfloat16* wq, \
                              int rank, int rot, int q_rank, int stride, int q_stride, int max_pos, float eps, int* err) { \
     pdl_wait();                                                                                                           \
-    norm_row(rows + (size_t)blockIdx.x * stride, wq, q_low + (size_t)blockIdx.x * q_stride, q_rank, eps);                 \
-    append_body<T>(rows + q_rank, cache, slots, w, rank, stride, eps, positions, cos_tab, sin_tab, rot, max_pos, err);    \
+    const bool vec = (rank | rot | q_rank | stride | q_stride) % 4 == 0 &&                                                \
+                     ((reinterpret_cast<uintptr_t>(rows) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(q_low) | \
+                       reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(wq)) & 15) == 0;                      \
+    if (vec)                                                                                                              \
+      prep_body<T, 4>(rows, cache, q_low, positions, slots, cos_tab, sin_tab, w, wq, rank, rot, q_rank, stride, q_stride, \
+                      max_pos, eps, err);                                                                                 \
+    else                                                                                                                  \
+      prep_body<T, 1>(rows, cache, q_low, positions, slots, cos_tab, sin_tab, w, wq, rank, rot, q_rank, stride, q_stride, \
+                      max_pos, eps, err);                                                                                 \
     pdl_launch_dependents();                                                                                              \
   }                                                                                                                       \
   LATENT_ATTN(T, SFX, 64)                                                                                                 \

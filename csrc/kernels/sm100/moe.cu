@@ -138,32 +138,48 @@ extern "C" __global__ void __launch_bounds__(128)
 // may be negative. `groups` equal groups of neighbours, a group's score the sum of its `group_top` largest c (1 or 2; its one, in
 // groups of one); the k largest c of the best `keep` groups are chosen (ties: the lower group, the lower id) and weigh s,
 // divided by their sum when `renorm`, times `scale`. One warp per token; E <= 1024, k <= 32, at most 64 groups.
-extern "C" __global__ void __launch_bounds__(128)
-    kern_moe_route_groups(const float* logits, const __nv_bfloat16* bias, int* topk_ids, float* topk_w, int tokens, int experts, int k,
-                          int groups, int keep, int softmax, int group_top, int renorm, float scale, int ld) {
+// A lane keeps the scores and choices of experts i * 32 + lane in registers; the choices also go through shared memory, for the
+// groups' scores.
+template <int PER>
+KERN_DEVICE void route_groups_body(const float* logits, const __nv_bfloat16* bias, int* topk_ids, float* topk_w, int tokens, int experts,
+                                   int k, int groups, int keep, int softmax, int group_top, int renorm, float scale, int ld) {
   extern __shared__ float route_sm[];      // [4][experts] choice scores, then [4][groups] group scores
-  pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp;
   if (t >= tokens) return;
   float* sc = route_sm + warp * experts;
   float* gs = route_sm + 4 * experts + warp * groups;
   const float* row = logits + (size_t)t * ld;
-  float mx = -INFINITY, over = 1.f;
+  float s[PER], c[PER], mx = -INFINITY;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    s[i] = i * 32 + lane < experts ? row[i * 32 + lane] : -INFINITY;
+    mx = fmaxf(mx, s[i]);
+  }
   if (softmax) {
-    for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, row[e]);
     mx = warp_max(mx);
     float sum = 0.f;
-    for (int e = lane; e < experts; e += 32) sum += exp2f((row[e] - mx) * 1.4426950408889634f);
-    over = 1.f / warp_sum(sum);
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      s[i] = exp2f((s[i] - mx) * 1.4426950408889634f);
+      sum += s[i];
+    }
+    const float over = 1.f / warp_sum(sum);
+#pragma unroll
+    for (int i = 0; i < PER; ++i) s[i] *= over;
+  } else {
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const float x = exp2f(-fabsf(s[i]) * 1.4426950408889634f);
+      s[i] = s[i] >= 0.f ? 1.f / (1.f + x) : x / (1.f + x);
+    }
   }
-  auto score = [&](int e) {
-    const float z = row[e];
-    if (softmax) return exp2f((z - mx) * 1.4426950408889634f) * over;
-    const float x = exp2f(-fabsf(z) * 1.4426950408889634f);
-    return z >= 0.f ? 1.f / (1.f + x) : x / (1.f + x);
-  };
-  for (int e = lane; e < experts; e += 32) sc[e] = score(e) + (bias ? __bfloat162float(bias[e]) : 0.f);
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int e = i * 32 + lane;
+    c[i] = -INFINITY;
+    if (e < experts) sc[e] = c[i] = s[i] + (bias ? __bfloat162float(bias[e]) : 0.f);
+  }
   __syncwarp();
   const int per = experts / groups;
   for (int g = lane; g < groups; g += 32) {
@@ -184,13 +200,20 @@ extern "C" __global__ void __launch_bounds__(128)
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) kept |= __shfl_xor_sync(0xffffffffu, kept, o);
-  float my_w = 0.f, sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int e = i * 32 + lane;
+    if (e < experts && !(kept >> (e / per) & 1)) c[i] = -INFINITY;
+  }
+  float my_w = 0.f;
   int my_id = 0;
   for (int j = 0; j < k; ++j) {
     float best = -INFINITY;
     int bi = 0x7fffffff;
-    for (int e = lane; e < experts; e += 32)
-      if ((kept >> (e / per) & 1) && sc[e] > best) { best = sc[e]; bi = e; }
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (c[i] > best) { best = c[i]; bi = i * 32 + lane; }
+#pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ob = __shfl_xor_sync(0xffffffffu, best, o);
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
@@ -198,16 +221,27 @@ extern "C" __global__ void __launch_bounds__(128)
     }
     const bool none = bi >= experts;      // no score is a number: still a valid row
     if (none) bi = 0;
-    __syncwarp();
-    if (lane == 0) sc[bi] = -INFINITY;
-    __syncwarp();
-    if (lane == j) { my_w = none ? 0.f : (bias ? score(bi) : best); my_id = bi; }
+    float w = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (i * 32 + lane == bi) { w = s[i]; c[i] = -INFINITY; }
+    w = __shfl_sync(0xffffffffu, w, bi & 31);
+    if (lane == j) { my_w = none ? 0.f : w; my_id = bi; }
   }
-  sum = warp_sum(my_w);
+  const float sum = warp_sum(my_w);
   if (lane < k) {
     topk_ids[(size_t)t * k + lane] = my_id;
     topk_w[(size_t)t * k + lane] = (renorm ? my_w / (sum + 1e-20f) : my_w) * scale;
   }
+}
+
+extern "C" __global__ void __launch_bounds__(128)
+    kern_moe_route_groups(const float* logits, const __nv_bfloat16* bias, int* topk_ids, float* topk_w, int tokens, int experts, int k,
+                          int groups, int keep, int softmax, int group_top, int renorm, float scale, int ld) {
+  pdl_wait();
+  if (experts <= 128) route_groups_body<4>(logits, bias, topk_ids, topk_w, tokens, experts, k, groups, keep, softmax, group_top, renorm, scale, ld);
+  else if (experts <= 512) route_groups_body<16>(logits, bias, topk_ids, topk_w, tokens, experts, k, groups, keep, softmax, group_top, renorm, scale, ld);
+  else route_groups_body<32>(logits, bias, topk_ids, topk_w, tokens, experts, k, groups, keep, softmax, group_top, renorm, scale, ld);
 }
 
 // Single CTA (block 1024). entries = tokens * k. Outputs:

@@ -120,54 +120,64 @@ KERN_DEVICE void mix_body(float* x, const T* y, const int* perm, const float* to
   if (!hidden) norm_out<T, V>(resid_sm, inv_rms(ss, width, eps), w_next, xn + (size_t)t * width, width);
 }
 
+// V values as they lie in memory: what waits for its turn takes no more registers than that
+template <typename T, int V> struct RawOf { T v[V]; };
+template <> struct __align__(8) RawOf<__nv_bfloat16, 4> { uint2 v; };
+template <> struct __align__(16) RawOf<float, 4> { float4 v; };
+template <int V, typename T> KERN_DEVICE RawOf<T, V> raw(const T* p) { return *reinterpret_cast<const RawOf<T, V>*>(p); }
+template <typename T, int V> KERN_DEVICE void add(Vec<V>& a, const RawOf<T, V>& r, float w) {
+  const Vec<V> b = ldv<V>(reinterpret_cast<const T*>(&r));
+#pragma unroll
+  for (int e = 0; e < V; ++e) a.v[e] += w * b.v[e];
+}
+
 // A sublayer's result: y, or with `perm` the weighted sum of a token's expert rows; choices without a row (perm < 0) are the
 // experts that hand back the input, xn as it is on entry. `shared` [rows][width] is weighed by sigmoid(gate[t gate_stride]).
-template <typename T, int V>
+template <typename T, int V, bool ROUTED>
 KERN_DEVICE void scale_body(float* x, const T* y, const int* perm, const float* topw, const T* shared, const float* gate,
                             const __nv_bfloat16* bias, const __nv_bfloat16* scale, const __nv_bfloat16* w_next, T* xn, float* hidden,
                             int width, int k, int gate_stride, float eps) {
   extern __shared__ __align__(16) float resid_sm[];
   __shared__ float tw[32];
-  __shared__ int tr[32];
+  __shared__ int tr[32], n_rows;
+  __shared__ float own_w;
   const int t = blockIdx.x;
-  if (perm) {
-    if (threadIdx.x < k) {
-      const int r = perm[(size_t)t * k + threadIdx.x];
-      const bool ok = r >= 0 && KERN_CHECK(y + (size_t)r * width, (size_t)width * sizeof(T), SITE_MOE_COMBINE);
-      tr[threadIdx.x] = ok ? r : -1;
-      tw[threadIdx.x] = topw[(size_t)t * k + threadIdx.x];
+  float self = 0.f;
+  if constexpr (ROUTED) {
+    if (threadIdx.x < 32) {      // the choices with a row to the front, then nothing
+      const int j = threadIdx.x;
+      int r = j < k ? perm[(size_t)t * k + j] : -1;
+      const float w = j < k ? topw[(size_t)t * k + j] : 0.f;
+      if (r >= 0 && !KERN_CHECK(y + (size_t)r * width, (size_t)width * sizeof(T), SITE_MOE_COMBINE)) r = -1;
+      const unsigned have = __ballot_sync(0xffffffffu, r >= 0);
+      if (r >= 0) { tr[__popc(have & ((1u << j) - 1))] = r; tw[__popc(have & ((1u << j) - 1))] = w; }
+      const float own = warp_sum(r < 0 ? w : 0.f);
+      if (j == 0) { n_rows = __popc(have); own_w = own; }
     }
     __syncthreads();
+    self = own_w;
   }
-  float self = 0.f;
-  if (perm)
-    for (int j = 0; j < k; ++j)
-      if (tr[j] < 0) self += tw[j];
   const float g = shared ? 1.f / (1.f + expf(-gate[(size_t)t * gate_stride])) : 0.f;
   float* xt = x + (size_t)t * width;
   T* xnt = xn + (size_t)t * width;
   float ss = 0.f;
   for (int i = threadIdx.x * V; i < width; i += 256 * V) {
     Vec<V> v = {};
-    if (perm) {
-      for (int j = 0; j < k; ++j) {
-        if (tr[j] < 0) continue;
-        const Vec<V> r = ldv<V>(y + (size_t)tr[j] * width + i);
-#pragma unroll
-        for (int e = 0; e < V; ++e) v.v[e] += tw[j] * r.v[e];
+    if constexpr (ROUTED) {
+      const int n = n_rows;
+      int j = 0;
+      for (; j + 4 <= n; j += 4) {      // four rows in flight
+        const RawOf<T, V> r0 = raw<V>(y + (size_t)tr[j] * width + i), r1 = raw<V>(y + (size_t)tr[j + 1] * width + i),
+                          r2 = raw<V>(y + (size_t)tr[j + 2] * width + i), r3 = raw<V>(y + (size_t)tr[j + 3] * width + i);
+        add(v, r0, tw[j]); add(v, r1, tw[j + 1]); add(v, r2, tw[j + 2]); add(v, r3, tw[j + 3]);
       }
-      if (self != 0.f) {
-        const Vec<V> h = ldv<V>(xnt + i);
-#pragma unroll
-        for (int e = 0; e < V; ++e) v.v[e] += self * h.v[e];
-      }
+      for (; j < n; ++j) add(v, raw<V>(y + (size_t)tr[j] * width + i), tw[j]);
+      if (self != 0.f) add(v, raw<V>(xnt + i), self);
     } else {
       v = ldv<V>(y + (size_t)t * width + i);
     }
     if (shared) {
-      const Vec<V> r = ldv<V>(shared + (size_t)t * width + i);
-#pragma unroll
-      for (int e = 0; e < V; ++e) v.v[e] += g * r.v[e];
+      add(v, raw<V>(shared + (size_t)t * width + i), g);
     }
     if (bias) {
       const Vec<V> r = ldv<V>(bias + i);
@@ -210,18 +220,25 @@ KERN_DEVICE void scale_body(float* x, const T* y, const int* perm, const float* 
     if (width % 4 == 0) mix_body<T, 4>(x, y, perm, topw, w_post, w_next, xn, hidden, width, k, eps);                      \
     else mix_body<T, 1>(x, y, perm, topw, w_post, w_next, xn, hidden, width, k, eps);                                     \
     pdl_launch_dependents();                                                                                              \
-  }                                                                                                                       \
-  extern "C" __global__ void __launch_bounds__(256)                                                                       \
-      kern_resid_scale_##SFX(float* x, const T* y, const int* perm, const float* topw, const T* shared, const float* gate, \
-                             const __nv_bfloat16* bias, const __nv_bfloat16* scale, const __nv_bfloat16* w_next, T* xn,   \
-                             float* hidden, int width, int k, int gate_stride, float eps) {                               \
-    pdl_wait();                                                                                                           \
-    if (width % 4 == 0)                                                                                                   \
-      scale_body<T, 4>(x, y, perm, topw, shared, gate, bias, scale, w_next, xn, hidden, width, k, gate_stride, eps);      \
-    else                                                                                                                  \
-      scale_body<T, 1>(x, y, perm, topw, shared, gate, bias, scale, w_next, xn, hidden, width, k, gate_stride, eps);      \
-    pdl_launch_dependents();                                                                                              \
   }
 
 RESID_ENTRIES(__nv_bfloat16, bf16)
 RESID_ENTRIES(float, f32)
+
+// the routed form has an entry of its own: its rows in flight would cost the plain one registers
+#define RESID_SCALE(NAME, T, ROUTED)                                                                                      \
+  extern "C" __global__ void __launch_bounds__(256)                                                                       \
+      NAME(float* x, const T* y, const int* perm, const float* topw, const T* shared, const float* gate,                  \
+           const __nv_bfloat16* bias, const __nv_bfloat16* scale, const __nv_bfloat16* w_next, T* xn, float* hidden,      \
+           int width, int k, int gate_stride, float eps) {                                                                \
+    pdl_wait();                                                                                                           \
+    if (width % 4 == 0)                                                                                                   \
+      scale_body<T, 4, ROUTED>(x, y, perm, topw, shared, gate, bias, scale, w_next, xn, hidden, width, k, gate_stride, eps); \
+    else                                                                                                                  \
+      scale_body<T, 1, ROUTED>(x, y, perm, topw, shared, gate, bias, scale, w_next, xn, hidden, width, k, gate_stride, eps); \
+    pdl_launch_dependents();                                                                                              \
+  }
+RESID_SCALE(kern_resid_scale_bf16, __nv_bfloat16, false)
+RESID_SCALE(kern_resid_scale_f32, float, false)
+RESID_SCALE(kern_resid_scale_routed_bf16, __nv_bfloat16, true)
+RESID_SCALE(kern_resid_scale_routed_f32, float, true)

@@ -286,10 +286,12 @@ def latent_prep_op(rank: int, rot: int, q_rank: int, stride: int, q_stride: int,
     Interface [rows, state, q latent, positions, slots, cos, sin, latent norm w, query norm w, err]."""
     if rot % 2 or not rot:
         raise ValueError(f"a rotated key part of {rot} columns")
+    if rank + q_rank > 50000:
+        raise ValueError(f"latents of {rank} and {q_rank} columns (at most 50000 together)")
     iface = [f"in buffer<{act}>", "inout state", f"out buffer<{act}>", "in buffer<i64>", "in buffer<i64>", "in buffer<f32>", "in buffer<f32>", "in buffer<bf16>",
              "in buffer<bf16>", "out buffer<i32>"]
-    return _op(iface, _launch("latent", f"kern_latent_prep_{act}", [128, 1, 1], ["tokens", 1, 1], iface[:9] + ["i32"] * 6 + ["f32", "out buffer<i32>"],
-                              [*map(P, range(9)), I(rank), I(rot), I(q_rank), I(stride), I(q_stride), I(max_pos), {"f32": eps}, P(9)]))
+    return _op(iface, _launch("latent", f"kern_latent_prep_{act}", [256, 1, 1], ["tokens", 1, 1], iface[:9] + ["i32"] * 6 + ["f32", "out buffer<i32>"],
+                              [*map(P, range(9)), I(rank), I(rot), I(q_rank), I(stride), I(q_stride), I(max_pos), {"f32": eps}, P(9)], shared_mem=(rank + q_rank) * 4))
 
 
 def latent_rot_attn_op(heads: int, rank: int, rot: int, scale: float, page_size: int, table_width: int, max_pos: int, rot_stride: int, ragged: bool,
@@ -356,7 +358,7 @@ def resid_scale_op(width: int, eps: float, act: str = "bf16", *, routed: int = 0
     else:
         tail = [(iface[3], P(3)), (iface[4], P(4)), NULL]
     parts = [(iface[0], P(0)), (iface[1], P(1)), *route, *sh, *b, (iface[2], P(2)), *tail]
-    return _op(iface, _launch("resid", f"kern_resid_scale_{act}", [256, 1, 1], ["tokens", 1, 1], [t for t, _ in parts] + ["i32", "i32", "i32", "f32"],
+    return _op(iface, _launch("resid", f"kern_resid_scale{'_routed' if routed else ''}_{act}", [256, 1, 1], ["tokens", 1, 1], [t for t, _ in parts] + ["i32", "i32", "i32", "f32"],
                               [a for _, a in parts] + [I(width), I(routed), I(shared_gate or 0), {"f32": eps}], shared_mem=width * 4))
 
 

@@ -568,7 +568,7 @@ for _a in ("bf16", "f32"):
     CPU_KERNELS.update({f"kern_hyper_embed_{_a}": k_hyper_embed, f"kern_row_norm_f32_{_a}": k_row_norm,
                         f"kern_rows_scatter_{_a}": k_rows_scatter, f"kern_gate_mul_{_a}": k_gate_mul,
                         f"kern_resid_embed_{_a}": k_resid_embed, f"kern_resid_mix_{_a}": k_resid_mix,
-                        f"kern_resid_scale_{_a}": k_resid_scale, f"kern_qk_prep_whole_{_a}": k_qk_prep_whole, f"kern_latent_prep_{_a}": k_latent_prep,
+                        f"kern_resid_scale_{_a}": k_resid_scale, f"kern_resid_scale_routed_{_a}": k_resid_scale, f"kern_qk_prep_whole_{_a}": k_qk_prep_whole, f"kern_latent_prep_{_a}": k_latent_prep,
                         f"kern_token_shift_{_a}": k_token_shift, f"kern_shift_state_{_a}": k_shift_state, f"kern_decay_{_a}": k_decay,
                         f"kern_lin_norm_gate_{_a}": k_lin_norm_gate, f"kern_qk_prep_{_a}": k_qk_prep,
                         f"kern_ssd_conv_{_a}": k_ssd_conv, f"kern_ssd_conv_state_{_a}": k_ssd_conv_state,
