@@ -17,7 +17,7 @@ def index(tmp_path, monkeypatch):
 
 def test_entries_come_from_the_sources_macros_included():
     gemv = R.entries_of(_build.KSRC / "gemv_bf16.cu")
-    assert {"kern_gemv_bf16_tn_m1", "kern_gemv_bf16_tn_swiglu_m8"} <= set(gemv) and len(gemv) == 20      # token-pasted names
+    assert {"kern_gemv_bf16_tn_m1", "kern_gemv_bf16_tn_swiglu_m8"} <= set(gemv) and len(gemv) == 24      # token-pasted names
     moe = R.entries_of(_build.KSRC / "moe.cu")
     assert "kern_ep_fc2_bf16_combine_n256" in moe and "kern_moe_plan_ep" in moe
     assert not any(e.startswith("kern_gemm_bf16_tn") for e in moe)          # the included GEMM source's own entries are switched off
