@@ -91,7 +91,7 @@ def from_config(doc: dict, ranks: list[int], **over) -> DideraxConfig:
     for i, b in enumerate(doc["layers"]):
         _check_mixer(i, b["type"], b["mixer"])
         _check_mlp(i, b["mlp"])
-    return DideraxConfig(name=over.pop("name", "diderax"), width=doc["width"], vocab=doc["vocab"], eps=doc["norm"]["eps"], blocks=doc["layers"],
+    return DideraxConfig(name=over.pop("name", "diderax"), width=doc["width"], vocab=doc["vocab"], eps=float(doc["norm"]["eps"]), blocks=doc["layers"],
                          ranks=list(ranks), **over)
 
 
@@ -160,7 +160,7 @@ def latent_sizes(m: dict) -> dict:
 def moe_sizes(f: dict) -> dict:
     r = f["router"]
     identity, g = r.get("identity", 0), r.get("groups", {"count": 1, "keep": 1})
-    return {"experts": r["experts"], "outputs": r["experts"] + identity, "top": r["top"], "groups": g["count"], "keep": g["keep"], "scale": r.get("scale", 1.0),
+    return {"experts": r["experts"], "outputs": r["experts"] + identity, "top": r["top"], "groups": g["count"], "keep": g["keep"], "scale": float(r.get("scale", 1.0)),
             "shared": f["shared"]["ff"] if f.get("shared") else 0}
 
 
@@ -271,9 +271,9 @@ def build_manifest(cfg: DideraxConfig) -> dict:
         states[kv] = {"bytes_per_token": z["token"] * es}
         w_in, qkg = m_.rows_weight(f"w.{p}qkg", d, [(p + "q", q), (p + "k", k), (p + "g", q)])
         room("qkg", qkg); room("attn", q); room("y", d)
-        cos_sin = m_.rotary(r["dims"], r["base"], r.get("scaling", {}).get("factor", 1.0))
+        cos_sin = m_.rotary(r["dims"], float(r["base"]), float((r.get("scaling") or {}).get("factor", 1.0)))
         prep = op(f"prep_whole_{hq}x{hk}x{dim}x{r['dims']}x{qkg}", lambda: K.qk_prep_whole_op(hq, hk, dim, dim, q, r["dims"], page, qkg, cfg.context, eps, A, halves=True))
-        attn = op(f"sink_attn{sfx}_{hq}x{hk}x{dim}x{qkg}_{m['scale']!r}", lambda: K.sink_attn_op(hq, hk, dim, dim, m["scale"], page, W, qkg, q, qkg, prefill, A, seqs_max=S))
+        attn = op(f"sink_attn{sfx}_{hq}x{hk}x{dim}x{qkg}_{m['scale']!r}", lambda: K.sink_attn_op(hq, hk, dim, dim, float(m["scale"]), page, W, qkg, q, qkg, prefill, A, seqs_max=S))
         lens, lists = B("seq_lens"), []
         if prefill and tiled[i]:
             lists = [B("cu_seqlens"), *m_.lists_of(hq, hk, dim)]
@@ -301,7 +301,7 @@ def build_manifest(cfg: DideraxConfig) -> dict:
         fill = [{"tensor": p + "uq", "rows": [0, 1]}] * (qc - rows)
         w_uq = weight(f"w.{p}uq", (qc, qr), *[head(h, 0, dim) for h in range(H)], *[head(h, dim, dim + rot) for h in range(H)], *fill)
         room("down", down); room("q_low", qr); room("q", qc); room("qlat", z["lat"]); room("olat", z["lat"]); room("attn", z["v"]); room("y", d)
-        cos, sin = m_.rotary(rot, m["rot"]["base"])
+        cos, sin = m_.rotary(rot, float(m["rot"]["base"]))
         prep = op(f"latent_prep_{rank}x{rot}x{qr}x{down}", lambda: K.latent_prep_op(rank, rot, qr, down, qr, cfg.context, eps, A))
         uk = same(p + "uk", (z["q"], rank))
         tiles = K.head_tiles(rank, dim, qc, z["lat"], A)
@@ -311,7 +311,7 @@ def build_manifest(cfg: DideraxConfig) -> dict:
         up = op(f"q_up_{H}x{dim}x{rank}x{qc}", lambda: K.head_linear_op(H, rank, dim, act=A, rows_max=T, lda=qc, ldc=z["lat"], transposed=not tiles))
         v_up = op(f"v_up_{H}x{vdim}x{rank}", lambda: K.head_linear_op(H, vdim, rank, act=A, rows_max=T, lda=z["lat"], ldc=z["v"]))
         attn = op(f"latent_attn{sfx}_{H}x{rank}x{rot}x{qc}_{m['scale']!r}",
-                  lambda: K.latent_rot_attn_op(H, rank, rot, m["scale"], page, W, cfg.context, qc, prefill, A, seqs_max=S))
+                  lambda: K.latent_rot_attn_op(H, rank, rot, float(m["scale"]), page, W, cfg.context, qc, prefill, A, seqs_max=S))
         lens = [B("row_len"), err, *m_.row_plan()] if prefill else [B("seq_lens"), err]
         return [
             linear("lin", down, d, B("xn"), w_in, B("down"), label=p + "down"),

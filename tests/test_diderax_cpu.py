@@ -72,6 +72,13 @@ def test_registry_reads_a_folder_and_refuses_what_it_does_not_know(tmp_path):
     m, errs = verify(build(got))
     assert m is not None, errs[:3]
     doc = json.loads((tmp_path / "config.json").read_text())
+    whole = json.loads(json.dumps(doc).replace("3.0", "3").replace("8.0", "8").replace("10000.0", "10000"))      # numbers without a point
+    whole["layers"][0]["mixer"]["scale"] = whole["layers"][2]["mixer"]["scale"] = whole["layers"][0]["mlp"]["router"]["scale"] = 1
+    whole["layers"][1]["mixer"]["tau"] = 4
+    (tmp_path / "config.json").write_text(json.dumps(whole))
+    for dtype in P.ACTS:
+        m, errs = verify(build(registry.from_folder(tmp_path, dtype=dtype)[0]))
+        assert m is not None, errs[:3]
     att, lat = doc["layers"][0], doc["layers"][2]
     for change in ({"architecture": "Other"}, {"layers": [dict(doc["layers"][1], type="gla2")]}, {"layers": [dict(att, mixer={"heads": 2})]},
                    {"layers": [dict(att, mlp={"kind": "other"})]}, {"layers": [dict(att, mixer={**att["mixer"], "vdim": 32})]},
