@@ -88,7 +88,7 @@ struct FmhaArgs {
 template <int D, int FN, int FORM = kAttnPlain>
 KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const int y) {
   using Cfg = FmhaCfg<D, FN>;
-  constexpr bool WIN = FORM == kAttnWindow;
+  constexpr bool POOL = FORM == kAttnPooled, WIN = FORM == kAttnWindow;
   constexpr int kStages = Cfg::kStages;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -131,8 +131,10 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
   const int valid_rows = tok_n * G;
   const int last_pos = L - R + tok_lo + tok_n - 1;
   // (WIN) the first tile that any row of this block sees; tile j of the walk starts at token tok_first + j FN
-  const int tok_first = WIN ? max(0, L - R + tok_lo - a.win.size + 1) / FN * FN : 0;
-  const int ntiles = (last_pos - tok_first) / FN + 1;
+  const int tok_first = WIN || POOL ? max(0, L - R + tok_lo - a.win.size + 1) / FN * FN : 0;
+  // (POOL) the walk begins with the tiles of pooled rows that any row sees
+  const int pooled_n = POOL ? pooled_seen(last_pos, a.win) : 0, pooled_tiles = (pooled_n + FN - 1) / FN;
+  const int ntiles = pooled_tiles + (last_pos - tok_first) / FN + 1;
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < kStages; ++s) {
@@ -146,6 +148,7 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
     *abort_flag = 0;
     mbar_fence_init();
     tma_prefetch_desc(kv_map);
+    if constexpr (POOL) tma_prefetch_desc(a.win.pool_map);
   }
   if (warp == 1) {
     tmem_alloc(tmem_slot, Cfg::kTmemCols);
@@ -173,7 +176,8 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
 
   if (warp == 0) {
     // ---------------- producer ----------------
-    if (lane == 0) {
+    // (POOL) pooled tiles come in many small boxes: the whole warp walks, and lane 0 alone where there is one wait or one page
+    if (POOL || lane == 0) {
       const int box_rows = a.page_size < 64 ? a.page_size : 64;
       const int boxes = FN / box_rows;
       // one half (K: which = 0, V: which = 1) of tile t into its stage, behind the half's own empty barrier
@@ -182,15 +186,35 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
         const uint32_t parity = ((t / kStages) & 1) ^ 1;
         uint64_t* empty = which ? &v_empty[stage] : &k_empty[stage];
         uint64_t* full = which ? &v_full[stage] : &k_full[stage];
-        if (!mbar_wait_ns(empty, parity, abort_flag)) {
-          set_error(a.err, ERR_WAIT_EMPTY);
-          *abort_flag = 1;
-          return false;
+        int ok = 1;
+        if (lane == 0) {
+          ok = mbar_wait_ns(empty, parity, abort_flag);
+          if (ok) {
+            mbar_expect_tx(full, Cfg::kTileBytes);
+          } else {
+            set_error(a.err, ERR_WAIT_EMPTY);
+            *abort_flag = 1;
+          }
         }
+        if constexpr (POOL) ok = __shfl_sync(0xffffffffu, ok, 0);
+        if (!ok) return false;
         uint8_t* dst = kv_s + stage * 2 * Cfg::kTileBytes + which * Cfg::kTileBytes;
-        mbar_expect_tx(full, Cfg::kTileBytes);
+        if constexpr (POOL) {
+          if (t < pooled_tiles) {
+            const int pbox = a.win.slots < 64 ? a.win.slots : 64;
+            const int* pages = a.block_table + (size_t)seq * a.max_pages;
+            for (int b = lane * pbox; b < FN; b += 32 * pbox) {
+              const int row = pooled_row(a.win, t * FN + b, pooled_n, pages, a.max_pages, a.page_size, a.pool_pages, which, a.hk, kvh, a.err);
+#pragma unroll
+              for (int cb = 0; cb < D / 64; ++cb) tma_load_2d(dst + cb * (FN * 128) + b * 128, a.win.pool_map, cb * 64, row, full);
+            }
+            __syncwarp();
+            return true;
+          }
+          if (lane != 0) return true;
+        }
         for (int b = 0; b < boxes; ++b) {
-          const int tok = tok_first + t * FN + b * box_rows;
+          const int tok = tok_first + (t - pooled_tiles) * FN + b * box_rows;
           int page = 0, in_page = 0;
           const int pidx = tok / a.page_size;
           if (tok < L && pidx < a.max_pages) {
@@ -272,7 +296,8 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
       if (!mbar_wait_ns(&s_full[j & 1], (j >> 1) & 1, abort_flag)) { set_error(a.err, ERR_WAIT_TMEM_FULL); *abort_flag = 1; ok = false; break; }
       tc_fence_after();
       const uint32_t s_tmem = tmem_base + lane_addr + (j & 1) * FN;
-      const int tok0 = tok_first + j * FN;
+      const bool pooled = POOL && j < pooled_tiles;                // tok0 then counts blocks
+      const int tok0 = pooled ? j * FN : tok_first + (j - pooled_tiles) * FN;
       const bool diag = tok0 + FN - 1 > pos;                        // some column of the tile is above this row's limit
       // pass 1: the row maximum of the tile. With 64-token tiles the row's 64 scores stay in registers for pass 2 (one
       // read of S instead of two), and the S buffer is handed back to the MMA warp at once.
@@ -284,7 +309,7 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
         for (int c = 0; c < FN / 32; ++c) tmem_ld_32x32(s_tmem + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&keep[c * 32]));
         tmem_ld_wait();
         if constexpr (WIN) {      // capped scores in base-2 units, then both edges of the window
-          static_assert(!WIN || kKeep, "the windowed form keeps a tile's scores in registers");
+          static_assert(kKeep, "the windowed form keeps a tile's scores in registers");
           float ab[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
           for (int i = 0; i < FN; ++i) ab[i & 3] = fmaxf(ab[i & 3], fabsf(__uint_as_float(keep[i])));
@@ -308,6 +333,13 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
 #pragma unroll
             for (int i = 0; i < FN; ++i)
               if (tok0 + i > pos || tok0 + i <= pos - a.win.size) keep[i] = 0xff800000u;
+          }
+        } else if constexpr (POOL) {      // this row's blocks, or both edges of its window
+          const int lo = pooled ? 0 : pos - a.win.size + 1, hi = pooled ? pooled_seen(pos, a.win) : pos + 1;
+          if (tok0 < lo || tok0 + FN > hi) {
+#pragma unroll
+            for (int i = 0; i < FN; ++i)
+              if (tok0 + i < lo || tok0 + i >= hi) keep[i] = 0xff800000u;
           }
         } else if (diag) {       // the causal limit, once, on the scores themselves (a per-row branch: no warp-wide instruction inside)
 #pragma unroll
@@ -405,7 +437,7 @@ KERN_DEVICE void fmha_body(const CUtensorMap* kv_map, const FmhaArgs& a, const i
       tc_fence_after();
       const uint32_t o_tmem = tmem_base + lane_addr + 2 * FN;
       float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-      if constexpr (FORM != kAttnPlain) inv = row < valid_rows ? sink_factor(m_ref, l_run, sink_of(a.win, kvh * G + row % G), a.win.out_scale) : 0.f;
+      if constexpr (FORM == kAttnWindow || FORM == kAttnSink) inv = row < valid_rows ? sink_factor(m_ref, l_run, sink_of(a.win, kvh * G + row % G), a.win.out_scale) : 0.f;
       __nv_bfloat16* dst = nullptr;
       const __nv_bfloat16* gate = nullptr;
       if (row < valid_rows) {
@@ -861,4 +893,16 @@ extern "C" __global__ void __launch_bounds__(192, 2)
   FmhaArgs a{q, out, block_table, seq_lens, cu_q, work, work_count, err, hq, hk, q_stride, out_stride, max_pages, page_size,
              pool_pages, scale_log2, {0, 0.f, 0.f, 1.f, sink, gate, gate_stride}};
   fmha_body<128, 64, kAttnSink>(&kv_map, a, (int)blockIdx.y);
+}
+
+// The 64-token form over a sliding window and the pooled rows before it (kAttnPooled in attn_paged.cu).
+extern "C" __global__ void __launch_bounds__(192, 2)
+    kern_attn_pooled_fmha_d128(const __grid_constant__ CUtensorMap kv_map, const __grid_constant__ CUtensorMap pool_map,
+                               const __nv_bfloat16* q, __nv_bfloat16* out, const int* block_table, const int* seq_lens,
+                               const int* cu_q, const int* work, const int* work_count, int hq, int hk, int q_stride,
+                               int out_stride, int max_pages, int page_size, int pool_pages, int* err, int window, int pool,
+                               int slots, float scale_log2) {
+  FmhaArgs a{q, out, block_table, seq_lens, cu_q, work, work_count, err, hq, hk, q_stride, out_stride, max_pages, page_size,
+             pool_pages, scale_log2, {window, 0.f, 0.f, 1.f, nullptr, nullptr, 0, &pool_map, pool, slots}};
+  fmha_body<128, 64, kAttnPooled>(&kv_map, a, (int)blockIdx.y);
 }

@@ -60,8 +60,8 @@ struct AttnCfg {
 };
 
 // The forms of the bodies here and in attn_fmha.cu: plain softmax; in a sliding window with capped scores and a sink; causal
-// with a sink.
-enum AttnForm : int { kAttnPlain = 0, kAttnWindow = 1, kAttnSink = 2 };
+// with a sink; in a sliding window with the mean keys and values of the blocks before it.
+enum AttnForm : int { kAttnPlain = 0, kAttnWindow = 1, kAttnSink = 2, kAttnPooled = 3 };
 
 // Attention in a sliding window with capped scores and a sink (kAttnWindow): a row at position i sees the keys j with
 // 0 <= i - j < size; a score is cap tanh(score / cap), computed as c2 (1 - 2 / (1 + 2^(c1 q.k))) with c1 = 2 log2(e) scale / cap
@@ -75,7 +75,32 @@ struct AttnWindow {
   const __nv_bfloat16* sink = nullptr;
   const __nv_bfloat16* gate = nullptr;
   int gate_stride = 0;
+  // kAttnPooled: a row at position i also sees the mean key and value of every block of `pool` tokens that ends at i - size or
+  // before. A page of this second cache holds the blocks that end in the page of the same number, `slots` of them at most:
+  // [page][k|v][head][slot][D].
+  const CUtensorMap* pool_map = nullptr;
+  int pool = 1, slots = 1;
 };
+// blocks that a row at position `pos` sees
+KERN_DEVICE int pooled_seen(int pos, const AttnWindow& w) { return pos - w.size + 1 > 0 ? (pos - w.size + 1) / w.pool : 0; }
+// Of a tile of pooled rows from block b0 on, one box: the row of its first block in the 2-D view ([page][k|v][head][slot]), or the
+// pool's first row for blocks that no row sees. Boxes hold min(slots, 64) blocks of one page.
+KERN_DEVICE int pooled_row(const AttnWindow& w, int b, int seen, const int* pages, int max_pages, int page_size, int pool_pages,
+                           int which, int hk, int head, int* err) {
+  int page = 0, slot = 0;
+  if (b < seen) {
+    const int pidx = (b * w.pool + w.pool - 1) / page_size;
+    if (pidx < max_pages) {
+      page = pages[pidx];
+      slot = b - pidx * page_size / w.pool;
+    }
+    if (page < 0 || page >= pool_pages) {
+      set_error(err, ERR_BOUNDS);
+      page = 0;
+    }
+  }
+  return ((page * 2 + which) * hk + head) * w.slots + slot;
+}
 constexpr float kLog2e = 1.4426950408889634f;
 KERN_DEVICE float capped_score(float qk, const AttnWindow& w) { return w.c2 - __fdividef(2.f * w.c2, 1.f + exp2f(qk * w.c1)); }
 KERN_DEVICE float sink_of(const AttnWindow& w, int head) { return w.sink ? __bfloat162float(w.sink[head]) : 0.f; }
@@ -120,7 +145,7 @@ struct AttnArgs {
 template <int D, bool PREFILL, int ST = 0, int FORM = kAttnPlain>
 KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const int y) {
   using Cfg = AttnCfg<D, PREFILL, ST>;
-  constexpr bool WIN = FORM == kAttnWindow;
+  constexpr bool POOL = FORM == kAttnPooled, WIN = FORM == kAttnWindow || POOL;
   constexpr int kStages = Cfg::kStages;
   constexpr int NT = PREFILL ? 8 : 2;        // 8-token n-tiles of S per warp per KV tile
   constexpr int ROWS = PREFILL ? 64 : 16;    // query rows per CTA
@@ -157,6 +182,7 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
     *abort_flag = 0;
     mbar_fence_init();
     tma_prefetch_desc(kv_map);
+    if constexpr (POOL) tma_prefetch_desc(a.win.pool_map);
   }
   __syncthreads();
   pdl_wait();
@@ -169,7 +195,9 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
   const int last_pos = L - R + tok_lo + tok_n - 1;
   // (WIN) no row of this block sees a key before `tile_first`
   const int tile_first = WIN ? max(0, L - R + tok_lo - a.win.size + 1) / TK : 0;
-  const int ntiles_all = last_pos / TK + 1 - tile_first;
+  // (POOL) the walk begins with the tiles of pooled rows that any row sees
+  const int pooled_n = POOL ? pooled_seen(last_pos, a.win) : 0, pooled_tiles = (pooled_n + TK - 1) / TK;
+  const int ntiles_all = pooled_tiles + last_pos / TK + 1 - tile_first;
   // `splits` packs three numbers: bits 0-7 the KV splits of this launch, bits 8-15 the first partial slot it writes,
   // bits 16-31 the partial slots per (row, head) in the workspace (0: same as the splits). A context-parallel rank
   // writes its partials into its own run of slots of a workspace that holds every rank's; one merge covers them all.
@@ -183,7 +211,7 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
     if (tile_hi < tile_lo) tile_hi = tile_lo;
   }
   const int ntiles = tile_hi - tile_lo;
-  tile_lo += tile_first;
+  if constexpr (!POOL) tile_lo += tile_first;
 
   // ---- q tile -> shared (all 5 warps help) ----
   for (int i = threadIdx.x; i < ROWS * (D / 8); i += kAttnThreads) {
@@ -200,9 +228,69 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
 
   if (warp == 4) {
     // ---------------- producer ----------------
-    if (lane == 0) {
-      const int box_rows = a.page_size < TK ? a.page_size : TK;
-      const int boxes = TK / box_rows;
+    const int box_rows = a.page_size < TK ? a.page_size : TK;
+    const int boxes = TK / box_rows;
+    auto raw_tile = [&](int tok0, uint8_t* sk, uint64_t* bar) {
+      uint8_t* sv = sk + Cfg::kTileBytes;
+      for (int b = 0; b < boxes; ++b) {
+        const int tok = tok0 + b * box_rows;
+        int page = 0, in_page = 0;
+        const int pidx = tok / a.page_size;
+        if (tok < L && pidx < a.max_pages) {
+          page = a.block_table[(size_t)seq * a.max_pages + pidx];
+          in_page = tok % a.page_size;
+        }
+        if (page < 0 || page >= a.pool_pages) {
+          set_error(a.err, ERR_BOUNDS);
+          page = 0;
+        }
+        // rows of the 2-D view: ((page*2 + kv)*HK + head)*page_size + offset
+        const int krow = ((page * 2 + 0) * a.hk + kvh) * a.page_size + in_page;
+        const int vrow = ((page * 2 + 1) * a.hk + kvh) * a.page_size + in_page;
+#pragma unroll
+        for (int cb = 0; cb < D / 64; ++cb) {
+          tma_load_2d(sk + cb * (TK * 128) + b * box_rows * 128, kv_map, cb * 64, krow, bar);
+          tma_load_2d(sv + cb * (TK * 128) + b * box_rows * 128, kv_map, cb * 64, vrow, bar);
+        }
+      }
+    };
+    if constexpr (POOL) {
+      // pooled tiles come in many small boxes: the whole warp issues them
+      const int pbox = a.win.slots < TK ? a.win.slots : TK;
+      int stage = 0;
+      uint32_t phase = 0;
+      for (int t = 0; t < ntiles; ++t) {
+        uint8_t* sk = stages + stage * Cfg::kStageBytes;
+        int ok = 1;
+        if (lane == 0) {
+          ok = mbar_wait(&empty_bar[stage], phase ^ 1, abort_flag);
+          if (ok) mbar_expect_tx(&full_bar[stage], Cfg::kStageBytes);
+        }
+        ok = __shfl_sync(0xffffffffu, ok, 0);
+        if (!ok) {
+          if (lane == 0) {
+            set_error(a.err, ERR_WAIT_EMPTY);
+            *abort_flag = 1;
+          }
+          break;
+        }
+        const int tile = tile_lo + t;
+        if (tile < pooled_tiles) {
+          const int* pages = a.block_table + (size_t)seq * a.max_pages;
+          for (int i = lane; i < 2 * (TK / pbox); i += 32) {
+            const int b = (i >> 1) * pbox, which = i & 1;
+            const int row = pooled_row(a.win, tile * TK + b, pooled_n, pages, a.max_pages, a.page_size, a.pool_pages, which, a.hk, kvh, a.err);
+#pragma unroll
+            for (int cb = 0; cb < D / 64; ++cb)
+              tma_load_2d(sk + which * Cfg::kTileBytes + cb * (TK * 128) + b * 128, a.win.pool_map, cb * 64, row, &full_bar[stage]);
+          }
+        } else if (lane == 0) {
+          raw_tile((tile - pooled_tiles + tile_first) * TK, sk, &full_bar[stage]);
+        }
+        __syncwarp();
+        if (++stage == kStages) { stage = 0; phase ^= 1; }
+      }
+    } else if (lane == 0) {
       int stage = 0;
       uint32_t phase = 0;
       for (int t = 0; t < ntiles; ++t) {
@@ -211,33 +299,8 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
           *abort_flag = 1;
           break;
         }
-        uint8_t* sk = stages + stage * Cfg::kStageBytes;
-        uint8_t* sv = sk + Cfg::kTileBytes;
         mbar_expect_tx(&full_bar[stage], Cfg::kStageBytes);
-        const int tok0 = (tile_lo + t) * TK;
-        for (int b = 0; b < boxes; ++b) {
-          const int tok = tok0 + b * box_rows;
-          int page = 0, in_page = 0;
-          const int pidx = tok / a.page_size;
-          if (tok < L && pidx < a.max_pages) {
-            page = a.block_table[(size_t)seq * a.max_pages + pidx];
-            in_page = tok % a.page_size;
-          }
-          if (page < 0 || page >= a.pool_pages) {
-            set_error(a.err, ERR_BOUNDS);
-            page = 0;
-          }
-          // rows of the 2-D view: ((page*2 + kv)*HK + head)*page_size + offset
-          const int krow = ((page * 2 + 0) * a.hk + kvh) * a.page_size + in_page;
-          const int vrow = ((page * 2 + 1) * a.hk + kvh) * a.page_size + in_page;
-#pragma unroll
-          for (int cb = 0; cb < D / 64; ++cb) {
-            tma_load_2d(sk + cb * (TK * 128) + b * box_rows * 128, kv_map, cb * 64, krow,
-                        &full_bar[stage]);
-            tma_load_2d(sv + cb * (TK * 128) + b * box_rows * 128, kv_map, cb * 64, vrow,
-                        &full_bar[stage]);
-          }
-        }
+        raw_tile((tile_lo + t) * TK, stages + stage * Cfg::kStageBytes, &full_bar[stage]);
         if (++stage == kStages) { stage = 0; phase ^= 1; }
       }
     }
@@ -266,12 +329,15 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
       }
       const uint32_t sk = smem_u32(stages + stage * Cfg::kStageBytes);
       const uint32_t sv = sk + Cfg::kTileBytes;
-      const int tok0 = (tile_lo + t) * TK;
+      const bool pooled = POOL && tile_lo + t < pooled_tiles;      // tok0 then counts blocks
+      const int tok0 = (POOL && !pooled ? tile_lo + t - pooled_tiles + tile_first : tile_lo + t) * TK;
       const int wtok = PREFILL ? 0 : warp * 16;   // this warp's token offset inside the tile
       // a whole tile above the causal limit of this warp's rows contributes nothing
       const int warp_max_pos = L - R + tok_lo + min(valid_rows - 1, qrow_base + 15) / G;
       bool skip = PREFILL && (tok0 > warp_max_pos || qrow_base >= valid_rows);
-      if constexpr (WIN)      // nor does one below the window of all of them
+      if (pooled)
+        skip = PREFILL && (tok0 >= pooled_seen(warp_max_pos, a.win) || qrow_base >= valid_rows);
+      else if constexpr (WIN)      // nor does one below the window of all of them
         skip = skip || tok0 + TK - 1 <= L - R + tok_lo + qrow_base / G - a.win.size;
       if (!skip) {
         // ---- S = Q K^T ----
@@ -295,10 +361,18 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
         }
         // ---- mask + online softmax (base-2) ----
         float mxA = -INFINITY, mxB = -INFINITY;
+        // (POOL) this thread's rows see columns loX .. hiX - 1 of the tile's numbering
+        const int loA = POOL && !pooled ? posA - a.win.size + 1 : 0, loB = POOL && !pooled ? posB - a.win.size + 1 : 0;
+        const int hiA = pooled ? pooled_seen(posA, a.win) : posA + 1, hiB = pooled ? pooled_seen(posB, a.win) : posB + 1;
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
           const int j = tok0 + wtok + n * 8 + 2 * (lane & 3);
-          if constexpr (WIN) {
+          if constexpr (POOL) {
+            s[n][0] = (j >= loA && j < hiA) ? s[n][0] * a.scale_log2 : -INFINITY;
+            s[n][1] = (j + 1 >= loA && j + 1 < hiA) ? s[n][1] * a.scale_log2 : -INFINITY;
+            s[n][2] = (j >= loB && j < hiB) ? s[n][2] * a.scale_log2 : -INFINITY;
+            s[n][3] = (j + 1 >= loB && j + 1 < hiB) ? s[n][3] * a.scale_log2 : -INFINITY;
+          } else if constexpr (WIN) {
             s[n][0] = (j <= posA && j > posA - a.win.size) ? capped_score(s[n][0], a.win) : -INFINITY;
             s[n][1] = (j + 1 <= posA && j + 1 > posA - a.win.size) ? capped_score(s[n][1], a.win) : -INFINITY;
             s[n][2] = (j <= posB && j > posB - a.win.size) ? capped_score(s[n][2], a.win) : -INFINITY;
@@ -402,7 +476,7 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
       const int tk = row0_tok + tok_lo + r / G, head = kvh * G + r % G;
       if (split_total == 1) {
         float v;
-        if constexpr (FORM != kAttnPlain) v = acc * sink_factor(m, l, sink_of(a.win, head), a.win.out_scale);
+        if constexpr (FORM == kAttnWindow || FORM == kAttnSink) v = acc * sink_factor(m, l, sink_of(a.win, head), a.win.out_scale);
         else v = l > 0.f ? acc / l : 0.f;
         if constexpr (FORM == kAttnSink)
           if (a.win.gate) v *= gate_factor(__bfloat162float(a.win.gate[(size_t)tk * a.win.gate_stride + (size_t)head * D + c]));
@@ -419,7 +493,7 @@ KERN_DEVICE void attn_body(const CUtensorMap* kv_map, const AttnArgs& a, const i
   } else if (warp < 4) {
     const int rA = warp * 16 + (lane >> 2), rB = rA + 8;
     float iA = l_run[0] > 0.f ? 1.f / l_run[0] : 0.f, iB = l_run[1] > 0.f ? 1.f / l_run[1] : 0.f;
-    if constexpr (FORM != kAttnPlain) {
+    if constexpr (FORM == kAttnWindow || FORM == kAttnSink) {
       if (rA < valid_rows) iA = sink_factor(m_run[0], l_run[0], sink_of(a.win, kvh * G + rA % G), a.win.out_scale);
       if (rB < valid_rows) iB = sink_factor(m_run[1], l_run[1], sink_of(a.win, kvh * G + rB % G), a.win.out_scale);
     }

@@ -102,27 +102,48 @@ extern "C" __global__ void __launch_bounds__(128)
   pdl_launch_dependents();
 }
 
-// cos/sin tables [max_pos][rot/2] in f32, angles evaluated in double so large positions stay exact.
-KERN_DEVICE void rope_table(float* cos_tab, float* sin_tab, int max_pos, int rot, double theta, double factor) {
+// cos/sin tables [max_pos][rot/2] in f32, angles evaluated in double so large positions stay exact. `freq(j, f)` scales the
+// plain frequency f = theta^(-2j / rot) of pair j; both tables are multiplied by `size`.
+template <typename F>
+KERN_DEVICE void rope_table(float* cos_tab, float* sin_tab, int max_pos, int rot, double theta, double size, F freq) {
   const int half = rot >> 1;
   const long long n = (long long)max_pos * half;
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n;
        i += (long long)gridDim.x * blockDim.x) {
     const int j = (int)(i % half);
     const long long p = i / half;
-    const double inv_freq = pow(theta, -2.0 * (double)j / (double)rot) / factor;
     double s, c;
-    sincos((double)p * inv_freq, &s, &c);
-    cos_tab[i] = (float)c;
-    sin_tab[i] = (float)s;
+    sincos((double)p * freq(j, pow(theta, -2.0 * (double)j / (double)rot)), &s, &c);
+    cos_tab[i] = (float)(c * size);
+    sin_tab[i] = (float)(s * size);
   }
 }
 extern "C" __global__ void kern_rope_table_f32(float* cos_tab, float* sin_tab, int max_pos, int rot,
                                                double theta) {
-  rope_table(cos_tab, sin_tab, max_pos, rot, theta, 1.0);
+  rope_table(cos_tab, sin_tab, max_pos, rot, theta, 1.0, [](int, double f) { return f; });
 }
 // linear scaling: every frequency divided by `factor`
 extern "C" __global__ void kern_rope_table_scaled_f32(float* cos_tab, float* sin_tab, int max_pos, int rot,
                                                       double theta, double factor) {
-  rope_table(cos_tab, sin_tab, max_pos, rot, theta, factor);
+  rope_table(cos_tab, sin_tab, max_pos, rot, theta, 1.0, [=](int, double f) { return f / factor; });
+}
+// scaling in bands of wavelengths: below original / high as they are, above original / low divided by `factor`, and from one to
+// the other in between
+extern "C" __global__ void kern_rope_table_banded_f32(float* cos_tab, float* sin_tab, int max_pos, int rot, double theta,
+                                                      double factor, double low, double high, double original) {
+  rope_table(cos_tab, sin_tab, max_pos, rot, theta, 1.0, [=](int, double f) {
+    const double wave = 6.283185307179586476925286766559 / f;
+    if (wave < original / high) return f;
+    if (wave > original / low) return f / factor;
+    const double u = (original / wave - low) / (high - low);
+    return (1.0 - u) * f / factor + u * f;
+  });
+}
+// scaling along a ramp over the pairs: up to pair `lo` as they are, from pair `hi` divided by `factor`
+extern "C" __global__ void kern_rope_table_ramp_f32(float* cos_tab, float* sin_tab, int max_pos, int rot, double theta,
+                                                    double factor, double lo, double hi, double size) {
+  rope_table(cos_tab, sin_tab, max_pos, rot, theta, size, [=](int j, double f) {
+    const double u = fmin(fmax(((double)j - lo) / fmax(hi - lo, 0.001), 0.0), 1.0);
+    return f / factor * u + f * (1.0 - u);
+  });
 }

@@ -1,12 +1,13 @@
 // build: precise
 // Latent attention whose keys and values are both linear maps of one cached row per token, in the absorbed form: per head,
 // score = (W_uk^T q) . c, and the weighted sum of the rows c goes through W_uv afterwards. A row may hold rotated key columns
-// behind the latent, one part for all heads, and a sink per head may join the denominator. These kernels take any latent width
+// behind the latent, one part for all heads; then a sink per head may join the denominator, a window may end a row's reach and a
+// gate per head may multiply its result. These kernels take any latent width
 // and either activation type; mla_decode.cu holds the tensor-core form.
 //   kern_latent_append_<act>   RMS norm of a token's latent, written to its row of the paged cache
 //   kern_latent_prep_<act>     the same with the rotated columns behind it, and the RMS norm of a low-rank query row
 //   kern_latent_attn_<act>     one (row, head) per block: softmax over the row's causal reach, f32 throughout
-//   kern_latent_rot_attn_<act> the same with rotated columns (turning the query's) and a sink
+//   kern_latent_rot_attn_<act> the same with rotated columns (turning the query's), a sink, a window, a gate
 #include "act.cuh"
 
 using namespace kern;
@@ -38,12 +39,12 @@ KERN_DEVICE void append_body(const T* lat, uint8_t* cache, const long long* slot
 }
 
 // Row [query latent | latent | rot columns]: the first normed to q_low, the second normed and the third turned by the token's
-// position (pairs i, i + rot / 2) to the token's cached row. Block 256, (q_rank + rank) floats of shared memory, V columns per
+// position (pairs i, i + rot / 2, or neighbours) to the token's cached row. Block 256, (q_rank + rank) floats of shared memory, V columns per
 // thread and step.
 template <typename T, int V>
 KERN_DEVICE void prep_body(const T* rows, uint8_t* cache, T* q_low, const long long* positions, const long long* slots,
                            const float* cos_tab, const float* sin_tab, const __nv_bfloat16* w, const __nv_bfloat16* wq, int rank,
-                           int rot, int q_rank, int stride, int q_stride, int max_pos, float eps, int* err) {
+                           int rot, int halves, int q_rank, int stride, int q_stride, int max_pos, float eps, int* err) {
   extern __shared__ __align__(16) float lat_sm[];
   __shared__ float part[2][8];
   const int t = blockIdx.x, n = q_rank + rank, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -86,9 +87,10 @@ KERN_DEVICE void prep_body(const T* rows, uint8_t* cache, T* q_low, const long l
   const int half = rot >> 1;
   if (store)
     for (int i = threadIdx.x; i < half; i += 256) {
-      const float a = ldf(x + n + i), b = ldf(x + n + half + i), c = cos_tab[pos * half + i], s = sin_tab[pos * half + i];
-      stf(dst + rank + i, a * c - b * s);
-      stf(dst + rank + half + i, b * c + a * s);
+      const int lo = halves ? i : 2 * i, hi = halves ? half + i : 2 * i + 1;
+      const float a = ldf(x + n + lo), b = ldf(x + n + hi), c = cos_tab[pos * half + i], s = sin_tab[pos * half + i];
+      stf(dst + rank + lo, a * c - b * s);
+      stf(dst + rank + hi, b * c + a * s);
     }
 }
 
@@ -99,6 +101,9 @@ struct RotArgs {      // as LatentExtra in mla_decode.cu
   const float* cos_tab = nullptr;
   const float* sin_tab = nullptr;
   const __nv_bfloat16* sink = nullptr;
+  int halves = 1, window = 0x7fffffff;
+  const T* gate = nullptr;
+  int gate_stride = 0;
 };
 
 // Four warps walk the keys (key j belongs to warp j % 4); a lane holds the columns i * 32 + lane of the query and of the
@@ -122,9 +127,10 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
     const int half = ex.rot >> 1, pos = min(L, ex.max_pos) - 1;
     const T* x = ex.q_rot + (size_t)r * ex.stride + (size_t)h * ex.rot;
     for (int i = threadIdx.x; i < half; i += 128) {
-      const float a = ldf(x + i), b = ldf(x + half + i), c = ex.cos_tab[(size_t)pos * half + i], s = ex.sin_tab[(size_t)pos * half + i];
-      turned[i] = a * c - b * s;
-      turned[half + i] = b * c + a * s;
+      const int lo = ex.halves ? i : 2 * i, hi = ex.halves ? half + i : 2 * i + 1;
+      const float a = ldf(x + lo), b = ldf(x + hi), c = ex.cos_tab[(size_t)pos * half + i], s = ex.sin_tab[(size_t)pos * half + i];
+      turned[lo] = a * c - b * s;
+      turned[hi] = b * c + a * s;
     }
     __syncthreads();
   }
@@ -136,7 +142,7 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
     o[i] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  for (int j = warp; j < L; j += 4) {
+  for (int j = (ROT ? max(0, L - ex.window) : 0) + warp; j < L; j += 4) {
     const int pi = j / page;
     if (pi >= max_pages) break;
     const T* row = rows + ((size_t)pages[pi] * page + j % page) * cols;
@@ -166,8 +172,9 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
     if (i * 32 + lane < rank) acc[warp * rank + i * 32 + lane] = o[i];
   __syncthreads();
   float mx = fmaxf(fmaxf(ms[0], ms[1]), fmaxf(ms[2], ms[3]));
-  float f[4], den = 0.f;
+  float f[4], den = 0.f, den_gate = 1.f;
   if constexpr (ROT) {
+    if (ex.gate) den_gate = 1.f + expf(-ldf(ex.gate + (size_t)r * ex.gate_stride + h));
     if (ex.sink) {
       const float sk = __bfloat162float(ex.sink[h]);
       mx = fmaxf(mx, sk);
@@ -180,7 +187,7 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
     float v = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) v += f[w] * acc[w * rank + c];
-    stf(out + ((size_t)r * heads + h) * rank + c, v / den);
+    stf(out + ((size_t)r * heads + h) * rank + c, v / (den * den_gate));
   }
 }
 
@@ -200,9 +207,10 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
       kern_latent_rot_attn_##SFX##_w##W(const T* q, const uint8_t* cache, T* out, const int* table, const int* lens,      \
                                         const int* row_seq, int heads, int rank, int max_pages, int page, float scale,    \
                                         int* err, const T* q_rot, const float* cos_tab, const float* sin_tab,             \
-                                        const __nv_bfloat16* sink, int rot_stride, int rot, int max_pos) {                \
+                                        const __nv_bfloat16* sink, const T* gate, int rot_stride, int rot, int max_pos,   \
+                                        int halves, int window, int gate_stride) {                                        \
     pdl_wait();                                                                                                           \
-    const RotArgs<T> ex{q_rot, rot_stride, rot, max_pos, cos_tab, sin_tab, sink};                                         \
+    const RotArgs<T> ex{q_rot, rot_stride, rot, max_pos, cos_tab, sin_tab, sink, halves, window, gate, gate_stride};      \
     attn_body<T, W / 32, true>(q, cache, out, table, lens, row_seq, heads, rank, max_pages, page, scale, err, ex);        \
   }
 #define LATENT_ENTRIES(T, SFX)                                                                                            \
@@ -215,16 +223,17 @@ KERN_DEVICE void attn_body(const T* q, const uint8_t* cache, T* out, const int* 
   extern "C" __global__ void __launch_bounds__(256)                                                                       \
       kern_latent_prep_##SFX(const T* rows, uint8_t* cache, T* q_low, const long long* positions, const long long* slots, \
                              const float* cos_tab, const float* sin_tab, const __nv_bfloat16* w, const __nv_bfloat16* wq, \
-                             int rank, int rot, int q_rank, int stride, int q_stride, int max_pos, float eps, int* err) { \
+                             int rank, int rot, int halves, int q_rank, int stride, int q_stride, int max_pos, float eps, \
+                             int* err) {                                                                                  \
     pdl_wait();                                                                                                           \
     const bool vec = (rank | rot | q_rank | stride | q_stride) % 4 == 0 &&                                                \
                      ((reinterpret_cast<uintptr_t>(rows) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(q_low) | \
                        reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(wq)) & 15) == 0;                      \
     if (vec)                                                                                                              \
-      prep_body<T, 4>(rows, cache, q_low, positions, slots, cos_tab, sin_tab, w, wq, rank, rot, q_rank, stride, q_stride, \
+      prep_body<T, 4>(rows, cache, q_low, positions, slots, cos_tab, sin_tab, w, wq, rank, rot, halves, q_rank, stride, q_stride, \
                       max_pos, eps, err);                                                                                 \
     else                                                                                                                  \
-      prep_body<T, 1>(rows, cache, q_low, positions, slots, cos_tab, sin_tab, w, wq, rank, rot, q_rank, stride, q_stride, \
+      prep_body<T, 1>(rows, cache, q_low, positions, slots, cos_tab, sin_tab, w, wq, rank, rot, halves, q_rank, stride, q_stride, \
                       max_pos, eps, err);                                                                                 \
     pdl_launch_dependents();                                                                                              \
   }                                                                                                                       \

@@ -31,14 +31,19 @@ constexpr int HM = 16;                   // heads per CTA
 constexpr int kPStride = TKM + 8, kPBytes = HM * kPStride * 2;
 constexpr int DQK = 576;                 // row of the 512 + 64 form
 
-// What a mixer with a rotated part and a sink adds: a head's rotated query columns are in a row of their own, not yet turned
-// (pairs i, i + rot / 2; a row's position is its length - 1), and `sink` (one per head) joins the denominator once, unscaled.
+// What a mixer with a rotated part adds: a head's rotated query columns are in a row of their own, not yet turned (pairs i,
+// i + rot / 2, or neighbours; a row's position is its length - 1). Where there are such, `sink` (one per head) joins the
+// denominator once, unscaled, a row sees the last `window` positions only, and sigmoid of `gate` (a column per head) multiplies
+// its heads' results.
 struct LatentExtra {
   const __nv_bfloat16* q_rot = nullptr;      // [rows][stride], head h at column h * rot
   int stride = 0, rot = 0, max_pos = 0;
   const float* cos_tab = nullptr;            // [max_pos][rot / 2]
   const float* sin_tab = nullptr;
   const __nv_bfloat16* sink = nullptr;
+  int halves = 1, window = 0x7fffffff;
+  const __nv_bfloat16* gate = nullptr;       // [rows][gate_stride]
+  int gate_stride = 0;
 };
 constexpr float kLog2eM = 1.4426950408889634f;
 
@@ -119,7 +124,8 @@ __device__ __forceinline__ void mla_body(const CUtensorMap* lat_map, const __nv_
   const int split_total = (splits >> 16) ? (splits >> 16) : nsplit;
   if (L <= 0 || valid_rows <= 0) return;       // uniform per CTA
   if (ex.rot > 0 && L > ex.max_pos && threadIdx.x == 0) set_error(err, ERR_BOUNDS);
-  const int ntiles_all = (L + TKM - 1) / TKM;
+  const int first_key = max(0, L - ex.window), tile_first = first_key / TKM;
+  const int ntiles_all = (L + TKM - 1) / TKM - tile_first;
   int tile_lo = 0, tile_hi = ntiles_all;
   if (nsplit > 1) {
     const int per = (ntiles_all + nsplit - 1) / nsplit;
@@ -128,6 +134,7 @@ __device__ __forceinline__ void mla_body(const CUtensorMap* lat_map, const __nv_
     if (tile_hi < tile_lo) tile_hi = tile_lo;
   }
   const int ntiles = tile_hi - tile_lo;
+  tile_lo += tile_first;
 
   // the 16 query rows (one per head) -> shared
   for (int i = threadIdx.x; i < HM * (QB * 8); i += blockDim.x) {
@@ -141,11 +148,21 @@ __device__ __forceinline__ void mla_body(const CUtensorMap* lat_map, const __nv_
       const float* cs = ex.cos_tab + (size_t)pos * half;
       const float* sn = ex.sin_tab + (size_t)pos * half;
       float f[8];
+      if (ex.halves) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        const int i = c * 8 - q_cols + e, j = i < half ? i : i - half;
-        const float a = __bfloat162float(x[i]), b = __bfloat162float(x[i < half ? i + half : j]);
-        f[e] = i < half ? a * cs[j] - b * sn[j] : a * cs[j] + b * sn[j];
+        for (int e = 0; e < 8; ++e) {
+          const int i = c * 8 - q_cols + e, j = i < half ? i : i - half;
+          const float a = __bfloat162float(x[i]), b = __bfloat162float(x[i < half ? i + half : j]);
+          f[e] = i < half ? a * cs[j] - b * sn[j] : a * cs[j] + b * sn[j];
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; e += 2) {
+          const int i = c * 8 - q_cols + e, j = i >> 1;
+          const float a = __bfloat162float(x[i]), b = __bfloat162float(x[i + 1]);
+          f[e] = a * cs[j] - b * sn[j];
+          f[e + 1] = b * cs[j] + a * sn[j];
+        }
       }
       v = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
     }
@@ -237,10 +254,11 @@ __device__ __forceinline__ void mla_body(const CUtensorMap* lat_map, const __nv_
 #pragma unroll
       for (int n = 0; n < 1; ++n) {
         const int j = tok0 + wtok + n * 8 + 2 * (lane & 3);
-        s[n][0] = (scoring && j < L) ? s[n][0] * scale_log2 : -INFINITY;
-        s[n][1] = (scoring && j + 1 < L) ? s[n][1] * scale_log2 : -INFINITY;
-        s[n][2] = (scoring && j < L) ? s[n][2] * scale_log2 : -INFINITY;
-        s[n][3] = (scoring && j + 1 < L) ? s[n][3] * scale_log2 : -INFINITY;
+        const bool in0 = scoring && j < L && j >= first_key, in1 = scoring && j + 1 < L && j + 1 >= first_key;
+        s[n][0] = in0 ? s[n][0] * scale_log2 : -INFINITY;
+        s[n][1] = in1 ? s[n][1] * scale_log2 : -INFINITY;
+        s[n][2] = in0 ? s[n][2] * scale_log2 : -INFINITY;
+        s[n][3] = in1 ? s[n][3] * scale_log2 : -INFINITY;
         mxA = fmaxf(mxA, fmaxf(s[n][0], s[n][1]));
         mxB = fmaxf(mxB, fmaxf(s[n][2], s[n][3]));
       }
@@ -319,6 +337,11 @@ __device__ __forceinline__ void mla_body(const CUtensorMap* lat_map, const __nv_
         iA = factor(m_run[0], lA, rA);
         iB = factor(m_run[1], lB, rB);
       }
+      if (ex.gate != nullptr) {
+        const __nv_bfloat16* g = ex.gate + (size_t)seq * ex.gate_stride + head0;
+        if (rA < valid_rows) iA /= 1.f + __expf(-__bfloat162float(g[rA]));
+        if (rB < valid_rows) iB /= 1.f + __expf(-__bfloat162float(g[rB]));
+      }
 #pragma unroll
       for (int i = 0; i < ON; ++i) {
         const int c = warp * (ON * 8) + i * 8 + 2 * (lane & 3);
@@ -385,8 +408,8 @@ KERN_LATENT_DECODE(8)
           float* ws_ml, const int* block_table, const int* seq_lens, int seqs, int heads, int q_stride, int out_stride,      \
           int max_pages, int page_size, int splits, int pool_pages, float scale_log2, int* err, const int* row_seq,          \
           int rank, const __nv_bfloat16* q_rot, const float* cos_tab, const float* sin_tab, const __nv_bfloat16* sink,       \
-          int rot_stride, int rot, int max_pos) {                                                                            \
-    const LatentExtra ex{q_rot, rot_stride, rot, max_pos, cos_tab, sin_tab, sink};                                           \
+          const __nv_bfloat16* gate, int rot_stride, int rot, int max_pos, int halves, int window, int gate_stride) {        \
+    const LatentExtra ex{q_rot, rot_stride, rot, max_pos, cos_tab, sin_tab, sink, halves, window, gate, gate_stride};        \
     mla_body<Q, B>(&lat_map, q, out, ws_o, ws_ml, block_table, seq_lens, seqs, heads, q_stride, out_stride, max_pages,       \
                    page_size, splits, pool_pages, scale_log2, err, row_seq, rank, rank, ex);                                 \
   }

@@ -3,6 +3,7 @@
 //   kern_moe_route_f32      router scores -> top-k expert ids and weights per token (sigmoid or softmax scoring,
 //                           optional selection bias, renormalise, scale)
 //   kern_moe_route_logits   the same by the logits plus a bias: top-k largest, softmax over the chosen
+//   kern_moe_route_table    the experts of every token id, read from a table, all with one weight
 //   kern_moe_route_groups   sigmoid or softmax scores, choices inside the best groups of neighbouring experts
 //   kern_moe_plan           counts per expert -> row offsets, the permuted row of every (token, choice), and the
 //                           M-tile table the grouped GEMM walks; experts outside [e_lo, e_hi) belong to another rank
@@ -87,6 +88,22 @@ extern "C" __global__ void __launch_bounds__(128)
     topk_ids[(size_t)t * k + lane] = my_id;
     topk_w[(size_t)t * k + lane] = w * scale;
   }
+}
+
+// No router: row `token` of the table [vocab][k] names the token's experts; each weighs 1 / k. grid = ceil(tokens k / 256).
+extern "C" __global__ void __launch_bounds__(256)
+    kern_moe_route_table(const long long* ids, const int* table, int* topk_ids, float* topk_w, int tokens, int experts, int k,
+                         int vocab, int* err) {
+  pdl_wait();
+  const int i = blockIdx.x * 256 + threadIdx.x;
+  if (i < tokens * k) {
+    const long long id = ids[i / k];
+    const int e = id >= 0 && id < vocab ? table[(size_t)id * k + i % k] : -1;
+    if (e < 0 || e >= experts) set_error(err, ERR_BOUNDS);
+    topk_ids[i] = e;
+    topk_w[i] = 1.f / (float)k;
+  }
+  pdl_launch_dependents();
 }
 
 // Routing on the logits themselves: z = logits + bias (bf16, one per expert, may be null), the k largest are chosen (ties:

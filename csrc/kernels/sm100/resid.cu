@@ -2,12 +2,15 @@
 // The residual of a decoder that norms a sublayer's result before adding it as well as the next sublayer's input:
 //     x <- x + rms(y) w_post;   xn = rms(x) w_next
 // x is f32 (one row per token), y the sublayer's result: a row of a plain buffer, or the weighted sum of a token's k
-// expert rows, summed here. Without `w_post` y is added as it is.
+// expert rows, summed here. Without `w_post` y is added as it is. A gated result is first multiplied, element by element, by
+// sigmoid(gate + gate_b). Where the next sublayer reads its input plus a short convolution of it over time, one row per sequence
+// (decode) is convolved here too (prompts: conv_add.cu).
 // or, in a decoder that only scales a sublayer's result, element by element:
 //     x <- x + s (y + bias + w_id h + sigmoid(gate) shared);   xn = rms(x) w_next
 // where h is the sublayer's own input, w_id the weight of the experts that hand it back, and `shared` an expert for every token.
-// kern_resid_embed  token row into x, and the first sublayer's normed input
-// kern_resid_scale  the second form; kern_resid_mix the first; with `hidden` the sum goes there instead and nothing is normed (the last sublayer)
+// kern_resid_embed  token row, times a factor, into x, and the first sublayer's normed input; kern_resid_embed_conv also convolves it
+// kern_resid_scale  the second form; kern_resid_mix the first, kern_resid_gate the first with a gate, kern_resid_gate_conv that and
+// the next input convolved; with `hidden` the sum goes there instead and nothing is normed (the last sublayer)
 // Residual, sums and norms are f32; activations are T (bf16, or f32 in the 32-bit form of a model).
 #include "act.cuh"
 
@@ -41,9 +44,74 @@ KERN_DEVICE void norm_out(const float* u, float inv, const __nv_bfloat16* w, T* 
   }
 }
 
+// out = h + conv(h) of one row per sequence, conv_t = sum_j w[c][j] h_(t - taps + 1 + j). `state` holds lines of the last
+// taps - 1 rows, which move on by one; line 0 is nobody's (zeros, and nothing is kept).
+template <typename T>
+struct ConvStep {
+  const __nv_bfloat16* w = nullptr;
+  T* out = nullptr;
+  uint8_t* state = nullptr;
+  const int* lines = nullptr;
+  int taps = 0;
+  long long line_bytes = 0;
+};
+
+// columns i .. of row t; h as the activations' type holds it
 template <typename T, int V>
+KERN_DEVICE void conv_step(const ConvStep<T>& cv, int line, int t, int i, const Vec<V>& h, int width) {
+  const int keep = cv.taps - 1;
+  T* win = reinterpret_cast<T*>(cv.state + (size_t)line * cv.line_bytes) + i;
+  const __nv_bfloat16* w = cv.w + (size_t)i * cv.taps;
+  Vec<V> acc = h;
+#pragma unroll
+  for (int e = 0; e < V; ++e) acc.v[e] += __bfloat162float(w[e * cv.taps + keep]) * h.v[e];
+  if (line > 0) {
+    Vec<V> past[3];      // the usual few taps: all rows in flight at once
+    const int few = min(keep, 3);
+#pragma unroll
+    for (int j = 0; j < 3; ++j)
+      if (j < few) past[j] = ldv<V>(win + (size_t)j * width);
+#pragma unroll
+    for (int j = 0; j < 3; ++j) {
+      if (j >= few) continue;
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc.v[e] += __bfloat162float(w[e * cv.taps + j]) * past[j].v[e];
+      if (j > 0) stv<V>(win + (size_t)(j - 1) * width, past[j]);
+    }
+    for (int j = 3; j < keep; ++j) {
+      const Vec<V> v = ldv<V>(win + (size_t)j * width);
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc.v[e] += __bfloat162float(w[e * cv.taps + j]) * v.v[e];
+      stv<V>(win + (size_t)(j - 1) * width, v);
+    }
+    if (keep > 0) stv<V>(win + (size_t)(keep - 1) * width, h);
+  }
+  stv<V>(cv.out + (size_t)t * width + i, acc);
+}
+
+// As norm_out, and the row's convolution
+template <typename T, int V>
+KERN_DEVICE void norm_conv_out(const float* u, float inv, const __nv_bfloat16* w, T* xn, const ConvStep<T>& cv, int width) {
+  const int t = blockIdx.x;
+  int line = cv.lines[t];
+  if (line <= 0 || !KERN_CHECK(cv.state + (size_t)line * cv.line_bytes, (size_t)cv.line_bytes, SITE_STATE_SLOT)) line = 0;
+  for (int i = threadIdx.x * V; i < width; i += 256 * V) {
+    const Vec<V> a = ldv<V>(u + i), b = ldv<V>(w + i);
+    T held[V];
+    Vec<V> o;
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      stf(held + e, a.v[e] * inv * b.v[e]);
+      o.v[e] = ldf(held + e);
+    }
+    stv<V>(xn + i, o);
+    conv_step<T, V>(cv, line, t, i, o, width);
+  }
+}
+
+template <typename T, int V, bool CONV>
 KERN_DEVICE void embed_body(const long long* ids, const __nv_bfloat16* table, const __nv_bfloat16* w_norm, float* x, T* xn,
-                            int width, int vocab, float eps, int* err) {
+                            int width, int vocab, float scale, float eps, int* err, const ConvStep<T>& cv) {
   extern __shared__ __align__(16) float resid_sm[];
   const int t = blockIdx.x;
   long long id = ids[t];
@@ -58,16 +126,22 @@ KERN_DEVICE void embed_body(const long long* ids, const __nv_bfloat16* table, co
     Vec<V> v = {};
     if (ok) v = ldv<V>(a + i);
 #pragma unroll
-    for (int j = 0; j < V; ++j) ss += v.v[j] * v.v[j];
+    for (int j = 0; j < V; ++j) {
+      v.v[j] *= scale;
+      ss += v.v[j] * v.v[j];
+    }
     stv<V>(x + (size_t)t * width + i, v);
     stv<V>(resid_sm + i, v);
   }
-  norm_out<T, V>(resid_sm, inv_rms(ss, width, eps), w_norm, xn + (size_t)t * width, width);
+  const float inv = inv_rms(ss, width, eps);
+  if constexpr (CONV) norm_conv_out<T, V>(resid_sm, inv, w_norm, xn + (size_t)t * width, cv, width);
+  else norm_out<T, V>(resid_sm, inv, w_norm, xn + (size_t)t * width, width);
 }
 
-template <typename T, int V>
-KERN_DEVICE void mix_body(float* x, const T* y, const int* perm, const float* topw, const __nv_bfloat16* w_post,
-                          const __nv_bfloat16* w_next, T* xn, float* hidden, int width, int k, float eps) {
+template <typename T, int V, bool GATED, bool CONV>
+KERN_DEVICE void mix_body(float* x, const T* y, const int* perm, const float* topw, const T* gate, const __nv_bfloat16* gate_b,
+                          const __nv_bfloat16* w_post, const __nv_bfloat16* w_next, T* xn, float* hidden, int width, int k,
+                          float eps, const ConvStep<T>& cv) {
   extern __shared__ __align__(16) float resid_sm[];
   __shared__ float tw[32];
   __shared__ int tr[32];
@@ -94,6 +168,11 @@ KERN_DEVICE void mix_body(float* x, const T* y, const int* perm, const float* to
     } else {
       v = ldv<V>(y + (size_t)t * width + i);
     }
+    if constexpr (GATED) {
+      const Vec<V> g = ldv<V>(gate + (size_t)t * width + i), b = ldv<V>(gate_b + i);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v.v[e] /= 1.f + expf(-(g.v[e] + b.v[e]));
+    }
 #pragma unroll
     for (int e = 0; e < V; ++e) ss += v.v[e] * v.v[e];
     stv<V>(resid_sm + i, v);
@@ -117,7 +196,10 @@ KERN_DEVICE void mix_body(float* x, const T* y, const int* perm, const float* to
       stv<V>(resid_sm + i, s);
     }
   }
-  if (!hidden) norm_out<T, V>(resid_sm, inv_rms(ss, width, eps), w_next, xn + (size_t)t * width, width);
+  if (hidden) return;
+  const float next = inv_rms(ss, width, eps);
+  if constexpr (CONV) norm_conv_out<T, V>(resid_sm, next, w_next, xn + (size_t)t * width, cv, width);
+  else norm_out<T, V>(resid_sm, next, w_next, xn + (size_t)t * width, width);
 }
 
 // V values as they lie in memory: what waits for its turn takes no more registers than that
@@ -204,22 +286,47 @@ KERN_DEVICE void scale_body(float* x, const T* y, const int* perm, const float* 
 }  // namespace
 
 // grid = rows, block 256, `width` floats of shared memory
+#define RESID_WIDTHS(call4, call1)                                                                                        \
+  pdl_wait();                                                                                                             \
+  if (width % 4 == 0) call4; else call1;                                                                                  \
+  pdl_launch_dependents();
 #define RESID_ENTRIES(T, SFX)                                                                                             \
   extern "C" __global__ void __launch_bounds__(256)                                                                       \
       kern_resid_embed_##SFX(const long long* ids, const __nv_bfloat16* table, const __nv_bfloat16* w_norm, float* x,     \
-                             T* xn, int width, int vocab, float eps, int* err) {                                          \
-    pdl_wait();                                                                                                           \
-    if (width % 4 == 0) embed_body<T, 4>(ids, table, w_norm, x, xn, width, vocab, eps, err);                              \
-    else embed_body<T, 1>(ids, table, w_norm, x, xn, width, vocab, eps, err);                                             \
-    pdl_launch_dependents();                                                                                              \
+                             T* xn, int width, int vocab, float scale, float eps, int* err) {                             \
+    RESID_WIDTHS((embed_body<T, 4, false>(ids, table, w_norm, x, xn, width, vocab, scale, eps, err, {})),                 \
+                 (embed_body<T, 1, false>(ids, table, w_norm, x, xn, width, vocab, scale, eps, err, {})))                 \
+  }                                                                                                                       \
+  extern "C" __global__ void __launch_bounds__(256)                                                                       \
+      kern_resid_embed_conv_##SFX(const long long* ids, const __nv_bfloat16* table, const __nv_bfloat16* w_norm,          \
+                                  float* x, T* xn, int width, int vocab, float scale, float eps, int* err,                \
+                                  const __nv_bfloat16* conv_w, T* conv_out, uint8_t* state, const int* lines, int taps,   \
+                                  long long line_bytes) {                                                                 \
+    const ConvStep<T> cv{conv_w, conv_out, state, lines, taps, line_bytes};                                               \
+    RESID_WIDTHS((embed_body<T, 4, true>(ids, table, w_norm, x, xn, width, vocab, scale, eps, err, cv)),                  \
+                 (embed_body<T, 1, true>(ids, table, w_norm, x, xn, width, vocab, scale, eps, err, cv)))                  \
   }                                                                                                                       \
   extern "C" __global__ void __launch_bounds__(256)                                                                       \
       kern_resid_mix_##SFX(float* x, const T* y, const int* perm, const float* topw, const __nv_bfloat16* w_post,         \
                            const __nv_bfloat16* w_next, T* xn, float* hidden, int width, int k, float eps) {              \
-    pdl_wait();                                                                                                           \
-    if (width % 4 == 0) mix_body<T, 4>(x, y, perm, topw, w_post, w_next, xn, hidden, width, k, eps);                      \
-    else mix_body<T, 1>(x, y, perm, topw, w_post, w_next, xn, hidden, width, k, eps);                                     \
-    pdl_launch_dependents();                                                                                              \
+    RESID_WIDTHS((mix_body<T, 4, false, false>(x, y, perm, topw, nullptr, nullptr, w_post, w_next, xn, hidden, width, k, eps, {})), \
+                 (mix_body<T, 1, false, false>(x, y, perm, topw, nullptr, nullptr, w_post, w_next, xn, hidden, width, k, eps, {}))) \
+  }                                                                                                                       \
+  extern "C" __global__ void __launch_bounds__(256)                                                                       \
+      kern_resid_gate_##SFX(float* x, const T* y, const int* perm, const float* topw, const __nv_bfloat16* w_post,        \
+                            const __nv_bfloat16* w_next, T* xn, float* hidden, int width, int k, float eps,               \
+                            const T* gate, const __nv_bfloat16* gate_b) {                                                 \
+    RESID_WIDTHS((mix_body<T, 4, true, false>(x, y, perm, topw, gate, gate_b, w_post, w_next, xn, hidden, width, k, eps, {})), \
+                 (mix_body<T, 1, true, false>(x, y, perm, topw, gate, gate_b, w_post, w_next, xn, hidden, width, k, eps, {}))) \
+  }                                                                                                                       \
+  extern "C" __global__ void __launch_bounds__(256)                                                                       \
+      kern_resid_gate_conv_##SFX(float* x, const T* y, const int* perm, const float* topw, const __nv_bfloat16* w_post,   \
+                                 const __nv_bfloat16* w_next, T* xn, int width, int k, float eps, const T* gate,          \
+                                 const __nv_bfloat16* gate_b, const __nv_bfloat16* conv_w, T* conv_out, uint8_t* state,   \
+                                 const int* lines, int taps, long long line_bytes) {                                      \
+    const ConvStep<T> cv{conv_w, conv_out, state, lines, taps, line_bytes};                                               \
+    RESID_WIDTHS((mix_body<T, 4, true, true>(x, y, perm, topw, gate, gate_b, w_post, w_next, xn, nullptr, width, k, eps, cv)), \
+                 (mix_body<T, 1, true, true>(x, y, perm, topw, gate, gate_b, w_post, w_next, xn, nullptr, width, k, eps, cv))) \
   }
 
 RESID_ENTRIES(__nv_bfloat16, bf16)

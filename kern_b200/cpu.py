@@ -232,14 +232,29 @@ def k_sample(g, logits, probs, out, temperature, top_k, top_p, min_p, seeds, off
     out[:r] = sample_rows(lv, temperature[:r], top_k[:r], top_p[:r], min_p[:r], seeds[:r], offsets[:r])
 
 
-def k_rope_table(g, cos, sin, max_pos, rot, theta_bits, factor_bits=None):
-    factor_bits = struct.unpack("<q", struct.pack("<d", 1.0))[0] if factor_bits is None else factor_bits
-    theta, factor = (struct.unpack("<d", struct.pack("<q", b))[0] for b in (theta_bits, factor_bits))
-    half = rot // 2
-    inv = theta ** (-torch.arange(0, half, dtype=torch.float64) * 2.0 / rot) / factor
-    ang = torch.arange(max_pos, dtype=torch.float64)[:, None] * inv[None]
-    cos.view(-1)[: max_pos * half] = ang.cos().float().reshape(-1)
-    sin.view(-1)[: max_pos * half] = ang.sin().float().reshape(-1)
+def _rope_table(scaled):
+    """`scaled(pairs, frequencies, *constants)` -> frequencies, and what both tables are multiplied by."""
+    def run(g, cos, sin, max_pos, rot, *bits):
+        theta, *constants = (struct.unpack("<d", struct.pack("<q", b))[0] for b in bits)
+        half = rot // 2
+        pairs = torch.arange(0, half, dtype=torch.float64)
+        inv, size = scaled(pairs, theta ** (-pairs * 2.0 / rot), *constants)
+        ang = torch.arange(max_pos, dtype=torch.float64)[:, None] * inv[None]
+        cos.view(-1)[: max_pos * half] = (ang.cos() * size).float().reshape(-1)
+        sin.view(-1)[: max_pos * half] = (ang.sin() * size).float().reshape(-1)
+    return run
+
+
+def _rope_banded(pairs, f, factor, low, high, original):
+    wave = 2 * math.pi / f
+    u = (original / wave - low) / (high - low)
+    between = (1 - u) * f / factor + u * f
+    return torch.where(wave < original / high, f, torch.where(wave > original / low, f / factor, between)), 1.0
+
+
+def _rope_ramp(pairs, f, factor, lo, hi, size):
+    u = ((pairs - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+    return f / factor * u + f * (1 - u), size
 
 
 def k_silu_mul(g, x, out, tokens, d):
@@ -401,7 +416,9 @@ CPU_KERNELS = {
     "kern_embedding_i64_bf16": k_embedding, "kern_embedding_i32_bf16": k_embedding,
     "kern_rms_norm_bf16": k_rms_norm, "kern_rms_norm_wide_bf16": k_rms_norm,
     "kern_fused_add_rms_norm_bf16": k_fused_add_rms_norm,
-    "kern_rope_kv_append_bf16": k_rope_append, "kern_rope_table_f32": k_rope_table, "kern_rope_table_scaled_f32": k_rope_table,
+    "kern_rope_kv_append_bf16": k_rope_append, "kern_rope_table_f32": _rope_table(lambda pairs, f: (f, 1.0)),
+    "kern_rope_table_scaled_f32": _rope_table(lambda pairs, f, factor: (f / factor, 1.0)),
+    "kern_rope_table_banded_f32": _rope_table(_rope_banded), "kern_rope_table_ramp_f32": _rope_table(_rope_ramp),
     "kern_attn_plan": k_attn_plan, "kern_attn_merge_splits": k_noop,
     "kern_last_row": k_last_row, "kern_argmax_partial_bf16": k_argmax_partial, "kern_argmax_partial_f32": k_argmax_partial,
     "kern_argmax_final_i64": k_argmax_final, "kern_sample_bf16": k_sample, "kern_sample_f32": k_sample,

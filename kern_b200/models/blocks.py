@@ -279,10 +279,10 @@ def latent_attn_op(heads: int, rank: int, scale: float, page_size: int, table_wi
                                {"f32": scale}, P(5)], shared_mem=(4 * rank + 8) * 4))
 
 
-# ---- latent attention with a rotated part and a sink ------------------------------------------------------------
-def latent_prep_op(rank: int, rot: int, q_rank: int, stride: int, q_stride: int, max_pos: int, eps: float, act: str = "bf16") -> dict:
+# ---- latent attention with a rotated part: sinks, windows, gates ------------------------------------------------------------
+def latent_prep_op(rank: int, rot: int, q_rank: int, stride: int, q_stride: int, max_pos: int, eps: float, act: str = "bf16", halves: bool = True) -> dict:
     """Of a projected row [query latent | latent | rotated key part]: the query latent normed into rows of its own, the latent
-    normed and the key part turned (pairs i, i + rot / 2) into a row of the paged cache.
+    normed and the key part turned (pairs i, i + rot / 2, or neighbours) into a row of the paged cache.
     Interface [rows, state, q latent, positions, slots, cos, sin, latent norm w, query norm w, err]."""
     if rot % 2 or not rot:
         raise ValueError(f"a rotated key part of {rot} columns")
@@ -290,35 +290,66 @@ def latent_prep_op(rank: int, rot: int, q_rank: int, stride: int, q_stride: int,
         raise ValueError(f"latents of {rank} and {q_rank} columns (at most 50000 together)")
     iface = [f"in buffer<{act}>", "inout state", f"out buffer<{act}>", "in buffer<i64>", "in buffer<i64>", "in buffer<f32>", "in buffer<f32>", "in buffer<bf16>",
              "in buffer<bf16>", "out buffer<i32>"]
-    return _op(iface, _launch("latent", f"kern_latent_prep_{act}", [256, 1, 1], ["tokens", 1, 1], iface[:9] + ["i32"] * 6 + ["f32", "out buffer<i32>"],
-                              [*map(P, range(9)), I(rank), I(rot), I(q_rank), I(stride), I(q_stride), I(max_pos), {"f32": eps}, P(9)], shared_mem=(rank + q_rank) * 4))
+    return _op(iface, _launch("latent", f"kern_latent_prep_{act}", [256, 1, 1], ["tokens", 1, 1], iface[:9] + ["i32"] * 7 + ["f32", "out buffer<i32>"],
+                              [*map(P, range(9)), I(rank), I(rot), I(int(halves)), I(q_rank), I(stride), I(q_stride), I(max_pos), {"f32": eps}, P(9)], shared_mem=(rank + q_rank) * 4))
 
 
 def latent_rot_attn_op(heads: int, rank: int, rot: int, scale: float, page_size: int, table_width: int, max_pos: int, rot_stride: int, ragged: bool,
-                       act: str = "bf16", seqs_max: int = 0) -> dict:
-    """`latent_attn_op` over rows with `rot` rotated key columns behind the latent, and a sink per head.
-    Interface [q, state, out, block_table, lens, err] (+ [row_seq] for ragged rows), then [q_rot, cos, sin, sink]."""
+                       act: str = "bf16", seqs_max: int = 0, *, sink: bool = True, halves: bool = True, window: int = C.I32_MAX, gate_stride: int = 0) -> dict:
+    """`latent_attn_op` over rows with `rot` rotated key columns behind the latent, with a sink per head, over the last `window`
+    positions, the result times sigmoid of a gate per head (`gate_stride`: the row stride of the gates; sinks and gates not both).
+    Interface [q, state, out, block_table, lens, err] (+ [row_seq] for ragged rows), then [q_rot, cos, sin], [sink], [gate]."""
     if act == "bf16" and tiles_fit(rank, rot) and rank <= 512 and rot <= 64 and (page_size % 64 == 0 or 64 % page_size == 0):
-        return C.mla_attn_op(heads, page_size, table_width, ragged, seqs_max=seqs_max, rank=rank, scale=scale, rot=rot, max_pos=max_pos, rot_stride=rot_stride)
+        return C.mla_attn_op(heads, page_size, table_width, ragged, seqs_max=seqs_max, rank=rank, scale=scale, rot=rot, max_pos=max_pos, rot_stride=rot_stride,
+                             sink=sink, halves=halves, window=window, gate_stride=gate_stride)
     if rank > 1024:
         raise ValueError(f"latent rows of {rank} columns (at most 1024)")
     iface = [f"in buffer<{act}>", "in state", f"out buffer<{act}>", "in buffer<i32>", "in buffer<i32>", "out buffer<i32>"]
     iface += ["in buffer<i32>"] if ragged else []
     o = len(iface)
-    iface += [f"in buffer<{act}>", "in buffer<f32>", "in buffer<f32>", "in buffer<bf16>"]
+    iface += [f"in buffer<{act}>", "in buffer<f32>", "in buffer<f32>"]
+    extra, more = C.latent_extra(iface, sink, gate_stride, act)
     w = next(n for n in (64, 128, 256, 512, 1024) if rank <= n)
     return _op(iface, _launch("latent", f"kern_latent_rot_attn_{act}_w{w}", [128, 1, 1], [heads, "tokens" if ragged else "seqs", 1],
-                              [*iface[:5], iface[6] if ragged else NULL[0], "i32", "i32", "i32", "i32", "f32", "out buffer<i32>", *iface[o:], "i32", "i32", "i32"],
+                              [*iface[:5], iface[6] if ragged else NULL[0], "i32", "i32", "i32", "i32", "f32", "out buffer<i32>", *iface[o:o + 3], *extra] + ["i32"] * 6,
                               [*map(P, range(5)), P(6) if ragged else NULL[1], I(heads), I(rank), I(table_width), I(page_size), {"f32": scale}, P(5),
-                               *map(P, range(o, o + 4)), I(rot_stride), I(rot), I(max_pos)], shared_mem=(4 * rank + 8 + rot) * 4))
+                               *map(P, range(o, o + 3)), *more, I(rot_stride), I(rot), I(max_pos), I(int(halves)), I(window), I(gate_stride)],
+                              shared_mem=(4 * rank + 8 + rot) * 4))
 
 
 # ---- a residual with norms on both sides of a sublayer -----------------------------------------------------
-def resid_embed_op(width: int, vocab: int, eps: float, act: str = "bf16") -> dict:
-    """Token row into the f32 residual, and the first sublayer's normed input. Interface [ids, table, next norm w, x, xn, err]."""
+def conv_line_bytes(width: int, taps: int, act: str = "bf16") -> int:
+    """Bytes of the state line of a convolution over a row's inputs: its last taps - 1 rows."""
+    return max(256, -(-(taps - 1) * width * ACT_BYTES[act] // 256) * 256)
+
+
+def _conv_step(conv: tuple[int, int], act: str, at: int):
+    """What a kernel that also convolves its row takes (`conv`: taps, bytes of a line): interface types, launch arguments."""
+    types = ["in buffer<bf16>", f"out buffer<{act}>", "inout state", "in buffer<i32>"]
+    return types, [(t, P(at + i)) for i, t in enumerate(types)] + [("i32", I(conv[0])), ("i64", L(conv[1]))]
+
+
+def conv_add_op(width: int, taps: int, line_bytes: int, act: str = "bf16") -> dict:
+    """Rows of a ragged call plus a causal convolution of them over time, channel by channel; the last taps - 1 rows of a sequence
+    stay in its state line. Interface [h, w, out, state, lines, cu_seqlens, seqs, rows]."""
+    iface = [f"in buffer<{act}>", "in buffer<bf16>", f"out buffer<{act}>", "inout state", "in buffer<i32>", "in buffer<i32>", "i32", "i32"]
+    conv = _launch("conv_add", f"kern_conv_add_{act}", [256, 1, 1], [{"ceil_div": ["tokens", 16]}, -(-width // (1024 if width % 4 == 0 else 256)), 1],
+                   [iface[0], iface[2], "in state", iface[4], iface[5], iface[1], "i32", "i32", "i32", "i32", "i64"],
+                   [P(0), P(2), P(3), P(4), P(5), P(1), P(6), P(7), I(width), I(taps), L(line_bytes)])
+    keep = _launch("conv_add", f"kern_conv_add_state_{act}", [256, 1, 1], ["seqs", -(-width // 256), 1], [iface[0], *iface[3:6], "i32", "i32", "i64"],
+                   [P(0), P(3), P(4), P(5), I(width), I(taps), L(line_bytes)])
+    return _op(iface, conv, *([keep] if taps > 1 else []))
+
+
+def resid_embed_op(width: int, vocab: int, eps: float, act: str = "bf16", scale: float = 1.0, conv: tuple[int, int] | None = None) -> dict:
+    """Token row times `scale` into the f32 residual, and the first sublayer's normed input.
+    Interface [ids, table, next norm w, x, xn, err]; `conv` (taps, bytes of a line; one row per sequence) also convolves the input:
+    [conv w, convolved, state, lines] at the end."""
     iface = ["in buffer<i64>", "in buffer<bf16>", "in buffer<bf16>", "out buffer<f32>", f"out buffer<{act}>", "out buffer<i32>"]
-    return _op(iface, _launch("resid", f"kern_resid_embed_{act}", [256, 1, 1], ["tokens", 1, 1], iface[:5] + ["i32", "i32", "f32", "out buffer<i32>"],
-                              [*map(P, range(5)), I(width), I(vocab), {"f32": eps}, P(5)], shared_mem=width * 4))
+    types, more = _conv_step(conv, act, 6) if conv else ([], [])
+    return _op(iface + types, _launch("resid", f"kern_resid_embed_{'conv_' if conv else ''}{act}", [256, 1, 1], ["tokens", 1, 1],
+                                      iface[:5] + ["i32", "i32", "f32", "f32", "out buffer<i32>"] + [t for t, _ in more],
+                                      [*map(P, range(5)), I(width), I(vocab), {"f32": scale}, {"f32": eps}, P(5), *(a for _, a in more)], shared_mem=width * 4))
 
 
 def resid_mix_op(width: int, eps: float, act: str = "bf16", routed: int = 0, last: bool = False) -> dict:
@@ -334,6 +365,25 @@ def resid_mix_op(width: int, eps: float, act: str = "bf16", routed: int = 0, las
     parts = [(iface[0], P(0)), (iface[1], P(1)), *route, (iface[2], P(2)), *tail]
     return _op(iface, _launch("resid", f"kern_resid_mix_{act}", [256, 1, 1], ["tokens", 1, 1], [t for t, _ in parts] + ["i32", "i32", "f32"],
                               [a for _, a in parts] + [I(width), I(routed), {"f32": eps}], shared_mem=width * 4))
+
+
+def resid_gate_op(width: int, eps: float, act: str = "bf16", routed: int = 0, last: bool = False, conv: tuple[int, int] | None = None) -> dict:
+    """`resid_mix_op` of a result gated element by element: x += rms(y sigmoid(gate + b)) w_post. Interface [x, y, w_post, w_next, xn,
+    gate, b] (`last`: [x, y, w_post, hidden, gate, b]), then with `routed` [perm, weights], with `conv` (taps, bytes of a line; one
+    row per sequence) the next input convolved as well: [conv w, convolved, state, lines]."""
+    iface = ["in buffer<f32>" if last else "inout buffer<f32>", f"in buffer<{act}>", "in buffer<bf16>"]
+    iface += ["out buffer<f32>"] if last else ["in buffer<bf16>", f"out buffer<{act}>"]
+    g = len(iface)
+    iface += [f"in buffer<{act}>", "in buffer<bf16>"]
+    n = len(iface)
+    iface += ["in buffer<i32>", "in buffer<f32>"] if routed else []
+    route = [(iface[n], P(n)), (iface[n + 1], P(n + 1))] if routed else [NULL, NULL]
+    types, more = _conv_step(conv, act, len(iface)) if conv else ([], [])
+    tail = [NULL, NULL, (iface[3], P(3))] if last else [(iface[3], P(3)), (iface[4], P(4))] + ([] if conv else [NULL])
+    parts = [(iface[0], P(0)), (iface[1], P(1)), *route, (iface[2], P(2)), *tail, ("i32", I(width)), ("i32", I(routed)), ("f32", {"f32": eps}),
+             (iface[g], P(g)), (iface[g + 1], P(g + 1)), *more]
+    return _op(iface + types, _launch("resid", f"kern_resid_gate_{'conv_' if conv else ''}{act}", [256, 1, 1], ["tokens", 1, 1], [t for t, _ in parts],
+                                      [a for _, a in parts], shared_mem=width * 4))
 
 
 def resid_scale_op(width: int, eps: float, act: str = "bf16", *, routed: int = 0, bias: bool = False, shared_gate: int | None = None,
@@ -492,6 +542,79 @@ def window_tiles(hq: int, hk: int, d: int, dv: int, page_size: int, act: str) ->
     return act == "bf16" and d == dv and d in (64, 128, 256) and hq // hk <= 16 and (page_size % 64 == 0 or (page_size % 8 == 0 and 64 % page_size == 0))
 
 
+def _split_ranges(hk: int, seqs_max: int, reach: int | None) -> list[tuple[int, int, int]]:
+    """(splits, fewest, most sequences) of a decode launch: enough sequences that heads x sequences x splits cover the SMs, and in a
+    reach of so many keys at least two tiles a split."""
+    ranges, hi, most = [], seqs_max, 8 if reach else 32
+    for splits in (1, 2, 4, 8, 16, 32)[: 4 if reach else 6]:
+        if reach and splits > 1 and splits * 128 > reach + 64:
+            break
+        lo = 1 if splits == most or (reach and 4 * splits * 64 > reach + 64) else max(1, -(-C.SMS // (hk * splits)))
+        if lo <= hi:
+            ranges.append((splits, lo, hi))
+            hi = lo - 1
+    if hi >= 1:
+        s, lo, top = ranges.pop() if ranges else (1, 1, seqs_max)
+        ranges.append((s, 1, top))
+    return ranges
+
+
+def _tiled_attn(form: str, iface: list, at: dict, maps: list, hq: int, hk: int, d: int, page_size: int, table_width: int, q_stride: int, out_stride: int, form_t: list,
+                form_a: list, ragged: bool, seqs_max: int, reach: int | None, merge) -> dict:
+    """The launches of one form (`window`, `sink`, `pooled`) of the paged attention bodies. `at`: where q, out, table and lens stand in
+    the interface; `form_t` / `form_a`: what the form's entries take at their end; `merge(splits, ws_o, ws_ml)`: the launch that puts
+    split keys together. Ragged calls add [cu_seqlens, work_p, count_p, work_d, count_d] to the interface."""
+    g, q, out, table, lens = hq // hk, *(P(at[k]) for k in ("q", "out", "table", "lens"))
+    q_t, out_t = iface[at["q"]], iface[at["out"]]
+    map_t = ["bytes<128>"] * len(maps)
+    lp = lambda ws, lists: map_t + [q_t, out_t] + (["out buffer<f32>"] * 2 if ws else ["i64"] * 2) + ["in buffer<i32>"] * 2 \
+        + (["in buffer<i32>"] * 3 if lists else ["i64"] * 3) + ["i32"] * 8 + form_t
+    sizes = lambda splits: [I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(splits), I(C.I32_MAX)]
+    if not ragged:
+        ranges = _split_ranges(hk, seqs_max, reach)
+        launches, most = [], max(s for s, _, _ in ranges)
+        for splits, lo, hi in ranges:
+            when = {"var": "seqs", **({"min": lo} if lo > 1 else {}), **({"max": hi} if hi < seqs_max else {})}
+            kw = {"when": when} if len(when) > 1 else {}
+            ws = [{"scratch": "ws_o"}, {"scratch": "ws_ml"}] if splits > 1 else [L(0), L(0)]
+            launches.append(_launch("attn_window", f"kern_attn_{form}_decode_d{d}", [160, 1, 1], [hk, "seqs", splits], lp(splits > 1, False),
+                                    [*maps, q, out, *ws, table, lens, L(0), L(0), L(0), *sizes(splits), *form_a], shared_mem=C.attn_smem(d), **kw))
+            if splits > 1:
+                launches.append(merge(splits, *ws) | kw)
+        scratch = {"scratch": {"ws_o": {"dtype": "f32", "shape": ["seqs", hq * most * d]}, "ws_ml": {"dtype": "f32", "shape": ["seqs", hq * most * 2]}}} if most > 1 else {}
+        return _op(iface, *launches, **scratch)
+    o = len(iface)
+    iface += ["in buffer<i32>"] * 5
+    lists = [P(o + i) for i in range(5)]
+    mode = C.attn_mode(hq, hk, d)
+    few = {"var": "seqs", "max": C.FMHA_SEQS}
+    many = {"var": "seqs", "min": C.FMHA_SEQS + 1}
+    grid = lambda rows: [hk, {"add": [{"ceil_div": ["tokens", rows // g]}, "seqs"]}, 1]
+    tail = [I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(C.I32_MAX), *form_a]
+    causal = lambda **kw: _launch("attn_fmha", f"kern_attn_{form}_fmha_d128", [192, 1, 1], grid(128), map_t + [q_t, out_t] + ["in buffer<i32>"] * 5 + ["i32"] * 7 + form_t,
+                                  [*maps, q, out, table, lens, *lists[:3], *tail], shared_mem=768 + 128 * d * 2 + 128 * 64 * 2 + 2 * 2 * (64 * d * 2) + 256, **kw)
+    listed = lambda kind, work, smem, g_, **kw: _launch("attn_window", f"kern_attn_{form}_{kind}_d{d}", [160, 1, 1], g_, lp(False, True),
+                                                        [*maps, q, out, L(0), L(0), table, lens, lists[0], lists[work], lists[work + 1], *sizes(1), *form_a],
+                                                        shared_mem=smem, **kw)
+    one = lambda **kw: _launch("attn_window", f"kern_attn_{form}_ragged_d{d}", [160, 1, 1], grid(64), map_t + [q_t, out_t] + ["in buffer<i32>"] * 7 + ["i32"] * 7 + form_t,
+                               [*maps, q, out, table, lens, *lists, *tail], shared_mem=C.attn_smem(d, prefill=True), **kw)
+    rows = lambda **kw: listed("decode", 3, C.attn_smem(d), [hk, "seqs", 1], **kw)
+    if mode == "auto":
+        return _op(iface, causal(when=few), rows(when=few), one(when=many))
+    if mode in ("fmha", "fmha2"):
+        return _op(iface, causal(), rows())
+    if mode == "ragged":
+        return _op(iface, one())
+    return _op(iface, listed("prefill", 1, C.attn_smem(d, prefill=True), grid(64)), rows())
+
+
+def _head_width(d: int, dv: int) -> int:
+    """The generic attention kernels' columns for heads of this size."""
+    if max(d, dv) > 512:
+        raise ValueError(f"heads of {d} / {dv} columns (at most 512)")
+    return next(n for n in (64, 128, 256, 512) if max(d, dv) <= n)
+
+
 def window_attn_op(hq: int, hk: int, d: int, dv: int, window: int, scale: float, cap: float, page_size: int, table_width: int, q_stride: int,
                    out_stride: int, out_scale: float, ragged: bool, act: str = "bf16", seqs_max: int = 0) -> dict:
     """Attention over the last `window` positions, capped scores, a sink per query head; rows times out_scale into columns of
@@ -502,68 +625,19 @@ def window_attn_op(hq: int, hk: int, d: int, dv: int, window: int, scale: float,
     iface = [f"in buffer<{act}>", "in state", f"out buffer<{act}>", "in buffer<i32>", "in buffer<i32>", "in buffer<bf16>", "out buffer<i32>"]
     if not window_tiles(hq, hk, d, dv, page_size, act):
         iface += ["in buffer<i32>"] if ragged else []
-        if max(d, dv) > 512:
-            raise ValueError(f"heads of {d} / {dv} columns (at most 512)")
-        w = next(n for n in (64, 128, 256, 512) if max(d, dv) <= n)
         row_t, row_a = (iface[7], P(7)) if ragged else NULL
-        return _op(iface, _launch("attn_window", f"kern_window_attn_{act}_w{w}", [128, 1, 1], [hq, "tokens" if ragged else "seqs", 1],
+        return _op(iface, _launch("attn_window", f"kern_window_attn_{act}_w{_head_width(d, dv)}", [128, 1, 1], [hq, "tokens" if ragged else "seqs", 1],
                                   [*iface[:5], row_t, iface[5], NULL[0]] + ["i32"] * 10 + ["f32"] * 3 + ["out buffer<i32>"],
                                   [*map(P, range(5)), row_a, P(5), NULL[1], I(hq), I(hk), I(d), I(dv), I(q_stride), I(out_stride), I(0), I(table_width), I(page_size),
                                    I(window), {"f32": scale}, {"f32": cap}, {"f32": out_scale}, P(6)], shared_mem=(4 * dv + 8) * 4))
-    g, kv = hq // hk, C._kv_map(d, page_size, 1)
     win_t = ["out buffer<i32>", "in buffer<bf16>", "i32", "f32", "f32", "f32"]
     win_a = [P(6), P(5), I(window), {"f32": 2 * LOG2E * scale / cap}, {"f32": cap * LOG2E}, {"f32": out_scale}]
-    lp = lambda ws, lists: ["bytes<128>", iface[0], iface[2]] + (["out buffer<f32>"] * 2 if ws else ["i64"] * 2) + ["in buffer<i32>"] * 2 \
-        + (["in buffer<i32>"] * 3 if lists else ["i64"] * 3) + ["i32"] * 8 + win_t
-    sizes = lambda splits: [I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(splits), I(C.I32_MAX)]
-    if not ragged:
-        ranges, hi = [], seqs_max
-        for splits in (1, 2, 4, 8):      # enough sequences that heads x sequences x splits cover the SMs; at least two tiles a split
-            if splits > 1 and splits * 128 > window + 64:
-                break
-            lo = max(1, -(-C.SMS // (hk * splits)))
-            if splits == 8 or 4 * splits * 64 > window + 64:
-                lo = 1
-            if lo <= hi:
-                ranges.append((splits, lo, hi))
-                hi = lo - 1
-        if hi >= 1:
-            s, lo, top = ranges.pop() if ranges else (1, 1, seqs_max)
-            ranges.append((s, 1, top))
-        launches, most = [], max(s for s, _, _ in ranges)
-        for splits, lo, hi in ranges:
-            when = {"var": "seqs", **({"min": lo} if lo > 1 else {}), **({"max": hi} if hi < seqs_max else {})}
-            kw = {"when": when} if len(when) > 1 else {}
-            ws = [{"scratch": "ws_o"}, {"scratch": "ws_ml"}] if splits > 1 else [L(0), L(0)]
-            launches.append(_launch("attn_window", f"kern_attn_window_decode_d{d}", [160, 1, 1], [hk, "seqs", splits], lp(splits > 1, False),
-                                    [kv, P(0), P(2), *ws, P(3), P(4), L(0), L(0), L(0), *sizes(splits), *win_a], shared_mem=C.attn_smem(d), **kw))
-            if splits > 1:
-                launches.append(_launch("attn_window", "kern_attn_window_merge", [min(256, d), 1, 1], [{"mul": ["seqs", hq]}, 1, 1],
-                                        ["in buffer<f32>", "in buffer<f32>", iface[2], "in buffer<bf16>", NULL[0]] + ["i32"] * 6 + ["f32"],
-                                        [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, P(2), P(5), NULL[1], I(0), I(C.I32_MAX), I(hq), I(d), I(splits), I(out_stride), {"f32": out_scale}], **kw))
-        scratch = {"scratch": {"ws_o": {"dtype": "f32", "shape": ["seqs", hq * most * d]}, "ws_ml": {"dtype": "f32", "shape": ["seqs", hq * most * 2]}}} if most > 1 else {}
-        return _op(iface, *launches, **scratch)
-    iface += ["in buffer<i32>"] * 5
-    mode = C.attn_mode(hq, hk, d)
-    few = {"var": "seqs", "max": C.FMHA_SEQS}
-    many = {"var": "seqs", "min": C.FMHA_SEQS + 1}
-    grid = lambda rows: [hk, {"add": [{"ceil_div": ["tokens", rows // g]}, "seqs"]}, 1]
-    causal = lambda **kw: _launch("attn_fmha", "kern_attn_window_fmha_d128", [192, 1, 1], grid(128), ["bytes<128>", iface[0], iface[2]] + ["in buffer<i32>"] * 5 + ["i32"] * 7 + win_t,
-                                  [kv, P(0), P(2), P(3), P(4), P(7), P(8), P(9), I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(C.I32_MAX), *win_a],
-                                  shared_mem=768 + 128 * d * 2 + 128 * 64 * 2 + 2 * 2 * (64 * d * 2) + 256, **kw)
-    listed = lambda kind, work, smem, g_, **kw: _launch("attn_window", f"kern_attn_window_{kind}_d{d}", [160, 1, 1], g_, lp(False, True),
-                                                        [kv, P(0), P(2), L(0), L(0), P(3), P(4), P(7), P(work), P(work + 1), *sizes(1), *win_a], shared_mem=smem, **kw)
-    one = lambda **kw: _launch("attn_window", f"kern_attn_window_ragged_d{d}", [160, 1, 1], grid(64), ["bytes<128>", iface[0], iface[2]] + ["in buffer<i32>"] * 7 + ["i32"] * 7 + win_t,
-                               [kv, P(0), P(2), P(3), P(4), P(7), P(8), P(9), P(10), P(11), I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(C.I32_MAX),
-                                *win_a], shared_mem=C.attn_smem(d, prefill=True), **kw)
-    rows = lambda **kw: listed("decode", 10, C.attn_smem(d), [hk, "seqs", 1], **kw)
-    if mode == "auto":
-        return _op(iface, causal(when=few), rows(when=few), one(when=many))
-    if mode in ("fmha", "fmha2"):
-        return _op(iface, causal(), rows())
-    if mode == "ragged":
-        return _op(iface, one())
-    return _op(iface, listed("prefill", 8, C.attn_smem(d, prefill=True), grid(64)), rows())
+    merge = lambda splits, ws_o, ws_ml: _launch(
+        "attn_window", "kern_attn_window_merge", [min(256, d), 1, 1], [{"mul": ["seqs", hq]}, 1, 1],
+        ["in buffer<f32>", "in buffer<f32>", iface[2], "in buffer<bf16>", NULL[0]] + ["i32"] * 6 + ["f32"],
+        [ws_o, ws_ml, P(2), P(5), NULL[1], I(0), I(C.I32_MAX), I(hq), I(d), I(splits), I(out_stride), {"f32": out_scale}])
+    return _tiled_attn("window", iface, {"q": 0, "out": 2, "table": 3, "lens": 4}, [C._kv_map(d, page_size, 1)], hq, hk, d, page_size, table_width, q_stride, out_stride,
+                       win_t, win_a, ragged, seqs_max, window, merge)
 
 
 # ---- attention with a sink and an output gate --------------------------------------------------------------------
@@ -580,64 +654,88 @@ def sink_attn_op(hq: int, hk: int, d: int, dv: int, scale: float, page_size: int
     sk, o = (("in buffer<bf16>", P(7)) if sink else NULL), len(iface)
     if not window_tiles(hq, hk, d, dv, page_size, act):
         iface += ["in buffer<i32>"] if ragged else []
-        if max(d, dv) > 512:
-            raise ValueError(f"heads of {d} / {dv} columns (at most 512)")
-        w = next(n for n in (64, 128, 256, 512) if max(d, dv) <= n)
         row_t, row_a = (iface[o], P(o)) if ragged else NULL
-        return _op(iface, _launch("attn_window", f"kern_window_attn_{act}_w{w}", [128, 1, 1], [hq, "tokens" if ragged else "seqs", 1],
+        return _op(iface, _launch("attn_window", f"kern_window_attn_{act}_w{_head_width(d, dv)}", [128, 1, 1], [hq, "tokens" if ragged else "seqs", 1],
                                   [*iface[:5], row_t, sk[0], iface[5]] + ["i32"] * 10 + ["f32"] * 3 + ["out buffer<i32>"],
                                   [*map(P, range(5)), row_a, sk[1], P(5), I(hq), I(hk), I(d), I(dv), I(q_stride), I(out_stride), I(gate_stride), I(table_width),
                                    I(page_size), I(C.I32_MAX), {"f32": scale}, {"f32": 0.0}, {"f32": 1.0}, P(6)], shared_mem=(4 * dv + 8) * 4))
-    g, kv = hq // hk, C._kv_map(d, page_size, 1)
     form_t, form_a = ["out buffer<i32>", sk[0], iface[5], "i32", "f32"], [P(6), sk[1], P(5), I(gate_stride), {"f32": scale * LOG2E}]
-    lp = lambda ws, lists: ["bytes<128>", iface[0], iface[2]] + (["out buffer<f32>"] * 2 if ws else ["i64"] * 2) + ["in buffer<i32>"] * 2 \
-        + (["in buffer<i32>"] * 3 if lists else ["i64"] * 3) + ["i32"] * 8 + form_t
-    sizes = lambda splits: [I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(splits), I(C.I32_MAX)]
+    merge = lambda splits, ws_o, ws_ml: _launch(
+        "attn_window", "kern_attn_window_merge", [min(256, d), 1, 1], [{"mul": ["seqs", hq]}, 1, 1],
+        ["in buffer<f32>", "in buffer<f32>", iface[2], sk[0], iface[5]] + ["i32"] * 6 + ["f32"],
+        [ws_o, ws_ml, P(2), sk[1], P(5), I(gate_stride), I(C.I32_MAX), I(hq), I(d), I(splits), I(out_stride), {"f32": 1.0}])
+    return _tiled_attn("sink", iface, {"q": 0, "out": 2, "table": 3, "lens": 4}, [C._kv_map(d, page_size, 1)], hq, hk, d, page_size, table_width, q_stride, out_stride,
+                       form_t, form_a, ragged, seqs_max, None, merge)
+
+
+# ---- attention in a window beside pooled blocks ------------------------------------------------------------------
+def pooled_sizes(hk: int, d: int, dv: int, pool: int, page_size: int, act: str = "bf16") -> dict:
+    """The second cache of attention with pooled blocks of `pool` tokens: a page of it holds the blocks that end in the page of the
+    same number. -> slots of a page, bytes per token (what a state declares), bytes of a page."""
+    slots = -(-page_size // pool)
+    per = -(-slots * hk * (d + dv) * ACT_BYTES[act] // page_size)
+    while per * page_size % 16:
+        per += 1
+    return {"slots": slots, "token": per, "page": per * page_size}
+
+
+def pooled_tiles(hq: int, hk: int, d: int, dv: int, pool: int, page_size: int, act: str) -> bool:
+    """Whether attention beside pooled blocks of this size runs on the tensor-core kernels: pages hold whole blocks or blocks whole
+    pages, without gaps."""
+    z = pooled_sizes(hk, d, dv, pool, page_size, act)
+    slots = z["slots"]
+    return window_tiles(hq, hk, d, dv, page_size, act) and (page_size % pool == 0 or pool % page_size == 0) and (slots % 64 == 0 or 64 % slots == 0) \
+        and slots * hk * 2 * d * ACT_BYTES[act] == z["page"]
+
+
+def qk_prep_pool_op(hq: int, hk: int, d: int, dv: int, rot: int, pool: int, page_size: int, table_width: int, row_stride: int, max_pos: int, ragged: bool,
+                    act: str = "bf16", halves: bool = False) -> dict:
+    """Rotary positions on the first `rot` columns of q and k, k and v into the paged cache, and the mean rows of the blocks that end
+    here into the second. Interface [qkv, state, pooled state, positions, slots, block_table, cos, sin, err] (+ [cu_seqlens, seqs,
+    rows] for ragged rows)."""
+    if rot % 2 or rot > d:
+        raise ValueError(f"rotary positions on {rot} of {d} columns")
+    z = pooled_sizes(hk, d, dv, pool, page_size, act)
+    iface = [f"inout buffer<{act}>", "inout state", "inout state", "in buffer<i64>", "in buffer<i64>", "in buffer<i32>", "in buffer<f32>", "in buffer<f32>",
+             "out buffer<i32>"]
+    smem = 8 * max(d, dv) * 4
     if not ragged:
-        ranges, hi = [], seqs_max
-        for splits in (1, 2, 4, 8, 16, 32):      # enough sequences that heads x sequences x splits cover the SMs
-            lo = 1 if splits == 32 else max(1, -(-C.SMS // (hk * splits)))
-            if lo <= hi:
-                ranges.append((splits, lo, hi))
-                hi = lo - 1
-            if hi < 1:
-                break
-        launches, most = [], max(s for s, _, _ in ranges)
-        for splits, lo, hi in ranges:
-            when = {"var": "seqs", **({"min": lo} if lo > 1 else {}), **({"max": hi} if hi < seqs_max else {})}
-            kw = {"when": when} if len(when) > 1 else {}
-            ws = [{"scratch": "ws_o"}, {"scratch": "ws_ml"}] if splits > 1 else [L(0), L(0)]
-            launches.append(_launch("attn_window", f"kern_attn_sink_decode_d{d}", [160, 1, 1], [hk, "seqs", splits], lp(splits > 1, False),
-                                    [kv, P(0), P(2), *ws, P(3), P(4), L(0), L(0), L(0), *sizes(splits), *form_a], shared_mem=C.attn_smem(d), **kw))
-            if splits > 1:
-                launches.append(_launch("attn_window", "kern_attn_window_merge", [min(256, d), 1, 1], [{"mul": ["seqs", hq]}, 1, 1],
-                                        ["in buffer<f32>", "in buffer<f32>", iface[2], sk[0], iface[5]] + ["i32"] * 6 + ["f32"],
-                                        [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, P(2), sk[1], P(5), I(gate_stride), I(C.I32_MAX), I(hq), I(d), I(splits), I(out_stride),
-                                         {"f32": 1.0}], **kw))
-        scratch = {"scratch": {"ws_o": {"dtype": "f32", "shape": ["seqs", hq * most * d]}, "ws_ml": {"dtype": "f32", "shape": ["seqs", hq * most * 2]}}} if most > 1 else {}
-        return _op(iface, *launches, **scratch)
-    iface += ["in buffer<i32>"] * 5
-    lists = [P(o + i) for i in range(5)]
-    mode = C.attn_mode(hq, hk, d)
-    few = {"var": "seqs", "max": C.FMHA_SEQS}
-    many = {"var": "seqs", "min": C.FMHA_SEQS + 1}
-    grid = lambda rows: [hk, {"add": [{"ceil_div": ["tokens", rows // g]}, "seqs"]}, 1]
-    tail = [I(hq), I(hk), I(q_stride), I(out_stride), I(table_width), I(page_size), I(C.I32_MAX), *form_a]
-    causal = lambda **kw: _launch("attn_fmha", "kern_attn_sink_fmha_d128", [192, 1, 1], grid(128), ["bytes<128>", iface[0], iface[2]] + ["in buffer<i32>"] * 5 + ["i32"] * 7 + form_t,
-                                  [kv, P(0), P(2), P(3), P(4), *lists[:3], *tail], shared_mem=768 + 128 * d * 2 + 128 * 64 * 2 + 2 * 2 * (64 * d * 2) + 256, **kw)
-    listed = lambda kind, work, smem, g_, **kw: _launch("attn_window", f"kern_attn_sink_{kind}_d{d}", [160, 1, 1], g_, lp(False, True),
-                                                        [kv, P(0), P(2), L(0), L(0), P(3), P(4), lists[0], lists[work], lists[work + 1], *sizes(1), *form_a],
-                                                        shared_mem=smem, **kw)
-    one = lambda **kw: _launch("attn_window", f"kern_attn_sink_ragged_d{d}", [160, 1, 1], grid(64), ["bytes<128>", iface[0], iface[2]] + ["in buffer<i32>"] * 7 + ["i32"] * 7 + form_t,
-                               [kv, P(0), P(2), P(3), P(4), *lists, *tail], shared_mem=C.attn_smem(d, prefill=True), **kw)
-    rows = lambda **kw: listed("decode", 3, C.attn_smem(d), [hk, "seqs", 1], **kw)
-    if mode == "auto":
-        return _op(iface, causal(when=few), rows(when=few), one(when=many))
-    if mode in ("fmha", "fmha2"):
-        return _op(iface, causal(), rows())
-    if mode == "ragged":
-        return _op(iface, one())
-    return _op(iface, listed("prefill", 1, C.attn_smem(d, prefill=True), grid(64)), rows())
+        return _op(iface, _launch("attn_window", f"kern_qk_prep_pool_{act}", [256, 1, 1], ["tokens", 1, 1], iface[:8] + ["i32"] * 11 + ["i64", "i32", "out buffer<i32>"],
+                                  [*map(P, range(8)), I(hq), I(hk), I(d), I(dv), I(rot), I(int(halves)), I(page_size), I(row_stride), I(max_pos), I(pool), I(z["slots"]),
+                                   L(z["page"]), I(table_width), P(8)], shared_mem=smem))
+    iface += ["in buffer<i32>", "i32", "i32"]
+    prep = _launch("attn_window", f"kern_qk_prep_{act}", [256, 1, 1], ["tokens", 1, 1],
+                   [*iface[:2], *iface[3:5], *iface[6:8], NULL[0], NULL[0]] + ["i32"] * 9 + ["f32", "out buffer<i32>"],
+                   [P(0), P(1), P(3), P(4), P(6), P(7), NULL[1], NULL[1], I(hq), I(hk), I(d), I(dv), I(rot), I(int(halves)), I(page_size), I(row_stride), I(max_pos),
+                    {"f32": 0.0}, P(8)], shared_mem=smem)
+    means = _launch("attn_window", f"kern_pool_blocks_{act}", [256, 1, 1], ["tokens", 1, 1],
+                    ["in state", "inout state", *iface[3:6], iface[9]] + ["i32"] * 8 + ["i64", "i32", "out buffer<i32>"],
+                    [P(1), P(2), P(3), P(4), P(5), P(9), P(10), P(11), I(hk), I(d), I(dv), I(page_size), I(pool), I(z["slots"]), L(z["page"]), I(table_width), P(8)])
+    return _op(iface, prep, means)
+
+
+def pooled_attn_op(hq: int, hk: int, d: int, dv: int, window: int, pool: int, scale: float, page_size: int, table_width: int, q_stride: int, out_stride: int,
+                   ragged: bool, act: str = "bf16", seqs_max: int = 0) -> dict:
+    """Attention over the last `window` positions and the mean rows of all blocks of `pool` tokens that end before them, in one
+    softmax. Interface [q, state, pooled state, out, block_table, lens, err], then for ragged rows on the tensor cores
+    (`pooled_tiles`) [cu_seqlens, work_p, count_p, work_d, count_d] (lens per sequence), else [row_seq] (lens per row)."""
+    if hq % hk:
+        raise ValueError(f"{hq} query heads over {hk} key heads")
+    z = pooled_sizes(hk, d, dv, pool, page_size, act)
+    iface = [f"in buffer<{act}>", "in state", "in state", f"out buffer<{act}>", "in buffer<i32>", "in buffer<i32>", "out buffer<i32>"]
+    if not pooled_tiles(hq, hk, d, dv, pool, page_size, act):
+        iface += ["in buffer<i32>"] if ragged else []
+        row_t, row_a = (iface[7], P(7)) if ragged else NULL
+        return _op(iface, _launch("attn_window", f"kern_pooled_attn_{act}_w{_head_width(d, dv)}", [128, 1, 1], [hq, "tokens" if ragged else "seqs", 1],
+                                  [*iface[:6], row_t] + ["i32"] * 11 + ["i64", "f32", "out buffer<i32>"],
+                                  [*map(P, range(6)), row_a, I(hq), I(hk), I(d), I(dv), I(q_stride), I(out_stride), I(table_width), I(page_size), I(window), I(pool),
+                                   I(z["slots"]), L(z["page"]), {"f32": scale}, P(6)], shared_mem=(4 * dv + 8) * 4))
+    form_t, form_a = ["out buffer<i32>", "i32", "i32", "i32", "f32"], [P(6), I(window), I(pool), I(z["slots"]), {"f32": scale * LOG2E}]
+    merge = lambda splits, ws_o, ws_ml: _launch(
+        "attn_paged", "kern_attn_merge_splits", [min(256, d), 1, 1], [{"mul": ["seqs", hq]}, 1, 1], ["in buffer<f32>", "in buffer<f32>", iface[3]] + ["i32"] * 5,
+        [ws_o, ws_ml, P(3), I(C.I32_MAX), I(hq), I(d), I(splits), I(out_stride)])
+    return _tiled_attn("pooled", iface, {"q": 0, "out": 3, "table": 4, "lens": 5}, [C._kv_map(d, page_size, 1), C._kv_map(d, z["slots"], 2)], hq, hk, d, page_size,
+                       table_width, q_stride, out_stride, form_t, form_a, ragged, seqs_max, window + table_width * page_size // pool, merge)
 
 
 # ---- routed experts ---------------------------------------------------------------------------------------
@@ -668,6 +766,16 @@ def route_groups_op(experts: int, top: int, groups: int = 1, keep: int = 1, reno
                               [iface[0], b_t, *iface[o:]] + ["i32"] * 7 + ["f32", "i32"],
                               [P(0), b_a, P(o), P(o + 1), P(o + 2), I(experts), I(top), I(groups), I(keep), I(int(softmax)), I(group_top), I(int(renorm)),
                                {"f32": scale}, I(ld or experts)], shared_mem=4 * (experts + groups) * 4))
+
+
+def route_table_op(experts: int, top: int, vocab: int) -> dict:
+    """No router: a table's row of the token id names its experts, each with weight 1 / top.
+    Interface [token ids, table, ids, weights, tokens, err]."""
+    if not 1 <= top <= min(32, experts):
+        raise ValueError(f"{top} of {experts} experts per token (at most 32)")
+    iface = ["in buffer<i64>", "in buffer<i32>", "out buffer<i32>", "out buffer<f32>", "i32", "out buffer<i32>"]
+    return _op(iface, _launch("moe", "kern_moe_route_table", [256, 1, 1], [{"ceil_div": [{"mul": ["tokens", top]}, 256]}, 1, 1], iface[:5] + ["i32"] * 3 + [iface[5]],
+                              [*map(P, range(5)), I(experts), I(top), I(vocab), P(5)]))
 
 
 def routed_tile_rows(act: str, width: int, ff: int) -> int:

@@ -9,6 +9,7 @@ program helper), tools/once.py (load programs), tools/toy/gen.py:238-246 (safete
 from __future__ import annotations
 
 import json
+import math
 import os
 import struct
 from pathlib import Path
@@ -638,14 +639,31 @@ def sample_op(vocab: int, dtype: str = "bf16") -> dict:
                                             {"i32": vocab}, {"i32": vocab}]}]}}
 
 
-def rope_table_op(max_pos: int, rot: int, theta: float, factor: float = 1.0) -> dict:
-    """Interface [cos, sin]: the `once` program's table of angles, position * theta^(-2i / rot) / factor."""
-    scaled = factor != 1.0
+def rope_table_op(max_pos: int, rot: int, theta: float, factor: float = 1.0, scaling: dict | None = None) -> dict:
+    """Interface [cos, sin]: the `once` program's table of angles, position * theta^(-2i / rot) / factor; or with `scaling`, the
+    frequencies scaled by the constants it holds: `banded_rope` or `ramped_rope`."""
+    kind, constants = ("scaled", [factor]) if factor != 1.0 else ("", [])
+    if scaling:
+        kind, constants = scaling["kind"], scaling["constants"]
     return {"params": ["out buffer<f32>", "out buffer<f32>"], "impl": {"launches": [{
-        "module": "attn_prep", "entry": "kern_rope_table_scaled_f32" if scaled else "kern_rope_table_f32", "block": [256, 1, 1],
+        "module": "attn_prep", "entry": "kern_rope_table_" + (kind + "_" if kind else "") + "f32", "block": [256, 1, 1],
         "grid": [min(1024, -(-max_pos * (rot // 2) // 256)), 1, 1],
-        "params": ["out buffer<f32>", "out buffer<f32>", "i32", "i32", "i64"] + ["i64"] * scaled,
-        "args": [{"param": 0}, {"param": 1}, {"i32": max_pos}, {"i32": rot}, {"i64": f64_bits(theta)}] + [{"i64": f64_bits(factor)}] * scaled}]}}
+        "params": ["out buffer<f32>", "out buffer<f32>", "i32", "i32", "i64"] + ["i64"] * len(constants),
+        "args": [{"param": 0}, {"param": 1}, {"i32": max_pos}, {"i32": rot}, {"i64": f64_bits(theta)}, *({"i64": f64_bits(c)} for c in constants)]}]}}
+
+
+def banded_rope(factor: float, low: float, high: float, original: float) -> dict:
+    """Frequencies by bands of wavelengths: shorter than original / high as they are, longer than original / low divided by
+    `factor`, and from one to the other in between (the scaling of Llama 3.1)."""
+    return {"kind": "banded", "constants": [factor, low, high, original]}
+
+
+def ramped_rope(rot: int, theta: float, factor: float, original: float, fast: float, slow: float) -> dict:
+    """Frequencies along a ramp over the pairs, from those that turn `fast` times in `original` positions (as they are) to those
+    that turn `slow` times (divided by `factor`); the tables grow by 0.1 ln(factor) + 1 (YaRN)."""
+    at = lambda turns: rot * math.log(original / (2 * math.pi * turns)) / (2 * math.log(theta))
+    lo, hi = max(math.floor(at(fast)), 0), min(math.ceil(at(slow)), rot - 1)
+    return {"kind": "ramp", "constants": [factor, lo, hi, 0.1 * math.log(factor) + 1]}
 
 
 # ---- tensor-parallel ops ---------------------------------------------------------------------------
@@ -1133,16 +1151,31 @@ def latent_smem(blocks: int) -> int:
     return 1024 + stages * 64 * blocks * 128 + 16 * (blocks * 64 + 8) * 2 + 16 * (64 + 8) * 2 + 2 * 8 * 16 * 4 + 256
 
 
+def latent_extra(iface: list, sink: bool, gate_stride: int, act: str) -> tuple[list, list]:
+    """The pointers [sink, gate] of a latent attention with rotated columns, each null where there is none; added to the interface."""
+    if sink and gate_stride:
+        raise ValueError("a latent attention with sinks and gates")
+    types, args = [], []
+    for there, t in ((sink, "in buffer<bf16>"), (gate_stride > 0, f"in buffer<{act}>")):
+        if there:
+            iface.append(t)
+        types.append(t if there else "i64")
+        args.append({"param": len(iface) - 1} if there else {"i64": 0})
+    return types, args
+
+
 def mla_attn_op(heads: int, page_size: int, table_width: int, ragged: bool, head_width: int = 192, seqs_max: int = 0,
-                sms: int = SMS, rank: int = 0, scale: float | None = None, rot: int = 0, max_pos: int = 0, rot_stride: int = 0) -> dict:
+                sms: int = SMS, rank: int = 0, scale: float | None = None, rot: int = 0, max_pos: int = 0, rot_stride: int = 0,
+                sink: bool = True, halves: bool = True, window: int = I32_MAX, gate_stride: int = 0) -> dict:
     """Absorbed latent attention: every head attends over the shared 576-wide latent rows, values their first 512
     columns. One row per sequence: interface [q, latent state, out, block_table, seq_lens, err], the context split over
     CTAs by `when` ranges of the batch (partials merged by a second launch) so that a few long sequences still fill
     the machine; ragged rows bring [.., row_len, err, row_seq] — a row reads its sequence's table row and attends over
     its own causal reach. `rank`: latent rows of that many columns (no rotary part), keys and values alike, scores times
-    `scale`; 0 is the 512 + 64 form. `rot`: as many rotated columns behind them; [q_rot, cos, sin, sink] then come at the end:
-    the heads' rotated query columns, not yet turned, in rows of their own `rot_stride` apart, tables of `max_pos` positions, and
-    a score per head that joins the denominator."""
+    `scale`; 0 is the 512 + 64 form. `rot`: as many rotated columns behind them; [q_rot, cos, sin] then come at the end:
+    the heads' rotated query columns, not yet turned (pairs of neighbours unless `halves`), in rows of their own `rot_stride` apart,
+    and tables of `max_pos` positions; then [sink], a score per head that joins the denominator, and with `gate_stride` [gate],
+    whose sigmoid multiplies a head's result. `window`: the positions a row sees."""
     dq, dv = (rank + rot, rank) if rank else (MLA_DQK, MLA_DV)
     scale = head_width ** -0.5 if scale is None else scale
     assert page_size % 64 == 0 or 64 % page_size == 0
@@ -1150,8 +1183,10 @@ def mla_attn_op(heads: int, page_size: int, table_width: int, ragged: bool, head
     if ragged:
         iface.append("in buffer<i32>")
     o = len(iface)
+    extra_t, extra_a = [], []
     if rot:
-        iface += ["in buffer<bf16>", "in buffer<f32>", "in buffer<f32>", "in buffer<bf16>"]
+        iface += ["in buffer<bf16>", "in buffer<f32>", "in buffer<f32>"]
+        extra_t, extra_a = latent_extra(iface, sink, gate_stride, "bf16")
     blocks = -(-heads // 16)
     qb, vb = -(-(rank + rot) // 64), -(-rank // 64)
     ranges, hi = [], seqs_max
@@ -1159,7 +1194,8 @@ def mla_attn_op(heads: int, page_size: int, table_width: int, ragged: bool, head
         ranges = [(1, 1, seqs_max)]
     else:
         for splits in (1, 2, 4, 8, 16, 32):
-            lo = 1 if splits == 32 else max(1, -(-sms // (blocks * splits)))
+            # at least two tiles a split
+            lo = 1 if splits == 32 or 4 * splits * 64 > window + 64 else max(1, -(-sms // (blocks * splits)))
             if lo <= hi:
                 ranges.append((splits, lo, hi))
                 hi = lo - 1
@@ -1185,8 +1221,8 @@ def mla_attn_op(heads: int, page_size: int, table_width: int, ragged: bool, head
         if rank:
             lp, args = lp + ["i32"], args + [{"i32": rank}]
         if rot:
-            lp = lp + iface[o:o + 4] + ["i32"] * 3
-            args = args + [{"param": o + i} for i in range(4)] + [{"i32": rot_stride}, {"i32": rot}, {"i32": max_pos}]
+            lp = lp + iface[o:o + 3] + extra_t + ["i32"] * 6
+            args = args + [{"param": o + i} for i in range(3)] + extra_a + [{"i32": v} for v in (rot_stride, rot, max_pos, int(halves), window, gate_stride)]
         entry = f"kern_latent_rot_decode_bf16_q{qb}_b{vb}" if rot else (f"kern_latent_decode_bf16_b{vb}" if rank else "kern_mla_decode_bf16")
         launch = {"module": "mla_decode", "entry": entry,
                   "block": [288, 1, 1], "grid": [blocks, "tokens" if ragged else "seqs", splits],
@@ -1196,7 +1232,12 @@ def mla_attn_op(heads: int, page_size: int, table_width: int, ragged: bool, head
                  "params": ["in buffer<f32>", "in buffer<f32>", "out buffer<bf16>", "i32", "i32", "i32", "i32", "i32"],
                  "args": [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, {"param": 2}, {"i32": I32_MAX}, {"i32": heads},
                           {"i32": dv}, {"i32": splits}, {"i32": heads * dv}]}
-        if rot:
+        if gate_stride:
+            merge = {"module": "attn_window", "entry": "kern_attn_gated_merge", "block": [256, 1, 1], "grid": [{"mul": ["tokens", heads]}, 1, 1],
+                     "params": ["in buffer<f32>", "in buffer<f32>", "out buffer<bf16>", "in buffer<bf16>"] + ["i32"] * 6,
+                     "args": [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, {"param": 2}, extra_a[1], {"i32": gate_stride}, {"i32": I32_MAX},
+                              {"i32": heads}, {"i32": dv}, {"i32": splits}, {"i32": heads * dv}]}
+        elif rot and sink:
             merge = {"module": "attn_window", "entry": "kern_attn_window_merge", "block": [256, 1, 1], "grid": [{"mul": ["tokens", heads]}, 1, 1],
                      "params": ["in buffer<f32>", "in buffer<f32>", "out buffer<bf16>", "in buffer<bf16>", "i64"] + ["i32"] * 6 + ["f32"],
                      "args": [{"scratch": "ws_o"}, {"scratch": "ws_ml"}, {"param": 2}, {"param": o + 3}, {"i64": 0}, {"i32": 0}, {"i32": I32_MAX},

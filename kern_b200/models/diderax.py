@@ -24,7 +24,7 @@ import torch
 from . import blocks as K
 from . import common as C
 from . import listed
-from .listed import Listed, gla_sizes, load_random
+from .listed import Listed, gla_sizes, latent_sizes, load_random
 
 
 @dataclass
@@ -152,11 +152,6 @@ def attention_sizes(m: dict) -> dict:
     return {"q": q, "k": k, "token": 2 * k}
 
 
-def latent_sizes(m: dict) -> dict:
-    H, r = m["heads"], m["kv_rank"]
-    return {"q": H * m["dim"], "rot": H * m["rot_dim"], "v": H * m["vdim"], "rank": r, "lat": H * r, "down": r + m["rot_dim"]}
-
-
 def moe_sizes(f: dict) -> dict:
     r = f["router"]
     identity, g = r.get("identity", 0), r.get("groups", {"count": 1, "keep": 1})
@@ -235,7 +230,7 @@ def save_folder(path, cfg: DideraxConfig, weights: dict[str, torch.Tensor]) -> N
 
 # ---- the manifest -------------------------------------------------------------------------------------------
 def build_manifest(cfg: DideraxConfig) -> dict:
-    d, A, S, T, W, page, eps = cfg.width, cfg.dtype, cfg.max_seqs, cfg.max_tokens, cfg.table_width, cfg.page_size, cfg.eps
+    d, A, S, W, page, eps = cfg.width, cfg.dtype, cfg.max_seqs, cfg.table_width, cfg.page_size, cfg.eps
     m_ = Listed(cfg)
     layers, es, bufs, states, err = cfg.depth, m_.es, m_.bufs, m_.states, m_.err
     B, V, op, room, weight, same, linear = m_.B, m_.V, m_.op, m_.room, m_.weight, m_.same, m_.linear
@@ -289,41 +284,8 @@ def build_manifest(cfg: DideraxConfig) -> dict:
         ]
 
     def latent(i: int, at: int, prefill: bool) -> list[dict]:
-        m, p, kv, sfx = layers[i]["mixer"], f"l{i}.mix.", f"kv.l{i}", "_p" if prefill else "_d"
-        z = latent_sizes(m)
-        H, dim, rot, vdim, rank, qr = m["heads"], m["dim"], m["rot_dim"], m["vdim"], z["rank"], m["q_rank"]
-        states[kv] = {"bytes_per_token": z["down"] * es}
-        w_in, down = m_.rows_weight(f"w.{p}down", d, [(p + "dq", qr), (p + "dkv", z["down"])])
-        # the unrotated rows of every head, then the rotated ones; filled up to whole 16-byte vectors of output
-        head = lambda h, lo, hi: {"tensor": p + "uq", "rows": [h * (dim + rot) + lo, h * (dim + rot) + hi]}
-        rows = z["q"] + z["rot"]
-        qc = -(-rows // 8) * 8
-        fill = [{"tensor": p + "uq", "rows": [0, 1]}] * (qc - rows)
-        w_uq = weight(f"w.{p}uq", (qc, qr), *[head(h, 0, dim) for h in range(H)], *[head(h, dim, dim + rot) for h in range(H)], *fill)
-        room("down", down); room("q_low", qr); room("q", qc); room("qlat", z["lat"]); room("olat", z["lat"]); room("attn", z["v"]); room("y", d)
-        cos, sin = m_.rotary(rot, float(m["rot"]["base"]))
-        prep = op(f"latent_prep_{rank}x{rot}x{qr}x{down}", lambda: K.latent_prep_op(rank, rot, qr, down, qr, cfg.context, eps, A))
-        uk = same(p + "uk", (z["q"], rank))
-        tiles = K.head_tiles(rank, dim, qc, z["lat"], A)
-        if tiles and f"ukt.l{i}" not in bufs:      # the tensor-core form wants W_uk with a latent column per row: turned once, at load
-            bufs[f"ukt.l{i}"] = {"dtype": "bf16", "shape": [H, rank, dim], "kind": "carry"}
-            m_.once.append({"op": op(f"transpose_{H}x{dim}x{rank}", lambda: K.transpose_heads_op(H, dim, rank)), "label": p + "ukt", "args": [uk, B(f"ukt.l{i}")]})
-        up = op(f"q_up_{H}x{dim}x{rank}x{qc}", lambda: K.head_linear_op(H, rank, dim, act=A, rows_max=T, lda=qc, ldc=z["lat"], transposed=not tiles))
-        v_up = op(f"v_up_{H}x{vdim}x{rank}", lambda: K.head_linear_op(H, vdim, rank, act=A, rows_max=T, lda=z["lat"], ldc=z["v"]))
-        attn = op(f"latent_attn{sfx}_{H}x{rank}x{rot}x{qc}_{m['scale']!r}",
-                  lambda: K.latent_rot_attn_op(H, rank, rot, float(m["scale"]), page, W, cfg.context, qc, prefill, A, seqs_max=S))
-        lens = [B("row_len"), err, *m_.row_plan()] if prefill else [B("seq_lens"), err]
-        return [
-            linear("lin", down, d, B("xn"), w_in, B("down"), label=p + "down"),
-            {"op": prep, "label": p + "prep", "args": [B("down"), {"state": kv}, B("q_low"), B("positions"), B("slot_mapping"), cos, sin, same(p + "dkv.norm", (rank,)),
-                                                       same(p + "dq.norm", (qr,)), err]},
-            linear("lin", qc, qr, B("q_low"), w_uq, B("q"), label=p + "uq"),
-            {"op": up, "label": p + "q_up", "args": [B("q"), B(f"ukt.l{i}") if tiles else uk, B("qlat"), V("tokens"), err]},
-            {"op": attn, "label": p + "attn", "args": [B("qlat"), {"state": kv}, B("olat"), B("block_table"), *lens, B("q", z["q"] * es), cos, sin, same(p + "sink", (H,))]},
-            {"op": v_up, "label": p + "v_up", "args": [B("olat"), same(p + "uv", (z["v"], rank)), B("attn"), V("tokens"), err]},
-            linear("lin", d, z["v"], B("attn"), same(p + "o", (d, z["v"])), B("y"), label=p + "o"),
-            finish(at, B("y"), p + "out"),
-        ]
+        m, p = layers[i]["mixer"], f"l{i}.mix."
+        return m_.latent(p, f"kv.l{i}", m, prefill, m_.rotary(m["rot_dim"], float(m["rot"]["base"])), sink=True) + [finish(at, B("y"), p + "out")]
 
     def dense(i: int, at: int) -> list[dict]:
         p = f"l{i}."

@@ -50,14 +50,14 @@ class Listed:
         have = self.bufs.get(name, {"shape": ["tokens", 0]})["shape"][1]
         self.bufs[name] = {"dtype": dtype or self.act, "shape": ["tokens", max(have, cols)], "kind": kind}
 
-    def weight(self, name: str, shape, *tensors) -> dict:
+    def weight(self, name: str, shape, *tensors, dtype: str = "bf16") -> dict:
         if name not in self.bufs:
-            self.bufs[name] = {"dtype": "bf16", "shape": list(shape), "kind": "weight",
+            self.bufs[name] = {"dtype": dtype, "shape": list(shape), "kind": "weight",
                                "bind": [t if isinstance(t, dict) else {"tensor": t} for t in tensors]}
         return self.B(name)
 
-    def same(self, name: str, shape) -> dict:
-        return self.weight("w." + name, shape, name)
+    def same(self, name: str, shape, dtype: str = "bf16") -> dict:
+        return self.weight("w." + name, shape, name, dtype=dtype)
 
     def rows_weight(self, name: str, width: int, parts: list[tuple[str, int]]) -> tuple[dict, int]:
         """Projections with one input as one matrix -> (the weight, its rows), filled up to whole 16-byte vectors of output with
@@ -115,15 +115,15 @@ class Listed:
                 "args": [B("positions"), B("cu_seqlens"), B("row_seq"), B("row_len"), V("seqs"), V("tokens")]}
 
     # ---- the first call, and what rides with it ----
-    def rotary(self, dims: int, base: float, factor: float = 1.0) -> list[dict]:
-        """The cos and sin tables of one rotation, written when the model is loaded."""
+    def rotary(self, dims: int, base: float, factor: float = 1.0, scaling: dict | None = None) -> list[dict]:
+        """The cos and sin tables of one rotation, written when the model is loaded; `scaling` as `rope_table_op` takes it."""
         context, B = self.cfg.context, self.B
-        tag = f"{dims}x{base!r}" + (f"x{factor!r}" if factor != 1.0 else "")
+        tag = f"{dims}x{base!r}" + (f"x{factor!r}" if factor != 1.0 else "") + ("_".join(["", scaling["kind"], *map(repr, scaling["constants"])]) if scaling else "")
         name = "rope." + tag
         if name + ".cos" not in self.bufs:
             for n in (".cos", ".sin"):
                 self.bufs[name + n] = {"dtype": "f32", "shape": [context, dims // 2], "kind": "carry"}
-            op = self.op("rope_" + tag, lambda: C.rope_table_op(context, dims, base, factor))
+            op = self.op("rope_" + tag, lambda: C.rope_table_op(context, dims, base, factor, scaling))
             self.once.append({"op": op, "label": name, "args": [B(name + ".cos"), B(name + ".sin")]})
         return [B(name + ".cos"), B(name + ".sin")]
 
@@ -147,14 +147,73 @@ class Listed:
             self.plans["rows"] = [self.B("row_seq")], self.ops.pop(c["op"]), c["args"]
         return self.plans["rows"][0]
 
-    def embed(self, next_norm: str, prefill: bool) -> dict:
-        """Token rows into the residual and the first sublayer's normed input; the plans in the same call, so that both programs
-        have as many calls to every layer."""
+    def embed(self, next_norm: str, prefill: bool, scale: float = 1.0, conv: dict | None = None) -> dict:
+        """Token rows, times `scale`, into the residual and the first sublayer's normed input, convolved where that reads it so (`conv`,
+        from `input_conv`); the plans in the same call, so that both programs have as many calls to every layer."""
         cfg, B, d = self.cfg, self.B, self.cfg.width
         args = [B("token_ids"), self.same("embed", (cfg.vocab, d)), self.same(next_norm, (d,)), B("x"), B("xn"), self.err]
-        first = self.plans.values() if prefill else ()
-        name = self.op("embed" + ("_p" if prefill else "_d"), lambda: K.chain_ops(K.resid_embed_op(d, cfg.vocab, cfg.eps, self.act), *[o for _, o, _ in first]))
-        return {"op": name, "label": "embed", "args": args + [a for _, _, more in first for a in more]}
+        first = [(o, more) for _, o, more in self.plans.values()] if prefill else []
+        own = lambda: K.resid_embed_op(d, cfg.vocab, cfg.eps, self.act, scale)
+        if conv and prefill:
+            first.insert(0, (conv["op"](), conv["args"]))
+        elif conv:
+            args, own = args + conv["args"], lambda: K.resid_embed_op(d, cfg.vocab, cfg.eps, self.act, scale, conv["fused"])
+        name = self.op("embed" + ("_p" if prefill else "_d"), lambda: K.chain_ops(own(), *[o for o, _ in first]))
+        return {"op": name, "label": "embed", "args": args + [a for _, more in first for a in more]}
+
+    # ---- a sublayer that reads its input plus a convolution of it ----
+    def input_conv(self, tensor: str, taps: int, st: str, prefill: bool) -> dict:
+        """xn -> `xc`, its last rows in lines `st`: in a decode call a part of the kernel that makes xn (`fused`: what its op takes,
+        `args`: at the end), in a ragged one an op behind it."""
+        cfg, d, A, B, V = self.cfg, self.cfg.width, self.act, self.B, self.V
+        line = K.conv_line_bytes(d, taps, A)
+        self.states[st] = {"bytes_per_seq": line}
+        self.room("xc", d)
+        tail = [self.same(tensor, (d, taps)), B("xc"), {"state": st}, B("lines")]
+        return {"tag": f"{taps}x{line}", "fused": (taps, line), "op": lambda: K.conv_add_op(d, taps, line, A),
+                "args": [B("xn"), *tail, B("cu_seqlens"), V("seqs"), V("tokens")] if prefill else tail}
+
+    # ---- latent attention with a rotated part ----
+    def latent(self, p: str, kv: str, m: dict, prefill: bool, tables: list[dict], *, x: str = "xn", halves: bool = True, sink: bool = False, gate: bool = False,
+               window: int = C.I32_MAX) -> list[dict]:
+        """Queries through a latent, one rotated key part for all heads, its rows in state `kv`: x -> y. `tables`: the rotation's;
+        `sink`: a score per head in the denominator; `gate`: a sigmoid per head on the results; `window`: positions a row sees."""
+        cfg, d, A, es, B, V, S, T = self.cfg, self.cfg.width, self.act, self.es, self.B, self.V, self.cfg.max_seqs, self.cfg.max_tokens
+        z, sfx, page, W, err, eps = latent_sizes(m), "_p" if prefill else "_d", cfg.page_size, cfg.table_width, self.err, cfg.eps
+        H, dim, rot, vdim, rank, qr = m["heads"], m["dim"], m["rot_dim"], m["vdim"], z["rank"], m["q_rank"]
+        self.states[kv] = {"bytes_per_token": z["down"] * es}
+        w_in, down = self.rows_weight(f"w.{p}down", d, [(p + "dq", qr), (p + "dkv", z["down"])] + ([(p + "g", H)] if gate else []))
+        # the unrotated rows of every head, then the rotated ones; filled up to whole 16-byte vectors of output
+        head = lambda h, lo, hi: {"tensor": p + "uq", "rows": [h * (dim + rot) + lo, h * (dim + rot) + hi]}
+        rows = z["q"] + z["rot"]
+        qc = -(-rows // 8) * 8
+        fill = [{"tensor": p + "uq", "rows": [0, 1]}] * (qc - rows)
+        w_uq = self.weight(f"w.{p}uq", (qc, qr), *[head(h, 0, dim) for h in range(H)], *[head(h, dim, dim + rot) for h in range(H)], *fill)
+        for name, cols in (("down", down), ("q_low", qr), ("q", qc), ("qlat", z["lat"]), ("olat", z["lat"]), ("attn", z["v"]), ("y", d)):
+            self.room(name, cols)
+        form = ("" if halves else "n") + ("" if window == C.I32_MAX else f"w{window}") + (f"g{down}" if gate else "")
+        prep = self.op(f"latent_prep_{rank}x{rot}x{qr}x{down}" + ("" if halves else "n"), lambda: K.latent_prep_op(rank, rot, qr, down, qr, cfg.context, eps, A, halves))
+        uk = self.same(p + "uk", (z["q"], rank))
+        tiles, ukt = K.head_tiles(rank, dim, qc, z["lat"], A), f"ukt.{p.split('.')[0]}"
+        if tiles and ukt not in self.bufs:      # the tensor-core form wants W_uk with a latent column per row: turned once, at load
+            self.bufs[ukt] = {"dtype": "bf16", "shape": [H, rank, dim], "kind": "carry"}
+            self.once.append({"op": self.op(f"transpose_{H}x{dim}x{rank}", lambda: K.transpose_heads_op(H, dim, rank)), "label": p + "ukt", "args": [uk, B(ukt)]})
+        up = self.op(f"q_up_{H}x{dim}x{rank}x{qc}", lambda: K.head_linear_op(H, rank, dim, act=A, rows_max=T, lda=qc, ldc=z["lat"], transposed=not tiles))
+        v_up = self.op(f"v_up_{H}x{vdim}x{rank}", lambda: K.head_linear_op(H, vdim, rank, act=A, rows_max=T, lda=z["lat"], ldc=z["v"]))
+        attn = self.op(f"latent_attn{sfx}_{H}x{rank}x{rot}x{qc}{form}_{m['scale']!r}", lambda: K.latent_rot_attn_op(
+            H, rank, rot, float(m["scale"]), page, W, cfg.context, qc, prefill, A, seqs_max=S, sink=sink, halves=halves, window=window, gate_stride=down if gate else 0))
+        lens = [B("row_len"), err, *self.row_plan()] if prefill else [B("seq_lens"), err]
+        extra = ([self.same(p + "sink", (H,))] if sink else []) + ([B("down", (qr + z["down"]) * es)] if gate else [])
+        return [
+            self.linear("lin", down, d, B(x), w_in, B("down"), label=p + "down"),
+            {"op": prep, "label": p + "prep", "args": [B("down"), {"state": kv}, B("q_low"), B("positions"), B("slot_mapping"), *tables, self.same(p + "dkv.norm", (rank,)),
+                                                       self.same(p + "dq.norm", (qr,)), err]},
+            self.linear("lin", qc, qr, B("q_low"), w_uq, B("q"), label=p + "uq"),
+            {"op": up, "label": p + "q_up", "args": [B("q"), B(ukt) if tiles else uk, B("qlat"), V("tokens"), err]},
+            {"op": attn, "label": p + "attn", "args": [B("qlat"), {"state": kv}, B("olat"), B("block_table"), *lens, B("q", z["q"] * es), *tables, *extra]},
+            {"op": v_up, "label": p + "v_up", "args": [B("olat"), self.same(p + "uv", (z["v"], rank)), B("attn"), V("tokens"), err]},
+            self.linear("lin", d, z["v"], B("attn"), self.same(p + "o", (d, z["v"])), B("y"), label=p + "o"),
+        ]
 
     # ---- linear attention with a decay per key channel ----
     def linear_attention(self, p: str, st: str, H: int, dk: int, dv: int, stride: int, ptrs, z, prefill: bool, norm, norm_shared: bool, u, q_scale, out, out_stride,
@@ -223,10 +282,25 @@ class Listed:
         """Routed experts up to their own rows: xn -> `moe.y` (expert-sorted), `moe.perm`, `moe.w`. `route(logits, ids, weights)` makes
         the call that picks them; an id from `experts` on has no row (`moe.perm` -1). `router`: a matrix of more rows than experts,
         and their number."""
-        cfg, d, B, V = self.cfg, self.cfg.width, self.B, self.V
+        d, B = self.cfg.width, self.B
+        w_router, outputs = router or (self.same(p + "mlp.router", (experts, d)), experts)
+        self.room("moe.logits", outputs, "f32"); self.room("moe.ids", top, "i32"); self.room("moe.w", top, "f32")
+        return [self.linear("router", outputs, d, B("xn"), w_router, B("moe.logits"), label=p + "router", epilogue="f32"), route(B("moe.logits"), B("moe.ids"), B("moe.w")),
+                *self.experts(p, experts, top, ff, glu, limit)]
+
+    def table_routed(self, p: str, experts: int, top: int, ff: int) -> list[dict]:
+        """As `routed` with no router: tensor `<p>mlp.table` names the experts of every token id, all with one weight."""
+        cfg, B = self.cfg, self.B
+        self.room("moe.ids", top, "i32"); self.room("moe.w", top, "f32")
+        op = self.op(f"moe_table_{experts}x{top}", lambda: K.route_table_op(experts, top, cfg.vocab))
+        return [{"op": op, "label": p + "route", "args": [B("token_ids"), self.same(p + "mlp.table", (cfg.vocab, top), "i32"), B("moe.ids"), B("moe.w"), self.V("tokens"),
+                                                          self.err]}, *self.experts(p, experts, top, ff)]
+
+    def experts(self, p: str, experts: int, top: int, ff: int, glu: str = "swiglu", limit: float = 0.0) -> list[dict]:
+        """The chosen experts (`moe.ids`) of every row."""
+        cfg, d, B = self.cfg, self.cfg.width, self.B
         E, k, T, A, err = experts, top, cfg.max_tokens, self.act, self.err
-        w_router, outputs = router or (self.same(p + "mlp.router", (E, d)), E)
-        self.room("moe.logits", outputs, "f32"); self.room("moe.ids", k, "i32"); self.room("moe.w", k, "f32"); self.room("moe.perm", k, "i32")
+        self.room("moe.perm", k, "i32")
         self.room("moe.x", k * d); self.room("moe.act", k * ff); self.room("moe.y", k * d)
         tiles = T * k // K.routed_tile_rows(A, d, ff) + E
         for name, shape in (("moe.offsets", [E + 1]), ("moe.tiles", [tiles, 4]), ("moe.tile_count", [1]), ("moe.rows", [1])):
@@ -240,8 +314,6 @@ class Listed:
         w1 = self.weight(f"w.{p}mlp.w1", (E, 2 * ff, d), *[f"{p}mlp.e{e}.{t}" for e in range(E) for t in ("gate", "up")])
         w2 = self.weight(f"w.{p}mlp.w2", (E, d, ff), *[f"{p}mlp.e{e}.down" for e in range(E)])
         return [
-            self.linear("router", outputs, d, B("xn"), w_router, B("moe.logits"), label=p + "router", epilogue="f32"),
-            route(B("moe.logits"), B("moe.ids"), B("moe.w")),
             {"op": f"moe_plan_{tag}", "label": p + "plan", "args": [B("moe.ids"), B("moe.perm"), B("moe.offsets"), B("moe.tiles"), B("moe.tile_count"), B("moe.rows"), n, err]},
             {"op": f"moe_gather_{tag}", "label": p + "gather", "args": [B("xn"), B("moe.perm"), B("moe.x"), n]},
             {"op": f"moe_fc1_{tag}", "label": p + "fc1", "args": [B("moe.x"), w1, B("moe.act"), B("moe.tiles"), B("moe.tile_count"), n, err]},
@@ -296,6 +368,11 @@ def gla_sizes(m: dict) -> dict:
     q, v = m["heads"] * m["dim"], m["heads"] * m["vdim"]
     line, s_off = K.lin_line_bytes(m["heads"], m["dim"], m["vdim"])
     return {"q": q, "v": v, "line": line, "s_off": s_off}
+
+
+def latent_sizes(m: dict) -> dict:
+    H, r = m["heads"], m["kv_rank"]
+    return {"q": H * m["dim"], "rot": H * m["rot_dim"], "v": H * m["vdim"], "rank": r, "lat": H * r, "down": r + m["rot_dim"]}
 
 
 # ---- checkpoints -------------------------------------------------------------------------------------------

@@ -8,7 +8,7 @@ import dataclasses
 import json
 from pathlib import Path
 
-ARCHITECTURES = {"Barotar": "barotar", "Diderax": "diderax", "Gafapel": "gafapel"}      # config.json's `architecture` -> the module of its family
+ARCHITECTURES = {"Barotar": "barotar", "Diderax": "diderax", "Fusasun": "fusasun", "Gafapel": "gafapel"}      # config.json's `architecture` -> the module of its family
 
 
 def is_folder(name: str) -> bool:
@@ -28,7 +28,7 @@ def from_folder(path, **overrides):
 
 
 def families() -> dict:
-    from . import barotar, dense, diderax, gafapel, hybrid, latent, moe
+    from . import barotar, dense, diderax, fusasun, gafapel, hybrid, latent, moe
 
     out = {}
     for cfg in (dense.TOY, dense.TINY, dense.DENSE_8B):
@@ -46,6 +46,8 @@ def families() -> dict:
         out[cfg.name] = (cfg, barotar.build_manifest, barotar.load_random_weights, barotar.random_weights)
     for cfg in (diderax.TINY_DIDERAX, diderax.DIDERAX_LARGE):
         out[cfg.name] = (cfg, diderax.build_manifest, diderax.load_random_weights, diderax.random_weights)
+    for cfg in (fusasun.TINY_FUSASUN, fusasun.FUSASUN_LARGE):
+        out[cfg.name] = (cfg, fusasun.build_manifest, fusasun.load_random_weights, fusasun.random_weights)
     from . import toy_int
 
     for lined in (False, True):

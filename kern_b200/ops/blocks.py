@@ -1,4 +1,4 @@
-"""CPU statements of the kernels in hyper.cu, resid.cu, linear.cu, ssd.cu, lin_attn.cu, latent.cu, attn_window.cu (and the forms
+"""CPU statements of the kernels in hyper.cu, resid.cu, linear.cu, ssd.cu, lin_attn.cu, latent.cu, attn_window.cu, conv_add.cu (and the forms
 of the same mechanisms in mla_decode.cu / moe.cu / ssd_chunk.cu / lin_attn_chunk.cu / attn_fmha.cu / gemm_bf16.cu):
 what each launch computes, over the same arguments, for `kern_b200.cpu.CpuRuntime`. Rounding follows the buffers' types."""
 from __future__ import annotations
@@ -66,28 +66,34 @@ def k_row_norm(g, src, cu, rows, w, y, src_rows, d, eps):
 
 
 # ---- the residual with norms on both sides ----
-def k_resid_embed(g, ids, table, w, x, xn, d, vocab, eps, err):
+def k_resid_embed(g, ids, table, w, x, xn, d, vocab, scale, eps, err):
     n = g[0]
     tok = ids[:n].long()
     if ((tok < 0) | (tok >= vocab)).any():
         err[0] = 300
-    e = _f(table[: vocab * d].view(vocab, d)[torch.where((tok < 0) | (tok >= vocab), 0, tok)])
+    e = _f(table[: vocab * d].view(vocab, d)[torch.where((tok < 0) | (tok >= vocab), 0, tok)]) * scale
     x[: n * d] = e.reshape(-1)
     xn[: n * d] = _norm(e, w[:d], eps).to(xn.dtype).reshape(-1)
 
 
-def k_resid_mix(g, x, y, perm, topw, w_post, w_next, xn, hidden, d, k, eps):
-    n = g[0]
+def _routed_rows(n, y, perm, topw, d, k):
     if isinstance(perm, T):
-        v = (_f(y.view(-1)[: n * k * d].view(-1, d)[perm[: n * k].long()]).view(n, k, d) * topw[: n * k].view(n, k, 1)).sum(1)
-    else:
-        v = _f(y[: n * d].view(n, d))
-    new = x[: n * d].view(n, d) + (_norm(v, w_post[:d], eps) if isinstance(w_post, T) else v)
+        return (_f(y.view(-1)[: n * k * d].view(-1, d)[perm[: n * k].long()]).view(n, k, d) * topw[: n * k].view(n, k, 1)).sum(1)
+    return _f(y[: n * d].view(n, d))
+
+
+def _resid_out(n, x, v, w_next, xn, hidden, d, eps):
+    new = x[: n * d].view(n, d) + v
     if isinstance(hidden, T):
         hidden[: n * d] = new.reshape(-1)
     else:
         x[: n * d] = new.reshape(-1)
         xn[: n * d] = _norm(new, w_next[:d], eps).to(xn.dtype).reshape(-1)
+
+
+def k_resid_mix(g, x, y, perm, topw, w_post, w_next, xn, hidden, d, k, eps):
+    v = _routed_rows(g[0], y, perm, topw, d, k)
+    _resid_out(g[0], x, _norm(v, w_post[:d], eps) if isinstance(w_post, T) else v, w_next, xn, hidden, d, eps)
 
 
 def k_resid_scale(g, x, y, perm, topw, shared, gate, bias, scale, w_next, xn, hidden, d, k, gs, eps):
@@ -325,6 +331,46 @@ def k_lin_norm_gate(g, o, gate, w, out, H, dv, gs, norm_step, os_, out_scale, ep
     _rows(out, n, H * dv, os_).copy_(y.reshape(n, -1) * F.silu(_f(_rows(gate, n, H * dv, gs))))
 
 
+# ---- a convolution added to its input ----
+def k_conv_add(g, h, out, state, lines, cu, w, seqs, rows, d, taps, line_bytes):
+    wt = _f(w[: d * taps].view(d, taps))
+    for s in range(seqs):
+        r0, r1 = _rows_of(cu, s)
+        if r1 <= r0:
+            continue
+        ln, n = int(lines[s]), r1 - r0
+        past = _f(_window(state, ln, line_bytes, taps - 1, d, h.dtype)) if ln > 0 else torch.zeros(taps - 1, d)
+        both = torch.cat([past, _f(h[r0 * d: r1 * d].view(n, d))])
+        out[r0 * d: r1 * d] = (both[taps - 1:] + sum(wt[:, j] * both[j: j + n] for j in range(taps))).to(out.dtype).reshape(-1)
+
+
+def k_conv_add_state(g, h, state, lines, cu, d, taps, line_bytes):
+    k_ssd_conv_state(g, h, state, lines, cu, g[0], d, taps, d, line_bytes)
+
+
+def _conv_rows(n, xn, w, out, state, lines, d, taps, line_bytes):
+    one = torch.arange(n + 1, dtype=torch.int32)
+    k_conv_add(None, xn, out, state, lines, one, w, n, n, d, taps, line_bytes)
+    k_conv_add_state((n,), xn, state, lines, one, d, taps, line_bytes)
+
+
+def k_resid_embed_conv(g, ids, table, w_norm, x, xn, d, vocab, scale, eps, err, *conv):
+    k_resid_embed(g, ids, table, w_norm, x, xn, d, vocab, scale, eps, err)
+    w, out, state, lines, taps, line_bytes = conv
+    _conv_rows(g[0], xn, w, out, state, lines, d, taps, line_bytes)
+
+
+def k_resid_gate(g, x, y, perm, topw, w_post, w_next, xn, hidden, d, k, eps, gate, gate_b):
+    n = g[0]
+    v = _routed_rows(n, y, perm, topw, d, k) * torch.sigmoid(_f(gate[: n * d].view(n, d)) + _f(gate_b[:d]))
+    _resid_out(n, x, _norm(v, w_post[:d], eps), w_next, xn, hidden, d, eps)
+
+
+def k_resid_gate_conv(g, x, y, perm, topw, w_post, w_next, xn, d, k, eps, gate, gate_b, w, out, state, lines, taps, line_bytes):
+    k_resid_gate(g, x, y, perm, topw, w_post, w_next, xn, 0, d, k, eps, gate, gate_b)
+    _conv_rows(g[0], xn, w, out, state, lines, d, taps, line_bytes)
+
+
 # ---- attention in a sliding window ----
 def _window_pool(cache, dt, hk, page, d, dv):
     pool = cache.view(dt).view(-1, hk * page * (d + dv))
@@ -340,7 +386,7 @@ def k_qk_prep(g, qkv, cache, positions, slots, cos, sin, qn, kn, hq, hk, d, dv, 
     c, s = (t.view(-1)[: max_pos * (rot // 2)].view(max_pos, rot // 2)[pos][:, None] for t in (cos, sin))
 
     def turned(x, w):
-        x = _norm(x, w[:d], eps)
+        x = _norm(x, w[:d], eps) if isinstance(w, T) else x
         a, b = (x[..., : rot // 2], x[..., rot // 2: rot]) if halves else (x[..., :rot:2], x[..., 1:rot:2])
         a, b = a * c - b * s, b * c + a * s
         return torch.cat([a, b, x[..., rot:]] if halves else [torch.stack([a, b], -1).flatten(-2), x[..., rot:]], -1)
@@ -468,6 +514,93 @@ def k_window_fmha(g, kv, q, out, table, lens, cu, work, count, hq, hk, qs, os_, 
     _window_listed(q, kv, out, table, lens, cu, work, count, 128 // (hq // hk), sink, hq, hk, 128, qs, os_, max_pages, page, window, c1, c2, out_scale)
 
 
+# ---- attention in a window beside pooled blocks ----
+def _pooled_pool(pooled, dt, hk, slots, d, dv, stride):
+    """(keys [pages, hk, slots, d], values) of the second cache, whose pages are `stride` bytes."""
+    es, n = dt.itemsize, hk * slots * (d + dv)
+    rows = torch.as_strided(pooled.view(dt), (pooled.numel() // stride, n), (stride // es, 1))
+    return rows[:, : hk * slots * d].unflatten(1, (hk, slots, d)), rows[:, hk * slots * d:].unflatten(1, (hk, slots, dv))
+
+
+def _pool_rows(n, cache, pooled, positions, slots, table, seq_of, hk, d, dv, page, pool, n_slots, stride, max_pages, dt):
+    ks, vs = _window_pool(cache, dt, hk, page, d, dv)
+    pk, pv = _pooled_pool(pooled, dt, hk, n_slots, d, dv, stride)
+    tb = table.view(-1, max_pages)
+    for t in range(n):
+        pos, slot = int(positions[t]), int(slots[t])
+        if slot < 0 or (pos + 1) % pool:
+            continue
+        b = pos // pool
+        at = torch.arange(b * pool, pos + 1)
+        pages, off = tb[seq_of(t)][at // page].long(), at % page
+        place = b - pos // page * page // pool
+        pk[slot // page, :, place] = _f(ks[pages, :, off]).mean(0).to(dt)
+        pv[slot // page, :, place] = _f(vs[pages, :, off]).mean(0).to(dt)
+
+
+def k_qk_prep_pool(g, qkv, cache, pooled, positions, slots, table, cos, sin, hq, hk, d, dv, rot, halves, page, stride, max_pos, pool, n_slots, pstride, max_pages, err):
+    k_qk_prep(g, qkv, cache, positions, slots, cos, sin, 0, 0, hq, hk, d, dv, rot, halves, page, stride, max_pos, 0.0, err)
+    _pool_rows(g[0], cache, pooled, positions, slots, table, lambda t: t, hk, d, dv, page, pool, n_slots, pstride, max_pages, qkv.dtype)
+
+
+def _k_pool_blocks(dt):
+    def run(g, cache, pooled, positions, slots, table, cu, seqs, rows, hk, d, dv, page, pool, n_slots, pstride, max_pages, err):
+        seq_of = torch.repeat_interleave(torch.arange(seqs), (cu[1: seqs + 1] - cu[:seqs]).long()).tolist()
+        _pool_rows(min(rows, len(seq_of)), cache, pooled, positions, slots, table, seq_of.__getitem__, hk, d, dv, page, pool, n_slots, pstride, max_pages, dt)
+    return run
+
+
+def _pooled_row(q, cache, pooled, out, pages, L, hq, hk, d, dv, page, window, pool, n_slots, pstride, scale):
+    """One row at position L - 1: the window, and the blocks that end before it."""
+    ks, vs = _window_pool(cache, q.dtype, hk, page, d, dv)
+    pk, pv = _pooled_pool(pooled, q.dtype, hk, n_slots, d, dv, pstride)
+    j = torch.arange(max(0, L - window), L)
+    b = torch.arange(max(0, L - window) // pool)
+    last = b * pool + pool - 1
+    ids = lambda x: pages[x // page].long()
+    place = b - last // page * page // pool
+    k, v = (torch.cat([_f(pt[ids(last), :, place]), _f(t[ids(j), :, j % page])]).repeat_interleave(hq // hk, 1) for pt, t in ((pk, ks), (pv, vs)))
+    s = torch.einsum("hd,lhd->hl", _f(q).view(hq, d), k) * scale
+    out.copy_(torch.einsum("hl,lhv->hv", torch.softmax(s, 1), v).reshape(-1))
+
+
+def k_pooled_attn(g, q, cache, pooled, out, table, lens, row_seq, hq, hk, d, dv, qs, os_, max_pages, page, window, pool, n_slots, pstride, scale, err):
+    tb = table.view(-1, max_pages)
+    for r in range(g[1]):
+        if int(lens[r]) > 0:
+            _pooled_row(q[r * qs: r * qs + hq * d], cache, pooled, out[r * os_: r * os_ + hq * dv], tb[int(row_seq[r]) if isinstance(row_seq, T) else r], int(lens[r]),
+                        hq, hk, d, dv, page, window, pool, n_slots, pstride, scale)
+
+
+def _pooled_listed(kv, pooled, q, out, table, lens, cu, work, count, tokens, hq, hk, d, qs, os_, max_pages, page, window, pool, n_slots, scale_log2):
+    tb, pstride = table.view(-1, max_pages), 2 * hk * n_slots * d * q.element_size()
+    for s, b in work.view(-1, 2)[: int(count[0])].tolist():
+        r0, r1 = int(cu[s]), int(cu[s + 1])
+        for t in range(b * tokens, min((b + 1) * tokens, r1 - r0)):
+            r = r0 + t
+            _pooled_row(q[r * qs: r * qs + hq * d], kv, pooled, out[r * os_: r * os_ + hq * d], tb[s], int(lens[s]) - (r1 - r0) + t + 1, hq, hk, d, d, page, window, pool,
+                        n_slots, pstride, scale_log2 / 1.4426950408889634)
+
+
+def _k_pooled(prefill, d):
+    def run(g, kv, pooled, q, out, ws_o, ws_ml, table, lens, cu, work, count, hq, hk, qs, os_, max_pages, page, splits, pool_pages, err, window, pool, n_slots, sl2):
+        # a split launch is followed by the merge; here it writes the finished rows and the merge is a no-op
+        rows = (cu, work, count, (64 if prefill else 16) // (hq // hk)) if isinstance(work, T) else (*_one_each(g[1], lens), 1)
+        _pooled_listed(kv, pooled, q, out, table, lens, *rows, hq, hk, d, qs, os_, max_pages, page, window, pool, n_slots, sl2)
+    return run
+
+
+def _k_pooled_ragged(d):
+    def run(g, kv, pooled, q, out, table, lens, cu, wp, cp, wd, cd, hq, hk, qs, os_, max_pages, page, pool_pages, err, window, pool, n_slots, sl2):
+        for w, c, rows in ((wp, cp, 64), (wd, cd, 16)):
+            _pooled_listed(kv, pooled, q, out, table, lens, cu, w, c, rows // (hq // hk), hq, hk, d, qs, os_, max_pages, page, window, pool, n_slots, sl2)
+    return run
+
+
+def k_pooled_fmha(g, kv, pooled, q, out, table, lens, cu, work, count, hq, hk, qs, os_, max_pages, page, pool_pages, err, window, pool, n_slots, sl2):
+    _pooled_listed(kv, pooled, q, out, table, lens, cu, work, count, 128 // (hq // hk), hq, hk, 128, qs, os_, max_pages, page, window, pool, n_slots, sl2)
+
+
 # ---- latent attention ----
 def k_latent_append(g, lat, cache, slots, w, rank, stride, eps):
     n = g[0]
@@ -499,26 +632,27 @@ def k_latent_decode(g, kv, q, out, ws_o, ws_ml, table, lens, seqs, heads, qs, os
     _attend(q, kv, out, table, lens, row_seq, g[1], heads, rank, max_pages, page, scale_log2 / 1.4426950408889634)
 
 
-def _turn_halves(x, pos, cos, sin, max_pos, rot):
-    """x [n, heads, rot], pairs (i, i + rot / 2), by the tables' rows `pos` [n]."""
+def _turn(x, pos, cos, sin, max_pos, rot, halves):
+    """x [n, heads, rot], pairs (i, i + rot / 2) or neighbours, by the tables' rows `pos` [n]."""
     c, s = (t.view(-1)[: max_pos * (rot // 2)].view(max_pos, rot // 2)[pos][:, None] for t in (cos, sin))
-    a, b = x[..., : rot // 2], x[..., rot // 2:]
-    return torch.cat([a * c - b * s, b * c + a * s], -1)
+    a, b = (x[..., : rot // 2], x[..., rot // 2:]) if halves else (x[..., ::2], x[..., 1::2])
+    a, b = a * c - b * s, b * c + a * s
+    return torch.cat([a, b], -1) if halves else torch.stack([a, b], -1).flatten(-2)
 
 
-def k_latent_prep(g, rows, cache, q_low, positions, slots, cos, sin, w, wq, rank, rot, q_rank, stride, qs, max_pos, eps, err):
+def k_latent_prep(g, rows, cache, q_low, positions, slots, cos, sin, w, wq, rank, rot, halves, q_rank, stride, qs, max_pos, eps, err):
     n = g[0]
     x, pos, sl = _f(_rows(rows, n, q_rank + rank + rot, stride)), positions[:n].long(), slots[:n].long()
     if ((pos < 0) | (pos >= max_pos)).any():
         err[0] = 300
     pos = torch.where((pos < 0) | (pos >= max_pos), 0, pos)
     _rows(q_low, n, q_rank, qs).copy_(_norm(x[:, :q_rank], wq[:q_rank], eps))
-    key = _turn_halves(x[:, None, q_rank + rank:], pos, cos, sin, max_pos, rot)[:, 0]
+    key = _turn(x[:, None, q_rank + rank:], pos, cos, sin, max_pos, rot, halves)[:, 0]
     new = torch.cat([_norm(x[:, q_rank: q_rank + rank], w[:rank], eps), key], -1).to(rows.dtype)
     cache.view(rows.dtype).view(-1, rank + rot)[sl[sl >= 0]] = new[sl >= 0]
 
 
-def _attend_rot(q, cache, out, table, lens, row_seq, n, heads, rank, rot, max_pages, page, scale, q_rot, cos, sin, sink, rs, max_pos, err):
+def _attend_rot(q, cache, out, table, lens, row_seq, n, heads, rank, rot, max_pages, page, scale, q_rot, cos, sin, sink, gate, rs, max_pos, halves, window, gs, err):
     pool = cache.view(q.dtype).view(-1, page, rank + rot)
     tb = table.view(-1, max_pages)
     for r in range(n):
@@ -527,21 +661,35 @@ def _attend_rot(q, cache, out, table, lens, row_seq, n, heads, rank, rot, max_pa
             continue
         if L > max_pos:
             err[0] = 300
-        c = _f(pool[tb[int(row_seq[r]) if isinstance(row_seq, T) else r, : -(-L // page)].long()]).reshape(-1, rank + rot)[:L]
-        turned = _turn_halves(_f(q_rot[r * rs: r * rs + heads * rot].view(1, heads, rot)), torch.tensor([min(L, max_pos) - 1]), cos, sin, max_pos, rot)[0]
+        c = _f(pool[tb[int(row_seq[r]) if isinstance(row_seq, T) else r, : -(-L // page)].long()]).reshape(-1, rank + rot)[max(0, L - window):L]
+        turned = _turn(_f(q_rot[r * rs: r * rs + heads * rot].view(1, heads, rot)), torch.tensor([min(L, max_pos) - 1]), cos, sin, max_pos, rot, halves)[0]
         qq = torch.cat([_f(q[r * heads * rank:(r + 1) * heads * rank].view(heads, rank)), turned.to(q.dtype).float()], -1)
-        p = torch.softmax(torch.cat([qq @ c.t() * scale, _f(sink[:heads])[:, None]], 1), -1)[:, :-1]
-        out[r * heads * rank:(r + 1) * heads * rank] = (p @ c[:, :rank]).to(out.dtype).reshape(-1)
+        s = qq @ c.t() * scale
+        p = torch.softmax(torch.cat([s, _f(sink[:heads])[:, None]], 1), -1)[:, :-1] if isinstance(sink, T) else torch.softmax(s, -1)
+        o = p @ c[:, :rank]
+        o = o * torch.sigmoid(_f(gate[r * gs: r * gs + heads]))[:, None] if isinstance(gate, T) else o
+        out[r * heads * rank:(r + 1) * heads * rank] = o.to(out.dtype).reshape(-1)
 
 
-def k_latent_rot_attn(g, q, cache, out, table, lens, row_seq, heads, rank, max_pages, page, scale, err, q_rot, cos, sin, sink, rs, rot, max_pos):
-    _attend_rot(q, cache, out, table, lens, row_seq, g[1], heads, rank, rot, max_pages, page, scale, q_rot, cos, sin, sink, rs, max_pos, err)
+def k_latent_rot_attn(g, q, cache, out, table, lens, row_seq, heads, rank, max_pages, page, scale, err, q_rot, cos, sin, sink, gate, rs, rot, max_pos, halves, window, gs):
+    _attend_rot(q, cache, out, table, lens, row_seq, g[1], heads, rank, rot, max_pages, page, scale, q_rot, cos, sin, sink, gate, rs, max_pos, halves, window, gs, err)
 
 
 def k_latent_rot_decode(g, kv, q, out, ws_o, ws_ml, table, lens, seqs, heads, qs, os_, max_pages, page, splits, pool_pages, scale_log2, err, row_seq, rank,
-                        q_rot, cos, sin, sink, rs, rot, max_pos):
+                        q_rot, cos, sin, sink, gate, rs, rot, max_pos, halves, window, gs):
     # a split launch is followed by the merge; here the first writes the finished rows and the merge is a no-op
-    _attend_rot(q, kv, out, table, lens, row_seq, g[1], heads, rank, rot, max_pages, page, scale_log2 / 1.4426950408889634, q_rot, cos, sin, sink, rs, max_pos, err)
+    _attend_rot(q, kv, out, table, lens, row_seq, g[1], heads, rank, rot, max_pages, page, scale_log2 / 1.4426950408889634, q_rot, cos, sin, sink, gate, rs, max_pos,
+                halves, window, gs, err)
+
+
+def k_route_table(g, ids, table, out, w, tokens, E, k, vocab, err):
+    tok = ids[:tokens].long()
+    ok = (tok >= 0) & (tok < vocab)
+    rows = torch.where(ok[:, None], table[: vocab * k].view(vocab, k)[torch.where(ok, tok, 0)], -1)
+    if ((rows < 0) | (rows >= E)).any():
+        err[0] = 300
+    out[: tokens * k] = rows.reshape(-1)
+    w[: tokens * k] = 1.0 / k
 
 
 def k_route_logits(g, logits, bias, ids, w, tokens, E, k, ld):
@@ -564,10 +712,13 @@ def k_route_groups(g, logits, bias, ids, w, tokens, E, k, groups, keep, softmax,
     w[: tokens * k] = ((top / (top.sum(-1, keepdim=True) + 1e-20) if renorm else top) * scale).reshape(-1)
 
 
-for _a in ("bf16", "f32"):
+_DT = {"bf16": torch.bfloat16, "f32": torch.float32}
+for _a in _DT:
     CPU_KERNELS.update({f"kern_hyper_embed_{_a}": k_hyper_embed, f"kern_row_norm_f32_{_a}": k_row_norm,
                         f"kern_rows_scatter_{_a}": k_rows_scatter, f"kern_gate_mul_{_a}": k_gate_mul,
-                        f"kern_resid_embed_{_a}": k_resid_embed, f"kern_resid_mix_{_a}": k_resid_mix,
+                        f"kern_resid_embed_{_a}": k_resid_embed, f"kern_resid_mix_{_a}": k_resid_mix, f"kern_resid_embed_conv_{_a}": k_resid_embed_conv,
+                        f"kern_resid_gate_{_a}": k_resid_gate, f"kern_resid_gate_conv_{_a}": k_resid_gate_conv, f"kern_conv_add_{_a}": k_conv_add,
+                        f"kern_conv_add_state_{_a}": k_conv_add_state, f"kern_qk_prep_pool_{_a}": k_qk_prep_pool, f"kern_pool_blocks_{_a}": _k_pool_blocks(_DT[_a]),
                         f"kern_resid_scale_{_a}": k_resid_scale, f"kern_resid_scale_routed_{_a}": k_resid_scale, f"kern_qk_prep_whole_{_a}": k_qk_prep_whole, f"kern_latent_prep_{_a}": k_latent_prep,
                         f"kern_token_shift_{_a}": k_token_shift, f"kern_shift_state_{_a}": k_shift_state, f"kern_decay_{_a}": k_decay,
                         f"kern_lin_norm_gate_{_a}": k_lin_norm_gate, f"kern_qk_prep_{_a}": k_qk_prep,
@@ -578,18 +729,20 @@ for _a in ("bf16", "f32"):
     CPU_KERNELS.update({f"kern_{k}_{_a}{'_' + e if e else ''}": f(e) for k, f in (("linear", _k_linear), ("linear_grouped", _k_grouped))
                         for e in ("", "swiglu", "geglu", "clamped")})
     CPU_KERNELS.update({f"kern_lin_rule_{_a}_r{r}_v{v}": k_lin_rule for r in (4, 8, 16, 32) for v in (1, 2, 4)})
-    CPU_KERNELS.update({f"kern_window_attn_{_a}_w{w}": k_window_attn for w in (64, 128, 256, 512)})
+    CPU_KERNELS.update({f"kern_{k}_attn_{_a}_w{w}": f for k, f in (("window", k_window_attn), ("pooled", k_pooled_attn)) for w in (64, 128, 256, 512)})
     CPU_KERNELS.update({f"kern_latent_{n}_{_a}_w{w}": f for n, f in (("attn", k_latent_attn), ("rot_attn", k_latent_rot_attn)) for w in (64, 128, 256, 512, 1024)})
 CPU_KERNELS.update({"kern_linear_bf16_f32": _k_linear(""), "kern_transpose_heads_bf16": k_transpose_heads, "kern_copy_cols_bf16": k_copy_cols,
                     "kern_moe_route_logits": k_route_logits, "kern_moe_route_groups": k_route_groups, "kern_attn_window_fmha_d128": k_window_fmha,
-                    "kern_attn_sink_fmha_d128": k_sink_fmha,
-                    "kern_attn_window_merge": lambda *a: None})
+                    "kern_attn_sink_fmha_d128": k_sink_fmha, "kern_attn_pooled_fmha_d128": k_pooled_fmha, "kern_moe_route_table": k_route_table,
+                    "kern_attn_window_merge": lambda *a: None, "kern_attn_gated_merge": lambda *a: None})
 CPU_KERNELS.update({f"kern_moe_gemm_bf16_{e}_n{n}": _k_moe_gemm(e) for e in ("geglu", "clamped") for n in (64, 128)})
 CPU_KERNELS.update({f"kern_lin_{k}_n{n}": f for k, f in (("prep", k_lin_prep), ("chunk", k_lin_chunk)) for n in (32, 64, 128, 256)})
 CPU_KERNELS.update({f"kern_attn_window_{k}_d{d}": _k_window(k == "prefill", d) for k in ("decode", "prefill") for d in (64, 128, 256)})
 CPU_KERNELS.update({f"kern_attn_window_ragged_d{d}": _k_window_ragged(d) for d in (64, 128)})
 CPU_KERNELS.update({f"kern_attn_sink_{k}_d{d}": _k_sink(k == "prefill", d) for k in ("decode", "prefill") for d in (64, 128, 256)})
 CPU_KERNELS.update({f"kern_attn_sink_ragged_d{d}": _k_sink_ragged(d) for d in (64, 128)})
+CPU_KERNELS.update({f"kern_attn_pooled_{k}_d{d}": _k_pooled(k == "prefill", d) for k in ("decode", "prefill") for d in (64, 128, 256)})
+CPU_KERNELS.update({f"kern_attn_pooled_ragged_d{d}": _k_pooled_ragged(d) for d in (64, 128)})
 CPU_KERNELS.update({f"kern_gemm_bf16_heads_n{n}": k_gemm_heads for n in (64, 128, 256)})
 CPU_KERNELS.update({f"kern_ssd_chunk_n{n}": k_ssd_chunk for n in (32, 64, 128, 256)})
 CPU_KERNELS.update({f"kern_latent_decode_bf16_b{b}": k_latent_decode for b in range(1, 9)})
