@@ -76,11 +76,11 @@ def main():
     ap.add_argument("--steps", type=int, default=256, help="timed steps (256 = every live sequence turns over once)")
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--config", default="b", choices=["b", "c", "d", "e", "gafapel", "barotar", "diderax", "toy"],
+    ap.add_argument("--config", default="b", choices=["b", "c", "d", "e", "gafapel", "barotar", "diderax", "fusasun", "toy"],
                     help="b: dense GQA 8B-class at concurrency 256 (the headline); c: the hybrid 27B-class decoder under agent-style "
                          "traffic on one GPU; d: decode of a routed-experts decoder with the experts sharded over the GPUs "
                          "(fused dispatch / combine); e: pipelined prefill of 32k-token prompts, then decode, over the KDA + latent-attention + "
-                         "routed-experts decoder, a stage per GPU; gafapel, barotar, diderax: prefill and decode of that decoder with listed layers beside it at equal size, "
+                         "routed-experts decoder, a stage per GPU; gafapel, barotar, diderax, fusasun: prefill and decode of that decoder with listed layers beside it at equal size, "
                          "call by call against the roofline (--layers, default 8); toy: the reference's own toy-paged package "
                          "(its manifest and cubin) served by this engine, the workload of the reference arm")
     ap.add_argument("--concurrency", type=int, default=256)
@@ -123,7 +123,7 @@ def main():
         return pp_pipeline_check.main(["--bench", "--json-line", "--model", "latent-48b-a3b", "--prompt", "32768", "--chunk", "2048",
                                        "--requests", str(max(1, min(args.concurrency, 4))), "--decode-steps", str(min(args.steps, 64)),
                                        "--timeout", "120"] + (["--layers", str(args.layers)] if args.layers != 36 else []))
-    if args.config in ("gafapel", "barotar", "diderax"):
+    if args.config in ("gafapel", "barotar", "diderax", "fusasun"):
         from kern_b200.testing import bench_layers
 
         return bench_layers.main(args)

@@ -173,13 +173,17 @@ KERN_DEVICE void pool_body(const T* cache, T* pooled, const int* pages, long lon
     const size_t base = (is_k ? 0 : (size_t)kcols * page) + (size_t)h * page * cols + i;
     T* dst = out + (is_k ? 0 : (size_t)kcols * slots) + ((size_t)h * slots + at) * cols + i;
     Vec<V> acc = {};
-#pragma unroll 4
-    for (int j = first; j < first + pool; ++j) {
-      const T* src = cache + (size_t)pages[j / page] * hk * page * (d + dv) + base + (size_t)(j % page) * cols;
-      if (!KERN_CHECK(src, V * sizeof(T), SITE_KV_ROW)) continue;
-      const Vec<V> a = ldv<V>(src);
+    for (int left = pool, pi = first / page, off = first % page; left > 0; ++pi, off = 0) {      // page by page
+      const int run = min(left, page - off);
+      const T* src = cache + (size_t)pages[pi] * hk * page * (d + dv) + base + (size_t)off * cols;
+      left -= run;
+      if (!KERN_CHECK(src, (size_t)run * cols * sizeof(T), SITE_KV_ROW)) continue;
+#pragma unroll 8
+      for (int j = 0; j < run; ++j) {
+        const Vec<V> a = ldv<V>(src + (size_t)j * cols);
 #pragma unroll
-      for (int e = 0; e < V; ++e) acc.v[e] += a.v[e];
+        for (int e = 0; e < V; ++e) acc.v[e] += a.v[e];
+      }
     }
     if (!KERN_CHECK(dst, V * sizeof(T), SITE_KV_APPEND)) continue;
 #pragma unroll

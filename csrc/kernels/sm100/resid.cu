@@ -44,6 +44,9 @@ KERN_DEVICE void norm_out(const float* u, float inv, const __nv_bfloat16* w, T* 
   }
 }
 
+// what a later pass over the row reads, on its way from memory while the first sums are made
+KERN_DEVICE void fetch(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
 // out = h + conv(h) of one row per sequence, conv_t = sum_j w[c][j] h_(t - taps + 1 + j). `state` holds lines of the last
 // taps - 1 rows, which move on by one; line 0 is nobody's (zeros, and nothing is kept).
 template <typename T>
@@ -89,12 +92,29 @@ KERN_DEVICE void conv_step(const ConvStep<T>& cv, int line, int t, int i, const 
   stv<V>(cv.out + (size_t)t * width + i, acc);
 }
 
+template <typename T>
+KERN_DEVICE int conv_line(const ConvStep<T>& cv, int t) {
+  const int line = cv.lines[t];
+  return line > 0 && KERN_CHECK(cv.state + (size_t)line * cv.line_bytes, (size_t)cv.line_bytes, SITE_STATE_SLOT) ? line : 0;
+}
+
+// the row's past and the norm's and the convolution's weights, 128 bytes a thread and step
+template <typename T>
+KERN_DEVICE void fetch_conv(const ConvStep<T>& cv, const __nv_bfloat16* w_post, const __nv_bfloat16* w_next, int width) {
+  const int line = conv_line(cv, blockIdx.x), step = threadIdx.x * 128;
+  auto span = [&](const void* p, int bytes) {
+    for (int i = step; i < bytes; i += 256 * 128) fetch(reinterpret_cast<const uint8_t*>(p) + i);
+  };
+  span(cv.w, width * cv.taps * 2);
+  span(w_next, width * 2);
+  if (w_post) span(w_post, width * 2);
+  if (line > 0) span(cv.state + (size_t)line * cv.line_bytes, (cv.taps - 1) * width * (int)sizeof(T));
+}
+
 // As norm_out, and the row's convolution
 template <typename T, int V>
 KERN_DEVICE void norm_conv_out(const float* u, float inv, const __nv_bfloat16* w, T* xn, const ConvStep<T>& cv, int width) {
-  const int t = blockIdx.x;
-  int line = cv.lines[t];
-  if (line <= 0 || !KERN_CHECK(cv.state + (size_t)line * cv.line_bytes, (size_t)cv.line_bytes, SITE_STATE_SLOT)) line = 0;
+  const int t = blockIdx.x, line = conv_line(cv, t);
   for (int i = threadIdx.x * V; i < width; i += 256 * V) {
     const Vec<V> a = ldv<V>(u + i), b = ldv<V>(w + i);
     T held[V];
@@ -119,6 +139,7 @@ KERN_DEVICE void embed_body(const long long* ids, const __nv_bfloat16* table, co
     if (threadIdx.x == 0) set_error(err, ERR_BOUNDS);
     id = 0;
   }
+  if constexpr (CONV) fetch_conv(cv, nullptr, w_norm, width);
   const __nv_bfloat16* a = table + (size_t)id * width;
   const bool ok = KERN_CHECK(a, (size_t)width * 2, SITE_EMBED_ROW);
   float ss = 0.f;
@@ -146,6 +167,7 @@ KERN_DEVICE void mix_body(float* x, const T* y, const int* perm, const float* to
   __shared__ float tw[32];
   __shared__ int tr[32];
   const int t = blockIdx.x;
+  if constexpr (CONV) fetch_conv(cv, w_post, w_next, width);
   if (perm) {
     if (threadIdx.x < k) {
       const int r = perm[(size_t)t * k + threadIdx.x];

@@ -1,11 +1,12 @@
 """Prefill and decode throughput of a decoder with listed layers beside the framework's closest model at equal size, with the
-time of every kind of kernel against its roofline: `python bench.py --config gafapel|barotar|diderax [--layers N]`.
+time of every kind of kernel against its roofline: `python bench.py --config gafapel|barotar|diderax|fusasun [--layers N]`.
 
 The decoders have the width, depth, vocabulary and routed experts of the 48B-A3B shape class and random weights. Gafapel has
 Mamba-2 and unrotated latent-attention layers over four residual streams, Barotar window attention beside time mixing and gated
 linear attention, Diderax gated linear attention, grouped-query attention and 512 + 64 latent attention with sinks; the model beside
 them per-key-decay delta-rule layers and 512 + 64 latent attention. Beside Barotar and Diderax there is also the routed decoder
-with grouped-query attention of the same head counts and dims, for its attention kernels. A point is timed end to end (CUDA events around the call, captured graphs for decode,
+with grouped-query attention of the same head counts and dims, for its attention kernels. Fusasun has window attention beside
+pooled blocks and 512 + 64 latent attention in a window; beside it Diderax, and Barotar for its window attention. A point is timed end to end (CUDA events around the call, captured graphs for decode,
 L2 flushed before every sample) and once more call by call, where a call's roofline is the larger of its bytes over the
 measured copy rate and its flops over the measured tensor rate.
 """
@@ -16,7 +17,7 @@ import re
 from pathlib import Path
 
 MODELS = {"gafapel": ("gafapel-48b-a3b", "latent-48b-a3b"), "barotar": ("barotar-48b-a3b", "latent-48b-a3b", "moe-30b-a3b"),
-          "diderax": ("diderax-48b-a3b", "latent-48b-a3b", "moe-30b-a3b")}
+          "diderax": ("diderax-48b-a3b", "latent-48b-a3b", "moe-30b-a3b"), "fusasun": ("fusasun-48b-a3b", "diderax-48b-a3b", "barotar-48b-a3b")}
 POINTS = ({"groups": 1, "chunk": 2048, "context": 2048}, {"groups": 4, "chunk": 512, "context": 2048},
           {"groups": 1, "rows": 1, "context": 1024}, {"groups": 16, "rows": 1, "context": 1024}, {"groups": 64, "rows": 1, "context": 1024})
 
@@ -55,11 +56,25 @@ def cost(doc: dict, call: dict, groups: int, rows: int, context: int) -> tuple[f
     for s in st:
         if s.get("bytes_per_seq"):
             tok += 2 * groups * s["bytes_per_seq"]
-    m = re.match(r"latent_attn_[pd]_(\d+)x(\d+)x(\d+)x", op)
-    if m:                                                   # heads, latent columns, rotated columns behind them
-        H, rank, rot = map(int, m.groups())
-        flops = 2.0 * n * H * (2 * rank + rot) * (context if rows == 1 else context - (rows - 1) / 2)
-        return n * H * (2 * rank + rot) * 2.0 + groups * context * (rank + rot) * 2.0, flops
+    m = re.match(r"latent_attn_[pd]_(\d+)x(\d+)x(\d+)x\d+n?(?:w(\d+))?", op)
+    if m:                                                   # heads, latent columns, rotated columns behind them, window
+        H, rank, rot = map(int, m.groups()[:3])
+        window = int(m.group(4) or 1 << 30)
+        flops = 2.0 * groups * H * (2 * rank + rot) * sum(min(p + 1, window) for p in range(context - rows, context))
+        return n * H * (2 * rank + rot) * 2.0 + groups * min(context, window + rows - 1) * (rank + rot) * 2.0, flops
+    if op.startswith("moe_table_"):                         # a row of the table, an expert and a weight per choice
+        return n * (8 + 12.0 * int(op.rsplit("x", 1)[1])), 0.0
+    m = re.match(r"prep_pool_[pd]_(\d+)x(\d+)x(\d+)x(\d+)x\d+x(\d+)x", op)
+    if m:                                                   # q read and written, keys and values read, written and read for their means
+        hq, hk, d, dv, pool = map(int, m.groups())
+        return n * 2.0 * (2 * hq * d + hk * (d + dv) * (3 + 1 / pool)), 0.0
+    m = re.match(r"pooled_attn_[pd]_(\d+)x(\d+)x(\d+)x(\d+)x(\d+)x(\d+)x", op)
+    if m:
+        hq, hk, d, dv, window, pool = map(int, m.groups())
+        seen_by = lambda p: min(p + 1, window) + max(0, p - window + 1) // pool
+        flops = 2.0 * groups * hq * (d + dv) * sum(seen_by(p) for p in range(context - rows, context))
+        keys = min(context, window + rows - 1) + max(0, context - window) // pool
+        return n * hq * (d + dv) * 2.0 + groups * keys * hk * (d + dv) * 2.0, flops
     m = re.match(r"prep_whole_(\d+)x(\d+)x(\d+)x", op)
     if m:                                                   # q read and written, k read, keys and values written
         hq, hk, d = map(int, m.groups())
