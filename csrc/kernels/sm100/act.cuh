@@ -35,4 +35,15 @@ template <int V> KERN_DEVICE void stv(__nv_bfloat16* p, const Vec<V>& r) {
   else *p = __float2bfloat16(r.v[0]);
 }
 
+// V values as they lie in memory: what waits for its turn takes no more registers than that
+template <typename T, int V> struct RawOf { T v[V]; };
+template <> struct __align__(8) RawOf<__nv_bfloat16, 4> { uint2 v; };
+template <> struct __align__(16) RawOf<float, 4> { float4 v; };
+template <int V, typename T> KERN_DEVICE RawOf<T, V> raw(const T* p) { return *reinterpret_cast<const RawOf<T, V>*>(p); }
+template <typename T, int V> KERN_DEVICE void add(Vec<V>& a, const RawOf<T, V>& r, float w) {
+  const Vec<V> b = ldv<V>(reinterpret_cast<const T*>(&r));
+#pragma unroll
+  for (int e = 0; e < V; ++e) a.v[e] += w * b.v[e];
+}
+
 }  // namespace kern

@@ -224,17 +224,6 @@ KERN_DEVICE void mix_body(float* x, const T* y, const int* perm, const float* to
   else norm_out<T, V>(resid_sm, next, w_next, xn + (size_t)t * width, width);
 }
 
-// V values as they lie in memory: what waits for its turn takes no more registers than that
-template <typename T, int V> struct RawOf { T v[V]; };
-template <> struct __align__(8) RawOf<__nv_bfloat16, 4> { uint2 v; };
-template <> struct __align__(16) RawOf<float, 4> { float4 v; };
-template <int V, typename T> KERN_DEVICE RawOf<T, V> raw(const T* p) { return *reinterpret_cast<const RawOf<T, V>*>(p); }
-template <typename T, int V> KERN_DEVICE void add(Vec<V>& a, const RawOf<T, V>& r, float w) {
-  const Vec<V> b = ldv<V>(reinterpret_cast<const T*>(&r));
-#pragma unroll
-  for (int e = 0; e < V; ++e) a.v[e] += w * b.v[e];
-}
-
 // A sublayer's result: y, or with `perm` the weighted sum of a token's expert rows; choices without a row (perm < 0) are the
 // experts that hand back the input, xn as it is on entry. `shared` [rows][width] is weighed by sigmoid(gate[t gate_stride]).
 template <typename T, int V, bool ROUTED>

@@ -1,7 +1,7 @@
 """Op builders of the decoder blocks that take any size and either activation type (bf16, or f32 in a model's 32-bit
 form): matrix products, hyper-connections, the residual with norms on both sides, the Mamba-2 mixer, linear attention with a
-decay per key channel, latent attention with or without rotated columns, attention in a sliding window or with a sink and an
-output gate, routed experts. Where a bf16 size fits the tensor-core kernels the op is the one `common.py` builds or the
+decay per key channel, latent attention with or without rotated columns, attention in a sliding window, beside pooled blocks, or
+with a sink and an output gate, a convolution added to its input, routed experts. Where a bf16 size fits the tensor-core kernels the op is the one `common.py` builds or the
 tensor-core form of the mechanism; the rest runs generic kernels. Weights are bf16 in both forms.
 """
 from __future__ import annotations
@@ -333,12 +333,9 @@ def conv_add_op(width: int, taps: int, line_bytes: int, act: str = "bf16") -> di
     """Rows of a ragged call plus a causal convolution of them over time, channel by channel; the last taps - 1 rows of a sequence
     stay in its state line. Interface [h, w, out, state, lines, cu_seqlens, seqs, rows]."""
     iface = [f"in buffer<{act}>", "in buffer<bf16>", f"out buffer<{act}>", "inout state", "in buffer<i32>", "in buffer<i32>", "i32", "i32"]
-    conv = _launch("conv_add", f"kern_conv_add_{act}", [256, 1, 1], [{"ceil_div": ["tokens", 16]}, -(-width // (1024 if width % 4 == 0 else 256)), 1],
-                   [iface[0], iface[2], "in state", iface[4], iface[5], iface[1], "i32", "i32", "i32", "i32", "i64"],
-                   [P(0), P(2), P(3), P(4), P(5), P(1), P(6), P(7), I(width), I(taps), L(line_bytes)])
-    keep = _launch("conv_add", f"kern_conv_add_state_{act}", [256, 1, 1], ["seqs", -(-width // 256), 1], [iface[0], *iface[3:6], "i32", "i32", "i64"],
-                   [P(0), P(3), P(4), P(5), I(width), I(taps), L(line_bytes)])
-    return _op(iface, conv, *([keep] if taps > 1 else []))
+    return _op(iface, _launch("conv_add", f"kern_conv_add_{act}", [256, 1, 1], [{"ceil_div": ["tokens", 4]}, -(-width // (1024 if width % 4 == 0 else 256)), 1],
+                              [iface[0], *iface[2:6], iface[1], "i32", "i32", "i32", "i32", "i64"],
+                              [P(0), *map(P, range(2, 6)), P(1), P(6), P(7), I(width), I(taps), L(line_bytes)]))
 
 
 def resid_embed_op(width: int, vocab: int, eps: float, act: str = "bf16", scale: float = 1.0, conv: tuple[int, int] | None = None) -> dict:

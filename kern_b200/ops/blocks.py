@@ -342,16 +342,11 @@ def k_conv_add(g, h, out, state, lines, cu, w, seqs, rows, d, taps, line_bytes):
         past = _f(_window(state, ln, line_bytes, taps - 1, d, h.dtype)) if ln > 0 else torch.zeros(taps - 1, d)
         both = torch.cat([past, _f(h[r0 * d: r1 * d].view(n, d))])
         out[r0 * d: r1 * d] = (both[taps - 1:] + sum(wt[:, j] * both[j: j + n] for j in range(taps))).to(out.dtype).reshape(-1)
-
-
-def k_conv_add_state(g, h, state, lines, cu, d, taps, line_bytes):
-    k_ssd_conv_state(g, h, state, lines, cu, g[0], d, taps, d, line_bytes)
+    k_ssd_conv_state(g, h, state, lines, cu, seqs, d, taps, d, line_bytes)
 
 
 def _conv_rows(n, xn, w, out, state, lines, d, taps, line_bytes):
-    one = torch.arange(n + 1, dtype=torch.int32)
-    k_conv_add(None, xn, out, state, lines, one, w, n, n, d, taps, line_bytes)
-    k_conv_add_state((n,), xn, state, lines, one, d, taps, line_bytes)
+    k_conv_add(None, xn, out, state, lines, torch.arange(n + 1, dtype=torch.int32), w, n, n, d, taps, line_bytes)
 
 
 def k_resid_embed_conv(g, ids, table, w_norm, x, xn, d, vocab, scale, eps, err, *conv):
@@ -718,7 +713,7 @@ for _a in _DT:
                         f"kern_rows_scatter_{_a}": k_rows_scatter, f"kern_gate_mul_{_a}": k_gate_mul,
                         f"kern_resid_embed_{_a}": k_resid_embed, f"kern_resid_mix_{_a}": k_resid_mix, f"kern_resid_embed_conv_{_a}": k_resid_embed_conv,
                         f"kern_resid_gate_{_a}": k_resid_gate, f"kern_resid_gate_conv_{_a}": k_resid_gate_conv, f"kern_conv_add_{_a}": k_conv_add,
-                        f"kern_conv_add_state_{_a}": k_conv_add_state, f"kern_qk_prep_pool_{_a}": k_qk_prep_pool, f"kern_pool_blocks_{_a}": _k_pool_blocks(_DT[_a]),
+                        f"kern_qk_prep_pool_{_a}": k_qk_prep_pool, f"kern_pool_blocks_{_a}": _k_pool_blocks(_DT[_a]),
                         f"kern_resid_scale_{_a}": k_resid_scale, f"kern_resid_scale_routed_{_a}": k_resid_scale, f"kern_qk_prep_whole_{_a}": k_qk_prep_whole, f"kern_latent_prep_{_a}": k_latent_prep,
                         f"kern_token_shift_{_a}": k_token_shift, f"kern_shift_state_{_a}": k_shift_state, f"kern_decay_{_a}": k_decay,
                         f"kern_lin_norm_gate_{_a}": k_lin_norm_gate, f"kern_qk_prep_{_a}": k_qk_prep,
